@@ -117,6 +117,48 @@ int b200_paged_attn_prefill(const void* q, const void* k_pool, const void* v_poo
                             int page_size, int num_blocks, int max_pages_per_seq, float scale, void* stream);
 
 /*
+ * b200_paged_attn_decode for models whose layers ask for more (no counterpart in the reference):
+ *   chunk  > 0: the positions of a sequence are cut into chunks of this many, counted from position 0, and a row sees
+ *          only the tokens of its own position's chunk: ctx_lens[b] = L attends to tokens [(L-1)/chunk*chunk, L).
+ *          0: all L tokens.  split_tokens counts from the page that holds the first token seen.
+ *   gate   [batch, num_q_heads] fp32 or NULL: the head's output is multiplied by sigmoid(gate).
+ * head_dim up to 1024 on the generic kernel; the split-K kernel also takes kv head counts other than 1, 2, 4, 8 (in
+ * groups of the largest of these that divides them).
+ */
+int b200_paged_attn_decode_chunked(const void* q, const void* k_pool, const void* v_pool,
+                                   const int32_t* block_table, const int32_t* ctx_lens, void* out,
+                                   void* workspace, size_t workspace_bytes, int batch, int num_q_heads,
+                                   int num_kv_heads, int head_dim, int page_size, int num_blocks,
+                                   int max_pages_per_seq, float scale, int split_tokens, int dtype, int chunk,
+                                   const float* gate, void* stream);
+
+/*
+ * b200_paged_attn_prefill with the same two options (gate: [num_tokens, num_q_heads]), always on the tcgen05 kernel:
+ * head_dim 64 or 128, any number of query heads per kv head up to 128; q, out and pools 16-byte aligned.
+ */
+int b200_paged_attn_prefill_chunked(const void* q, const void* k_pool, const void* v_pool,
+                                    const int32_t* block_table_row, void* out, void* status_word, int num_tokens,
+                                    int first_position, int num_q_heads, int num_kv_heads, int head_dim,
+                                    int page_size, int num_blocks, int max_pages_per_seq, float scale, int chunk,
+                                    const float* gate, void* stream);
+
+/*
+ * Decode attention over a cache of latents: one vector c of `rank` numbers per token, shared by all heads as key and
+ * as value (the heads' key map is already applied to the queries, their value map is applied to the result):
+ *   out[b, h] = sigmoid(gate[b, h]) * sum_j softmax_j(scale * q[b, h] . c_j) c_j   over j < ctx_lens[b]
+ *   q, out     [batch, num_heads, rank] bf16
+ *   c_pool     [num_blocks, page_size, rank] bf16
+ *   workspace  b200_paged_attn_workspace_bytes(batch, num_heads, rank, ...) bytes
+ *   gate       [batch, num_heads] fp32 or NULL
+ * page_size 16, rank 64, 128, 192, 256, 384 or 512 (b200_latent_attn_supported).
+ */
+int b200_latent_attn_supported(int rank, int page_size);
+int b200_latent_attn_decode(const void* q, const void* c_pool, const int32_t* block_table, const int32_t* ctx_lens,
+                            void* out, void* workspace, size_t workspace_bytes, int batch, int num_heads, int rank,
+                            int page_size, int num_blocks, int max_pages_per_seq, float scale, int split_tokens,
+                            const float* gate, void* stream);
+
+/*
  * Paged decode attention for callers that cannot allocate device memory.
  * No counterpart in the reference: it exists for hosts of this library that own
  * no allocator at the point of the call - a server whose device memory was
@@ -191,6 +233,50 @@ size_t b200_dense_gemm_workspace_bytes(int num_rows, int out_features);
 int b200_dense_gemm_bf16(const void* x, const void* w, void* y, void* workspace, size_t workspace_bytes,
                          void* status_word, int num_rows, int out_features, int in_features, int k_split,
                          void* stream);
+
+/* b200_dense_gemm_bf16 with the fp32 accumulators written as they are (logits). */
+int b200_dense_gemm_bf16_f32(const void* x, const void* w, float* y, void* workspace, size_t workspace_bytes,
+                             void* status_word, int num_rows, int out_features, int in_features, int k_split,
+                             void* stream);
+
+/*
+ * `groups` products side by side (one per attention head) in one launch:
+ *   y[m, g*y_step + n] = sum_k x[m, g*x_step + k] * w[g*w_step + n, k],  k < in_features, n < out_features
+ *   x [num_rows, x_cols] bf16, w [(groups-1)*w_step + out_features, in_features] bf16, y [num_rows, y_cols] bf16.
+ *   in_features, x_step and x_cols multiples of 8; x and w 16-byte aligned; x finite.
+ */
+int b200_dense_gemm_grouped(const void* x, const void* w, void* y, void* status_word, int num_rows, int groups,
+                            int out_features, int in_features, int x_step, int w_step, int y_step, int x_cols,
+                            int y_cols, void* stream);
+
+/*
+ * A projection whose output goes to up to four places, split by ranges of features (segment i = features
+ * [seg_end[i-1], seg_end[i])), each feature first multiplied by col_scale[n] in fp32 when col_scale is given:
+ *   kind 0  bf16 rows [num_rows, width of the segment]          kind 1  the same in fp32
+ *   kind 2  page slots of a pool [num_blocks, heads, page_size, dim] bf16, heads * dim = width: row m goes to
+ *           position positions[m] of the sequence whose pages are block_table[m] (positions NULL: position m;
+ *           block_table NULL: page p of the sequence is block p)
+ * seg_* are HOST arrays; seg_ptr holds device pointers.  x [num_rows, in_features], w [seg_end[last], in_features].
+ */
+int b200_proj_split_gemm(const void* x, const void* w, const float* col_scale, const int32_t* seg_end,
+                         const int32_t* seg_kind, const int32_t* seg_heads, const int32_t* seg_dim,
+                         void* const* seg_ptr, int num_segs, const int32_t* positions, const int32_t* block_table,
+                         void* status_word, int num_rows, int in_features, int page_size, int num_blocks,
+                         int max_pages_per_seq, void* stream);
+
+/*
+ * Gate and up projection of a dense feed-forward with the clamped gated unit in the epilogue:
+ *   g = min(x Wg, limit), u = clamp(x Wu, -limit, limit), y = g * sigmoid(alpha g) * (u + 1)
+ *   w_interleaved [2*inter, in_features] bf16: alternating blocks of 128 gate rows and the 128 up rows of the same
+ *   features; inter a multiple of 128; y [num_rows, inter] bf16.
+ */
+int b200_dense_glu_gemm(const void* x, const void* w_interleaved, void* y, void* status_word, int num_rows, int inter,
+                        int in_features, float limit, float alpha, void* stream);
+
+/* fp32 products (true fp32 multiply-add, no reduced-precision mode), grouped like b200_dense_gemm_grouped; in_features,
+ * x_step and x_cols multiples of 4. */
+int b200_gemm_f32(const float* x, const float* w, float* y, int num_rows, int groups, int out_features, int in_features,
+                  int x_step, int w_step, int y_step, int x_cols, int y_cols, void* stream);
 
 /*
  * Replaces, in one kernel: the fused q/k/v projection of an attention block and what follows it before the
@@ -281,6 +367,55 @@ int b200_add_rmsnorm_route(void* x, const void* delta, const void* norm_weight, 
                            const void* router_weight, int num_rows, int hidden, int num_experts, int top_k,
                            int renormalize, const int32_t* num_valid_rows, void* normed_out, int32_t* topk_ids,
                            float* topk_weights, float* logits_out, void* stream);
+
+/* ------------------------------------------ glue of layer-list decoders -- */
+/* dtype: the activations' type (B200_DTYPE_*); the residual stream x is always fp32.  No counterparts in the
+ * reference. */
+
+/* x[m, i] = embed[tokens[m], i] + sinusoid(positions[m])_i for i < width, 0 for width <= i < ld.  The sinusoid comes from
+ * two fp32 tables by the addition theorem: lo [64, ld] holds (sin, cos) pairs of positions 0..63, hi [n_hi, ld] those of
+ * the multiples of 64. */
+int b200_embed_sinusoid(const int64_t* tokens, const int32_t* positions, const void* embed, const float* lo,
+                        const float* hi, float* x, void* status_word, int num_rows, int width, int ld, int vocab,
+                        int n_hi, int dtype, void* stream);
+
+/* x += delta (when given), out = weight * x / rms, the RMS taken over each of `groups` equal parts of the first `width`
+ * columns (rows are ld wide, the rest is zero).
+ * With taps > 0 also the short causal convolution of a decode step, row m being the token at positions[m] of its own
+ * sequence: out += sum_j conv_w[j] * h(position - taps + 1 + j), h the normed row rounded to dtype, zeros before the
+ * start.  The earlier h come from the pages: hist [num_blocks, min(taps-1, page), ld] keeps for every page the last rows
+ * written in it (position p in slot p % page % rows), and the row's own h is written there. */
+int b200_group_rmsnorm(float* x, const void* delta, const void* weight, float eps, int num_rows, int width, int ld,
+                       int groups, void* out, const void* conv_w, int taps, void* hist, const int32_t* positions,
+                       const int32_t* block_table, int page_size, int num_blocks, int max_pages_per_seq,
+                       void* status_word, int dtype, void* stream);
+
+/* The same convolution for num_rows consecutive tokens of ONE sequence starting at first_position: h [num_rows, ld] ->
+ * out, earlier rows from hist, hist updated. */
+int b200_short_conv(const void* h, const void* conv_w, int taps, void* hist, const int32_t* block_table_row,
+                    int num_rows, int first_position, int ld, void* out, int page_size, int num_blocks,
+                    int max_pages_per_seq, void* status_word, int dtype, void* stream);
+
+/* RMS norm of raw [num_rows, ld] fp32 over its first `rank` columns, written into the latents' page slots:
+ * c_pool [num_blocks, page_size, ld]. */
+int b200_latent_norm_append(const float* raw, const void* weight, float eps, int num_rows, int rank, int ld,
+                            void* c_pool, const int32_t* positions, const int32_t* block_table, int page_size,
+                            int num_blocks, int max_pages_per_seq, void* status_word, int dtype, void* stream);
+
+/* out[i] = row i of a sequence's latents, i < num_tokens: c_pool [num_blocks, page_size, ld] -> [num_tokens, ld]. */
+int b200_gather_pages(const void* c_pool, const int32_t* block_table_row, void* out, int num_tokens, int ld,
+                      int page_size, int num_blocks, int max_pages_per_seq, void* status_word, int dtype, void* stream);
+
+/* Unfused forms, for fp32: the split store of b200_proj_split_gemm on a finished fp32 product y [num_rows, n] (segment
+ * kinds 0 and 2 in dtype), the clamped gated unit on gate/up columns interleaved in blocks of 128, and the arg-max of
+ * fp32 logits (ties to the lower index). */
+int b200_split_store(const float* y, const float* col_scale, const int32_t* seg_end, const int32_t* seg_kind,
+                     const int32_t* seg_heads, const int32_t* seg_dim, void* const* seg_ptr, int num_segs,
+                     const int32_t* positions, const int32_t* block_table, void* status_word, int num_rows,
+                     int page_size, int num_blocks, int max_pages_per_seq, int dtype, void* stream);
+int b200_clamped_glu(const void* gate_up, void* out, int num_rows, int inter, float limit, float alpha, int dtype,
+                     void* stream);
+int b200_argmax_rows(const float* logits, int64_t* out, int num_rows, int n, void* stream);
 
 /* ------------------------------------------------------------------- MoE -- */
 

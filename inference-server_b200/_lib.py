@@ -26,11 +26,32 @@ SIGNATURES = {
         [c_void_p] * 7 + [c_size_t] + [c_int] * 7 + [c_float, c_int, c_int, c_void_p],
     ),
     "b200_paged_attn_decode_pairs": (c_int, [c_void_p] * 7 + [c_size_t] + [c_int] * 7 + [c_float, c_int, c_void_p]),
+    "b200_paged_attn_decode_chunked": (
+        c_int, [c_void_p] * 7 + [c_size_t] + [c_int] * 7 + [c_float] + [c_int] * 3 + [c_void_p] * 2),
+    "b200_paged_attn_prefill_chunked": (c_int, [c_void_p] * 6 + [c_int] * 8 + [c_float, c_int] + [c_void_p] * 2),
+    "b200_latent_attn_supported": (c_int, [c_int, c_int]),
+    "b200_latent_attn_decode": (c_int, [c_void_p] * 6 + [c_size_t] + [c_int] * 6 + [c_float, c_int] + [c_void_p] * 2),
     "b200_paged_attn_prefill": (c_int, [c_void_p] * 6 + [c_int] * 8 + [c_float, c_void_p]),
     "b200_paged_attn_decode_static": (c_int, [c_void_p] * 7 + [c_int] * 7 + [c_float, c_int, c_void_p]),
     "b200_kv_append": (c_int, [c_void_p] * 7 + [c_int] * 7 + [c_void_p]),
     "b200_dense_gemm_workspace_bytes": (c_size_t, [c_int, c_int]),
     "b200_dense_gemm_bf16": (c_int, [c_void_p] * 4 + [c_size_t, c_void_p] + [c_int] * 4 + [c_void_p]),
+    "b200_dense_gemm_bf16_f32": (c_int, [c_void_p] * 4 + [c_size_t, c_void_p] + [c_int] * 4 + [c_void_p]),
+    "b200_dense_gemm_grouped": (c_int, [c_void_p] * 4 + [c_int] * 9 + [c_void_p]),
+    "b200_proj_split_gemm": (c_int, [c_void_p] * 8 + [c_int] + [c_void_p] * 3 + [c_int] * 5 + [c_void_p]),
+    "b200_dense_glu_gemm": (c_int, [c_void_p] * 4 + [c_int] * 3 + [c_float] * 2 + [c_void_p]),
+    "b200_gemm_f32": (c_int, [c_void_p] * 3 + [c_int] * 9 + [c_void_p]),
+    "b200_embed_sinusoid": (c_int, [c_void_p] * 7 + [c_int] * 6 + [c_void_p]),
+    "b200_group_rmsnorm": (c_int, [c_void_p] * 3 + [c_float] + [c_int] * 4 + [c_void_p] * 2 + [c_int] + [c_void_p] * 3
+                           + [c_int] * 3 + [c_void_p, c_int, c_void_p]),
+    "b200_short_conv": (c_int, [c_void_p] * 2 + [c_int] + [c_void_p] * 2 + [c_int] * 3 + [c_void_p] + [c_int] * 3
+                        + [c_void_p, c_int, c_void_p]),
+    "b200_latent_norm_append": (c_int, [c_void_p] * 2 + [c_float] + [c_int] * 3 + [c_void_p] * 3 + [c_int] * 3
+                                + [c_void_p, c_int, c_void_p]),
+    "b200_gather_pages": (c_int, [c_void_p] * 3 + [c_int] * 5 + [c_void_p, c_int, c_void_p]),
+    "b200_split_store": (c_int, [c_void_p] * 7 + [c_int] + [c_void_p] * 3 + [c_int] * 5 + [c_void_p]),
+    "b200_clamped_glu": (c_int, [c_void_p] * 2 + [c_int] * 2 + [c_float] * 2 + [c_int, c_void_p]),
+    "b200_argmax_rows": (c_int, [c_void_p] * 2 + [c_int] * 2 + [c_void_p]),
     "b200_qkv_rope_append_supported": (c_int, [c_int, c_int]),
     "b200_qkv_rope_append_gemm": (c_int, [c_void_p] * 12 + [c_int] * 5 + [c_float] + [c_int] * 4 + [c_void_p]),
     "b200_lm_head_argmax_workspace_bytes": (c_size_t, []),
@@ -74,6 +95,19 @@ SIGNATURES = {
 }
 
 _lib = None
+_path = LIB_PATH
+_partial = False
+
+
+def use(path: str) -> None:
+    """Load this library file instead of the full one: `path` may hold a subset of the entry points (build.SUBSETS), and
+    calling one that is not in it raises.  Before the first load() of the process."""
+    global _path, _partial
+    if _lib is not None:
+        if os.path.realpath(path) != os.path.realpath(_path):
+            raise RuntimeError(f"{_path} is already loaded")
+        return
+    _path, _partial = path, os.path.realpath(path) != os.path.realpath(LIB_PATH)
 
 
 class B200Error(RuntimeError):
@@ -90,17 +124,19 @@ def load() -> ctypes.CDLL:
     global _lib
     if _lib is not None:
         return _lib
-    if not os.path.exists(LIB_PATH):
+    if not os.path.exists(_path):
         raise RuntimeError(
-            f"{LIB_PATH} is missing. Build it with `python inference-server_b200/build.py` "
+            f"{_path} is missing. Build it with `python inference-server_b200/build.py` "
             "(needs nvcc); there is no fallback implementation."
         )
-    lib = ctypes.CDLL(LIB_PATH)
+    lib = ctypes.CDLL(_path)
     for name, (restype, argtypes) in SIGNATURES.items():
         try:
             fn = getattr(lib, name)
         except AttributeError as e:
-            raise RuntimeError(f"{LIB_PATH} does not export {name}; rebuild the library") from e
+            if _partial:
+                continue
+            raise RuntimeError(f"{_path} does not export {name}; rebuild the library") from e
         fn.restype = restype
         fn.argtypes = argtypes
     _lib = lib

@@ -1,8 +1,8 @@
 """Builds libb200decode.so (the C-ABI library) in-tree with nvcc for sm_100a.
 
 Run as a script (``python inference-server_b200/build.py``) or call
-:func:`build_library`.  The library is rebuilt only when a source is newer than
-the existing binary.  nvcc cross-compiles without a GPU present.
+:func:`build_library`.  Only what is older than its source is compiled
+again.  nvcc cross-compiles without a GPU present.
 """
 from __future__ import annotations
 
@@ -17,7 +17,14 @@ CSRC = os.path.join(PKG_DIR, "csrc")
 INCLUDE = os.path.join(ROOT_DIR, "include")
 LIB_PATH = os.path.join(PKG_DIR, "libb200decode.so")
 SOURCES = ["host.cu", "paged_attn.cu", "paged_prefill.cu", "paged_prefill_tc.cu", "decode_glue.cu", "dense_gemm.cu", "router_fused.cu", "moe_route.cu", "moe_gemm.cu",
-           "moe_layer.cu", "ep_p2p.cu"]
+           "moe_layer.cu", "ep_p2p.cu", "latent_attn.cu", "layer_glue.cu"]
+# Parts of the library that are enough for some model families, each with a library file of its own, for a process that
+# has to build before it can run and needs no more than that.
+SUBSETS = {
+    "layered": ["host.cu", "paged_attn.cu", "paged_prefill.cu", "paged_prefill_tc.cu", "dense_gemm.cu", "latent_attn.cu",
+                "layer_glue.cu"],
+}
+HEADERS = ["common.cuh", "host.h"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "-I", INCLUDE, "-I", CSRC,
@@ -31,44 +38,70 @@ def _nvcc() -> str:
     return exe
 
 
-def _stale() -> bool:
-    if not os.path.exists(LIB_PATH):
-        return True
-    built = os.path.getmtime(LIB_PATH)
-    deps = [os.path.join(CSRC, f) for f in os.listdir(CSRC)] + [os.path.join(INCLUDE, "b200_decode.h")]
-    return any(os.path.getmtime(d) > built for d in deps)
+def _mtime(path: str) -> float:
+    return os.path.getmtime(path) if os.path.exists(path) else 0.0
 
 
-def build_library(force: bool = False, verbose: bool = False) -> str:
-    """Compile every .cu under csrc/ and link the shared library. Returns its path."""
-    if not force and not _stale():
-        return LIB_PATH
+def _header_time() -> float:
+    return max(_mtime(os.path.join(CSRC, h)) for h in HEADERS) if HEADERS else 0.0
+
+
+def _newest(sources: list[str]) -> float:
+    return max([_mtime(os.path.join(CSRC, f)) for f in sources]
+               + [_header_time(), _mtime(os.path.join(INCLUDE, "b200_decode.h"))])
+
+
+def _fresh(path: str, sources: list[str]) -> bool:
+    return _mtime(path) >= _newest(sources)
+
+
+def subset_path(subset: str) -> str:
+    return LIB_PATH.replace(".so", f"_{subset}.so")
+
+
+def build_library(force: bool = False, verbose: bool = False, subset: str | None = None) -> str:
+    """Compile what is out of date of the .cu files under csrc/ (of one of SUBSETS if given) and link the shared library.
+    Returns its path."""
+    sources, lib_path = (SOURCES, LIB_PATH) if subset is None else (SUBSETS[subset], subset_path(subset))
+    if not force and _fresh(lib_path, sources):
+        return lib_path
     nvcc = _nvcc()
     obj_dir = os.path.join(ROOT_DIR, "build")
     os.makedirs(obj_dir, exist_ok=True)
     objs = []
     procs = []
-    for src in SOURCES:
+    for src in sources:
         obj = os.path.join(obj_dir, src.replace(".cu", ".o"))
-        cmd = [nvcc, *NVCC_FLAGS, "-c", os.path.join(CSRC, src), "-o", obj]
+        objs.append(obj)
+        if not force and _fresh(obj, [src]):
+            continue
+        cmd = [nvcc, *NVCC_FLAGS, "-c", os.path.join(CSRC, src), "-o", obj + ".tmp.o"]
         if verbose:
             cmd.insert(1, "-Xptxas")
             cmd.insert(2, "-v")
-        procs.append((src, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
-        objs.append(obj)
-    for src, proc in procs:
+        procs.append((src, obj, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
+    for src, obj, proc in procs:
         out, _ = proc.communicate()
         if verbose and out:
             print(out)
         if proc.returncode != 0:
             raise RuntimeError(f"nvcc failed on {src}:\n{out}")
-    tmp = LIB_PATH + ".tmp"
+        os.replace(obj + ".tmp.o", obj)
+    tmp = lib_path + ".tmp"
     link = [nvcc, "-shared", "-o", tmp, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
     res = subprocess.run(link, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)
     if res.returncode != 0:
         raise RuntimeError(f"link failed:\n{res.stdout}")
-    os.replace(tmp, LIB_PATH)
-    return LIB_PATH
+    os.replace(tmp, lib_path)
+    return lib_path
+
+
+def library_for(subset: str) -> str:
+    """Path of an up-to-date library with the entry points of `subset`: the full one if it is there, else the subset's,
+    built now if need be."""
+    if _fresh(LIB_PATH, SOURCES):
+        return LIB_PATH
+    return build_library(subset=subset)
 
 
 if __name__ == "__main__":

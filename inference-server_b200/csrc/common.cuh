@@ -247,6 +247,37 @@ __device__ __forceinline__ float warp_sum(float v) {
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
   return v;
 }
+// First token a row at position L - 1 sees when positions are cut into chunks of `chunk` (0: all of them).
+__device__ __forceinline__ int first_visible(int L, int chunk) {
+  return chunk > 0 && L > 0 ? (L - 1) / chunk * chunk : 0;
+}
+// Output gate of a (row, head): sigmoid of its fp32 logit, 1 without a gate.
+__device__ __forceinline__ float head_gate(const float* gate, size_t i) {
+  return gate == nullptr ? 1.f : 1.f / (1.f + expf(-gate[i]));
+}
+// Clamped gated unit: g * sigmoid(alpha g) * (u + 1) with g capped at `limit` and u held to +-limit.
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
+__device__ __forceinline__ float clamped_glu_fast(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);
+}
+template <typename T>
+__device__ __forceinline__ float to_f32(T v);
+template <>
+__device__ __forceinline__ float to_f32<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ float to_f32<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T>
+__device__ __forceinline__ T from_f32(float v);
+template <>
+__device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 __device__ __forceinline__ uint8_t to_e4m3(float v) {
   return static_cast<uint8_t>(__nv_cvt_float_to_fp8(v, __NV_SATFINITE, __NV_E4M3));
 }

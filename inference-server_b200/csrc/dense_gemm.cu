@@ -39,7 +39,15 @@
 //               128-row tiles of W against one X box (two accumulators), which halves how often X
 //               is pulled from L2, and walks its share of the vocabulary persistently.
 //
-// Epilogues: bf16 store, or (lm_head) a running arg-max: every epilogue thread owns one feature of
+// Groups: a launch may cover several independent products that sit side by side (one per attention head): group g
+// multiplies the columns [g * x_step, + K) of X with the weight rows [g * w_step, + N) into the columns
+// [g * y_step, + N) of Y.  K may then be any multiple of 8: what a 64-wide K block holds past a group's K is the next
+// group's data in X but zero fill in W, whose rows are K long.
+//
+// Epilogues: bf16 (or fp32) store; a split store (kEpiSplit), which sends consecutive ranges of features to different
+// places - rows of their own, bf16 or fp32, or the page slots of a K/V pool -, each feature first multiplied by a number
+// of its own; the clamped gated unit of a dense feed-forward (kEpiGlu: the two W tiles of an item are the gate and the
+// up rows of the same 128 features); or (lm_head) a running arg-max: every epilogue thread owns one feature of
 // the current weight tile and keeps, for each of its 128 rows of X, the largest logit it has seen over
 // all the tiles of the CTA as one integer key in a register; the warp-wide maximum is taken once, after
 // the last tile.  The [M, vocab] logits are never written; a small second kernel folds the per-warp
@@ -60,7 +68,15 @@ constexpr int kDenseXBytesMax = 256 * 128;        // largest X box of a stage
 constexpr int kDenseThreads = 10 * 32;           // TMA warp, MMA warp, 8 epilogue warps
 constexpr int kDenseMaxRows = 256;                // rows of X per MMA (its N)
 
-enum : int { kEpiStore = 0, kEpiArgmax = 1, kEpiQkvRope = 2 };
+enum : int { kEpiStore = 0, kEpiArgmax = 1, kEpiQkvRope = 2, kEpiSplit = 3, kEpiGlu = 4 };
+enum : int { kSegBf16 = 0, kSegF32 = 1, kSegPages = 2 };
+constexpr int kMaxSegs = 4;
+// kEpiSplit: features [end of the segment before, end) go to `ptr`.
+struct DenseSeg {
+  int end, kind;
+  int heads, dim;  // kSegPages: pool [num_blocks, heads, page, dim]
+  void* ptr;       // kSegBf16 / kSegF32: [M, end - begin]
+};
 constexpr int kQkvStageBytes = kDenseMaxRows * 128 * 2;  // kEpiQkvRope: one head of up to 256 rows, bf16
 
 template <int A_TILES, int EPI = kEpiStore>
@@ -74,7 +90,15 @@ struct DenseCfg {
 };
 
 struct DenseParams {
-  __nv_bfloat16* y;   // kEpiStore: [M, N]
+  __nv_bfloat16* y;   // kEpiStore, kEpiGlu: [M, ldy]
+  float* y_f32;       // kEpiStore: instead of y
+  int ldy;            // row pitch of y
+  int groups, x_step, w_step, y_step;
+  // kEpiSplit (positions, block_table, page, num_blocks, max_pages below serve its page segments; positions NULL =
+  // row m is position m, block_table NULL = page p of the sequence is block p)
+  const float* col_scale;  // [N] or NULL
+  DenseSeg segs[kMaxSegs];
+  float glu_limit, glu_alpha;  // kEpiGlu
   float* part_val;    // kEpiArgmax: [grid * 4, 256] candidates per TMEM lane quarter
   int* part_idx;
   float* exchange;    // kEpiStore, split K: [tile][finishing CTA][source CTA][rows_per][128] fp32
@@ -186,8 +210,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
   grid_dep_launch();
 
   const int ks = p.ksplit;
-  const int kb_per = p.K / kDenseBlockK / ks;  // K blocks of one work item
-  const int total = p.n_tiles * p.m_tiles * ks;
+  const int kb_per = (p.K + kDenseBlockK - 1) / kDenseBlockK / ks;  // K blocks of one work item
+  const int total = p.groups * p.n_tiles * p.m_tiles * ks;
   const uint32_t stage_tx = A_TILES * kDenseWBytes + static_cast<uint32_t>(p.xbox) * 128u;
 
   if (warp == 0) {
@@ -197,7 +221,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
       bool alive = true;
       for (int w = blockIdx.x; w < total && alive; w += gridDim.x) {
         const int tile = w / ks, kidx = w - tile * ks;
-        const int nt = tile / p.m_tiles, mt = tile - nt * p.m_tiles;
+        const int gn = tile / p.m_tiles, mt = tile - gn * p.m_tiles;
+        const int g = gn / p.n_tiles, nt = gn - g * p.n_tiles;
         for (int kb = 0; kb < kb_per; ++kb, ++it) {
           const uint32_t slot = it % kStages, phase = (it / kStages) & 1;
           alive = mbar_wait(bar_empty + 8 * slot, phase ^ 1, p.err);
@@ -207,8 +232,9 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           mbar_arrive_expect_tx(bar_full + 8 * slot, stage_tx);
 #pragma unroll
           for (int a = 0; a < A_TILES; ++a)
-            tma_load_2d(sw + a * kDenseWBytes, &w_map, bar_full + 8 * slot, kx, (nt * A_TILES + a) * 128);
-          tma_load_2d(sx, &x_map, bar_full + 8 * slot, kx, mt * p.xbox);
+            tma_load_2d(sw + a * kDenseWBytes, &w_map, bar_full + 8 * slot, kx,
+                        g * p.w_step + (nt * A_TILES + a) * 128);
+          tma_load_2d(sx, &x_map, bar_full + 8 * slot, g * p.x_step + kx, mt * p.xbox);
         }
       }
     }
@@ -266,7 +292,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
     bool alive = true;
     for (int w = blockIdx.x; w < total && alive; w += gridDim.x, ++item) {
       const int tile = w / ks;
-      const int nt = tile / p.m_tiles, mt = tile - nt * p.m_tiles;
+      const int gn = tile / p.m_tiles, mt = tile - gn * p.m_tiles;
+      const int g = gn / p.n_tiles, nt = gn - g * p.n_tiles;
       const uint32_t buf = item % kBufs, aphase = (item / kBufs) & 1;
       const int m0 = mt * p.xbox;
       // kEpiQkvRope: position and page of the rows this warp will finish (lane i: row (warp - 2) + 8 i of the
@@ -288,9 +315,106 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           }
         }
       }
+      // kEpiSplit: where this thread's feature goes, and the page and slot of the rows of this warp's chunks (lane i:
+      // row i of the chunk), fetched while the MMAs of the item are still running; page -1 = not written
+      int seg_kind = -1, seg_page_stride = 0, seg_dim = 0, seg_ld = 0, row_page4[4], row_slot4[4];
+      void* seg_ptr = nullptr;
+      float seg_scale = 1.f;
+      if (EPI == kEpiSplit) {
+        const int n = nt * 128 + t;
+        int begin = 0;
+        bool pages = false;
+#pragma unroll
+        for (int e = 0; e < kMaxSegs; ++e) {
+          const DenseSeg& sg = p.segs[e];
+          pages = pages || (sg.kind == kSegPages && sg.end > begin && begin < (nt + 1) * 128 && sg.end > nt * 128);
+          if (n >= begin && n < sg.end) {
+            const int local = n - begin;
+            seg_kind = sg.kind;
+            if (sg.kind == kSegPages) {
+              const int head = local / sg.dim;
+              seg_dim = sg.dim;
+              seg_page_stride = sg.heads * p.page * sg.dim;
+              seg_ptr = static_cast<__nv_bfloat16*>(sg.ptr) + static_cast<size_t>(head) * p.page * sg.dim + (local - head * sg.dim);
+            } else {
+              seg_ld = sg.end - begin;
+              seg_ptr = sg.kind == kSegF32 ? static_cast<void*>(static_cast<float*>(sg.ptr) + local)
+                                           : static_cast<void*>(static_cast<__nv_bfloat16*>(sg.ptr) + local);
+            }
+          }
+          begin = max(begin, sg.end);
+        }
+        if (p.col_scale != nullptr && n < p.N) seg_scale = p.col_scale[n];
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) {
+          row_page4[cc] = -1;
+          row_slot4[cc] = 0;
+          const int r = (cc * 2 + half) * 32 + lane, m = m0 + r;
+          if (pages && r < p.xbox && m < p.M) {
+            const int ps = p.positions != nullptr ? p.positions[m] : m;
+            if (ps < 0 || ps >= p.max_pages * p.page) {
+              set_error(p.err, kErrDevBadCtxLen);
+            } else {
+              const int pg = ps / p.page;
+              const int id = p.block_table != nullptr ? p.block_table[static_cast<size_t>(m) * p.max_pages + pg] : pg;
+              if (id < 0 || id >= p.num_blocks) {
+                set_error(p.err, kErrDevBadBlockId);
+              } else {
+                row_page4[cc] = id;
+                row_slot4[cc] = ps - pg * p.page;
+              }
+            }
+          }
+        }
+      }
       alive = mbar_wait(bar_tfull + 8 * buf, aphase, p.err);
       if (!alive) break;
       tc_fence_after();
+      if (EPI == kEpiSplit) {
+        const uint32_t t0 = lane_addr + buf * kDenseMaxRows;
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) {
+          const int c = cc * 2 + half;
+          if (c >= chunks) break;
+          uint32_t v[32];
+          tmem_ld32(t0 + c * 32, v);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const int m = m0 + c * 32 + i;
+            const int page = __shfl_sync(0xffffffffu, row_page4[cc], i), slot = __shfl_sync(0xffffffffu, row_slot4[cc], i);
+            const float f = __uint_as_float(v[i]) * seg_scale;
+            if (m < p.M) {
+              if (seg_kind == kSegPages) {
+                if (page >= 0)
+                  static_cast<__nv_bfloat16*>(seg_ptr)[static_cast<size_t>(page) * seg_page_stride + slot * seg_dim] =
+                      __float2bfloat16(f);
+              } else if (seg_kind == kSegBf16) {
+                static_cast<__nv_bfloat16*>(seg_ptr)[static_cast<size_t>(m) * seg_ld] = __float2bfloat16(f);
+              } else if (seg_kind == kSegF32) {
+                static_cast<float*>(seg_ptr)[static_cast<size_t>(m) * seg_ld] = f;
+              }
+            }
+          }
+        }
+      } else if (EPI == kEpiGlu) {
+        const int n = nt * 128 + t;
+        for (int c = half; c < chunks; c += 2) {
+          uint32_t v[32], u[32];
+          tmem_ld32(lane_addr + c * 32, v);
+          tmem_ld32(lane_addr + (A_TILES > 1 ? kDenseMaxRows : 0) + c * 32, u);
+          tmem_ld_wait();
+          if (n < p.N) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const int m = m0 + c * 32 + i;
+              if (m < p.M)
+                p.y[static_cast<size_t>(m) * p.ldy + n] = __float2bfloat16(clamped_glu_fast(
+                    __uint_as_float(v[i]), __uint_as_float(u[i]), p.glu_limit, p.glu_alpha));
+            }
+          }
+        }
+      } else
 #pragma unroll
       for (int a = 0; a < A_TILES; ++a) {
         const int n = (nt * A_TILES + a) * 128 + t;
@@ -315,7 +439,11 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
 #pragma unroll
               for (int i = 0; i < 32; ++i) {
                 const int m = m0 + c * 32 + i;
-                if (m < p.M) p.y[static_cast<size_t>(m) * p.N + n] = __float2bfloat16(__uint_as_float(v[i]));
+                const size_t at = static_cast<size_t>(m) * p.ldy + g * p.y_step + n;
+                if (m < p.M) {
+                  if (p.y_f32 != nullptr) p.y_f32[at] = __uint_as_float(v[i]);
+                  else p.y[at] = __float2bfloat16(__uint_as_float(v[i]));
+                }
               }
             }
           }
@@ -518,7 +646,11 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           const int m = mt * p.xbox + static_cast<int>(me) * rows_per + r, n = nt * 128 + g4;
           if (m < p.M) {
             __nv_bfloat16* dst = p.y + static_cast<size_t>(m) * p.N + n;
-            if (n + 3 < p.N && (p.N & 3) == 0) {
+            if (p.y_f32 != nullptr) {
+              const float a4[4] = {acc.x, acc.y, acc.z, acc.w};
+              for (int e = 0; e < 4; ++e)
+                if (n + e < p.N) p.y_f32[static_cast<size_t>(m) * p.N + n + e] = a4[e];
+            } else if (n + 3 < p.N && (p.N & 3) == 0) {
               uint2 o;
               o.x = pack_bf16x2(acc.x, acc.y);
               o.y = pack_bf16x2(acc.z, acc.w);
@@ -708,9 +840,9 @@ extern "C" size_t b200_dense_gemm_workspace_bytes(int num_rows, int out_features
   return rows * n_tiles * 128 * 4 * 8;
 }
 
-extern "C" int b200_dense_gemm_bf16(const void* x, const void* w, void* y, void* workspace, size_t workspace_bytes,
-                                    void* status_word, int num_rows, int out_features, int in_features,
-                                    int k_split, void* stream) {
+static int dense_gemm_any(const void* x, const void* w, void* y, bool y_is_f32, void* workspace, size_t workspace_bytes,
+                          void* status_word, int num_rows, int out_features, int in_features, int k_split,
+                          void* stream) {
   int rc = dense_args_ok(x, w, num_rows, out_features, in_features, "dense_gemm_bf16");
   if (rc) return rc;
   B200_REQUIRE(y && (reinterpret_cast<uintptr_t>(y) & 7) == 0, "dense_gemm_bf16: output must be 8-byte aligned");
@@ -720,7 +852,12 @@ extern "C" int b200_dense_gemm_bf16(const void* x, const void* w, void* y, void*
   rc = device_sm_count(&sms);
   if (rc) return rc;
   DenseParams p{};
-  p.y = static_cast<__nv_bfloat16*>(y);
+  if (y_is_f32)
+    p.y_f32 = static_cast<float*>(y);
+  else
+    p.y = static_cast<__nv_bfloat16*>(y);
+  p.groups = 1;
+  p.ldy = out_features;
   p.err = static_cast<int*>(status_word);
   p.M = num_rows;
   p.N = out_features;
@@ -761,6 +898,166 @@ extern "C" int b200_dense_gemm_bf16(const void* x, const void* w, void* y, void*
   return launch_dense<1, kEpiStore>(w_map, x_map, p, grid, as_stream(stream));
 }
 
+extern "C" int b200_dense_gemm_bf16(const void* x, const void* w, void* y, void* workspace, size_t workspace_bytes,
+                                    void* status_word, int num_rows, int out_features, int in_features,
+                                    int k_split, void* stream) {
+  return dense_gemm_any(x, w, y, false, workspace, workspace_bytes, status_word, num_rows, out_features, in_features,
+                        k_split, stream);
+}
+
+extern "C" int b200_dense_gemm_bf16_f32(const void* x, const void* w, float* y, void* workspace, size_t workspace_bytes,
+                                        void* status_word, int num_rows, int out_features, int in_features, int k_split,
+                                        void* stream) {
+  return dense_gemm_any(x, w, y, true, workspace, workspace_bytes, status_word, num_rows, out_features, in_features,
+                        k_split, stream);
+}
+
+namespace b200 {
+
+// Rows per work item without a K split: the width that needs the fewest waves of CTAs, then the least data per CTA.
+static int pick_xbox_waves(int num_rows, int tiles, int w_rows, int sms) {
+  int pick = pick_xbox(num_rows);
+  double best = 1e30;
+  for (int xbox = pick; xbox >= 32; xbox -= 32) {
+    const int items = tiles * ((num_rows + xbox - 1) / xbox);
+    const double cost = static_cast<double>((items + sms - 1) / sms) * (static_cast<double>(w_rows) + xbox) + xbox * 0.25;
+    if (cost < best) {
+      best = cost;
+      pick = xbox;
+    }
+  }
+  return pick;
+}
+
+}  // namespace b200
+
+extern "C" int b200_dense_gemm_grouped(const void* x, const void* w, void* y, void* status_word, int num_rows, int groups,
+                                       int out_features, int in_features, int x_step, int w_step, int y_step, int x_cols,
+                                       int y_cols, void* stream) {
+  B200_REQUIRE(x && w && y, "dense_gemm_grouped: null pointer");
+  B200_REQUIRE(num_rows > 0 && groups > 0 && out_features > 0 && in_features > 0 && in_features % 8 == 0 &&
+                   x_step % 8 == 0 && x_step >= 0 && w_step >= out_features && y_step >= out_features,
+               "dense_gemm_grouped: rows %d, groups %d, N %d, K %d (K and x_step must be multiples of 8)", num_rows, groups,
+               out_features, in_features);
+  B200_REQUIRE(x_cols % 8 == 0 && (groups - 1) * x_step + in_features <= x_cols &&
+                   (groups - 1) * y_step + out_features <= y_cols,
+               "dense_gemm_grouped: the groups do not fit %d input and %d output columns", x_cols, y_cols);
+  B200_REQUIRE(((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0,
+               "dense_gemm_grouped: x and w must be 16-byte aligned");
+  int rc = check_device(nullptr);
+  if (rc) return rc;
+  int sms = 148;
+  rc = device_sm_count(&sms);
+  if (rc) return rc;
+  DenseParams p{};
+  p.y = static_cast<__nv_bfloat16*>(y);
+  p.ldy = y_cols;
+  p.groups = groups;
+  p.x_step = x_step;
+  p.w_step = w_step;
+  p.y_step = y_step;
+  p.err = static_cast<int*>(status_word);
+  p.M = num_rows;
+  p.N = out_features;
+  p.K = in_features;
+  p.n_tiles = (out_features + 127) / 128;
+  p.ksplit = 1;
+  p.xbox = pick_xbox_waves(num_rows, groups * p.n_tiles, 128, sms);
+  p.m_tiles = (num_rows + p.xbox - 1) / p.xbox;
+  CUtensorMap w_map, x_map;
+  rc = get_tensor_map_2d(w, static_cast<uint64_t>(groups - 1) * w_step + out_features, in_features, 2, 128, 64, &w_map);
+  if (rc) return rc;
+  rc = get_tensor_map_2d(x, num_rows, x_cols, 2, p.xbox, 64, &x_map);
+  if (rc) return rc;
+  const int items = groups * p.n_tiles * p.m_tiles;
+  return launch_dense<1, kEpiStore>(w_map, x_map, p, items < sms ? items : sms, as_stream(stream));
+}
+
+extern "C" int b200_proj_split_gemm(const void* x, const void* w, const float* col_scale, const int32_t* seg_end,
+                                    const int32_t* seg_kind, const int32_t* seg_heads, const int32_t* seg_dim,
+                                    void* const* seg_ptr, int num_segs, const int32_t* positions,
+                                    const int32_t* block_table, void* status_word, int num_rows, int in_features,
+                                    int page_size, int num_blocks, int max_pages_per_seq, void* stream) {
+  B200_REQUIRE(seg_end && seg_kind && seg_heads && seg_dim && seg_ptr && num_segs >= 1 && num_segs <= kMaxSegs,
+               "proj_split_gemm: 1 to %d segments", kMaxSegs);
+  DenseParams p{};
+  int begin = 0;
+  for (int i = 0; i < kMaxSegs; ++i) {
+    p.segs[i].end = begin;  // unused segments are empty
+    if (i >= num_segs) continue;
+    B200_REQUIRE(seg_end[i] > begin && seg_ptr[i], "proj_split_gemm: segment %d is empty or has no target", i);
+    B200_REQUIRE(seg_kind[i] >= kSegBf16 && seg_kind[i] <= kSegPages, "proj_split_gemm: segment kind %d", seg_kind[i]);
+    if (seg_kind[i] == kSegPages)
+      B200_REQUIRE(seg_heads[i] > 0 && seg_dim[i] > 0 && seg_heads[i] * seg_dim[i] == seg_end[i] - begin && page_size > 0 &&
+                       num_blocks > 0 && max_pages_per_seq > 0,
+                   "proj_split_gemm: page segment %d does not match its pool", i);
+    p.segs[i] = DenseSeg{seg_end[i], seg_kind[i], seg_heads[i], seg_dim[i], seg_ptr[i]};
+    begin = seg_end[i];
+  }
+  int rc = dense_args_ok(x, w, num_rows, begin, in_features, "proj_split_gemm");
+  if (rc) return rc;
+  rc = check_device(nullptr);
+  if (rc) return rc;
+  int sms = 148;
+  rc = device_sm_count(&sms);
+  if (rc) return rc;
+  p.groups = 1;
+  p.err = static_cast<int*>(status_word);
+  p.M = num_rows;
+  p.N = begin;
+  p.K = in_features;
+  p.n_tiles = (begin + 127) / 128;
+  p.ksplit = 1;
+  p.xbox = pick_xbox_waves(num_rows, p.n_tiles, 128, sms);
+  p.m_tiles = (num_rows + p.xbox - 1) / p.xbox;
+  p.col_scale = col_scale;
+  p.positions = positions;
+  p.block_table = block_table;
+  p.page = page_size;
+  p.num_blocks = num_blocks;
+  p.max_pages = max_pages_per_seq;
+  CUtensorMap w_map, x_map;
+  rc = get_tensor_map_2d(w, p.N, in_features, 2, 128, 64, &w_map);
+  if (rc) return rc;
+  rc = get_tensor_map_2d(x, num_rows, in_features, 2, p.xbox, 64, &x_map);
+  if (rc) return rc;
+  const int items = p.n_tiles * p.m_tiles;
+  return launch_dense<1, kEpiSplit>(w_map, x_map, p, items < sms ? items : sms, as_stream(stream));
+}
+
+extern "C" int b200_dense_glu_gemm(const void* x, const void* w_interleaved, void* y, void* status_word, int num_rows,
+                                   int inter, int in_features, float limit, float alpha, void* stream) {
+  int rc = dense_args_ok(x, w_interleaved, num_rows, 2 * inter, in_features, "dense_glu_gemm");
+  if (rc) return rc;
+  B200_REQUIRE(y && inter % 128 == 0, "dense_glu_gemm: %d inner features (a multiple of 128)", inter);
+  rc = check_device(nullptr);
+  if (rc) return rc;
+  int sms = 148;
+  rc = device_sm_count(&sms);
+  if (rc) return rc;
+  DenseParams p{};
+  p.y = static_cast<__nv_bfloat16*>(y);
+  p.ldy = inter;
+  p.groups = 1;
+  p.err = static_cast<int*>(status_word);
+  p.M = num_rows;
+  p.N = inter;
+  p.K = in_features;
+  p.n_tiles = inter / 128;
+  p.ksplit = 1;
+  p.xbox = pick_xbox_waves(num_rows, p.n_tiles, 256, sms);
+  p.m_tiles = (num_rows + p.xbox - 1) / p.xbox;
+  p.glu_limit = limit;
+  p.glu_alpha = alpha;
+  CUtensorMap w_map, x_map;
+  rc = get_tensor_map_2d(w_interleaved, static_cast<uint64_t>(2) * inter, in_features, 2, 128, 64, &w_map);
+  if (rc) return rc;
+  rc = get_tensor_map_2d(x, num_rows, in_features, 2, p.xbox, 64, &x_map);
+  if (rc) return rc;
+  const int items = p.n_tiles * p.m_tiles;
+  return launch_dense<2, kEpiGlu>(w_map, x_map, p, items < sms ? items : sms, as_stream(stream));
+}
+
 extern "C" int b200_qkv_rope_append_supported(int head_dim, int in_features) {
   return head_dim == 128 && in_features > 0 && in_features % kDenseBlockK == 0;
 }
@@ -791,23 +1088,12 @@ extern "C" int b200_qkv_rope_append_gemm(const void* x, const void* wqkv, const 
   DenseParams p{};
   p.err = static_cast<int*>(status_word);
   p.M = num_rows;
+  p.groups = 1;
   p.N = heads * head_dim;
   p.K = in_features;
   p.n_tiles = heads;
   p.ksplit = 1;
-  // rows per item: the width that needs the fewest waves of CTAs, then the least data per CTA
-  p.xbox = pick_xbox(num_rows);
-  {
-    double best = 1e30;
-    for (int xbox = p.xbox; xbox >= 32; xbox -= 32) {  // any multiple of 32 here: this epilogue has no K split
-      const int items = heads * ((num_rows + xbox - 1) / xbox);
-      const double cost = static_cast<double>((items + sms - 1) / sms) * (128.0 + xbox) + xbox * 0.25;
-      if (cost < best) {
-        best = cost;
-        p.xbox = xbox;
-      }
-    }
-  }
+  p.xbox = pick_xbox_waves(num_rows, heads, 128, sms);  // this epilogue has no K split
   p.m_tiles = (num_rows + p.xbox - 1) / p.xbox;
   p.q_norm_w = static_cast<const __nv_bfloat16*>(q_norm_weight);
   p.k_norm_w = static_cast<const __nv_bfloat16*>(k_norm_weight);
@@ -859,6 +1145,7 @@ extern "C" int b200_lm_head_argmax(const void* x, const void* w, int64_t* next_t
   DenseParams p{};
   p.err = static_cast<int*>(status_word);
   p.M = num_rows;
+  p.groups = 1;
   p.N = vocab_size;
   p.K = hidden;
   p.m_tiles = 1;

@@ -60,6 +60,27 @@ inline cudaError_t launch_overlapped(void (*kernel)(KArgs...), dim3 grid, dim3 b
   return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
 }
 
+// Split partials of the decode attention kernels inside a caller workspace: the status word, then (m, l) and the
+// unnormalised fp32 output per (row, head, split).
+struct AttnWorkspace {
+  int* err;
+  float2* ml;
+  float* o;
+  size_t bytes;
+};
+inline AttnWorkspace carve(void* ws, int batch, int hq, int D, int max_splits) {
+  AttnWorkspace w;
+  uint8_t* p = static_cast<uint8_t*>(ws);
+  w.err = reinterpret_cast<int*>(p);
+  size_t off = 256;
+  w.ml = reinterpret_cast<float2*>(p + off);
+  off += (static_cast<size_t>(batch) * hq * max_splits * sizeof(float2) + 255) & ~size_t(255);
+  w.o = reinterpret_cast<float*>(p + off);
+  off += static_cast<size_t>(batch) * hq * max_splits * D * sizeof(float);
+  w.bytes = off;
+  return w;
+}
+
 }  // namespace b200
 
 #define B200_REQUIRE(cond, ...)            \

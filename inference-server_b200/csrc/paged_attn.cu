@@ -28,6 +28,15 @@
 //           kernel folds the splits in split order and writes bf16.
 // The kernel is HBM-bound: per token and kv head it reads 2*D*2 bytes once.
 //
+// Two things a model may ask for on top, both run-time arguments of every kernel here:
+//   chunk   positions are cut into chunks of `chunk` counted from the sequence's start, and a row sees only the
+//           tokens of its own position's chunk (0 = no chunks, all tokens).  The splits then start at the page that
+//           holds the chunk's first token, so pages before it are never read.
+//   gate    an fp32 number per (row, query head); the head's output is multiplied by its sigmoid where the
+//           row is normalised.
+// Other kv head counts than 1, 2, 4, 8 run as groups of the largest of these that divides them (grid.z), each CTA
+// with the heads of its group.
+//
 // Generic kernel: any head_dim <= 256, any page size, fp32 or bf16 pools, no
 // split, fp32 arithmetic throughout.  It serves shapes the main kernel does not
 // (the tiny fp32 parity model) and is not tuned.
@@ -67,8 +76,9 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap k_map,
                          const int* __restrict__ ctx_lens,
                          float* __restrict__ part_o, float2* __restrict__ part_ml,
                          __nv_bfloat16* __restrict__ out,
-                         int* __restrict__ err, int batch, int num_q_heads, int num_blocks, int max_pages,
-                         int split_tokens, int max_splits, float scale_log2) {
+                         int* __restrict__ err, int batch, int num_q_heads, int num_kv_heads, int num_blocks,
+                         int max_pages, int split_tokens, int max_splits, float scale_log2, int chunk,
+                         const float* __restrict__ gate) {
 #ifdef B200_DEVICE_OK
   grid_dep_wait();    // the context lengths, the query rows and the new K/V rows come from the kernels before
   grid_dep_launch();
@@ -79,7 +89,7 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap k_map,
 
   const int b = PAIRS ? 2 * blockIdx.x : blockIdx.x, split = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int group = num_q_heads / HKV;
+  const int group = num_q_heads / num_kv_heads;
   const bool has1 = PAIRS && b + 1 < batch;  // the pair's second row exists
 
   int L = ctx_lens[b];
@@ -106,9 +116,11 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap k_map,
     }
     L = max(L0, L1);
   }
-  const int start = split * split_tokens;
+  const int lo = first_visible(L, chunk);  // tokens lo .. L-1 are seen
+  const int range0 = lo & ~(kPage - 1);    // the splits count from the page that holds the first of them
+  const int start = range0 + split * split_tokens;
   if (start >= L) {  // uniform for the whole CTA
-    if (!PAIRS && L == 0 && split == 0)  // a row with no context attends to nothing: zeros
+    if (!PAIRS && L == 0 && split == 0 && blockIdx.z == 0)  // a row with no context attends to nothing: zeros
       for (int i = threadIdx.x; i < num_q_heads * D; i += blockDim.x)
         out[static_cast<size_t>(b) * num_q_heads * D + i] = __float2bfloat16(0.f);
     return;
@@ -155,14 +167,15 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap k_map,
       __syncwarp();
       if (issuer) {
         const uint32_t dst = ring + slot * Cfg::kStageBytes + (lkv * Cfg::kHalves + lh) * Cfg::kBoxAll;
-        tma_load_2d(dst, lkv ? &v_map : &k_map, bars + 8 * slot, lh * 64, id * (HKV * kPage));
+        tma_load_2d(dst, lkv ? &v_map : &k_map, bars + 8 * slot, lh * 64,
+                    (id * num_kv_heads + static_cast<int>(blockIdx.z) * HKV) * kPage);
       }
     }
     return;
   }
 
   // --------------------------------------------------------------- consumers --
-  const int kvh = warp;      // this warp's kv head
+  const int kvh = blockIdx.z * HKV + warp;  // this warp's kv head
   const int gq = lane >> 2;  // fragment row (query head inside the kv group)
   const int tq = lane & 3;
   const bool hi_rows = PAIRS ? has1 : group > 8;
@@ -205,7 +218,7 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap k_map,
     const uint32_t phase = (i / STAGES) & 1;
     alive = mbar_wait(bars + 8 * slot, phase, err);
     if (alive) {
-      const uint32_t kbase = ring + slot * Cfg::kStageBytes + kvh * Cfg::kHeadBytes;
+      const uint32_t kbase = ring + slot * Cfg::kStageBytes + warp * Cfg::kHeadBytes;
       const uint32_t vbase = kbase + Cfg::kHalves * Cfg::kBoxAll;
 
       float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
@@ -237,6 +250,12 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap k_map,
         if (tok0 + 1 >= L) s0[1] = s0[3] = -INFINITY;
         if (tok0 + 8 >= L) s1[0] = s1[2] = -INFINITY;
         if (tok0 + 9 >= L) s1[1] = s1[3] = -INFINITY;
+      }
+      if (start + i * kPage < lo) {  // the chunk begins inside this page (its first token is here, so a row keeps one)
+        if (tok0 < lo) s0[0] = s0[2] = -INFINITY;
+        if (tok0 + 1 < lo) s0[1] = s0[3] = -INFINITY;
+        if (tok0 + 8 < lo) s1[0] = s1[2] = -INFINITY;
+        if (tok0 + 9 < lo) s1[1] = s1[3] = -INFINITY;
       }
 
       // online softmax, log2 domain; rows gq (index 0,1) and gq + 8 (index 2,3)
@@ -330,11 +349,13 @@ paged_attn_decode_kernel(const __grid_constant__ CUtensorMap k_map,
     return;
   }
 
-  const int nsplits = (L + split_tokens - 1) / split_tokens;  // CTAs working on this sequence
+  const int nsplits = (L - range0 + split_tokens - 1) / split_tokens;  // CTAs working on this sequence
   if (nsplits == 1) {
     // The whole sequence was this CTA's: normalise and write the result, no partials.
-    const float i0 = 1.f / l0, i1 = hi_rows ? 1.f / l1 : 0.f;
-    __nv_bfloat16* o0 = out + (static_cast<size_t>(b) * num_q_heads + kvh * group + gq) * D;
+    const size_t orow = static_cast<size_t>(b) * num_q_heads + kvh * group + gq;
+    const float i0 = (gq < group ? head_gate(gate, orow) : 1.f) / l0;
+    const float i1 = hi_rows ? (gq + 8 < group ? head_gate(gate, orow + 8) : 1.f) / l1 : 0.f;
+    __nv_bfloat16* o0 = out + orow * D;
     __nv_bfloat16* o1 = o0 + static_cast<size_t>(8) * D;
 #pragma unroll
     for (int n = 0; n < D / 8; ++n) {
@@ -370,7 +391,8 @@ template <int D>
 __global__ void __launch_bounds__(128)
 paged_attn_reduce_kernel(const float* __restrict__ part_o, const float2* __restrict__ part_ml,
                          const int* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out,
-                         int rows_total, int num_q_heads, int max_splits, int split_tokens, int max_ctx) {
+                         int rows_total, int num_q_heads, int max_splits, int split_tokens, int max_ctx, int chunk,
+                         const float* __restrict__ gate) {
   grid_dep_wait();
   grid_dep_launch();
   const int row = blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -379,7 +401,7 @@ paged_attn_reduce_kernel(const float* __restrict__ part_o, const float2* __restr
   const int b = row / num_q_heads;
   int L = ctx_lens[b];
   L = L < 0 ? 0 : (L > max_ctx ? max_ctx : L);
-  const int n = (L + split_tokens - 1) / split_tokens;
+  const int n = (L - (first_visible(L, chunk) & ~(kPage - 1)) + split_tokens - 1) / split_tokens;
   if (n <= 1) return;
   const size_t base = static_cast<size_t>(row) * max_splits;
   constexpr int V = D / 32;  // floats per lane
@@ -440,7 +462,7 @@ paged_attn_reduce_kernel(const float* __restrict__ part_o, const float2* __restr
     }
   }
   den = warp_sum(den);
-  const float inv = 1.f / den;
+  const float inv = head_gate(gate, row) / den;
   __nv_bfloat16* dst = out + static_cast<size_t>(row) * D + lane * V;
 #pragma unroll
   for (int j = 0; j < V; j += 2)
@@ -448,30 +470,18 @@ paged_attn_reduce_kernel(const float* __restrict__ part_o, const float2* __restr
 }
 
 // ------------------------------------------------------------ generic path --
-template <typename T>
-__device__ __forceinline__ float to_f32(T v);
-template <>
-__device__ __forceinline__ float to_f32<float>(float v) { return v; }
-template <>
-__device__ __forceinline__ float to_f32<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-template <typename T>
-__device__ __forceinline__ T from_f32(float v);
-template <>
-__device__ __forceinline__ float from_f32<float>(float v) { return v; }
-template <>
-__device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
-
 constexpr int kGenWarps = 4;
-constexpr int kGenMaxPerLane = 8;  // head_dim <= 256
+constexpr int kGenMaxD = 1024;
 
-template <typename T>
+// PER: elements of head_dim per lane (head_dim <= 32 * PER).
+template <typename T, int PER>
 __global__ void __launch_bounds__(kGenWarps * 32)
 paged_attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool,
                           const T* __restrict__ v_pool, const int* __restrict__ block_table,
                           const int* __restrict__ ctx_lens, T* __restrict__ out,
                           int* __restrict__ err, int num_q_heads, int num_kv_heads, int D, int page,
-                          int num_blocks, int max_pages, float scale) {
-  __shared__ float o_sm[kGenWarps][256];
+                          int num_blocks, int max_pages, float scale, int chunk, const float* __restrict__ gate) {
+  __shared__ float o_sm[kGenWarps][32 * PER];
   __shared__ float m_sm[kGenWarps], l_sm[kGenWarps];
   const int h = blockIdx.x, b = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -481,15 +491,15 @@ paged_attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool,
     if (threadIdx.x == 0) set_error(err, kErrDevBadCtxLen);
     L = L < 0 ? 0 : max_pages * page;
   }
-  float qr[kGenMaxPerLane], acc[kGenMaxPerLane];
+  float qr[PER], acc[PER];
 #pragma unroll
-  for (int j = 0; j < kGenMaxPerLane; ++j) {
+  for (int j = 0; j < PER; ++j) {
     const int d = lane + 32 * j;
     qr[j] = d < D ? to_f32<T>(q[(static_cast<size_t>(b) * num_q_heads + h) * D + d]) : 0.f;
     acc[j] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int tok = warp; tok < L; tok += kGenWarps) {
+  for (int tok = first_visible(L, chunk) + warp; tok < L; tok += kGenWarps) {
     int id = block_table[static_cast<size_t>(b) * max_pages + tok / page];
     if (id < 0 || id >= num_blocks) {
       set_error(err, kErrDevBadBlockId);
@@ -498,7 +508,7 @@ paged_attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool,
     const size_t base = ((static_cast<size_t>(id) * num_kv_heads + kvh) * page + tok % page) * D;
     float dot = 0.f;
 #pragma unroll
-    for (int j = 0; j < kGenMaxPerLane; ++j) {
+    for (int j = 0; j < PER; ++j) {
       const int d = lane + 32 * j;
       if (d < D) dot += qr[j] * to_f32<T>(k_pool[base + d]);
     }
@@ -508,13 +518,13 @@ paged_attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool,
     m = mn;
     l = l * a + p;
 #pragma unroll
-    for (int j = 0; j < kGenMaxPerLane; ++j) {
+    for (int j = 0; j < PER; ++j) {
       const int d = lane + 32 * j;
       if (d < D) acc[j] = acc[j] * a + p * to_f32<T>(v_pool[base + d]);
     }
   }
 #pragma unroll
-  for (int j = 0; j < kGenMaxPerLane; ++j) {
+  for (int j = 0; j < PER; ++j) {
     const int d = lane + 32 * j;
     if (d < D) o_sm[warp][d] = acc[j];
   }
@@ -532,7 +542,8 @@ paged_attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool,
       num += wgt * o_sm[w][d];
       den += wgt * l_sm[w];
     }
-    out[(static_cast<size_t>(b) * num_q_heads + h) * D + d] = from_f32<T>(den > 0.f ? num / den : 0.f);
+    const size_t orow = static_cast<size_t>(b) * num_q_heads + h;
+    out[orow * D + d] = from_f32<T>(den > 0.f ? head_gate(gate, orow) * num / den : 0.f);
   }
 }
 
@@ -568,38 +579,19 @@ __global__ void kv_append_kernel(const T* __restrict__ k_new, const T* __restric
 }
 
 // ------------------------------------------------------------------ launch --
-struct AttnWorkspace {
-  int* err;
-  float2* ml;
-  float* o;
-  size_t bytes;
-};
-
 static int max_splits_of(int max_pages, int page, int split_tokens) {
   return (max_pages * page + split_tokens - 1) / split_tokens;
-}
-
-static AttnWorkspace carve(void* ws, int batch, int hq, int D, int max_splits) {
-  AttnWorkspace w;
-  uint8_t* p = static_cast<uint8_t*>(ws);
-  w.err = reinterpret_cast<int*>(p);
-  size_t off = 256;
-  w.ml = reinterpret_cast<float2*>(p + off);
-  off += (static_cast<size_t>(batch) * hq * max_splits * sizeof(float2) + 255) & ~size_t(255);
-  w.o = reinterpret_cast<float*>(p + off);
-  off += static_cast<size_t>(batch) * hq * max_splits * D * sizeof(float);
-  w.bytes = off;
-  return w;
 }
 
 template <int D, int HKV, int STAGES, int CTAS, bool PAIRS = false>
 static int launch_main(const void* q, const void* k_pool, const void* v_pool,
                        const int* block_table, const int* ctx_lens, void* out,
-                       const AttnWorkspace& w, int batch, int hq, int num_blocks, int max_pages,
-                       float scale, int split_tokens, int max_splits, cudaStream_t stream) {
+                       const AttnWorkspace& w, int batch, int hq, int hkv, int num_blocks, int max_pages,
+                       float scale, int split_tokens, int max_splits, int chunk, const float* gate,
+                       cudaStream_t stream) {
   using Cfg = AttnCfg<D, HKV, STAGES, CTAS>;
   CUtensorMap kmap, vmap;
-  const uint64_t rows = static_cast<uint64_t>(num_blocks) * HKV * kPage;
+  const uint64_t rows = static_cast<uint64_t>(num_blocks) * hkv * kPage;
   int rc = get_tensor_map_2d(k_pool, rows, D, 2, HKV * kPage, 64, &kmap);
   if (rc) return rc;
   rc = get_tensor_map_2d(v_pool, rows, D, 2, HKV * kPage, 64, &vmap);
@@ -607,17 +599,17 @@ static int launch_main(const void* q, const void* k_pool, const void* v_pool,
   rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&paged_attn_decode_kernel<D, HKV, STAGES, CTAS, PAIRS>),
                            Cfg::kSmemBytes);
   if (rc) return rc;
-  dim3 grid(PAIRS ? (batch + 1) / 2 : batch, max_splits);
+  dim3 grid(PAIRS ? (batch + 1) / 2 : batch, max_splits, hkv / HKV);
   const float scale_log2 = scale * 1.4426950408889634f;
   B200_CUDA(launch_overlapped(paged_attn_decode_kernel<D, HKV, STAGES, CTAS, PAIRS>, grid, dim3(Cfg::kThreads),
                               Cfg::kSmemBytes, stream, kmap, vmap, static_cast<const __nv_bfloat16*>(q), block_table,
-                              ctx_lens, w.o, w.ml, static_cast<__nv_bfloat16*>(out), w.err, batch, hq, num_blocks,
-                              max_pages, split_tokens, max_splits, scale_log2));
+                              ctx_lens, w.o, w.ml, static_cast<__nv_bfloat16*>(out), w.err, batch, hq, hkv,
+                              num_blocks, max_pages, split_tokens, max_splits, scale_log2, chunk, gate));
   if (max_splits > 1) {
     const int rows = batch * hq;
     B200_CUDA(launch_overlapped(paged_attn_reduce_kernel<D>, dim3((rows + 3) / 4), dim3(128), 0, stream, w.o, w.ml,
                                 ctx_lens, static_cast<__nv_bfloat16*>(out), rows, hq, max_splits, split_tokens,
-                                max_pages * kPage));
+                                max_pages * kPage, chunk, gate));
   }
   return 0;
 }
@@ -636,12 +628,43 @@ extern "C" size_t b200_paged_attn_workspace_bytes(int batch, int num_q_heads, in
   return carve(nullptr, batch, num_q_heads, head_dim, ms).bytes;
 }
 
-extern "C" int b200_paged_attn_decode(const void* q, const void* k_pool, const void* v_pool,
-                                      const int32_t* block_table, const int32_t* ctx_lens,
-                                      void* out, void* workspace, size_t workspace_bytes, int batch,
-                                      int num_q_heads, int num_kv_heads, int head_dim,
-                                      int page_size, int num_blocks, int max_pages_per_seq,
-                                      float scale, int split_tokens, int dtype, void* stream) {
+namespace b200 {
+
+// Splits of the longest range one row can see.
+static int max_splits_chunked(int max_pages, int page, int split_tokens, int chunk) {
+  const long long all = static_cast<long long>(max_pages) * page;
+  long long seen = chunk > 0 ? (static_cast<long long>(chunk) + page - 1) / page * page + page : all;
+  if (seen > all) seen = all;
+  return static_cast<int>((seen + split_tokens - 1) / split_tokens);
+}
+
+template <typename T>
+static int launch_generic(const void* q, const void* k_pool, const void* v_pool, const int* block_table,
+                          const int* ctx_lens, void* out, int* err, int batch, int hq, int hkv, int D, int page,
+                          int num_blocks, int max_pages, float scale, int chunk, const float* gate, cudaStream_t st) {
+  dim3 grid(hq, batch);
+#define B200_GEN_ARGS                                                                                                \
+  static_cast<const T*>(q), static_cast<const T*>(k_pool), static_cast<const T*>(v_pool), block_table, ctx_lens,     \
+      static_cast<T*>(out), err, hq, hkv, D, page, num_blocks, max_pages, scale, chunk, gate
+  if (D <= 256)
+    paged_attn_generic_kernel<T, 8><<<grid, kGenWarps * 32, 0, st>>>(B200_GEN_ARGS);
+  else if (D <= 512)
+    paged_attn_generic_kernel<T, 16><<<grid, kGenWarps * 32, 0, st>>>(B200_GEN_ARGS);
+  else
+    paged_attn_generic_kernel<T, 32><<<grid, kGenWarps * 32, 0, st>>>(B200_GEN_ARGS);
+#undef B200_GEN_ARGS
+  B200_CUDA(cudaGetLastError());
+  return 0;
+}
+
+}  // namespace b200
+
+extern "C" int b200_paged_attn_decode_chunked(const void* q, const void* k_pool, const void* v_pool,
+                                              const int32_t* block_table, const int32_t* ctx_lens, void* out,
+                                              void* workspace, size_t workspace_bytes, int batch, int num_q_heads,
+                                              int num_kv_heads, int head_dim, int page_size, int num_blocks,
+                                              int max_pages_per_seq, float scale, int split_tokens, int dtype,
+                                              int chunk, const float* gate, void* stream) {
   B200_REQUIRE(q && k_pool && v_pool && block_table && ctx_lens && out && workspace,
                "paged_attn_decode: null pointer");
   B200_REQUIRE(batch > 0 && num_q_heads > 0 && num_kv_heads > 0 && num_blocks > 0 &&
@@ -649,7 +672,9 @@ extern "C" int b200_paged_attn_decode(const void* q, const void* k_pool, const v
                "paged_attn_decode: non-positive dimension");
   B200_REQUIRE(num_q_heads % num_kv_heads == 0, "paged_attn_decode: q heads %d not a multiple of kv heads %d",
                num_q_heads, num_kv_heads);
-  B200_REQUIRE(head_dim > 0 && head_dim <= 256, "paged_attn_decode: head_dim %d outside (0, 256]", head_dim);
+  B200_REQUIRE(head_dim > 0 && head_dim <= kGenMaxD, "paged_attn_decode: head_dim %d outside (0, %d]", head_dim,
+               kGenMaxD);
+  B200_REQUIRE(chunk >= 0, "paged_attn_decode: chunk %d is negative", chunk);
   B200_REQUIRE(dtype == 0 || dtype == 1, "paged_attn_decode: dtype %d is neither 0 (bf16) nor 1 (f32)", dtype);
   B200_REQUIRE(workspace_bytes >= 256, "paged_attn_decode: workspace smaller than the status word block");
   int dev = 0;
@@ -658,8 +683,7 @@ extern "C" int b200_paged_attn_decode(const void* q, const void* k_pool, const v
   cudaStream_t st = as_stream(stream);
   const int group = num_q_heads / num_kv_heads;
   const bool fast = dtype == 0 && page_size == kPage && (head_dim == 64 || head_dim == 128) &&
-                    group <= 16 && split_tokens > 0 &&
-                    (num_kv_heads == 1 || num_kv_heads == 2 || num_kv_heads == 4 || num_kv_heads == 8);
+                    group <= 16 && split_tokens > 0;
   if (fast) {
     B200_REQUIRE(split_tokens % kPage == 0, "paged_attn_decode: split_tokens %d not a multiple of %d",
                  split_tokens, kPage);
@@ -667,17 +691,18 @@ extern "C" int b200_paged_attn_decode(const void* q, const void* k_pool, const v
                      (reinterpret_cast<uintptr_t>(v_pool) & 15) == 0 &&
                      (reinterpret_cast<uintptr_t>(q) & 3) == 0,
                  "paged_attn_decode: pools must be 16-byte aligned");
-    const int ms = max_splits_of(max_pages_per_seq, page_size, split_tokens);
+    const int ms = max_splits_chunked(max_pages_per_seq, page_size, split_tokens, chunk);
     B200_REQUIRE(ms <= 65535, "paged_attn_decode: grid too large");
     AttnWorkspace w = carve(workspace, batch, num_q_heads, head_dim, ms);
     if (workspace_bytes < w.bytes) {
       set_detail("paged_attn_decode: workspace %zu < required %zu", workspace_bytes, w.bytes);
       return -kErrWorkspace;
     }
-#define B200_ATTN_ARGS q, k_pool, v_pool, block_table, ctx_lens, out, w, batch, num_q_heads, num_blocks, \
-                       max_pages_per_seq, scale, split_tokens, ms, st
+#define B200_ATTN_ARGS q, k_pool, v_pool, block_table, ctx_lens, out, w, batch, num_q_heads, num_kv_heads, num_blocks, \
+                       max_pages_per_seq, scale, split_tokens, ms, chunk, gate, st
+    const int heads = num_kv_heads % 8 == 0 ? 8 : num_kv_heads % 4 == 0 ? 4 : num_kv_heads % 2 == 0 ? 2 : 1;
     if (head_dim == 128) {
-      switch (num_kv_heads) {
+      switch (heads) {
         case 1: return launch_main<128, 1, 8, 4>(B200_ATTN_ARGS);
         case 2: return launch_main<128, 2, 6, 2>(B200_ATTN_ARGS);
         case 4:
@@ -688,7 +713,7 @@ extern "C" int b200_paged_attn_decode(const void* q, const void* k_pool, const v
         default: return launch_main<128, 8, 3, 1>(B200_ATTN_ARGS);
       }
     }
-    switch (num_kv_heads) {
+    switch (heads) {
       case 1: return launch_main<64, 1, 8, 4>(B200_ATTN_ARGS);
       case 2: return launch_main<64, 2, 6, 4>(B200_ATTN_ARGS);
       case 4: return launch_main<64, 4, 6, 2>(B200_ATTN_ARGS);
@@ -696,21 +721,25 @@ extern "C" int b200_paged_attn_decode(const void* q, const void* k_pool, const v
     }
 #undef B200_ATTN_ARGS
   }
+  B200_REQUIRE(batch <= 65535, "paged_attn_decode: grid too large");
   int* err = static_cast<int*>(workspace);
-  dim3 grid(num_q_heads, batch);
   if (dtype == 0)
-    paged_attn_generic_kernel<__nv_bfloat16><<<grid, kGenWarps * 32, 0, st>>>(
-        static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_pool),
-        static_cast<const __nv_bfloat16*>(v_pool), block_table, ctx_lens,
-        static_cast<__nv_bfloat16*>(out), err, num_q_heads, num_kv_heads, head_dim, page_size,
-        num_blocks, max_pages_per_seq, scale);
-  else
-    paged_attn_generic_kernel<float><<<grid, kGenWarps * 32, 0, st>>>(
-        static_cast<const float*>(q), static_cast<const float*>(k_pool),
-        static_cast<const float*>(v_pool), block_table, ctx_lens, static_cast<float*>(out), err,
-        num_q_heads, num_kv_heads, head_dim, page_size, num_blocks, max_pages_per_seq, scale);
-  B200_CUDA(cudaGetLastError());
-  return 0;
+    return launch_generic<__nv_bfloat16>(q, k_pool, v_pool, block_table, ctx_lens, out, err, batch, num_q_heads,
+                                         num_kv_heads, head_dim, page_size, num_blocks, max_pages_per_seq, scale, chunk,
+                                         gate, st);
+  return launch_generic<float>(q, k_pool, v_pool, block_table, ctx_lens, out, err, batch, num_q_heads, num_kv_heads,
+                               head_dim, page_size, num_blocks, max_pages_per_seq, scale, chunk, gate, st);
+}
+
+extern "C" int b200_paged_attn_decode(const void* q, const void* k_pool, const void* v_pool,
+                                      const int32_t* block_table, const int32_t* ctx_lens,
+                                      void* out, void* workspace, size_t workspace_bytes, int batch,
+                                      int num_q_heads, int num_kv_heads, int head_dim,
+                                      int page_size, int num_blocks, int max_pages_per_seq,
+                                      float scale, int split_tokens, int dtype, void* stream) {
+  return b200_paged_attn_decode_chunked(q, k_pool, v_pool, block_table, ctx_lens, out, workspace, workspace_bytes, batch,
+                                        num_q_heads, num_kv_heads, head_dim, page_size, num_blocks, max_pages_per_seq,
+                                        scale, split_tokens, dtype, 0, nullptr, stream);
 }
 
 /* Prompt form: rows 2i and 2i+1 are two consecutive tokens of one sequence and share block_table row 2i. */
@@ -747,9 +776,11 @@ extern "C" int b200_paged_attn_decode_pairs(const void* q, const void* k_pool, c
   cudaStream_t st = as_stream(stream);
   if (head_dim == 128)
     return launch_main<128, 4, 3, 2, true>(q, k_pool, v_pool, block_table, ctx_lens, out, w, batch, num_q_heads,
-                                           num_blocks, max_pages_per_seq, scale, split_tokens, ms, st);
+                                           num_kv_heads, num_blocks, max_pages_per_seq, scale, split_tokens, ms, 0,
+                                           nullptr, st);
   return launch_main<64, 2, 6, 4, true>(q, k_pool, v_pool, block_table, ctx_lens, out, w, batch, num_q_heads,
-                                        num_blocks, max_pages_per_seq, scale, split_tokens, ms, st);
+                                        num_kv_heads, num_blocks, max_pages_per_seq, scale, split_tokens, ms, 0,
+                                        nullptr, st);
 }
 
 extern "C" int b200_kv_append(const void* k_new, const void* v_new, void* k_pool, void* v_pool,
@@ -867,8 +898,8 @@ extern "C" int b200_paged_attn_decode_static(const void* q, const void* k_pool, 
   w.o = reinterpret_cast<float*>(static_cast<unsigned char*>(scratch) + ml_bytes);
   w.bytes = ml_bytes + o_bytes;
   cudaStream_t st = as_stream(stream);
-#define B200_ATTN_ARGS q, k_pool, v_pool, block_table, ctx_lens, out, w, batch, num_q_heads, num_blocks, \
-                       max_pages_per_seq, scale, split_tokens, ms, st
+#define B200_ATTN_ARGS q, k_pool, v_pool, block_table, ctx_lens, out, w, batch, num_q_heads, num_kv_heads, num_blocks, \
+                       max_pages_per_seq, scale, split_tokens, ms, 0, nullptr, st
   if (head_dim == 128) {
     switch (num_kv_heads) {
       case 1: return launch_main<128, 1, 8, 4>(B200_ATTN_ARGS);

@@ -307,7 +307,8 @@ static int launch_prefill(const void* q, const void* k_pool, const void* v_pool,
 
 // paged_prefill_tc.cu
 int launch_prefill_tc(const void* q, const void* k_pool, const void* v_pool, const int* table_row, void* out, int* err,
-                      int num_tokens, int first_pos, int hq, int hkv, int num_blocks, float scale, cudaStream_t st);
+                      int num_tokens, int first_pos, int hq, int hkv, int head_dim, int num_blocks, float scale,
+                      int chunk, const float* gate, cudaStream_t st);
 
 // The tcgen05 kernel serves head_dim 128 unless the environment variable B200_PREFILL_MMA_SYNC is set to a
 // non-zero value (read once), which keeps every shape on the mma.sync kernel of this file.
@@ -354,9 +355,35 @@ extern "C" int b200_paged_attn_prefill(const void* q, const void* k_pool, const 
   if (head_dim == 128 && prefill_tc_enabled() &&
       ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out)) & 15) == 0)
     return launch_prefill_tc(q, k_pool, v_pool, block_table_row, out, err, num_tokens, first_position, num_q_heads,
-                             num_kv_heads, num_blocks, scale, st);
+                             num_kv_heads, head_dim, num_blocks, scale, 0, nullptr, st);
   if (head_dim == 128 && group == 8) return launch_prefill<128, 8>(B200_PF_ARGS);
   if (head_dim == 128) return launch_prefill<128, 16>(B200_PF_ARGS);
   return launch_prefill<64, 4>(B200_PF_ARGS);
 #undef B200_PF_ARGS
+}
+
+extern "C" int b200_paged_attn_prefill_chunked(const void* q, const void* k_pool, const void* v_pool,
+                                               const int32_t* block_table_row, void* out, void* status_word,
+                                               int num_tokens, int first_position, int num_q_heads, int num_kv_heads,
+                                               int head_dim, int page_size, int num_blocks, int max_pages_per_seq,
+                                               float scale, int chunk, const float* gate, void* stream) {
+  B200_REQUIRE(q && k_pool && v_pool && block_table_row && out, "paged_attn_prefill_chunked: null pointer");
+  B200_REQUIRE(num_tokens > 0 && first_position >= 0 && num_q_heads > 0 && num_kv_heads > 0 && num_blocks > 0 &&
+                   max_pages_per_seq > 0 && chunk >= 0,
+               "paged_attn_prefill_chunked: non-positive dimension");
+  B200_REQUIRE(page_size == kPfPage, "paged_attn_prefill_chunked: page_size %d must be %d", page_size, kPfPage);
+  B200_REQUIRE(num_q_heads % num_kv_heads == 0 && num_q_heads / num_kv_heads <= 128 && num_kv_heads <= 65535,
+               "paged_attn_prefill_chunked: %d query heads over %d kv heads", num_q_heads, num_kv_heads);
+  B200_REQUIRE(head_dim == 64 || head_dim == 128, "paged_attn_prefill_chunked: head_dim %d is not 64 or 128", head_dim);
+  B200_REQUIRE(first_position + num_tokens <= max_pages_per_seq * kPfPage,
+               "paged_attn_prefill_chunked: positions up to %d do not fit %d pages", first_position + num_tokens,
+               max_pages_per_seq);
+  B200_REQUIRE(((reinterpret_cast<uintptr_t>(k_pool) | reinterpret_cast<uintptr_t>(v_pool) |
+                 reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(out)) & 15) == 0,
+               "paged_attn_prefill_chunked: buffers must be 16-byte aligned");
+  int rc = check_device(nullptr);
+  if (rc) return rc;
+  return launch_prefill_tc(q, k_pool, v_pool, block_table_row, out, static_cast<int*>(status_word), num_tokens,
+                           first_position, num_q_heads, num_kv_heads, head_dim, num_blocks, scale, chunk, gate,
+                           as_stream(stream));
 }

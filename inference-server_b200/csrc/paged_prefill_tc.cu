@@ -1,5 +1,5 @@
 // Tiled causal attention over KV pages for a chunk of prompt tokens on the tcgen05 tensor cores (sm_100a),
-// head_dim 128 with 8 or 16 query heads per kv head.  Same operation, arguments and row order as
+// head_dim 64 or 128, up to 128 query heads per kv head.  Same operation, arguments and row order as
 // paged_attn_prefill_kernel (paged_prefill.cu), which stays for the other head shapes; what it replaces in the
 // reference is described there (src/inference_server/kv_cache/hf_format.py:21-45 gather +
 // src/inference_server/backends/torch_backend.py:107-147 chunk forward).
@@ -31,7 +31,17 @@
 //            after the final division by the sum taken against the same max.
 //   out      O / l as bf16, each thread 128 contiguous bytes of its row.
 //
-// TMEM: S0 columns 0-127, S1 128-255, O 256-383 (512 allocated).  Shared memory: Q 32 KiB, P 32 KiB,
+// With 8 or 16 query heads per kv head the Q tile comes by TMA; with any other number G the softmax warps copy it
+// (128 - 128 % G rows are used, the rest are zero rows that are never written out).
+//
+// Two run-time options, as in the decode kernel (paged_attn.cu): `chunk` > 0 cuts the sequence's positions into
+// chunks counted from position 0, and a row sees only the keys of its own chunk - the CTA's walk then begins at the
+// key tile that holds the first key its first row sees, and a tile's two mask edges (the row's chunk start, the row
+// itself) are both per row; `gate` multiplies a row's output by the sigmoid of an fp32 number per (token, head).
+// In this form a row may find its first tiles fully masked: its running maximum stays -inf, its exponentials are taken
+// against 0 (and are all 0), and the first tile it does see rescales by 0 what is an exact 0.
+//
+// TMEM: S0 columns 0-127, S1 128-255, O 256-383 (512 allocated).  Shared memory (head_dim 128): Q 32 KiB, P 32 KiB,
 // K ring 2 x 32 KiB, V ring 2 x 32 KiB.  Every mbarrier wait is bounded; a wait that runs out records
 // kErrDevWaitTimeout and the thread stops waiting but keeps the loop structure (the named barriers between
 // partner warps are still met), so the kernel ends.
@@ -45,15 +55,18 @@ constexpr int kTcPage = 16;
 constexpr int kTcRows = 128;                 // score rows per CTA = M of the MMAs
 constexpr int kTcKeys = 128;                 // keys per tile = N of S, K of P V
 constexpr int kTcPages = kTcKeys / kTcPage;
-constexpr int kTcD = 128;
 constexpr int kTcHalfBytes = 128 * 128;      // 128 rows x 64 bf16: one swizzled column half of a tile
-constexpr int kTcTileBytes = 2 * kTcHalfBytes;
+constexpr int kTcPBytes = 2 * kTcHalfBytes;  // P: 128 rows x 128 keys
 constexpr int kTcSoftmaxWarps = 8;
 constexpr int kTcThreads = (3 + kTcSoftmaxWarps) * 32;
-constexpr int kTcSmemTiles = 6;              // Q, P, K0, K1, V0, V1
 constexpr int kTcExtraBytes = 256 /* barriers, tmem base */ + 2 * 2 * kTcRows * 4 /* max exchange */ +
                               2 * kTcRows * 4 /* sum exchange */;
-constexpr int kTcSmemBytes = kTcSmemTiles * kTcTileBytes + 1024 + kTcExtraBytes;
+template <int D>
+struct TcCfg {
+  static constexpr int kTileBytes = D / 64 * kTcHalfBytes;                 // Q, and one stage of K or V
+  static constexpr int kRingBytes = 5 * kTileBytes + kTcPBytes;            // Q, P, K0, K1, V0, V1
+  static constexpr int kSmemBytes = kRingBytes + 1024 + kTcExtraBytes;
+};
 constexpr float kTcRescaleLog2 = 8.f;        // rescale O when the max grew by more than this (log2 domain)
 
 // bf16 x bf16 -> f32; A K-major; B K-major or (b_mn) MN-major.
@@ -111,21 +124,25 @@ __device__ __forceinline__ void pair_barrier(int quarter) {
   }
 }
 
-// G: query heads per kv head (8 or 16).
-template <int G>
+// G: query heads per kv head (8 or 16, Q tile by TMA); 0 = `group` of them.
+template <int D, int G>
 __global__ void __launch_bounds__(kTcThreads, 1)
 paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                              const __grid_constant__ CUtensorMap v_map, const int* __restrict__ table_row,
                              __nv_bfloat16* __restrict__ out, int* __restrict__ err, int num_tokens, int first_pos,
-                             int num_q_heads, int num_kv_heads, int num_blocks, float scale_log2) {
+                             int num_q_heads, int num_kv_heads, int num_blocks, float scale_log2, int group, int chunk,
+                             const float* __restrict__ gate, const __nv_bfloat16* __restrict__ q) {
 #ifdef B200_DEVICE_OK
-  constexpr int QT = kTcRows / G;  // prompt positions per CTA
+  constexpr int kTcTileBytes = TcCfg<D>::kTileBytes;
+  constexpr int kHalves = D / 64;
+  const int gr = G > 0 ? G : group;
+  const int QT = kTcRows / gr;  // prompt positions per CTA
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* base_ptr = smem_raw + (base - smem_u32(smem_raw));
   const uint32_t q_sm = base, p_sm = base + kTcTileBytes;
-  const uint32_t k_sm = base + 2 * kTcTileBytes, v_sm = base + 4 * kTcTileBytes;  // two stages each
-  const uint32_t bars = base + kTcSmemTiles * kTcTileBytes;
+  const uint32_t k_sm = p_sm + kTcPBytes, v_sm = k_sm + 2 * kTcTileBytes;  // two stages each
+  const uint32_t bars = base + TcCfg<D>::kRingBytes;
   const uint32_t bar_q = bars;                                   // Q tile landed
   const uint32_t bar_kfull = bars + 8, bar_kempty = bars + 24;   // [2] each
   const uint32_t bar_vfull = bars + 40, bar_vempty = bars + 56;  // [2] each
@@ -136,19 +153,19 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
   // rescale can get here for tile j + 1 before a warp of another quarter has arrived for tile j; it cannot get
   // to tile j + 2 before that (its P half waits for the product of tile j, which waits for this barrier).
   const uint32_t bar_rescaled = bars + 136;
-  uint8_t* extra = base_ptr + kTcSmemTiles * kTcTileBytes;
+  uint8_t* extra = base_ptr + TcCfg<D>::kRingBytes;
   uint32_t* tmem_base_sm = reinterpret_cast<uint32_t*>(extra + 192);
   float* mx_sm = reinterpret_cast<float*>(extra + 256);          // [2 tiles][2 halves][128 rows]
   float* l_sm = mx_sm + 2 * 2 * kTcRows;                         // [2 halves][128 rows]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 32) {
-    tma_prefetch_desc(&q_map);
+    if (G > 0) tma_prefetch_desc(&q_map);
     tma_prefetch_desc(&k_map);
     tma_prefetch_desc(&v_map);
   }
   if (threadIdx.x == 0) {
-    mbar_init(bar_q, 1);
+    mbar_init(bar_q, G > 0 ? 1 : kTcSoftmaxWarps);
     for (int s = 0; s < 2; ++s) {
       mbar_init(bar_kfull + 8 * s, 1);
       mbar_init(bar_kempty + 8 * s, 1);
@@ -178,20 +195,23 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
   const int t0 = qt * QT;
   const int t_end = min(t0 + QT, num_tokens);       // one past the tile's last real prompt token
   const int last_pos = first_pos + t_end - 1;       // last position any row of this CTA sees
-  const int n_tiles = last_pos / kTcKeys + 1;
+  const int kt0 = first_visible(first_pos + t0 + 1, chunk) / kTcKeys;  // key tile of the first key any row sees
+  const int n_tiles = last_pos / kTcKeys - kt0 + 1;
   const int last_page = last_pos / kTcPage;
 
   if (warp == 0) {
     // ------------------------------------------------------------ TMA ------
-    // Lanes 0-15 each own one box of a tile: page lane >> 1, column half lane & 1.
-    if (lane == 0) mbar_arrive_expect_tx(bar_q, kTcTileBytes);
-    __syncwarp();
-    for (int i = lane; i < 2 * QT; i += 32) {
-      const int tl = i >> 1, hf = i & 1;
-      tma_load_2d(q_sm + hf * kTcHalfBytes + tl * G * 128, &q_map, bar_q, hf * 64,
-                  (t0 + tl) * num_q_heads + h * G);  // rows past the chunk are filled with zeros
+    // The first 8 * kHalves lanes each own one box of a tile: page lane / kHalves, column half lane % kHalves.
+    if (G > 0) {
+      if (lane == 0) mbar_arrive_expect_tx(bar_q, kTcTileBytes);
+      __syncwarp();
+      for (int i = lane; i < kHalves * QT; i += 32) {
+        const int tl = i / kHalves, hf = i % kHalves;
+        tma_load_2d(q_sm + hf * kTcHalfBytes + tl * gr * 128, &q_map, bar_q, hf * 64,
+                    (t0 + tl) * num_q_heads + h * gr);  // rows past the chunk are filled with zeros
+      }
     }
-    const int pg = (lane >> 1) & 7, hf = lane & 1;
+    const int pg = (lane / kHalves) & 7, hf = lane % kHalves;
     bool alive = true;
 #pragma unroll 1
     for (int j = 0; j < n_tiles; ++j) {
@@ -199,7 +219,7 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
       const uint32_t ph = (j >> 1) & 1;
       // pages past the tile's last position hold nothing this CTA may read; the last valid page stands in so that
       // every stage is the same number of bytes and holds finite numbers (their scores are masked)
-      int page = __ldg(table_row + min(j * kTcPages + pg, last_page));
+      int page = __ldg(table_row + min((kt0 + j) * kTcPages + pg, last_page));
       if (page < 0 || page >= num_blocks) {
         set_error(err, kErrDevBadBlockId);
         page = 0;
@@ -210,12 +230,12 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
       if (!__all_sync(0xffffffffu, alive)) break;
       if (lane == 0) mbar_arrive_expect_tx(bar_kfull + 8 * st, kTcTileBytes);
       __syncwarp();
-      if (lane < 16) tma_load_2d(k_sm + dst, &k_map, bar_kfull + 8 * st, hf * 64, row);
+      if (lane < 8 * kHalves) tma_load_2d(k_sm + dst, &k_map, bar_kfull + 8 * st, hf * 64, row);
       if (alive) alive = mbar_wait(bar_vempty + 8 * st, ph ^ 1, err);
       if (!__all_sync(0xffffffffu, alive)) break;
       if (lane == 0) mbar_arrive_expect_tx(bar_vfull + 8 * st, kTcTileBytes);
       __syncwarp();
-      if (lane < 16) tma_load_2d(v_sm + dst, &v_map, bar_vfull + 8 * st, hf * 64, row);
+      if (lane < 8 * kHalves) tma_load_2d(v_sm + dst, &v_map, bar_vfull + 8 * st, hf * 64, row);
     }
   } else if (warp == 1) {
     // ---------------------------------------------------- S = Q K^T ------
@@ -234,7 +254,7 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
         tc_fence_after();
         const uint64_t b0 = umma_desc_k128(k_sm + st * kTcTileBytes);
 #pragma unroll
-        for (int k = 0; k < 8; ++k) {  // 16 of the 128 head dimensions each
+        for (int k = 0; k < D / 16; ++k) {  // 16 of the head dimensions each
           const uint32_t off = ((k >> 2) * kTcHalfBytes + (k & 3) * 32) >> 4;
           tc_mma_f16(tmem_base + st * kTcKeys, a0 + off, b0 + off, idesc_s, k > 0 ? 1u : 0u);
         }
@@ -245,7 +265,7 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
   } else if (warp == 2) {
     // ---------------------------------------------------- O += P V ------
     if (lane == 0) {
-      constexpr uint32_t idesc_o = tc_idesc_bf16(kTcRows, kTcD, 1);  // B = V, MN-major
+      constexpr uint32_t idesc_o = tc_idesc_bf16(kTcRows, D, 1);  // B = V, MN-major
       const uint32_t tmem_o = tmem_base + 2 * kTcKeys;
       bool alive = true;
 #pragma unroll 1
@@ -279,10 +299,24 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
     const int quarter = warp & 3;            // TMEM lanes this warp may touch
     const int r = quarter * 32 + lane;       // score row
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16);
-    const uint32_t tmem_o = lane_addr + 2 * kTcKeys + hf * 64;
-    const int tl = r / G;
-    const bool real = t0 + tl < num_tokens;
+    const uint32_t tmem_o = lane_addr + 2 * kTcKeys + hf * (D / 2);
+    const int tl = r / gr;
+    const bool real = tl < QT && t0 + tl < num_tokens;
     const int pos = first_pos + min(t0 + tl, t_end - 1);  // the last key this row may see
+    const int row_lo = first_visible(pos + 1, chunk);     // and the first one
+    if (G == 0) {  // copy the Q tile: 16-byte pieces, neighbouring threads neighbouring pieces of a row
+      for (int i = sw * 32 + lane; i < kTcRows * (D / 8); i += kTcSoftmaxWarps * 32) {
+        const int qr = i / (D / 8), ch = i % (D / 8), qt_l = qr / gr;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (qt_l < QT && t0 + qt_l < num_tokens)
+          v = *reinterpret_cast<const uint4*>(
+              q + (static_cast<size_t>(t0 + qt_l) * num_q_heads + h * gr + (qr - qt_l * gr)) * D + ch * 8);
+        *reinterpret_cast<uint4*>(base_ptr + (ch >> 3) * kTcHalfBytes + swz128(qr, ch & 7)) = v;
+      }
+      fence_proxy_async();  // the tensor core reads Q through the async proxy
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar_q);
+    }
     uint8_t* p_half = base_ptr + kTcTileBytes + hf * kTcHalfBytes;
     float m_run = -INFINITY, l_run = 0.f;
     bool alive = true;
@@ -303,12 +337,12 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
       __syncwarp();
       if (lane == 0) mbar_arrive(bar_sempty + 8 * buf);  // this S accumulator may be overwritten
       float s[64];
-      const int kbase = j * kTcKeys + hf * 64;
+      const int kbase = (kt0 + j) * kTcKeys + hf * 64;
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      if (kbase + 63 > pos) {  // the causal edge runs through this half row
+      if (kbase + 63 > pos || kbase < row_lo) {  // the causal edge or the chunk's start runs through this half row
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
-          s[c] = kbase + c > pos ? -INFINITY : __uint_as_float(raw[c]);
+          s[c] = kbase + c > pos || kbase + c < row_lo ? -INFINITY : __uint_as_float(raw[c]);
           mx4[c & 3] = fmaxf(mx4[c & 3], s[c]);
         }
       } else {
@@ -329,11 +363,12 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
           // O may be touched once both products of the tile before have finished
           if (alive) alive = mbar_wait(bar_odone + 8 * (hf ^ 1), (j - 1) & 1, err);
           if (alive) alive = mbar_wait(bar_odone + 8 * hf, (j - 1) & 1, err);
-          const float alpha = fast_exp2((m_run - m_new) * scale_log2);
+          // a row that has seen no key yet holds exact zeros
+          const float alpha = m_new == -INFINITY ? 1.f : fast_exp2((m_run - m_new) * scale_log2);
           l_run *= alpha;
           tc_fence_after();
 #pragma unroll
-          for (int c0 = 0; c0 < 64; c0 += 32) {
+          for (int c0 = 0; c0 < D / 2; c0 += 32) {
             uint32_t o[32];
             tmem_ld32(tmem_o + c0, o);
             tmem_ld_wait();
@@ -350,7 +385,7 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
       if (lane == 0) mbar_arrive(bar_rescaled + 8 * buf);
       // this half of the P tile was last read by the product of the tile before
       if (j > 0 && alive) alive = mbar_wait(bar_odone + 8 * hf, (j - 1) & 1, err);
-      const float mb = m_run * scale_log2;
+      const float mb = m_run == -INFINITY ? 0.f : m_run * scale_log2;
       float sum4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int ch = 0; ch < 8; ++ch) {
@@ -376,10 +411,11 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
     tc_fence_after();
     l_sm[hf * kTcRows + r] = l_run;
     pair_barrier(quarter);
-    const float inv = 1.f / (l_run + l_sm[(hf ^ 1) * kTcRows + r]);
-    __nv_bfloat16* orow = out + (static_cast<size_t>(t0 + tl) * num_q_heads + h * G + (r - tl * G)) * kTcD + hf * 64;
+    const size_t oidx = static_cast<size_t>(t0 + tl) * num_q_heads + h * gr + (r - tl * gr);
+    const float inv = (real ? head_gate(gate, oidx) : 1.f) / (l_run + l_sm[(hf ^ 1) * kTcRows + r]);
+    __nv_bfloat16* orow = out + oidx * D + hf * (D / 2);
 #pragma unroll
-    for (int c0 = 0; c0 < 64; c0 += 32) {
+    for (int c0 = 0; c0 < D / 2; c0 += 32) {
       uint32_t o[32];
       tmem_ld32(tmem_o + c0, o);
       tmem_ld_wait();
@@ -406,43 +442,47 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __
 #endif
 }
 
-static int launch_prefill_tc_g(int group, const CUtensorMap& qmap, const CUtensorMap& kmap, const CUtensorMap& vmap,
+template <int D, int G>
+static int launch_prefill_tc_g(const CUtensorMap& qmap, const CUtensorMap& kmap, const CUtensorMap& vmap, const void* q,
                                const int* table_row, void* out, int* err, int num_tokens, int first_pos, int hq, int hkv,
-                               int num_blocks, float scale, cudaStream_t st) {
-  const float sl = scale * 1.4426950408889634f;
-  const int qt = kTcRows / group;
+                               int num_blocks, float scale, int chunk, const float* gate, cudaStream_t st) {
+  const int group = hq / hkv, qt = kTcRows / group;
   const dim3 grid((num_tokens + qt - 1) / qt, hkv);
-  if (group == 8) {
-    int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&paged_attn_prefill_tc_kernel<8>), kTcSmemBytes);
-    if (rc) return rc;
-    B200_CUDA(launch_overlapped(paged_attn_prefill_tc_kernel<8>, grid, dim3(kTcThreads), kTcSmemBytes, st, qmap, kmap,
-                                vmap, table_row, static_cast<__nv_bfloat16*>(out), err, num_tokens, first_pos, hq, hkv,
-                                num_blocks, sl));
-  } else {
-    int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&paged_attn_prefill_tc_kernel<16>), kTcSmemBytes);
-    if (rc) return rc;
-    B200_CUDA(launch_overlapped(paged_attn_prefill_tc_kernel<16>, grid, dim3(kTcThreads), kTcSmemBytes, st, qmap, kmap,
-                                vmap, table_row, static_cast<__nv_bfloat16*>(out), err, num_tokens, first_pos, hq, hkv,
-                                num_blocks, sl));
-  }
+  int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&paged_attn_prefill_tc_kernel<D, G>), TcCfg<D>::kSmemBytes);
+  if (rc) return rc;
+  B200_CUDA(launch_overlapped(paged_attn_prefill_tc_kernel<D, G>, grid, dim3(kTcThreads), TcCfg<D>::kSmemBytes, st, qmap,
+                              kmap, vmap, table_row, static_cast<__nv_bfloat16*>(out), err, num_tokens, first_pos, hq,
+                              hkv, num_blocks, scale * 1.4426950408889634f, group, chunk, gate,
+                              static_cast<const __nv_bfloat16*>(q)));
   return 0;
 }
 
-// The tcgen05 form of the prompt attention: head_dim 128, 8 or 16 query heads per kv head, q and out 16-byte
-// aligned.  Arguments as launch_prefill in paged_prefill.cu, which has checked them.
+// The tcgen05 form of the prompt attention: head_dim 64 or 128, 1 to 128 query heads per kv head, at most 65535 kv
+// heads, q and out 16-byte aligned.  Arguments as launch_prefill in paged_prefill.cu, which has checked them.
 int launch_prefill_tc(const void* q, const void* k_pool, const void* v_pool, const int* table_row, void* out, int* err,
-                      int num_tokens, int first_pos, int hq, int hkv, int num_blocks, float scale, cudaStream_t st) {
+                      int num_tokens, int first_pos, int hq, int hkv, int head_dim, int num_blocks, float scale,
+                      int chunk, const float* gate, cudaStream_t st) {
   const int group = hq / hkv;
   CUtensorMap qmap, kmap, vmap;
   const uint64_t rows = static_cast<uint64_t>(num_blocks) * hkv * kTcPage;
-  int rc = get_tensor_map_2d(k_pool, rows, kTcD, 2, kTcPage, 64, &kmap);
+  int rc = get_tensor_map_2d(k_pool, rows, head_dim, 2, kTcPage, 64, &kmap);
   if (rc) return rc;
-  rc = get_tensor_map_2d(v_pool, rows, kTcD, 2, kTcPage, 64, &vmap);
+  rc = get_tensor_map_2d(v_pool, rows, head_dim, 2, kTcPage, 64, &vmap);
   if (rc) return rc;
-  rc = get_tensor_map_2d(q, static_cast<uint64_t>(num_tokens) * hq, kTcD, 2, group, 64, &qmap);
-  if (rc) return rc;
-  return launch_prefill_tc_g(group, qmap, kmap, vmap, table_row, out, err, num_tokens, first_pos, hq, hkv, num_blocks,
-                             scale, st);
+  const bool q_tma = head_dim == 128 && (group == 8 || group == 16);
+  if (q_tma) {
+    rc = get_tensor_map_2d(q, static_cast<uint64_t>(num_tokens) * hq, head_dim, 2, group, 64, &qmap);
+    if (rc) return rc;
+  } else {
+    qmap = kmap;  // not read
+  }
+#define B200_TC_ARGS qmap, kmap, vmap, q, table_row, out, err, num_tokens, first_pos, hq, hkv, num_blocks, scale, chunk, \
+                     gate, st
+  if (q_tma && group == 8) return launch_prefill_tc_g<128, 8>(B200_TC_ARGS);
+  if (q_tma) return launch_prefill_tc_g<128, 16>(B200_TC_ARGS);
+  if (head_dim == 128) return launch_prefill_tc_g<128, 0>(B200_TC_ARGS);
+  return launch_prefill_tc_g<64, 0>(B200_TC_ARGS);
+#undef B200_TC_ARGS
 }
 
 }  // namespace b200

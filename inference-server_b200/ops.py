@@ -344,6 +344,353 @@ def qk_norm_rope_append(qkv, q_norm_w, k_norm_w, cos, sin, positions, block_tabl
     return q_out
 
 
+# ------------------------------------------- layer-list decoders (layered.py)
+
+SEG_ROWS, SEG_F32, SEG_PAGES = 0, 1, 2
+
+
+def paged_attn_decode_chunked(q, k_pool, v_pool, block_table, ctx_lens, scale: float, split_tokens: int, workspace, chunk: int = 0,
+                              gate=None, out=None):
+    """`paged_attn_decode` with two options: `chunk` > 0 limits a row to the tokens of its own chunk of positions, and
+    `gate` [B, Hq] fp32 multiplies every head's output by its sigmoid.  bf16 or fp32."""
+    _need(q, "q")
+    _need(k_pool, "k_pool", q.dtype)
+    _need(v_pool, "v_pool", q.dtype)
+    _need(block_table, "block_table", torch.int32)
+    _need(ctx_lens, "ctx_lens", torch.int32)
+    if gate is not None:
+        _need(gate, "gate", torch.float32)
+    B, Hq, D = q.shape
+    nb, Hkv, page, D2 = k_pool.shape
+    if D2 != D or v_pool.shape != k_pool.shape or block_table.shape[0] != B or ctx_lens.shape[0] != B:
+        raise ValueError("pools, block table or lengths do not match q")
+    if gate is not None and gate.numel() != B * Hq:
+        raise ValueError("gate does not match q")
+    if out is None:
+        out = torch.empty_like(q)
+    rc = _lib.load().b200_paged_attn_decode_chunked(
+        _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), _ptr(ctx_lens), _ptr(out), _ptr(workspace), workspace.numel(),
+        B, Hq, Hkv, D, page, nb, block_table.shape[1], float(scale), int(split_tokens), DTYPE_CODE[q.dtype], int(chunk),
+        _ptr(gate), _stream())
+    check(rc, "b200_paged_attn_decode_chunked")
+    return out
+
+
+def paged_attn_prefill_chunked_supported(num_q_heads: int, num_kv_heads: int, head_dim: int, dtype) -> bool:
+    return dtype == torch.bfloat16 and head_dim in (64, 128) and num_q_heads // num_kv_heads <= 128
+
+
+def paged_attn_prefill_chunked(q, k_pool, v_pool, table_row, first_pos: int, scale: float, status=None, chunk: int = 0, gate=None,
+                               out=None):
+    """`paged_attn_prefill` with the options of `paged_attn_decode_chunked`; head_dim 64 or 128, any head grouping."""
+    _need(q, "q", torch.bfloat16)
+    _need(k_pool, "k_pool", torch.bfloat16)
+    _need(v_pool, "v_pool", torch.bfloat16)
+    _need(table_row, "table_row", torch.int32)
+    if gate is not None:
+        _need(gate, "gate", torch.float32)
+    R, Hq, D = q.shape
+    nb, Hkv, page, D2 = k_pool.shape
+    if D2 != D or v_pool.shape != k_pool.shape or (gate is not None and gate.numel() != R * Hq):
+        raise ValueError("pools or gate do not match q")
+    if out is None:
+        out = torch.empty_like(q)
+    _need(out, "out", torch.bfloat16)
+    rc = _lib.load().b200_paged_attn_prefill_chunked(
+        _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(table_row), _ptr(out), _ptr(status), R, int(first_pos), Hq, Hkv, D, page, nb,
+        table_row.numel(), float(scale), int(chunk), _ptr(gate), _stream())
+    check(rc, "b200_paged_attn_prefill_chunked")
+    return out
+
+
+def latent_attn_supported(rank: int, page_size: int, dtype) -> bool:
+    return dtype == torch.bfloat16 and bool(_lib.load().b200_latent_attn_supported(int(rank), int(page_size)))
+
+
+def latent_split_tokens(batch: int, max_ctx: int, num_sms: int = 148) -> int:
+    """Tokens per split of the latent decode kernel (all heads of a row in one CTA): enough CTAs to fill the GPU about
+    twice over, splits no shorter than 256 tokens."""
+    per_row = max(1, -(-2 * num_sms // max(1, batch)))
+    split = -(-max(1, max_ctx) // per_row)
+    return int(min(4096, max(256, -(-split // 64) * 64)))
+
+
+def latent_attn_decode(q, c_pool, block_table, ctx_lens, scale: float, split_tokens: int, workspace, gate=None, out=None):
+    """Attention of projected queries q [B, H, rank] over a cache of latents c_pool [num_blocks, page, rank], which are keys
+    and values at once; returns weighted sums of latents [B, H, rank]."""
+    _need(q, "q", torch.bfloat16)
+    _need(c_pool, "c_pool", torch.bfloat16)
+    _need(block_table, "block_table", torch.int32)
+    _need(ctx_lens, "ctx_lens", torch.int32)
+    if gate is not None:
+        _need(gate, "gate", torch.float32)
+    B, H, R = q.shape
+    nb, page, R2 = c_pool.shape
+    if R2 != R or block_table.shape[0] != B or ctx_lens.shape[0] != B or (gate is not None and gate.numel() != B * H):
+        raise ValueError("pool, block table, lengths or gate do not match q")
+    if out is None:
+        out = torch.empty_like(q)
+    rc = _lib.load().b200_latent_attn_decode(
+        _ptr(q), _ptr(c_pool), _ptr(block_table), _ptr(ctx_lens), _ptr(out), _ptr(workspace), workspace.numel(), B, H, R, page, nb,
+        block_table.shape[1], float(scale), int(split_tokens), _ptr(gate), _stream())
+    check(rc, "b200_latent_attn_decode")
+    return out
+
+
+def dense_gemm_f32_out(x, w, status=None, workspace=None, out=None):
+    """y = x w^T with bf16 operands and the fp32 accumulators as the result (logits)."""
+    _need(x, "x", torch.bfloat16)
+    _need(w, "w", torch.bfloat16)
+    M, K = x.shape
+    N = w.shape[0]
+    if w.shape[1] != K:
+        raise ValueError(f"x has {K} columns, w has {w.shape[1]}")
+    if out is None:
+        out = torch.empty(M, N, dtype=torch.float32, device=x.device)
+    if M == 0:
+        return out
+    rc = _lib.load().b200_dense_gemm_bf16_f32(_ptr(x), _ptr(w), _ptr(out), _ptr(workspace),
+                                              0 if workspace is None else workspace.numel(), _ptr(status), M, N, K,
+                                              0 if workspace is not None else 1, _stream())
+    check(rc, "b200_dense_gemm_bf16_f32")
+    return out
+
+
+def grouped_gemm(x, w, groups: int, out=None, status=None):
+    """Per group (head) g: y[:, g] = x[:, g] w[g]^T for x [M, groups, K], w [groups, N, K] -> [M, groups, N].  bf16 on the
+    tensor cores, fp32 in true fp32."""
+    _need(x, "x")
+    _need(w, "w", x.dtype)
+    M, G, K = x.shape
+    N = w.shape[1]
+    if G != groups or w.shape[0] != groups or w.shape[2] != K:
+        raise ValueError("x and w do not match")
+    if out is None:
+        out = torch.empty(M, groups, N, dtype=x.dtype, device=x.device)
+    if M == 0:
+        return out
+    lib = _lib.load()
+    if x.dtype == torch.bfloat16:
+        rc = lib.b200_dense_gemm_grouped(_ptr(x), _ptr(w), _ptr(out), _ptr(status), M, groups, N, K, K, N, N, groups * K,
+                                         groups * N, _stream())
+        check(rc, "b200_dense_gemm_grouped")
+    else:
+        _need(x, "x", torch.float32)
+        rc = lib.b200_gemm_f32(_ptr(x), _ptr(w), _ptr(out), M, groups, N, K, K, N, N, groups * K, groups * N, _stream())
+        check(rc, "b200_gemm_f32")
+    return out
+
+
+def gemm_f32(x, w, out=None):
+    """y = x w^T in true fp32."""
+    _need(x, "x", torch.float32)
+    _need(w, "w", torch.float32)
+    M, K = x.shape
+    N = w.shape[0]
+    if w.shape[1] != K:
+        raise ValueError(f"x has {K} columns, w has {w.shape[1]}")
+    if out is None:
+        out = torch.empty(M, N, dtype=torch.float32, device=x.device)
+    if M:
+        check(_lib.load().b200_gemm_f32(_ptr(x), _ptr(w), _ptr(out), M, 1, N, K, 0, N, 0, K, N, _stream()), "b200_gemm_f32")
+    return out
+
+
+def _segments(segs):
+    """segs: (kind, target) or (SEG_PAGES, pool, heads, dim) in feature order -> ctypes arrays."""
+    import ctypes
+    n = len(segs)
+    end, kind, heads, dim = ((ctypes.c_int32 * n)() for _ in range(4))
+    ptr = (ctypes.c_void_p * n)()
+    at = 0
+    for i, s in enumerate(segs):
+        t = s[1]
+        if not t.is_cuda or not t.is_contiguous():
+            raise ValueError("segment targets must be contiguous CUDA tensors")
+        if s[0] == SEG_PAGES:
+            heads[i], dim[i] = t.shape[1], t.shape[3]
+            width = t.shape[1] * t.shape[3]
+        else:
+            width = t[0].numel() if t.shape[0] else 0
+        at += width
+        end[i], kind[i], ptr[i] = at, s[0], t.data_ptr()
+    return end, kind, heads, dim, ptr, n, at
+
+
+def _segment_pages(segs):
+    for s in segs:
+        if s[0] == SEG_PAGES:
+            return s[1].shape[2], s[1].shape[0]
+    return 1, 1
+
+
+def proj_split(x, w, segs, col_scale=None, positions=None, block_table=None, status=None, max_pages: int | None = None):
+    """x w^T with consecutive ranges of output features sent to different places: segs lists (SEG_ROWS, bf16/fp32 tensor
+    [M, ...] of x's dtype), (SEG_F32, fp32 tensor [M, ...]) and (SEG_PAGES, pool [blocks, heads, page, dim], written at
+    positions[m] of the sequence block_table[m]; both None: row m of page-contiguous scratch).  `col_scale` multiplies the
+    features in fp32.  One kernel in bf16; in fp32 a product and a store kernel."""
+    _need(x, "x")
+    _need(w, "w", x.dtype)
+    M, K = x.shape
+    if M == 0:
+        return
+    end, kind, heads, dim, ptr, n, total = _segments(segs)
+    if w.shape != (total, K):
+        raise ValueError(f"w is {tuple(w.shape)}, the segments need {(total, K)}")
+    if col_scale is not None:
+        _need(col_scale, "col_scale", torch.float32)
+    page, nb = _segment_pages(segs)
+    if positions is not None:
+        _need(positions, "positions", torch.int32)
+    if block_table is not None:
+        _need(block_table, "block_table", torch.int32)
+        max_pages = block_table.shape[1]
+    elif max_pages is None:
+        max_pages = nb
+    lib = _lib.load()
+    if x.dtype == torch.bfloat16:
+        rc = lib.b200_proj_split_gemm(_ptr(x), _ptr(w), _ptr(col_scale), end, kind, heads, dim, ptr, n, _ptr(positions),
+                                      _ptr(block_table), _ptr(status), M, K, page, nb, max_pages, _stream())
+        check(rc, "b200_proj_split_gemm")
+    else:
+        split_store(gemm_f32(x, w), segs, col_scale, positions, block_table, status, torch.float32, max_pages)
+
+
+def split_store(y, segs, col_scale=None, positions=None, block_table=None, status=None, dtype=torch.float32,
+                max_pages: int | None = None):
+    """The store of `proj_split` on a finished fp32 product y [M, N]."""
+    _need(y, "y", torch.float32)
+    end, kind, heads, dim, ptr, n, total = _segments(segs)
+    if y.shape[1] != total:
+        raise ValueError(f"y has {y.shape[1]} columns, the segments {total}")
+    page, nb = _segment_pages(segs)
+    if block_table is not None:
+        max_pages = block_table.shape[1]
+    rc = _lib.load().b200_split_store(_ptr(y), _ptr(col_scale), end, kind, heads, dim, ptr, n, _ptr(positions),
+                                      _ptr(block_table), _ptr(status), y.shape[0], page, nb, max_pages or nb, DTYPE_CODE[dtype],
+                                      _stream())
+    check(rc, "b200_split_store")
+
+
+def glu_proj(x, w_interleaved, limit: float, alpha: float, status=None, out=None):
+    """Gate and up projection + clamped gated unit; w rows alternate in blocks of 128 gate / 128 up features.  One kernel in
+    bf16; in fp32 a product and an element-wise kernel."""
+    _need(x, "x")
+    _need(w_interleaved, "w", x.dtype)
+    M, K = x.shape
+    F = w_interleaved.shape[0] // 2
+    if w_interleaved.shape[1] != K:
+        raise ValueError("x and w do not match")
+    if out is None:
+        out = torch.empty(M, F, dtype=x.dtype, device=x.device)
+    if M == 0:
+        return out
+    if x.dtype == torch.bfloat16:
+        rc = _lib.load().b200_dense_glu_gemm(_ptr(x), _ptr(w_interleaved), _ptr(out), _ptr(status), M, F, K, float(limit),
+                                             float(alpha), _stream())
+        check(rc, "b200_dense_glu_gemm")
+        return out
+    return clamped_glu(gemm_f32(x, w_interleaved), limit, alpha, out)
+
+
+def clamped_glu(gate_up, limit: float, alpha: float, out=None):
+    """The gated unit alone on gate/up columns interleaved in blocks of 128."""
+    _need(gate_up, "gate_up")
+    M, F = gate_up.shape[0], gate_up.shape[1] // 2
+    if out is None:
+        out = torch.empty(M, F, dtype=gate_up.dtype, device=gate_up.device)
+    check(_lib.load().b200_clamped_glu(_ptr(gate_up), _ptr(out), M, F, float(limit), float(alpha), DTYPE_CODE[gate_up.dtype],
+                                       _stream()), "b200_clamped_glu")
+    return out
+
+
+def embed_sinusoid(tokens, positions, embed, tables, width: int, status=None):
+    """fp32 residual rows embed[token] + sinusoid(position); tables = (lo, hi) as `layered.sinusoid_tables` makes them."""
+    _need(tokens, "tokens", torch.int64)
+    _need(positions, "positions", torch.int32)
+    _need(embed, "embed")
+    lo, hi = tables
+    M, ld = tokens.shape[0], embed.shape[1]
+    x = torch.empty(M, ld, dtype=torch.float32, device=embed.device)
+    rc = _lib.load().b200_embed_sinusoid(_ptr(tokens), _ptr(positions), _ptr(embed), _ptr(lo), _ptr(hi), _ptr(x), _ptr(status), M,
+                                         int(width), ld, embed.shape[0], hi.shape[0], DTYPE_CODE[embed.dtype], _stream())
+    check(rc, "b200_embed_sinusoid")
+    return x
+
+
+def group_rmsnorm(x, delta, weight, eps: float, width: int, groups: int, conv_w=None, hist=None, positions=None,
+                  block_table=None, page: int = 16, status=None, out=None):
+    """x (fp32) += delta in place; returns weight * x / rms per group of columns, in weight's dtype.  With conv_w [taps, ld]
+    the rows are decode rows and the short causal convolution over the pages' history `hist` is added."""
+    _need(x, "x", torch.float32)
+    _need(weight, "weight")
+    if delta is not None:
+        _need(delta, "delta", weight.dtype)
+    M, ld = x.shape
+    if out is None:
+        out = torch.empty(M, ld, dtype=weight.dtype, device=x.device)
+    taps = 0 if conv_w is None else conv_w.shape[0]
+    nb = 1 if hist is None else hist.shape[0]
+    if taps and block_table is not None and hist is None:
+        nb = 2**31 - 1
+    rc = _lib.load().b200_group_rmsnorm(_ptr(x), _ptr(delta), _ptr(weight), float(eps), M, int(width), ld, int(groups), _ptr(out),
+                                        _ptr(conv_w), taps, _ptr(hist), _ptr(positions), _ptr(block_table), page, nb,
+                                        1 if block_table is None else block_table.shape[1], _ptr(status),
+                                        DTYPE_CODE[weight.dtype], _stream())
+    check(rc, "b200_group_rmsnorm")
+    return out
+
+
+def short_conv(h, conv_w, hist, table_row, first_pos: int, page: int = 16, status=None, out=None):
+    """h + causal convolution for consecutive tokens of one sequence; earlier rows come from, and the last rows go to, the
+    pages' history."""
+    _need(h, "h")
+    _need(conv_w, "conv_w", h.dtype)
+    _need(table_row, "table_row", torch.int32)
+    M, ld = h.shape
+    if out is None:
+        out = torch.empty_like(h)
+    nb = hist.shape[0] if hist is not None else 2**31 - 1
+    rc = _lib.load().b200_short_conv(_ptr(h), _ptr(conv_w), conv_w.shape[0], _ptr(hist), _ptr(table_row), M, int(first_pos), ld,
+                                     _ptr(out), page, nb, table_row.numel(), _ptr(status), DTYPE_CODE[h.dtype], _stream())
+    check(rc, "b200_short_conv")
+    return out
+
+
+def latent_norm_append(raw, weight, eps: float, rank: int, c_pool, positions, block_table, status=None):
+    """RMS norm of fp32 latents [M, ld] over their first `rank` columns, written into the page slots of c_pool."""
+    _need(raw, "raw", torch.float32)
+    _need(c_pool, "c_pool", weight.dtype)
+    nb, page, ld = c_pool.shape
+    if raw.shape[1] != ld:
+        raise ValueError("raw does not match the pool")
+    rc = _lib.load().b200_latent_norm_append(_ptr(raw), _ptr(weight), float(eps), raw.shape[0], int(rank), ld, _ptr(c_pool),
+                                             _ptr(positions), _ptr(block_table), page, nb, block_table.shape[1], _ptr(status),
+                                             DTYPE_CODE[weight.dtype], _stream())
+    check(rc, "b200_latent_norm_append")
+
+
+def gather_pages(c_pool, table_row, num_tokens: int, status=None):
+    """The first num_tokens rows of a sequence's pages [num_blocks, page, ld] as one [num_tokens, ld] tensor."""
+    _need(c_pool, "c_pool")
+    nb, page, ld = c_pool.shape
+    out = torch.empty(num_tokens, ld, dtype=c_pool.dtype, device=c_pool.device)
+    rc = _lib.load().b200_gather_pages(_ptr(c_pool), _ptr(table_row), _ptr(out), num_tokens, ld, page, nb, table_row.numel(),
+                                       _ptr(status), DTYPE_CODE[c_pool.dtype], _stream())
+    check(rc, "b200_gather_pages")
+    return out
+
+
+def argmax_rows(logits, out=None):
+    """Arg-max of fp32 rows, ties to the lower index."""
+    _need(logits, "logits", torch.float32)
+    if out is None:
+        out = torch.empty(logits.shape[0], dtype=torch.int64, device=logits.device)
+    _need(out, "out", torch.int64)
+    check(_lib.load().b200_argmax_rows(_ptr(logits), _ptr(out), logits.shape[0], logits.shape[1], _stream()), "b200_argmax_rows")
+    return out
+
+
 # ------------------------------------------------------------------------ MoE
 
 
