@@ -383,7 +383,7 @@ int b200_embed_sinusoid(const int64_t* tokens, const int32_t* positions, const v
  * columns (rows are ld wide, the rest is zero).
  * With taps > 0 also the short causal convolution of a decode step, row m being the token at positions[m] of its own
  * sequence: out += sum_j conv_w[j] * h(position - taps + 1 + j), h the normed row rounded to dtype, zeros before the
- * start.  The earlier h come from the pages: hist [num_blocks, min(taps-1, page), ld] keeps for every page the last rows
+ * start.  The earlier h come from the pages: hist [num_blocks, min(taps, page), ld] keeps for every page the last rows
  * written in it (position p in slot p % page % rows), and the row's own h is written there. */
 int b200_group_rmsnorm(float* x, const void* delta, const void* weight, float eps, int num_rows, int width, int ld,
                        int groups, void* out, const void* conv_w, int taps, void* hist, const int32_t* positions,

@@ -84,6 +84,7 @@ class B200Backend:
 
     cache_adapter = None
     last_cache_hit_tokens: int = 0
+    last_logits = None  # prefill_chunk(..., want=...)
 
     def __init__(self, engine=None, eos_ids: set[int] | None = None, max_new_tokens: int = 256):
         self.engine = engine
@@ -105,6 +106,10 @@ class B200Backend:
         eng = self.engine
         if bm is None or eng is None or not getattr(bm, "k_pools", None):
             return
+        if not getattr(eng, "takes_reference_pools", True):
+            # its layers keep other state than K/V pairs of one shape (latents, convolution history), which the
+            # manager neither stores nor finds again
+            raise ValueError("this model's cache does not fit a reference CacheManager's K/V pools; serve it without one")
         want = (eng.cfg.kv_heads, PAGE, eng.cfg.head_dim)
         ok = (len(bm.k_pools) == eng.cfg.layers and all(
             tuple(p.shape[1:]) == want and p.dtype == torch.bfloat16 and p.device.type == torch.device(eng.device).type
@@ -119,28 +124,39 @@ class B200Backend:
         self._alloc = None  # pages now come from the reference BlockManager
 
     def load_model(self, model_name: str, num_blocks: int = 4096, max_batch: int = 64,
-                   max_pages_per_seq: int = 256) -> None:
-        """Load a Qwen3-MoE checkpoint as TorchBackend.load_model does (torch_backend.py:33-53):
+                   max_pages_per_seq: int = 256, **engine_args) -> None:
+        """Load a model: a folder whose config.json names an architecture of ``registry`` (layer-list decoders: their own
+        tensors, EOS ids from the config's ``eos_token_id`` if it has one), a Qwen3-MoE checkpoint, or a built-in shape.
+        ``engine_args`` go to the engine (``dtype``, ``keep_logits``, ...).
+        A Qwen3-MoE checkpoint is loaded as TorchBackend.load_model does (torch_backend.py:33-53):
         ``AutoModelForCausalLM.from_pretrained(model_name, dtype=bfloat16)``, EOS ids from the model
         config; the weights are then converted to the engine's run-time formats (``engine_from_hf``: dense
         weights bf16, experts e4m3 with 128x128 block scales - taken as stored when the checkpoint is FP8).
-        One of the built-in shape names (``engine.CONFIGS``) builds a random-init engine of that shape
+        One of the built-in shape names (``engine.CONFIGS``, ``layered.CONFIGS``) builds a random-init engine of that shape
         instead, for benchmarks without a checkpoint.  Needs a CUDA device either way."""
-        from . import engine as eng_mod
+        from . import registry
 
-        if model_name in eng_mod.CONFIGS:
-            self.engine = eng_mod.DecodeEngine(eng_mod.CONFIGS[model_name], num_blocks=num_blocks, max_batch=max_batch,
-                                               max_pages_per_seq=max_pages_per_seq)
+        sizes = dict(num_blocks=num_blocks, max_batch=max_batch, max_pages_per_seq=max_pages_per_seq)
+        shape, folder = registry.shape_family(model_name), registry.folder_family(model_name)
+        if shape is not None:
+            self.engine = shape[0].from_shape(shape[1], **sizes, **engine_args)
+        elif folder is not None:
+            family, config = folder
+            self._eos_ids = self._eos_of(config.get("eos_token_id"))
+            self.engine = family.from_folder(model_name, config, **sizes, **engine_args)
         else:
             model, self.tokenizer = self._read_checkpoint(model_name)
-            eos = model.config.eos_token_id
-            self._eos_ids = set(eos) if isinstance(eos, (list, tuple)) else ({eos} if eos is not None else set())
+            self._eos_ids = self._eos_of(model.config.eos_token_id)
             self.engine = self._engine_from_model(model, num_blocks, max_batch, max_pages_per_seq)
             del model
         self._alloc = _FreeListAllocator(self.engine.num_blocks)
         self._table_cpu = self._lens_cpu = self._synced_batch = None
         if self.cache_adapter is not None:
             self.set_cache_adapter(self.cache_adapter)
+
+    @staticmethod
+    def _eos_of(eos) -> set[int]:
+        return set(eos) if isinstance(eos, (list, tuple)) else ({eos} if eos is not None else set())
 
     @staticmethod
     def _read_checkpoint(model_name: str):
@@ -190,11 +206,13 @@ class B200Backend:
 
     def kv_shape_per_layer(self) -> list[tuple[int, int]]:
         cfg = self.engine.cfg
+        if not getattr(self.engine, "takes_reference_pools", True):
+            raise ValueError("this model's layers do not all keep K/V pairs of one shape")
         return [(cfg.kv_heads, cfg.head_dim)] * cfg.layers
 
     @property
     def kv_dtype(self) -> torch.dtype:
-        return torch.bfloat16
+        return getattr(self.engine, "dtype", torch.bfloat16)
 
     @property
     def device(self):
@@ -355,9 +373,10 @@ class B200Backend:
             raise
         return kv, matched
 
-    def prefill_chunk(self, chunk_token_ids: list[int], partial_kv):
+    def prefill_chunk(self, chunk_token_ids: list[int], partial_kv, want: list[int] | None = None):
         """Forward one chunk on top of partial_kv (base.py:71-78).  If the chunk cannot run, the pages taken
-        for it go back; the partial KV of the earlier chunks stays as it was."""
+        for it go back; the partial KV of the earlier chunks stays as it was.  With `want` (places in the chunk) the
+        logits there are kept in ``last_logits`` [len(want), vocab], on the device."""
         kv = partial_kv if partial_kv is not None else SeqKV(block_ids=[], ctx_len=0)
         new_len = kv.ctx_len + len(chunk_token_ids)
         total_pages = (new_len + self.max_new_tokens + PAGE - 1) // PAGE
@@ -368,7 +387,8 @@ class B200Backend:
         try:
             # only the tokens past `cached_tokens` are embedded; the earlier ones are already pages
             tokens = [0] * kv.ctx_len + list(chunk_token_ids)
-            last, _ = self.engine.prefill(tokens, kv.block_ids + ids, cached_tokens=kv.ctx_len)
+            asked = {} if want is None else {"want": [kv.ctx_len + w for w in want]}
+            last, self.last_logits = self.engine.prefill(tokens, kv.block_ids + ids, cached_tokens=kv.ctx_len, **asked)
             self._check_status("prefill_chunk")
         except BaseException:
             self._give_back(handles)

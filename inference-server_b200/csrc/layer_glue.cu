@@ -4,8 +4,10 @@
 // convolutions are fp32; T is the type of the activations between kernels (bf16 or fp32).
 //
 // The convolution's history lives in the pages, beside the K/V or latents of the same tokens: per layer
-// hist [num_blocks, min(taps - 1, page), ld], position p of a sequence in its page p / page, slot (p % page) % rows.
+// hist [num_blocks, min(taps, page), ld], position p of a sequence in its page p / page, slot (p % page) % rows.
 // The taps - 1 rows before any position are then always to be found: each is among the last `rows` written in its page.
+// One row more than the convolution looks back makes a step repeatable: writing position p overwrites none of the rows
+// that p itself reads (a CUDA graph's warm-up runs the same step several times).
 // A sequence's state is taken, moved and given back with its pages, and there is no slot to manage.
 
 #include <initializer_list>
@@ -136,7 +138,7 @@ __global__ void group_rmsnorm_kernel(float* __restrict__ x, const T* __restrict_
     pos = positions[m];
     const int* table_row = block_table + static_cast<size_t>(m) * pm.max_pages;
     page = page_of(pm, table_row, pos);
-    rows = min(taps - 1, pm.page);
+    rows = taps > 1 ? min(taps, pm.page) : 0;
     if (in && page >= 0) {
       load8<T>(conv_w + static_cast<size_t>(taps - 1) * ld + col, wlast);
       for (int j = 0; j + 1 < taps; ++j) {
@@ -212,7 +214,7 @@ short_conv_kernel(const T* __restrict__ h, const T* __restrict__ conv_w, int tap
   if (col >= ld) return;
   const int pg0 = first_pos / pm.page + static_cast<int>(blockIdx.x);
   const int lo = max(first_pos, pg0 * pm.page), hi = min(first_pos + num_rows, (pg0 + 1) * pm.page);
-  const int rows = min(taps - 1, pm.page);
+  const int rows = taps > 1 ? min(taps, pm.page) : 0;
 #pragma unroll 2
   for (int p = lo; p < hi; ++p) {
     float acc[8], hv[8], cw[8];

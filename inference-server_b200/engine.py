@@ -135,18 +135,28 @@ def engine_from_hf(model, num_blocks: int, max_batch: int, max_pages_per_seq: in
                         final_norm=model.model.norm.weight.detach().to(device=device, dtype=bf).contiguous(), **kw)
 
 
-class DecodeEngine:
-    """Owns weights, KV page pools and the per-batch-size CUDA graphs of the decode step."""
+class PagedEngine:
+    """What every model's engine is: the static step state (tokens, context lengths, block table of up to `max_batch` rows),
+    the decode step as CUDA graphs per batch size, the prompt pass in chunks and the merged pass.  A model adds its
+    weights, its page pools (`num_blocks` pages per layer, one more as scratch page) and five hooks:
 
-    def __init__(self, cfg: ModelConfig, num_blocks: int, max_batch: int, max_pages_per_seq: int,
-                 device: str | torch.device = "cuda", seed: int = 0, layers: list[LayerWeights] | None = None,
-                 embed: torch.Tensor | None = None, lm_head: torch.Tensor | None = None,
-                 final_norm: torch.Tensor | None = None, k_pools=None, v_pools=None, use_graphs: bool = True,
-                 split_tokens: int | None = None, ep_group=None, ep_capacity: int | None = None,
-                 ep_transport: str = "p2p", graph_buckets: bool = True, keep_logits: bool = False):
+      _decode_hidden(B)                        final normed hidden rows of one decode step of rows [0, B)
+      _begin_prompt(chunk) -> chunk            buffers for prompt passes of up to `chunk` tokens
+      _prompt_hidden(token_ids, row, lo, chunk)     hidden rows of one chunk at positions lo.. of the sequence with table `row`
+      _mixed_hidden(tokens, pos, table, first_pos, n, B)   rows of a chunk (first n) and of a decode step (the rest)
+      _pick(h, out) / _logits(h)               next tokens (arg-max) / logits of hidden rows
+    """
+
+    prompt_chunk = 1024       # tokens of a prompt pass unless the caller says otherwise
+    ep_state = None           # expert parallelism (DecodeEngine)
+    round_hook = None
+    takes_reference_pools = False  # whether a reference BlockManager's K/V pools can stand in for the engine's own
+    logits_dtype = torch.bfloat16
+
+    def _init_step_state(self, num_blocks: int, max_batch: int, max_pages_per_seq: int, device, use_graphs: bool,
+                         keep_logits: bool, scratch_page: bool) -> None:
         if not torch.cuda.is_available():
-            raise RuntimeError("DecodeEngine needs a CUDA device; this path has no CPU implementation")
-        self.cfg = cfg
+            raise RuntimeError(f"{type(self).__name__} needs a CUDA device; this path has no CPU implementation")
         self.device = torch.device(device)
         # The step picks its next tokens inside the lm_head kernel and never writes the [batch, vocab] logits.
         # With keep_logits they are computed as well, by a second pass over lm_head, into `last_logits` (for
@@ -157,6 +167,221 @@ class DecodeEngine:
         self.max_pages = max_pages_per_seq
         self.num_blocks = num_blocks
         self.use_graphs = use_graphs
+        # Pools the engine allocates itself get one block more than the caller may hand out: the scratch page
+        # that the padding rows of a bucketed CUDA graph write their state to (see step).
+        self.scratch_block = num_blocks if scratch_page else None
+        self.tokens = torch.zeros(max_batch, dtype=torch.int64, device=self.device)
+        self.ctx_lens = torch.zeros(max_batch, dtype=torch.int32, device=self.device)
+        self.block_table = torch.zeros(max_batch, max_pages_per_seq, dtype=torch.int32, device=self.device)
+        self.next_tokens = torch.zeros(max_batch, dtype=torch.int64, device=self.device)
+        self._graphs: dict[int, torch.cuda.CUDAGraph] = {}
+        self._graph_logits: dict[int, torch.Tensor] = {}
+
+    # ------------------------------------------------------------------ step
+    def _step_eager(self, B: int) -> None:
+        """One decode step over rows [0, B) of the static buffers; advances ctx_lens by one."""
+        h = self._decode_hidden(B)
+        if self.keep_logits:
+            self.last_logits = self._logits(h)
+        self._pick(h, self.next_tokens[:B])
+        self.ctx_lens[:B] += 1
+
+    GRAPH_BUCKETS = (1, 2, 4, 8, 16, 24, 32, 48, 64, 96, 128, 192, 256, 384, 512, 768, 1024)
+
+    def graph_batch(self, B: int) -> int:
+        """Rows the captured graph for a batch of B runs: B itself, or with a scratch page the next bucket, so
+        that a batch whose size changes with every admitted and finished request reuses a handful of graphs."""
+        if self.ep_state is not None:
+            if self.scratch_block is None and B != self.max_batch:
+                raise ValueError("this expert-parallel engine reads pools it does not own (no scratch page for "
+                                 "padding rows), so it can only step at its full batch")
+            return self.max_batch  # the exchange has one shape; fewer rows are padded up to it
+        if self.scratch_block is None:
+            return B
+        for b in self.GRAPH_BUCKETS:
+            if b >= B:
+                return min(b, self.max_batch)
+        return self.max_batch
+
+    def _pad_rows(self, lo: int, hi: int) -> None:
+        """Make rows [lo, hi) of the static state padding rows: token 0 at position 0 of a sequence whose only
+        page is the scratch page."""
+        if hi > lo:
+            self.tokens[lo:hi] = 0
+            self.ctx_lens[lo:hi] = 0
+            self.block_table[lo:hi, 0] = self.scratch_block
+
+    def _build_graph(self, B: int, pad_from: int | None = None) -> torch.cuda.CUDAGraph:
+        """Capture the step for B rows (two eager warm-up runs, then the capture).  `pad_from`: rows from
+        there on are set up as padding rows first."""
+        if pad_from is not None:
+            self._pad_rows(pad_from, B)
+            self.n_valid.fill_(pad_from)
+        saved = self.ctx_lens.clone()
+        stream = torch.cuda.Stream(device=self.device)
+        stream.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(stream):
+            for _ in range(2):  # warm-up: library handles, function attributes, tensor maps
+                self._step_eager(B)
+                # every warm-up run writes the K/V slot of the CURRENT position only (the one the real step
+                # will overwrite): a run that advanced could cross into a page the row does not own yet
+                self.ctx_lens.copy_(saved)
+        torch.cuda.current_stream().wait_stream(stream)
+        torch.cuda.synchronize()
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            self._step_eager(B)
+        self.ctx_lens.copy_(saved)  # warm-up and capture advanced nothing the caller asked for
+        torch.cuda.synchronize()
+        self._graphs[B] = g
+        if self.keep_logits:
+            self._graph_logits[B] = self.last_logits
+        return g
+
+    def step(self, B: int, joined: bool = False) -> torch.Tensor:
+        """Run one decode step for the first B rows of the static state; returns next tokens (device).
+        On an expert-parallel engine B may be anything from 0 (an idle rank keeping the exchange company) to
+        the full batch; `joined` says the caller has already agreed the round with the other ranks."""
+        lowest = 0 if self.ep_state is not None else 1
+        if B < lowest or B > self.max_batch:
+            raise ValueError(f"batch {B} outside [{lowest}, {self.max_batch}]")
+        if not self.use_graphs and self.ep_state is None:
+            self._step_eager(B)
+            return self.next_tokens[:B]
+        rows = self.graph_batch(B)
+        if self.ep_state is not None:
+            if self.round_hook is not None and not joined:
+                self.round_hook()
+            self.n_valid.fill_(B)
+        if rows > B:
+            # padding rows: reset every step because the graph advances their lengths like everyone's
+            self._pad_rows(B, rows)
+        real, B = B, rows
+        if not self.use_graphs:
+            self._step_eager(B)
+            return self.next_tokens[:real]
+        g = self._graphs.get(B)
+        if g is None:
+            g = self._build_graph(B)
+        g.replay()
+        if self.keep_logits:
+            self.last_logits = self._graph_logits[B]  # the buffer this graph writes
+        return self.next_tokens[:real]
+
+    def idle_pass(self) -> None:
+        """Expert parallelism: take part in one exchange round without any rows of one's own."""
+        self.step(0, joined=True)
+
+    # --------------------------------------------------------------- prefill
+    @torch.no_grad()
+    def prefill(self, token_ids: list[int], block_ids: list[int], cached_tokens: int = 0,
+                chunk: int | None = None, want: list[int] | None = None) -> tuple[int, torch.Tensor]:
+        """Prompt pass for one sequence; writes K/V of tokens [cached_tokens, n) into `block_ids` pages.
+
+        Runs in chunks of `chunk` prompt tokens through the same projection, glue and MoE kernels as decode
+        (every token of a chunk is a row with its own position); attention reads the sequence's pages in place,
+        cached prefix pages included - there is no dense gather of the KV as in the reference
+        (src/inference_server/kv_cache/hf_format.py:21-45).  The K/V of a whole chunk are written to their page
+        slots before the chunk's attention runs.  Attention is the tiled causal kernel
+        (b200_paged_attn_prefill: a page fetched once per 128 score rows); for head shapes it is not built for,
+        the decode kernel with one row per token (two rows per CTA: b200_paged_attn_decode_pairs), where
+        row i only looks at positions <= its own, which is the causal mask.
+        Under expert parallelism a chunk is one exchange round like a decode step: it is padded to the
+        exchange's fixed shape (the engine's full batch) with rows that route nowhere, and the other ranks spend
+        the round on a decode step, a chunk of their own or an idle pass.
+        Returns (first generated token, logits): the last position's, None unless the engine was built with keep_logits;
+        or, with `want`, a [len(want), vocab] tensor of the logits at those positions (at or after cached_tokens)."""
+        n = len(token_ids)
+        if n == 0 or cached_tokens >= n:
+            raise ValueError("prefill needs at least one uncached token")
+        if len(block_ids) * PAGE < n:
+            raise ValueError("not enough pages for the prompt")
+        if len(block_ids) > self.max_pages:
+            raise ValueError("sequence needs more pages than the block table is wide")
+        chunk = self._begin_prompt(chunk or self.prompt_chunk)
+        row = torch.zeros(self.max_pages, dtype=torch.int32)
+        row[: len(block_ids)] = torch.tensor(block_ids, dtype=torch.int32)
+        row = row.to(self.device)
+        h_last = None
+        if want and not all(cached_tokens <= p < n for p in want):
+            raise ValueError("logits can be asked for at the positions that are run")
+        wanted = None if want is None else torch.empty(len(want), self.vocab_size, dtype=self.logits_dtype, device=self.device)
+        for lo in range(cached_tokens, n, chunk):
+            hi = min(n, lo + chunk)
+            h = self._prompt_hidden(token_ids[lo:hi], row, lo, chunk)
+            here = [i for i, p in enumerate(want or ()) if lo <= p < hi]
+            if here:
+                logits = self._logits(h[torch.tensor([want[i] - lo for i in here], device=self.device)])
+                wanted[torch.tensor(here, device=self.device)] = logits
+            h_last = h[hi - lo - 1:hi - lo].contiguous()
+        first = self._pick(h_last)
+        if want is not None:
+            return int(first[0]), wanted
+        # the logits cost a second pass over lm_head: only for engines built to keep them (tests, debugging)
+        return int(first[0]), self._logits(h_last)[0] if self.keep_logits else None
+
+    @torch.no_grad()
+    def mixed_step(self, B: int, chunk_token_ids: list[int], block_ids: list[int], first_pos: int,
+                   want_first: bool = True) -> tuple[torch.Tensor, int | None, torch.Tensor | None]:
+        """One pass that is a decode step for rows [0, B) of the static state AND a prompt chunk of one other
+        sequence: its tokens `chunk_token_ids` sit at positions first_pos.. of the sequence whose pages are
+        `block_ids` (earlier positions already written).  The reference runs the two as separate forwards
+        (src/inference_server/scheduler.py:312-353 then :379-402) and names the merged form as the next step
+        (docs/arch-scheduler.html:269-270); merged, the projections' and the experts' weights are streamed once
+        for both, which is most of what a decode step costs.  The chunk's rows come first; every kernel but
+        attention treats the rows alike, and attention runs as the tiled causal kernel for the chunk and the
+        decode kernel for the rest.
+        Returns (next tokens of the B decode rows (device), token after the chunk's last position, its logits);
+        the last two are None unless `want_first` (the logits also unless the engine was built with keep_logits).
+        Advances ctx_lens of the decode rows by one."""
+        n = len(chunk_token_ids)
+        if self.ep_state is not None:
+            raise ValueError("mixed passes are not built for expert-parallel engines: run the chunk and the step as "
+                             "two rounds")
+        if n == 0 or B < 1 or B > self.max_batch:
+            raise ValueError(f"mixed pass needs a chunk and 1..{self.max_batch} decode rows (got {n} and {B})")
+        if len(block_ids) * PAGE < first_pos + n or len(block_ids) > self.max_pages:
+            raise ValueError("the chunk's sequence needs more pages than it was given or than the block table is wide")
+        row = torch.zeros(self.max_pages, dtype=torch.int32)
+        row[: len(block_ids)] = torch.tensor(block_ids, dtype=torch.int32)
+        row = row.to(self.device)
+        tokens = torch.cat([torch.tensor(chunk_token_ids, device=self.device), self.tokens[:B]])
+        pos = torch.cat([torch.arange(first_pos, first_pos + n, device=self.device, dtype=torch.int32), self.ctx_lens[:B]])
+        table = torch.cat([row.unsqueeze(0).expand(n, -1), self.block_table[:B]])
+        h = self._mixed_hidden(tokens, pos, table, first_pos, n, B)
+        first = logits = None
+        if want_first:
+            # the chunk's last row and the decode rows are neighbours: lm_head is streamed once for both
+            nxt = self._pick(h[n - 1:])
+            self.next_tokens[:B].copy_(nxt[1:])
+            first = int(nxt[0])
+        else:
+            self._pick(h[n:], self.next_tokens[:B])
+        if want_first and self.keep_logits:
+            logits = self._logits(h[n - 1:n])[0]
+        self.ctx_lens[:B] += 1
+        return self.next_tokens[:B], first, logits
+
+
+class DecodeEngine(PagedEngine):
+    """The Qwen3-MoE engine: owns weights, KV page pools and the per-batch-size CUDA graphs of the decode step."""
+
+    takes_reference_pools = True
+
+    def __init__(self, cfg: ModelConfig, num_blocks: int, max_batch: int, max_pages_per_seq: int,
+                 device: str | torch.device = "cuda", seed: int = 0, layers: list[LayerWeights] | None = None,
+                 embed: torch.Tensor | None = None, lm_head: torch.Tensor | None = None,
+                 final_norm: torch.Tensor | None = None, k_pools=None, v_pools=None, use_graphs: bool = True,
+                 split_tokens: int | None = None, ep_group=None, ep_capacity: int | None = None,
+                 ep_transport: str = "p2p", graph_buckets: bool = True, keep_logits: bool = False):
+        # Pools given from outside (a reference BlockManager's) have no scratch page; graphs are then captured per
+        # exact batch size, and an expert-parallel engine (whose exchange always runs at the full shape) can only
+        # step at its full batch.
+        own_pools = k_pools is None and v_pools is None
+        self._init_step_state(num_blocks, max_batch, max_pages_per_seq, device, use_graphs, keep_logits,
+                              own_pools and graph_buckets)
+        self.cfg = cfg
+        self.vocab_size = cfg.vocab_size
         bf = torch.bfloat16
         gen = torch.Generator(device=self.device).manual_seed(seed)
         # expert parallelism: this rank owns experts [rank * E / W, (rank + 1) * E / W) of every layer
@@ -176,12 +401,6 @@ class DecodeEngine:
         self.lm_head = lm_head if lm_head is not None else (
             torch.randn(cfg.vocab_size, cfg.hidden, device=self.device, generator=gen) * std).to(bf)
         self.final_norm = final_norm if final_norm is not None else torch.ones(cfg.hidden, device=self.device, dtype=bf)
-        # Pools the engine allocates itself get one block more than the caller may hand out: the scratch page
-        # that the padding rows of a bucketed CUDA graph write their K/V to (see step).  Pools given from outside
-        # (a reference BlockManager's) have no such page; graphs are then captured per exact batch size, and an
-        # expert-parallel engine (whose exchange always runs at the full shape) can only step at its full batch.
-        own_pools = k_pools is None and v_pools is None
-        self.scratch_block = num_blocks if (own_pools and graph_buckets) else None
         shape = (num_blocks + (1 if self.scratch_block is not None else 0), cfg.kv_heads, PAGE, cfg.head_dim)
         self.k_pools = k_pools if k_pools is not None else [torch.zeros(shape, device=self.device, dtype=bf) for _ in range(cfg.layers)]
         self.v_pools = v_pools if v_pools is not None else [torch.zeros(shape, device=self.device, dtype=bf) for _ in range(cfg.layers)]
@@ -190,11 +409,6 @@ class DecodeEngine:
         self._fixed_split = split_tokens
         self.split_tokens = split_tokens or ops.default_split_tokens(max_batch, cfg.kv_heads, max_pages_per_seq * PAGE)
 
-        # static step state (read by the captured graphs)
-        self.tokens = torch.zeros(max_batch, dtype=torch.int64, device=self.device)
-        self.ctx_lens = torch.zeros(max_batch, dtype=torch.int32, device=self.device)
-        self.block_table = torch.zeros(max_batch, max_pages_per_seq, dtype=torch.int32, device=self.device)
-        self.next_tokens = torch.zeros(max_batch, dtype=torch.int64, device=self.device)
         self.attn_ws = ops.paged_attn_workspace(max_batch, cfg.q_heads, cfg.head_dim, max_pages_per_seq, PAGE,
                                                 self.split_tokens, self.device)
         self.moe_ws = ops.moe_fp8_workspace(max_batch, cfg.experts, cfg.top_k, cfg.hidden, cfg.moe_inter, self.device)
@@ -204,7 +418,6 @@ class DecodeEngine:
         widest = max((cfg.q_heads + 2 * cfg.kv_heads) * cfg.head_dim, cfg.hidden, cfg.experts)
         self.gemm_ws = ops.dense_gemm_workspace(min(max_batch, 256), widest, self.device)  # K-split partial tiles
         self.argmax_ws = ops.lm_head_argmax_workspace(self.device)
-        self._graphs: dict[int, torch.cuda.CUDAGraph] = {}
         # rows of the current pass that are real (expert parallelism only): the router gives the rows beyond
         # it no expert, so they send nothing and receive nothing
         self.n_valid = torch.zeros(1, dtype=torch.int32, device=self.device)
@@ -235,7 +448,6 @@ class DecodeEngine:
         # Expert parallelism: every rank must run the same number of exchange passes.  `round_hook`, when set,
         # is called before every pass that has work (a decode step, a prompt chunk) and is where the ranks agree
         # that a round runs (ep.RoundGate); a rank without work answers with `idle_pass`.
-        self.round_hook = None
         if self.ep_state is not None and self.use_graphs and self.scratch_block is not None:
             # The exchange has one shape, so there is one graph; it is built here, where every rank is (its
             # warm-up runs are real exchanges and must happen on all ranks together), with padding rows only.
@@ -355,33 +567,6 @@ class DecodeEngine:
                                    f"{st.C} rows; the dropped (token, expert) pairs were left out of the result. "
                                    "Build the engine with a larger ep_capacity.")
 
-    def copy_kv_tokens(self, src: list[tuple[int, int]], dst: list[tuple[int, int]]) -> None:
-        """Copy the K/V of single tokens between page slots, in every layer: src[i] = (block, slot) ->
-        dst[i].  Used when a prefix-cache hit ends in, or runs through, a partially filled block: those tokens
-        are compacted into the row's own pages instead of being recomputed."""
-        if len(src) != len(dst):
-            raise ValueError("src and dst must list the same number of tokens")
-        if not src:
-            return
-        dev = self.k_pools[0].device
-        sb = torch.tensor([b for b, _ in src], device=dev)
-        ss = torch.tensor([s for _, s in src], device=dev)
-        db = torch.tensor([b for b, _ in dst], device=dev)
-        ds = torch.tensor([s for _, s in dst], device=dev)
-        for kp, vp in zip(self.k_pools, self.v_pools):
-            kp[db, :, ds, :] = kp[sb, :, ss, :]
-            vp[db, :, ds, :] = vp[sb, :, ss, :]
-
-    def _step_eager(self, B: int) -> None:
-        """One decode step over rows [0, B) of the static buffers; advances ctx_lens by one."""
-        split, attn_ws = self._attn_for(B)
-        h = self._forward(self.tokens[:B], self.ctx_lens[:B], self.block_table[:B], attn_ws, self.moe_ws,
-                          split, self.ep_state is not None)
-        if self.keep_logits:
-            self.last_logits = ops.dense_gemm(h, self.lm_head, status=self.gemm_status)
-        ops.lm_head_argmax(h, self.lm_head, self.argmax_ws, out=self.next_tokens[:B], status=self.gemm_status)
-        self.ctx_lens[:B] += 1
-
     def _ep_moe(self, h2, logits, w: LayerWeights, x, next_norm, B: int, routing=None) -> torch.Tensor:
         """Expert-parallel MoE layer: dispatch and combine around the local grouped GEMMs, by NCCL all-to-all
         or, with a peer arena, by stores into the other ranks' memory.  The exchange has one fixed shape (the
@@ -397,113 +582,19 @@ class DecodeEngine:
                                  lambda o, i: dist.all_to_all_single(o, i, group=st.group), residual=x,
                                  norm_weight=next_norm, eps=self.cfg.rms_eps, n_valid=self.n_valid, routing=routing)
 
-    GRAPH_BUCKETS = (1, 2, 4, 8, 16, 24, 32, 48, 64, 96, 128, 192, 256, 384, 512, 768, 1024)
+    # ----------------------------------------------------------------- hooks
+    def _decode_hidden(self, B: int) -> torch.Tensor:
+        split, attn_ws = self._attn_for(B)
+        return self._forward(self.tokens[:B], self.ctx_lens[:B], self.block_table[:B], attn_ws, self.moe_ws,
+                             split, self.ep_state is not None)
 
-    def graph_batch(self, B: int) -> int:
-        """Rows the captured graph for a batch of B runs: B itself, or with a scratch page the next bucket, so
-        that a batch whose size changes with every admitted and finished request reuses a handful of graphs."""
-        if self.ep_state is not None:
-            if self.scratch_block is None and B != self.max_batch:
-                raise ValueError("this expert-parallel engine reads pools it does not own (no scratch page for "
-                                 "padding rows), so it can only step at its full batch")
-            return self.max_batch  # the exchange has one shape; fewer rows are padded up to it
-        if self.scratch_block is None:
-            return B
-        for b in self.GRAPH_BUCKETS:
-            if b >= B:
-                return min(b, self.max_batch)
-        return self.max_batch
+    def _pick(self, h, out=None) -> torch.Tensor:
+        return ops.lm_head_argmax(h, self.lm_head, self.argmax_ws, out=out, status=self.gemm_status)
 
-    def _pad_rows(self, lo: int, hi: int) -> None:
-        """Make rows [lo, hi) of the static state padding rows: token 0 at position 0 of a sequence whose only
-        page is the scratch page."""
-        if hi > lo:
-            self.tokens[lo:hi] = 0
-            self.ctx_lens[lo:hi] = 0
-            self.block_table[lo:hi, 0] = self.scratch_block
+    def _logits(self, h) -> torch.Tensor:
+        return ops.dense_gemm(h, self.lm_head, status=self.gemm_status)
 
-    def _build_graph(self, B: int, pad_from: int | None = None) -> torch.cuda.CUDAGraph:
-        """Capture the step for B rows (two eager warm-up runs, then the capture).  `pad_from`: rows from
-        there on are set up as padding rows first."""
-        if pad_from is not None:
-            self._pad_rows(pad_from, B)
-            self.n_valid.fill_(pad_from)
-        saved = self.ctx_lens.clone()
-        stream = torch.cuda.Stream(device=self.device)
-        stream.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(stream):
-            for _ in range(2):  # warm-up: library handles, function attributes, tensor maps
-                self._step_eager(B)
-                # every warm-up run writes the K/V slot of the CURRENT position only (the one the real step
-                # will overwrite): a run that advanced could cross into a page the row does not own yet
-                self.ctx_lens.copy_(saved)
-        torch.cuda.current_stream().wait_stream(stream)
-        torch.cuda.synchronize()
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            self._step_eager(B)
-        self.ctx_lens.copy_(saved)  # warm-up and capture advanced nothing the caller asked for
-        torch.cuda.synchronize()
-        self._graphs[B] = g
-        return g
-
-    def step(self, B: int, joined: bool = False) -> torch.Tensor:
-        """Run one decode step for the first B rows of the static state; returns next tokens (device).
-        On an expert-parallel engine B may be anything from 0 (an idle rank keeping the exchange company) to
-        the full batch; `joined` says the caller has already agreed the round with the other ranks."""
-        lowest = 0 if self.ep_state is not None else 1
-        if B < lowest or B > self.max_batch:
-            raise ValueError(f"batch {B} outside [{lowest}, {self.max_batch}]")
-        if not self.use_graphs and self.ep_state is None:
-            self._step_eager(B)
-            return self.next_tokens[:B]
-        rows = self.graph_batch(B)
-        if self.ep_state is not None:
-            if self.round_hook is not None and not joined:
-                self.round_hook()
-            self.n_valid.fill_(B)
-        if rows > B:
-            # padding rows: reset every step because the graph advances their lengths like everyone's
-            self._pad_rows(B, rows)
-        real, B = B, rows
-        if not self.use_graphs:
-            self._step_eager(B)
-            return self.next_tokens[:real]
-        g = self._graphs.get(B)
-        if g is None:
-            g = self._build_graph(B)
-        g.replay()
-        return self.next_tokens[:real]
-
-    def idle_pass(self) -> None:
-        """Expert parallelism: take part in one exchange round without any rows of one's own."""
-        self.step(0, joined=True)
-
-    # --------------------------------------------------------------- prefill
-    @torch.no_grad()
-    def prefill(self, token_ids: list[int], block_ids: list[int], cached_tokens: int = 0,
-                chunk: int = 1024) -> tuple[int, torch.Tensor]:
-        """Prompt pass for one sequence; writes K/V of tokens [cached_tokens, n) into `block_ids` pages.
-
-        Runs in chunks of `chunk` prompt tokens through the same projection, glue and MoE kernels as decode
-        (every token of a chunk is a row with its own position); attention reads the sequence's pages in place,
-        cached prefix pages included - there is no dense gather of the KV as in the reference
-        (src/inference_server/kv_cache/hf_format.py:21-45).  The K/V of a whole chunk are written to their page
-        slots before the chunk's attention runs.  Attention is the tiled causal kernel
-        (b200_paged_attn_prefill: a page fetched once per 128 score rows); for head shapes it is not built for,
-        the decode kernel with one row per token (two rows per CTA: b200_paged_attn_decode_pairs), where
-        row i only looks at positions <= its own, which is the causal mask.
-        Under expert parallelism a chunk is one exchange round like a decode step: it is padded to the
-        exchange's fixed shape (the engine's full batch) with rows that route nowhere, and the other ranks spend
-        the round on a decode step, a chunk of their own or an idle pass.
-        Returns (first generated token, last-position logits - None unless the engine was built with keep_logits)."""
-        n = len(token_ids)
-        if n == 0 or cached_tokens >= n:
-            raise ValueError("prefill needs at least one uncached token")
-        if len(block_ids) * PAGE < n:
-            raise ValueError("not enough pages for the prompt")
-        if len(block_ids) > self.max_pages:
-            raise ValueError("sequence needs more pages than the block table is wide")
+    def _begin_prompt(self, chunk: int) -> int:
         ep = self.ep_state is not None
         if ep:
             if self.scratch_block is None:
@@ -523,57 +614,31 @@ class DecodeEngine:
             self._prefill_moe_ws = None if ep else ops.moe_fp8_workspace(chunk, cfg.experts, cfg.top_k, cfg.hidden,
                                                                          cfg.moe_inter, self.device)
         # consecutive prompt tokens share the table, so the row-per-token form takes them two rows per CTA where it can
-        pairs = not tiled and ops.paged_attn_pairs_supported(cfg.q_heads, cfg.kv_heads, cfg.head_dim, PAGE, torch.bfloat16)
-        row = torch.zeros(self.max_pages, dtype=torch.int32)
-        row[: len(block_ids)] = torch.tensor(block_ids, dtype=torch.int32)
-        row = row.to(self.device)
-        h_last = None
-        for lo in range(cached_tokens, n, chunk):
-            hi = min(n, lo + chunk)
-            tokens = torch.tensor(token_ids[lo:hi], device=self.device)
-            pos = torch.arange(lo, hi, device=self.device, dtype=torch.int32)
-            table = row.unsqueeze(0).expand(hi - lo, -1).contiguous()
-            if ep:
-                pad = chunk - (hi - lo)
-                if pad:
-                    tokens = torch.cat([tokens, tokens.new_zeros(pad)])
-                    pos = torch.cat([pos, pos.new_zeros(pad)])
-                    scratch = torch.zeros(pad, self.max_pages, dtype=torch.int32, device=self.device)
-                    scratch[:, 0] = self.scratch_block
-                    table = torch.cat([table, scratch])
-                if self.round_hook is not None:
-                    self.round_hook()
-                self.n_valid.fill_(hi - lo)
-            h = self._forward(tokens, pos, table, self._prefill_attn_ws, self._prefill_moe_ws, self._prefill_split,
-                              ep, pairs=pairs, chunk_of=(lo, hi - lo) if tiled else None)
-            h_last = h[hi - lo - 1:hi - lo].contiguous()
-        first = ops.lm_head_argmax(h_last, self.lm_head, self.argmax_ws, status=self.gemm_status)
-        # the logits cost a second pass over lm_head: only for engines built to keep them (tests, debugging)
-        logits = ops.dense_gemm(h_last, self.lm_head, status=self.gemm_status)[0] if self.keep_logits else None
-        return int(first[0]), logits
+        self._prefill_tiled = tiled
+        self._prefill_pairs = not tiled and ops.paged_attn_pairs_supported(cfg.q_heads, cfg.kv_heads, cfg.head_dim, PAGE, torch.bfloat16)
+        return chunk
 
-    @torch.no_grad()
-    def mixed_step(self, B: int, chunk_token_ids: list[int], block_ids: list[int], first_pos: int,
-                   want_first: bool = True) -> tuple[torch.Tensor, int | None, torch.Tensor | None]:
-        """One pass that is a decode step for rows [0, B) of the static state AND a prompt chunk of one other
-        sequence: its tokens `chunk_token_ids` sit at positions first_pos.. of the sequence whose pages are
-        `block_ids` (earlier positions already written).  The reference runs the two as separate forwards
-        (src/inference_server/scheduler.py:312-353 then :379-402) and names the merged form as the next step
-        (docs/arch-scheduler.html:269-270); merged, the projections' and the experts' weights are streamed once
-        for both, which is most of what a decode step costs.  The chunk's rows come first; every kernel but
-        attention treats the rows alike, and attention runs as the tiled causal kernel for the chunk and the
-        decode kernel for the rest.
-        Returns (next tokens of the B decode rows (device), token after the chunk's last position, its logits);
-        the last two are None unless `want_first` (the logits also unless the engine was built with keep_logits).
-        Advances ctx_lens of the decode rows by one."""
-        n = len(chunk_token_ids)
-        if self.ep_state is not None:
-            raise ValueError("mixed passes are not built for expert-parallel engines: run the chunk and the step as "
-                             "two rounds")
-        if n == 0 or B < 1 or B > self.max_batch:
-            raise ValueError(f"mixed pass needs a chunk and 1..{self.max_batch} decode rows (got {n} and {B})")
-        if len(block_ids) * PAGE < first_pos + n or len(block_ids) > self.max_pages:
-            raise ValueError("the chunk's sequence needs more pages than it was given or than the block table is wide")
+    def _prompt_hidden(self, token_ids: list[int], row: torch.Tensor, lo: int, chunk: int) -> torch.Tensor:
+        hi = lo + len(token_ids)
+        ep = self.ep_state is not None
+        tokens = torch.tensor(token_ids, device=self.device)
+        pos = torch.arange(lo, hi, device=self.device, dtype=torch.int32)
+        table = row.unsqueeze(0).expand(hi - lo, -1).contiguous()
+        if ep:
+            pad = chunk - (hi - lo)
+            if pad:
+                tokens = torch.cat([tokens, tokens.new_zeros(pad)])
+                pos = torch.cat([pos, pos.new_zeros(pad)])
+                scratch = torch.zeros(pad, self.max_pages, dtype=torch.int32, device=self.device)
+                scratch[:, 0] = self.scratch_block
+                table = torch.cat([table, scratch])
+            if self.round_hook is not None:
+                self.round_hook()
+            self.n_valid.fill_(hi - lo)
+        return self._forward(tokens, pos, table, self._prefill_attn_ws, self._prefill_moe_ws, self._prefill_split,
+                          ep, pairs=self._prefill_pairs, chunk_of=(lo, hi - lo) if self._prefill_tiled else None)
+
+    def _mixed_hidden(self, tokens, pos, table, first_pos: int, n: int, B: int) -> torch.Tensor:
         cfg = self.cfg
         if not ops.paged_attn_prefill_supported(cfg.q_heads, cfg.kv_heads, cfg.head_dim, PAGE, torch.bfloat16):
             raise ValueError("mixed passes need the tiled prompt-attention kernel, which is not built for this head shape")
@@ -583,26 +648,25 @@ class DecodeEngine:
             self._mixed_moe_ws = ops.moe_fp8_workspace(self._mixed_rows, cfg.experts, cfg.top_k, cfg.hidden,
                                                        cfg.moe_inter, self.device)
             self._mixed_attn_ws = torch.zeros(256, dtype=torch.uint8, device=self.device)  # status word only
-        row = torch.zeros(self.max_pages, dtype=torch.int32)
-        row[: len(block_ids)] = torch.tensor(block_ids, dtype=torch.int32)
-        row = row.to(self.device)
-        tokens = torch.cat([torch.tensor(chunk_token_ids, device=self.device), self.tokens[:B]])
-        pos = torch.cat([torch.arange(first_pos, first_pos + n, device=self.device, dtype=torch.int32), self.ctx_lens[:B]])
-        table = torch.cat([row.unsqueeze(0).expand(n, -1), self.block_table[:B]])
-        h = self._forward(tokens, pos, table, self._mixed_attn_ws, self._mixed_moe_ws, 0, False, chunk_of=(first_pos, n),
-                          decode_attn=self._attn_for(B))
-        first = logits = None
-        if want_first:
-            # the chunk's last row and the decode rows are neighbours: lm_head is streamed once for both
-            nxt = ops.lm_head_argmax(h[n - 1:], self.lm_head, self.argmax_ws, status=self.gemm_status)
-            self.next_tokens[:B].copy_(nxt[1:])
-            first = int(nxt[0])
-        else:
-            ops.lm_head_argmax(h[n:], self.lm_head, self.argmax_ws, out=self.next_tokens[:B], status=self.gemm_status)
-        if want_first and self.keep_logits:
-            logits = ops.dense_gemm(h[n - 1:n], self.lm_head, status=self.gemm_status)[0]
-        self.ctx_lens[:B] += 1
-        return self.next_tokens[:B], first, logits
+        return self._forward(tokens, pos, table, self._mixed_attn_ws, self._mixed_moe_ws, 0, False, chunk_of=(first_pos, n),
+                             decode_attn=self._attn_for(B))
+
+    def copy_kv_tokens(self, src: list[tuple[int, int]], dst: list[tuple[int, int]]) -> None:
+        """Copy the K/V of single tokens between page slots, in every layer: src[i] = (block, slot) ->
+        dst[i].  Used when a prefix-cache hit ends in, or runs through, a partially filled block: those tokens
+        are compacted into the row's own pages instead of being recomputed."""
+        if len(src) != len(dst):
+            raise ValueError("src and dst must list the same number of tokens")
+        if not src:
+            return
+        dev = self.k_pools[0].device
+        sb = torch.tensor([b for b, _ in src], device=dev)
+        ss = torch.tensor([s for _, s in src], device=dev)
+        db = torch.tensor([b for b, _ in dst], device=dev)
+        ds = torch.tensor([s for _, s in dst], device=dev)
+        for kp, vp in zip(self.k_pools, self.v_pools):
+            kp[db, :, ds, :] = kp[sb, :, ss, :]
+            vp[db, :, ds, :] = vp[sb, :, ss, :]
 
     # ------------------------------------------------------------- accounting
     def weight_bytes_per_step(self, experts_hit_per_layer: float | None = None) -> dict:
