@@ -101,15 +101,15 @@ class B200Backend:
     # ------------------------------------------------------------ lifecycle
     def set_cache_adapter(self, adapter) -> None:
         """Attach a reference CacheManager (base.py:16-18) and adopt its pools when they fit."""
-        self.cache_adapter = adapter
         bm = getattr(adapter, "block_manager", None)
         eng = self.engine
-        if bm is None or eng is None or not getattr(bm, "k_pools", None):
-            return
-        if not getattr(eng, "takes_reference_pools", True):
+        if adapter is not None and eng is not None and not getattr(eng, "takes_reference_pools", True):
             # its layers keep other state than K/V pairs of one shape (latents, convolution history), which the
             # manager neither stores nor finds again
             raise ValueError("this model's cache does not fit a reference CacheManager's K/V pools; serve it without one")
+        self.cache_adapter = adapter
+        if bm is None or eng is None or not getattr(bm, "k_pools", None):
+            return
         want = (eng.cfg.kv_heads, PAGE, eng.cfg.head_dim)
         ok = (len(bm.k_pools) == eng.cfg.layers and all(
             tuple(p.shape[1:]) == want and p.dtype == torch.bfloat16 and p.device.type == torch.device(eng.device).type
