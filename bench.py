@@ -509,7 +509,9 @@ def main():
     ap.add_argument("--steps", type=int, default=32)
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--model", default="qwen3-30b-a3b")
+    ap.add_argument("--model", default="qwen3-30b-a3b",
+                    help="a built-in shape; a layer-list shape (sulepel-2048, sulepel-4096) measures decode, prefill and "
+                         "every kernel beside Qwen3-MoE of the same size (bench_layered.py)")
     ap.add_argument("--batch", type=int, default=256, help="concurrent sequences per GPU")
     ap.add_argument("--gen-tokens", type=int, default=256)
     ap.add_argument("--ctx-min", type=int, default=512, help="shortest prompt (tokens)")
@@ -538,6 +540,13 @@ def main():
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
+    if args.model not in pkg("engine").CONFIGS and args.model in pkg("layered").CONFIGS:
+        # a layer-list decoder: decode, prefill and every kernel beside the closest other model, one GPU
+        if world > 1 or args.impl != "b200":
+            raise SystemExit(f"--model {args.model} measures this build on one GPU")
+        import bench_layered
+        bench_layered.run(args, build_workload, ClockSampler)
+        return
     cfg = pkg("engine").CONFIGS[args.model]
     balance = world > 1 and args.ep and not args.no_balance
     prompt_lens, table, num_blocks, max_pages = build_workload(cfg, args.batch, args.gen_tokens, seed=rank,

@@ -379,23 +379,30 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           uint32_t v[32];
           tmem_ld32(t0 + c * 32, v);
           tmem_ld_wait();
+          const int left = p.M - (m0 + c * 32);  // rows of this chunk that exist
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const int m = m0 + c * 32 + i;
-            const int page = __shfl_sync(0xffffffffu, row_page4[cc], i), slot = __shfl_sync(0xffffffffu, row_slot4[cc], i);
-            const float f = __uint_as_float(v[i]) * seg_scale;
-            if (m < p.M) {
-              if (seg_kind == kSegPages) {
-                if (page >= 0)
-                  static_cast<__nv_bfloat16*>(seg_ptr)[static_cast<size_t>(page) * seg_page_stride + slot * seg_dim] =
-                      __float2bfloat16(f);
-              } else if (seg_kind == kSegBf16) {
-                static_cast<__nv_bfloat16*>(seg_ptr)[static_cast<size_t>(m) * seg_ld] = __float2bfloat16(f);
-              } else if (seg_kind == kSegF32) {
-                static_cast<float*>(seg_ptr)[static_cast<size_t>(m) * seg_ld] = f;
-              }
+          for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * seg_scale);
+          if (__any_sync(0xffffffffu, seg_kind == kSegPages)) {
+            __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(seg_ptr);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const int page = __shfl_sync(0xffffffffu, row_page4[cc], i), slot = __shfl_sync(0xffffffffu, row_slot4[cc], i);
+              if (seg_kind == kSegPages && page >= 0 && i < left)
+                dst[static_cast<size_t>(page) * seg_page_stride + slot * seg_dim] = __float2bfloat16(__uint_as_float(v[i]));
             }
           }
+          if (seg_kind == kSegBf16) {
+            __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(seg_ptr) + static_cast<size_t>(m0 + c * 32) * seg_ld;
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (i < left) dst[static_cast<size_t>(i) * seg_ld] = __float2bfloat16(__uint_as_float(v[i]));
+          } else if (seg_kind == kSegF32) {
+            float* dst = static_cast<float*>(seg_ptr) + static_cast<size_t>(m0 + c * 32) * seg_ld;
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (i < left) dst[static_cast<size_t>(i) * seg_ld] = __uint_as_float(v[i]);
+          }
+          __syncwarp();
         }
       } else if (EPI == kEpiGlu) {
         const int n = nt * 128 + t;

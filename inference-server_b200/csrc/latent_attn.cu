@@ -10,20 +10,23 @@
 //
 // A page [16, rank] is fetched once for all heads and serves as K and as V: rank * 2 bytes per token.
 //
-//   grid     (batch, splits, head groups of 16 * MT)
-//   load     tiles of 64 tokens by TMA (4 pages x NW boxes of 16 tokens x 128 B, 128-byte swizzle, one box per lane of
-//            warp 0) into a ring of stages; a stage is refilled right after the barrier that every warp reaches only when
-//            it is done with the tile before, so no "empty" barriers and no producer warp are needed (a ninth warp
-//            would cut the registers of the other eight from 255 to 168)
-//   warps 0..NW-1 (NW = rank / 64)
-//     scores     the 8 groups of 8 tokens of a tile are dealt to the warps; S[heads x 8 tokens] over the whole rank by
-//                mma.sync m16n8k16.  The projected queries stay in registers, or in shared memory where they do not fit.
-//     softmax    row maxima meet in shared memory (barrier), exponentials in fp32 against the common running maximum,
-//                P in bf16 to shared memory (barrier)
-//     values     warp w owns columns [64 w, 64 w + 64) of the output: O += P C over the tile's 64 tokens
+//   grid     (batch x head groups of 16 * MT, splits): the head groups of a row are neighbours, so the second finds the
+//            row's pages in L2
+//   load     tiles of tokens by TMA (boxes of 16 tokens x 128 B, 128-byte swizzle, one box per lane of warp 0) into a ring
+//            of stages; a stage is refilled right after the barrier that every warp reaches only when it is done with the
+//            tile before, so no "empty" barriers and no producer warp are needed
+//   scores   the groups of 8 tokens of a tile are dealt to the warps; S[heads x 8 tokens] over the whole rank by mma.sync
+//            m16n8k16.  The projected queries stay in registers, or in shared memory where they do not fit.
+//   softmax  exponentials in fp32 against the common running maximum; the warps' row maxima meet in shared memory, P in
+//            bf16 goes to shared memory
+//   values   warp w owns rank / warps columns of the output: O += P C over the tile's tokens
+//   None of the units is near its limit here - what costs is the chain score -> maximum -> exponential -> value with two
+//   barriers per tile -, so two CTAs of four warps share an SM where registers and shared memory allow.  (A loop skewed by
+//   one tile, with the next tile's scores ahead of a single barrier, was slower: it needs every tile one step earlier, and
+//   the ring is only three tiles deep.)
 //   out      as in paged_attn.cu: bf16 straight from registers when the row fits one split, else fp32 partials that
 //            a second kernel folds in split order.
-// HBM-bound for up to 16 heads; every wait is bounded.
+// Every wait is bounded.
 
 #include "common.cuh"
 #include "host.h"
@@ -31,45 +34,50 @@
 namespace b200 {
 
 constexpr int kLatPage = 16;
-constexpr int kLatTile = 64;                   // tokens per pipeline stage
-constexpr int kLatPages = kLatTile / kLatPage;
-constexpr int kLatHalf = kLatTile * 128;       // 64 tokens x 64 latent columns
 
-template <int NW, int MT>
+// R: rank.  MT: head tiles of 16 per CTA.  WARPS: each owns R / WARPS columns of the output.  TILE: tokens per pipeline
+// stage.  CTAS: CTAs per SM aimed for.
+template <int R_, int MT_, int WARPS_, int TILE_, int STAGES_, int CTAS_>
 struct LatentCfg {
-  static constexpr bool kQRegs = NW * MT <= 8;
-  static constexpr int kStageBytes = NW * kLatHalf;
-  static constexpr int kStages = NW <= 2 ? 4 : (NW * MT > 12 ? 2 : 3);
-  static constexpr int kCtas = NW <= 2 ? 3 : (NW <= 4 ? 2 : 1);
-  static constexpr int kQBytes = kQRegs ? 0 : MT * 16 * NW * 128;
+  static constexpr int R = R_, MT = MT_, kWarps = WARPS_, kTile = TILE_, kStages = STAGES_, kCtas = CTAS_;
+  static constexpr int kPages = kTile / kLatPage;
+  static constexpr int kHalf = kTile * 128;  // 64 columns of a tile
+  static constexpr int kHalves = R / 64;
+  static constexpr bool kQRegs = R * MT <= 512;
+  static constexpr int kStageBytes = kHalves * kHalf;
+  static constexpr int kQBytes = kQRegs ? 0 : MT * 16 * R * 2;
   static constexpr int kPBytes = MT * 16 * 128;
-  static constexpr int kRedBytes = NW * MT * 16 * 4;
+  static constexpr int kRedBytes = kWarps * MT * 16 * 4;
   static constexpr int kSmemBytes = 1024 + kStages * kStageBytes + kQBytes + kPBytes + kRedBytes + 8 * kStages;
-  static constexpr int kThreads = NW * 32;
+  static constexpr int kThreads = kWarps * 32;
+  static_assert(kPages * kHalves <= 32, "one TMA box per lane");
+  static_assert(!kQRegs || MT * 16 * R * 2 <= kStageBytes, "the queries pass through the last stage");
+
+  static_assert(kTile <= 64 && kTile % 16 == 0 && R % (kWarps * 16) == 0, "tile shape");
 };
 
-template <int NW, int MT>
-__global__ void __launch_bounds__(NW * 32, LatentCfg<NW, MT>::kCtas)
+template <class Cfg>
+__global__ void __launch_bounds__(Cfg::kThreads, Cfg::kCtas)
 latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_bfloat16* __restrict__ q,
                           const int* __restrict__ block_table, const int* __restrict__ ctx_lens,
                           float* __restrict__ part_o, float2* __restrict__ part_ml, __nv_bfloat16* __restrict__ out,
                           int* __restrict__ err, int heads, int num_blocks, int max_pages, int split_tokens,
-                          int max_splits, float scale_log2, const float* __restrict__ gate) {
+                          int max_splits, float scale_log2, const float* __restrict__ gate, int head_groups) {
 #ifdef B200_DEVICE_OK
   grid_dep_wait();
   grid_dep_launch();
-  using Cfg = LatentCfg<NW, MT>;
-  constexpr int R = NW * 64, STAGES = Cfg::kStages;
+  constexpr int R = Cfg::R, MT = Cfg::MT, NW = Cfg::kWarps, STAGES = Cfg::kStages;
+  constexpr int kLatTile = Cfg::kTile, kLatHalf = Cfg::kHalf, kLatPages = Cfg::kPages, kHalves = Cfg::kHalves;
+  constexpr int kCols = R / NW, kNt = kCols / 8;  // output columns of a warp, n tiles of 8
   extern __shared__ uint8_t smem_raw[];
   const uint32_t ring = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* base_ptr = smem_raw + (ring - smem_u32(smem_raw));
-  const uint32_t q_sm = ring + STAGES * Cfg::kStageBytes;
-  const uint32_t p_sm = q_sm + Cfg::kQBytes;
+  const uint32_t p_sm = ring + STAGES * Cfg::kStageBytes + Cfg::kQBytes;
   uint8_t* p_ptr = base_ptr + STAGES * Cfg::kStageBytes + Cfg::kQBytes;
   float* red = reinterpret_cast<float*>(p_ptr + Cfg::kPBytes);  // [NW][MT * 16]
   const uint32_t bars = p_sm + Cfg::kPBytes + Cfg::kRedBytes;   // full[STAGES]
 
-  const int b = blockIdx.x, split = blockIdx.y, h0 = blockIdx.z * (16 * MT);
+  const int b = blockIdx.x / head_groups, split = blockIdx.y, h0 = (blockIdx.x - b * head_groups) * (16 * MT);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   int L = ctx_lens[b];
   if (L < 0 || L > max_pages * kLatPage) {
@@ -92,14 +100,15 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
     fence_mbar_init();
     fence_proxy_async();
   }
-  if (!Cfg::kQRegs) {  // projected queries to shared memory, [64-column half][head][128 B] swizzled
-    for (int i = threadIdx.x; i < MT * 16 * (R / 8); i += blockDim.x) {
-      const int row = i / (R / 8), ch = i % (R / 8);
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (h0 + row < heads)
-        v = *reinterpret_cast<const uint4*>(q + (static_cast<size_t>(b) * heads + h0 + row) * R + ch * 8);
-      *reinterpret_cast<uint4*>(base_ptr + STAGES * Cfg::kStageBytes + (ch >> 3) * (MT * 16 * 128) + swz128(row, ch & 7)) = v;
-    }
+  // projected queries to shared memory, [64-column half][head][128 B] swizzled: to stay there, or on their way to registers
+  // in the last stage, which the first tiles do not use
+  constexpr uint32_t kQOff = Cfg::kQRegs ? (STAGES - 1) * Cfg::kStageBytes : STAGES * Cfg::kStageBytes;
+  for (int i = threadIdx.x; i < MT * 16 * (R / 8); i += blockDim.x) {
+    const int row = i / (R / 8), ch = i % (R / 8);
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (h0 + row < heads)
+      v = *reinterpret_cast<const uint4*>(q + (static_cast<size_t>(b) * heads + h0 + row) * R + ch * 8);
+    *reinterpret_cast<uint4*>(base_ptr + kQOff + (ch >> 3) * (MT * 16 * 128) + swz128(row, ch & 7)) = v;
   }
   __syncthreads();
 
@@ -107,8 +116,8 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
   // Lane of warp 0 -> one box of a tile.  The page id of the next tile to load is fetched one step ahead.  Pages past the
   // split's end hold nothing that may be read; the last valid page stands in (its scores are masked).
   const int* table_row = block_table + static_cast<size_t>(b) * max_pages;
-  const int pg = lane / NW, half = lane % NW;
-  const bool issuer = warp == 0 && lane < kLatPages * NW;
+  const int pg = lane / kHalves, half = lane % kHalves;
+  const bool issuer = warp == 0 && lane < kLatPages * kHalves;
   int next_id = 0;
   auto fetch_id = [&](int tile) {
     if (issuer) next_id = table_row[min(first_page + tile * kLatPages + pg, last_page)];
@@ -138,55 +147,50 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
   const int gq = lane >> 2, tq = lane & 3, lj = lane >> 3, lr = lane & 7;
   const int v_tok = (lj & 1) * 8 + lr, v_sub = lj >> 1;
   uint32_t qa[Cfg::kQRegs ? MT : 1][Cfg::kQRegs ? R / 16 : 1][4];
+  auto q_frag = [&](int mt, int ks, uint32_t (&a)[4]) {
+    const int c = ks * 2 + (lj >> 1);
+    ldmatrix_x4(ring + kQOff + (c >> 3) * (MT * 16 * 128) + swz128(mt * 16 + (lj & 1) * 8 + lr, c & 7), a[0], a[1], a[2], a[3]);
+  };
   if (Cfg::kQRegs) {
 #pragma unroll
-    for (int mt = 0; mt < (Cfg::kQRegs ? MT : 1); ++mt) {
-      const int ha = h0 + mt * 16 + gq;
-      const __nv_bfloat16* r0 = q + (static_cast<size_t>(b) * heads + ha) * R + 2 * tq;
+    for (int mt = 0; mt < (Cfg::kQRegs ? MT : 1); ++mt)
 #pragma unroll
-      for (int ks = 0; ks < (Cfg::kQRegs ? R / 16 : 1); ++ks) {
-        const uint32_t* a0 = reinterpret_cast<const uint32_t*>(r0 + ks * 16);
-        const uint32_t* a1 = reinterpret_cast<const uint32_t*>(r0 + 8 * R + ks * 16);
-        qa[mt][ks][0] = ha < heads ? __ldg(a0) : 0u;
-        qa[mt][ks][1] = ha + 8 < heads ? __ldg(a1) : 0u;
-        qa[mt][ks][2] = ha < heads ? __ldg(a0 + 4) : 0u;
-        qa[mt][ks][3] = ha + 8 < heads ? __ldg(a1 + 4) : 0u;
-      }
-    }
+      for (int ks = 0; ks < (Cfg::kQRegs ? R / 16 : 1); ++ks) q_frag(mt, ks, qa[mt][ks]);
+    fence_proxy_async();  // read before the copies that will refill the stage (ordered by the loop's first barrier)
   }
-  float o[MT][8][4];
+  float o[MT][kNt][4];
   float m_run[MT][2], l_run[MT][2];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
-    for (int n = 0; n < 8; ++n) o[mt][n][0] = o[mt][n][1] = o[mt][n][2] = o[mt][n][3] = 0.f;
+    for (int n = 0; n < kNt; ++n) o[mt][n][0] = o[mt][n][1] = o[mt][n][2] = o[mt][n][3] = 0.f;
     m_run[mt][0] = m_run[mt][1] = -INFINITY;
     l_run[mt][0] = l_run[mt][1] = 0.f;
   }
-  constexpr int kMine = (8 + NW - 1) / NW;  // groups of 8 tokens per warp (some warps may have one less)
+  constexpr int kGroups = kLatTile / 8;                  // groups of 8 tokens, dealt to the warps
+  constexpr int kMine = (kGroups + NW - 1) / NW;         // per warp (some warps may have one less)
+  constexpr int kChains = MT == 1 && R % 64 == 0 ? 4 : 2;  // independent accumulators: short chains of dependent MMAs
   bool alive = true;
-#pragma unroll 1
-  for (int i = 0; i < n_tiles; ++i) {
-    const int slot = i % STAGES;
-    const uint32_t phase = (i / STAGES) & 1;
-    if (alive) alive = mbar_wait(bars + 8 * slot, phase, err);
-    const uint32_t cbase = ring + slot * Cfg::kStageBytes;
-    const int left = end - (start + i * kLatTile);  // tokens of this tile that exist
-
-    float s[kMine][MT][4];
+  float s[kMine][MT][4];
+  auto wait_tile = [&](int t) {
+    if (alive) alive = mbar_wait(bars + 8 * (t % STAGES), (t / STAGES) & 1, err);
+  };
+  // scores of tile t into s (log2 domain), this warp's row maxima to shared memory
+  auto score = [&](int t) {
+    const uint32_t cbase = ring + (t % STAGES) * Cfg::kStageBytes;
+    const int left = end - (start + t * kLatTile);  // tokens of the tile that exist
     float mx[MT][2];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) mx[mt][0] = mx[mt][1] = -INFINITY;
 #pragma unroll
     for (int g = 0; g < kMine; ++g) {
       const int n8 = warp + g * NW;
-      // two independent accumulators per tile keep the chain of dependent MMAs short
-      float acc[2][MT][4];
+      float acc[kChains][MT][4];
 #pragma unroll
-      for (int e = 0; e < 2; ++e)
+      for (int e = 0; e < kChains; ++e)
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) acc[e][mt][0] = acc[e][mt][1] = acc[e][mt][2] = acc[e][mt][3] = 0.f;
-      if (n8 < 8) {
+      if (n8 < kGroups) {
 #pragma unroll
         for (int kk = 0; kk < R / 32; ++kk) {  // 32 latent columns: two k steps
           uint32_t b0, b1, b2, b3;
@@ -195,16 +199,14 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
 #pragma unroll
           for (int mt = 0; mt < MT; ++mt) {
             if (Cfg::kQRegs) {
-              mma_bf16_16816(acc[0][mt], qa[Cfg::kQRegs ? mt : 0][Cfg::kQRegs ? 2 * kk : 0], b0, b1);
-              mma_bf16_16816(acc[1][mt], qa[Cfg::kQRegs ? mt : 0][Cfg::kQRegs ? 2 * kk + 1 : 0], b2, b3);
+              mma_bf16_16816(acc[(2 * kk) % kChains][mt], qa[Cfg::kQRegs ? mt : 0][Cfg::kQRegs ? 2 * kk : 0], b0, b1);
+              mma_bf16_16816(acc[(2 * kk + 1) % kChains][mt], qa[Cfg::kQRegs ? mt : 0][Cfg::kQRegs ? 2 * kk + 1 : 0], b2, b3);
             } else {
-              const int qr = mt * 16 + (lj & 1) * 8 + lr;
               uint32_t a[4], a2[4];
-              const int c0 = kk * 4 + (lj >> 1), c1 = c0 + 2;
-              ldmatrix_x4(q_sm + (c0 >> 3) * (MT * 16 * 128) + swz128(qr, c0 & 7), a[0], a[1], a[2], a[3]);
-              ldmatrix_x4(q_sm + (c1 >> 3) * (MT * 16 * 128) + swz128(qr, c1 & 7), a2[0], a2[1], a2[2], a2[3]);
-              mma_bf16_16816(acc[0][mt], a, b0, b1);
-              mma_bf16_16816(acc[1][mt], a2, b2, b3);
+              q_frag(mt, 2 * kk, a);
+              q_frag(mt, 2 * kk + 1, a2);
+              mma_bf16_16816(acc[(2 * kk) % kChains][mt], a, b0, b1);
+              mma_bf16_16816(acc[(2 * kk + 1) % kChains][mt], a2, b2, b3);
             }
           }
         }
@@ -214,13 +216,16 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
       for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const bool seen = n8 < 8 && tok + (e & 1) < left;
-          s[g][mt][e] = seen ? (acc[0][mt][e] + acc[1][mt][e]) * scale_log2 : -INFINITY;
+          const bool seen = n8 < kGroups && tok + (e & 1) < left;
+          float sum = acc[0][mt][e] + acc[1][mt][e];
+          if (kChains == 4) sum += acc[kChains - 2][mt][e] + acc[kChains - 1][mt][e];
+          s[g][mt][e] = seen ? sum * scale_log2 : -INFINITY;
         }
         mx[mt][0] = fmaxf(mx[mt][0], fmaxf(s[g][mt][0], s[g][mt][1]));
         mx[mt][1] = fmaxf(mx[mt][1], fmaxf(s[g][mt][2], s[g][mt][3]));
       }
     }
+    float* mine = red + warp * (MT * 16);
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -228,14 +233,20 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
         float v = mx[mt][hf];
         v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 1));
         v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 2));
-        if (tq == 0) red[warp * (MT * 16) + mt * 16 + hf * 8 + gq] = v;
+        if (tq == 0) mine[mt * 16 + hf * 8 + gq] = v;
       }
+  };
+#pragma unroll 1
+  for (int i = 0; i < n_tiles; ++i) {
+    wait_tile(i);
+    score(i);
     // every warp's maxima are written, and every warp is done with the P and the latents of the tile before
     __syncthreads();
     if (warp == 0 && i + STAGES - 1 < n_tiles) {
       load_tile(i + STAGES - 1);
       fetch_id(i + STAGES);
     }
+    const uint32_t cbase = ring + (i % STAGES) * Cfg::kStageBytes;
     float alpha[MT][2];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
@@ -251,7 +262,7 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
 #pragma unroll
     for (int g = 0; g < kMine; ++g) {
       const int n8 = warp + g * NW;
-      if (n8 < 8) {
+      if (n8 < kGroups) {
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -270,7 +281,7 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-        for (int n = 0; n < 8; ++n) {
+        for (int n = 0; n < kNt; ++n) {
           o[mt][n][0] *= alpha[mt][0];
           o[mt][n][1] *= alpha[mt][0];
           o[mt][n][2] *= alpha[mt][1];
@@ -284,9 +295,10 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
       for (int mt = 0; mt < MT; ++mt)
         ldmatrix_x4(p_sm + swz128(mt * 16 + (lj & 1) * 8 + lr, ks * 2 + (lj >> 1)), pa[mt][0], pa[mt][1], pa[mt][2], pa[mt][3]);
 #pragma unroll
-      for (int np = 0; np < 4; ++np) {
+      for (int np = 0; np < kNt / 2; ++np) {
         uint32_t v0, v1, v2, v3;
-        ldmatrix_x4_trans(cbase + warp * kLatHalf + swz128(ks * 16 + v_tok, np * 2 + v_sub), v0, v1, v2, v3);
+        const int ch = warp * (kCols / 8) + np * 2 + v_sub;
+        ldmatrix_x4_trans(cbase + (ch >> 3) * kLatHalf + swz128(ks * 16 + v_tok, ch & 7), v0, v1, v2, v3);
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
           mma_bf16_16816(o[mt][2 * np], pa[mt], v0, v1);
@@ -321,15 +333,15 @@ latent_attn_decode_kernel(const __grid_constant__ CUtensorMap c_map, const __nv_
       const size_t row = static_cast<size_t>(b) * heads + h;
       if (nsplits == 1) {
         const float inv = head_gate(gate, row) / l;
-        __nv_bfloat16* od = out + row * R + warp * 64 + 2 * tq;
+        __nv_bfloat16* od = out + row * R + warp * kCols + 2 * tq;
 #pragma unroll
-        for (int n = 0; n < 8; ++n)
+        for (int n = 0; n < kNt; ++n)
           *reinterpret_cast<uint32_t*>(od + n * 8) = pack_bf16x2(o[mt][n][2 * hf] * inv, o[mt][n][2 * hf + 1] * inv);
       } else {
         const size_t prow = row * max_splits + split;
-        float* od = part_o + prow * R + warp * 64 + 2 * tq;
+        float* od = part_o + prow * R + warp * kCols + 2 * tq;
 #pragma unroll
-        for (int n = 0; n < 8; ++n)
+        for (int n = 0; n < kNt; ++n)
           *reinterpret_cast<float2*>(od + n * 8) = make_float2(o[mt][n][2 * hf], o[mt][n][2 * hf + 1]);
         if (warp == 0 && tq == 0) part_ml[prow] = make_float2(m_run[mt][hf], l);
       }
@@ -373,25 +385,25 @@ latent_attn_reduce_kernel(const float* __restrict__ part_o, const float2* __rest
   *reinterpret_cast<uint2*>(out + row * rank + col) = r;
 }
 
-template <int NW, int MT>
+template <class Cfg>
 static int launch_latent(const void* q, const void* c_pool, const int* block_table, const int* ctx_lens, void* out,
                          const AttnWorkspace& w, int batch, int heads, int num_blocks, int max_pages, float scale,
                          int split_tokens, int max_splits, const float* gate, cudaStream_t st) {
-  using Cfg = LatentCfg<NW, MT>;
   static_assert(Cfg::kSmemBytes <= 232448, "more shared memory than a CTA may have");
   CUtensorMap cmap;
-  int rc = get_tensor_map_2d(c_pool, static_cast<uint64_t>(num_blocks) * kLatPage, NW * 64, 2, kLatPage, 64, &cmap);
+  int rc = get_tensor_map_2d(c_pool, static_cast<uint64_t>(num_blocks) * kLatPage, Cfg::R, 2, kLatPage, 64, &cmap);
   if (rc) return rc;
-  rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&latent_attn_decode_kernel<NW, MT>), Cfg::kSmemBytes);
+  rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&latent_attn_decode_kernel<Cfg>), Cfg::kSmemBytes);
   if (rc) return rc;
-  const dim3 grid(batch, max_splits, (heads + 16 * MT - 1) / (16 * MT));
-  B200_CUDA(launch_overlapped(latent_attn_decode_kernel<NW, MT>, grid, dim3(Cfg::kThreads), Cfg::kSmemBytes, st, cmap,
+  const int head_groups = (heads + 16 * Cfg::MT - 1) / (16 * Cfg::MT);
+  const dim3 grid(batch * head_groups, max_splits);
+  B200_CUDA(launch_overlapped(latent_attn_decode_kernel<Cfg>, grid, dim3(Cfg::kThreads), Cfg::kSmemBytes, st, cmap,
                               static_cast<const __nv_bfloat16*>(q), block_table, ctx_lens, w.o, w.ml,
                               static_cast<__nv_bfloat16*>(out), w.err, heads, num_blocks, max_pages, split_tokens,
-                              max_splits, scale * 1.4426950408889634f, gate));
+                              max_splits, scale * 1.4426950408889634f, gate, head_groups));
   if (max_splits > 1)
     B200_CUDA(launch_overlapped(latent_attn_reduce_kernel, dim3(batch * heads), dim3(128), 0, st, w.o, w.ml, ctx_lens,
-                                static_cast<__nv_bfloat16*>(out), heads, NW * 64, max_splits, split_tokens,
+                                static_cast<__nv_bfloat16*>(out), heads, Cfg::R, max_splits, split_tokens,
                                 max_pages * kLatPage, gate));
   return 0;
 }
@@ -430,17 +442,21 @@ extern "C" int b200_latent_attn_decode(const void* q, const void* c_pool, const 
   cudaStream_t st = as_stream(stream);
 #define B200_LAT_ARGS q, c_pool, block_table, ctx_lens, out, w, batch, num_heads, num_blocks, max_pages_per_seq, scale, \
                       split_tokens, ms, gate, st
-#define B200_LAT_CASE(NW)                                                \
-  case NW * 64:                                                          \
-    return num_heads > 16 ? launch_latent<NW, 2>(B200_LAT_ARGS) : launch_latent<NW, 1>(B200_LAT_ARGS)
+  //                    rank MT warps tile stages CTAs
+  const bool two = num_heads > 16;
   switch (rank) {
-    B200_LAT_CASE(1);
-    B200_LAT_CASE(2);
-    B200_LAT_CASE(3);
-    B200_LAT_CASE(4);
-    B200_LAT_CASE(6);
-    default: return num_heads > 16 ? launch_latent<8, 2>(B200_LAT_ARGS) : launch_latent<8, 1>(B200_LAT_ARGS);
+    case 64: return two ? launch_latent<LatentCfg<64, 2, 1, 64, 4, 3>>(B200_LAT_ARGS)
+                        : launch_latent<LatentCfg<64, 1, 1, 64, 4, 3>>(B200_LAT_ARGS);
+    case 128: return two ? launch_latent<LatentCfg<128, 2, 2, 64, 4, 3>>(B200_LAT_ARGS)
+                         : launch_latent<LatentCfg<128, 1, 2, 64, 4, 3>>(B200_LAT_ARGS);
+    case 192: return two ? launch_latent<LatentCfg<192, 2, 3, 48, 4, 2>>(B200_LAT_ARGS)
+                         : launch_latent<LatentCfg<192, 1, 3, 48, 4, 2>>(B200_LAT_ARGS);
+    case 256: return two ? launch_latent<LatentCfg<256, 2, 4, 64, 3, 2>>(B200_LAT_ARGS)
+                         : launch_latent<LatentCfg<256, 1, 4, 64, 3, 2>>(B200_LAT_ARGS);
+    case 384: return two ? launch_latent<LatentCfg<384, 2, 6, 48, 4, 1>>(B200_LAT_ARGS)
+                         : launch_latent<LatentCfg<384, 1, 3, 32, 4, 2>>(B200_LAT_ARGS);
+    default: return two ? launch_latent<LatentCfg<512, 2, 4, 32, 2, 2>>(B200_LAT_ARGS)
+                        : launch_latent<LatentCfg<512, 1, 4, 32, 3, 2>>(B200_LAT_ARGS);
   }
-#undef B200_LAT_CASE
 #undef B200_LAT_ARGS
 }

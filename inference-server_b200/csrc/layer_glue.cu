@@ -18,6 +18,7 @@
 namespace b200 {
 
 constexpr int kGlueMaxSegs = 4;
+constexpr int kFastTaps = 5;  // convolutions of up to this many taps keep their rows in registers
 
 template <typename T>
 __device__ __forceinline__ void load8(const T* p, float (&f)[8]);
@@ -56,6 +57,38 @@ __device__ __forceinline__ void store8<float>(float* p, const float (&f)[8]) {
 }
 template <typename T>
 __device__ __forceinline__ float round_to(float v) { return to_f32<T>(from_f32<T>(v)); }
+
+// Eight columns as they lie in memory, so that several rows can be asked for before the first is used.
+template <typename T>
+struct Raw8;
+template <>
+struct Raw8<__nv_bfloat16> {
+  uint4 v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void zero() { v = make_uint4(0u, 0u, 0u, 0u); }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 t = __bfloat1622float2(h[j]);
+      f[2 * j] = t.x;
+      f[2 * j + 1] = t.y;
+    }
+  }
+};
+template <>
+struct Raw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) {
+    a = reinterpret_cast<const float4*>(p)[0];
+    b = reinterpret_cast<const float4*>(p)[1];
+  }
+  __device__ __forceinline__ void zero() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+    f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  }
+};
 
 // Where the pages of a row or sequence are; -1 and a status code for anything outside.
 struct PageMap {
@@ -104,8 +137,9 @@ __global__ void embed_sinusoid_kernel(const long long* __restrict__ tokens, cons
 }
 
 // One CTA per row, 8 columns per thread.  WIDE: a group's width is a multiple of 256, so every warp lies in one group.
-template <typename T, bool WIDE>
-__global__ void group_rmsnorm_kernel(float* __restrict__ x, const T* __restrict__ delta, const T* __restrict__ weight,
+template <typename T, bool WIDE, int MAXT>
+__global__ void __launch_bounds__(MAXT)
+group_rmsnorm_kernel(float* __restrict__ x, const T* __restrict__ delta, const T* __restrict__ weight,
                                      float eps, int width, int ld, int groups, T* __restrict__ out,
                                      const T* __restrict__ conv_w, int taps, T* __restrict__ hist,
                                      const int* __restrict__ positions, const int* __restrict__ block_table, PageMap pm) {
@@ -120,6 +154,17 @@ __global__ void group_rmsnorm_kernel(float* __restrict__ x, const T* __restrict_
   float f[8], w[8], acc[8];
 #pragma unroll
   for (int j = 0; j < 8; ++j) f[j] = w[j] = acc[j] = 0.f;
+  // the convolution's earlier rows do not depend on this row: their pages are looked up first, the rows themselves asked
+  // for before the statistics
+  int pos = 0, page = -1, before = -1, rows = 0;
+  const int* table_row = nullptr;
+  if (taps > 0) {
+    pos = positions[m];
+    table_row = block_table + static_cast<size_t>(m) * pm.max_pages;
+    page = page_of(pm, table_row, pos);
+    if (pos >= pm.page) before = page_of(pm, table_row, pos - pm.page);
+    rows = taps > 1 ? min(taps, pm.page) : 0;
+  }
   if (in) {
     load8<float>(x + at, f);
     load8<T>(weight + col, w);
@@ -131,16 +176,36 @@ __global__ void group_rmsnorm_kernel(float* __restrict__ x, const T* __restrict_
       store8<float>(x + at, f);
     }
   }
-  // the convolution's earlier rows do not depend on this row: fetched before the statistics
-  int pos = 0, page = -1, rows = 0;
   float wlast[8];
   if (taps > 0) {
-    pos = positions[m];
-    const int* table_row = block_table + static_cast<size_t>(m) * pm.max_pages;
-    page = page_of(pm, table_row, pos);
-    rows = taps > 1 ? min(taps, pm.page) : 0;
     if (in && page >= 0) {
       load8<T>(conv_w + static_cast<size_t>(taps - 1) * ld + col, wlast);
+    }
+    if (taps <= kFastTaps && taps - 1 <= pm.page) {
+      // the earlier rows lie in this page and the one before: all rows and weights are in flight together
+      const int slot0 = pos % pm.page;
+      Raw8<T> hv[kFastTaps - 1], cw[kFastTaps - 1];
+#pragma unroll
+      for (int j = 0; j < kFastTaps - 1; ++j) {
+        const int s = pos - taps + 1 + j;
+        const int back = slot0 - (taps - 1 - j);  // slot in this page, negative: in the page before
+        const int pg = back >= 0 ? page : before;
+        hv[j].zero();
+        cw[j].zero();
+        if (in && j + 1 < taps && s >= 0 && pg >= 0) {
+          hv[j].load(hist + (static_cast<size_t>(pg) * rows + (back >= 0 ? back : back + pm.page) % rows) * ld + col);
+          cw[j].load(conv_w + static_cast<size_t>(j) * ld + col);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < kFastTaps - 1; ++j) {
+        float a[8], b[8];
+        hv[j].get(a);
+        cw[j].get(b);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] = fmaf(b[e], a[e], acc[e]);
+      }
+    } else if (in && page >= 0) {
       for (int j = 0; j + 1 < taps; ++j) {
         const int s = pos - taps + 1 + j;
         if (s < 0) continue;
@@ -203,7 +268,8 @@ __global__ void group_rmsnorm_kernel(float* __restrict__ x, const T* __restrict_
 // Rows of one page of the sequence per CTA (blockIdx.x), 8 columns per thread.  The only rows read from the history
 // lie before the chunk; a page's history is written by the CTA of that page alone, each column by the thread that has
 // read it, so the first page's writes come after its reads.  Reads further back are of pages that nobody writes.
-template <typename T>
+// TAPS > 0: that many, the rows of the window kept in registers; 0: `taps`, each row read again for every tap.
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(64)
 short_conv_kernel(const T* __restrict__ h, const T* __restrict__ conv_w, int taps, T* __restrict__ hist,
                   const int* __restrict__ table_row, int num_rows, int first_pos, int ld, T* __restrict__ out,
@@ -215,6 +281,43 @@ short_conv_kernel(const T* __restrict__ h, const T* __restrict__ conv_w, int tap
   const int pg0 = first_pos / pm.page + static_cast<int>(blockIdx.x);
   const int lo = max(first_pos, pg0 * pm.page), hi = min(first_pos + num_rows, (pg0 + 1) * pm.page);
   const int rows = taps > 1 ? min(taps, pm.page) : 0;
+  if (TAPS > 1) {
+    float w[TAPS > 1 ? TAPS : 1][8], win[TAPS > 1 ? TAPS - 1 : 1][8];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load8<T>(conv_w + static_cast<size_t>(j) * ld + col, w[j]);
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j) {
+      const int s = lo - TAPS + 1 + j;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) win[j][e] = 0.f;
+      if (s >= first_pos) {
+        load8<T>(h + static_cast<size_t>(s - first_pos) * ld + col, win[j]);
+      } else if (s >= 0) {
+        const int pg = page_of(pm, table_row, s);
+        if (pg >= 0) load8<T>(hist + (static_cast<size_t>(pg) * rows + (s % pm.page) % rows) * ld + col, win[j]);
+      }
+    }
+#pragma unroll 4
+    for (int p = lo; p < hi; ++p) {
+      float hv[8], acc[8];
+      load8<T>(h + static_cast<size_t>(p - first_pos) * ld + col, hv);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] = fmaf(w[j][e], win[j][e], acc[e]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[e] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][e], hv[e], acc[e]) + hv[e];
+#pragma unroll
+      for (int j = 0; j + 2 < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) win[j][e] = win[j + 1][e];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) win[TAPS > 1 ? TAPS - 2 : 0][e] = hv[e];
+      store8<T>(out + static_cast<size_t>(p - first_pos) * ld + col, acc);
+    }
+  } else
 #pragma unroll 2
   for (int p = lo; p < hi; ++p) {
     float acc[8], hv[8], cw[8];
@@ -434,11 +537,34 @@ static int launch_group_rmsnorm(float* x, const void* delta, const void* weight,
 #define B200_NORM_ARGS                                                                                              \
   x, static_cast<const T*>(delta), static_cast<const T*>(weight), eps, width, ld, groups, static_cast<T*>(out),      \
       static_cast<const T*>(conv_w), taps, static_cast<T*>(hist), positions, block_table, pm
-  if (wide)
-    B200_CUDA(launch_overlapped(group_rmsnorm_kernel<T, true>, dim3(rows), dim3(threads), smem, st, B200_NORM_ARGS));
-  else
-    B200_CUDA(launch_overlapped(group_rmsnorm_kernel<T, false>, dim3(rows), dim3(threads), smem, st, B200_NORM_ARGS));
+  if (threads <= 512) {
+    if (wide)
+      B200_CUDA(launch_overlapped(group_rmsnorm_kernel<T, true, 512>, dim3(rows), dim3(threads), smem, st, B200_NORM_ARGS));
+    else
+      B200_CUDA(launch_overlapped(group_rmsnorm_kernel<T, false, 512>, dim3(rows), dim3(threads), smem, st, B200_NORM_ARGS));
+  } else if (wide) {
+    B200_CUDA(launch_overlapped(group_rmsnorm_kernel<T, true, 1024>, dim3(rows), dim3(threads), smem, st, B200_NORM_ARGS));
+  } else {
+    B200_CUDA(launch_overlapped(group_rmsnorm_kernel<T, false, 1024>, dim3(rows), dim3(threads), smem, st, B200_NORM_ARGS));
+  }
 #undef B200_NORM_ARGS
+  return 0;
+}
+
+template <typename T>
+static int launch_short_conv(const void* h, const void* conv_w, int taps, void* hist, const int* table_row, int rows,
+                             int first_pos, int ld, void* out, const PageMap& pm, dim3 grid, cudaStream_t st) {
+#define B200_CONV_CASE(TAPS)                                                                                             \
+  B200_CUDA(launch_overlapped(short_conv_kernel<T, TAPS>, grid, dim3(64), 0, st, static_cast<const T*>(h),               \
+                              static_cast<const T*>(conv_w), taps, static_cast<T*>(hist), table_row, rows, first_pos, ld, \
+                              static_cast<T*>(out), pm))
+  switch (taps) {
+    case 2: B200_CONV_CASE(2); break;
+    case 3: B200_CONV_CASE(3); break;
+    case 4: B200_CONV_CASE(4); break;
+    default: B200_CONV_CASE(0); break;
+  }
+#undef B200_CONV_CASE
   return 0;
 }
 
@@ -511,15 +637,10 @@ extern "C" int b200_short_conv(const void* h, const void* conv_w, int taps, void
   const int pages = (first_position + num_rows - 1) / page_size - first_position / page_size + 1;
   const dim3 grid(pages, (ld / 8 + 63) / 64);
   if (dtype == 0)
-    B200_CUDA(launch_overlapped(short_conv_kernel<__nv_bfloat16>, grid, dim3(64), 0, as_stream(stream),
-                                static_cast<const __nv_bfloat16*>(h), static_cast<const __nv_bfloat16*>(conv_w), taps,
-                                static_cast<__nv_bfloat16*>(hist), block_table_row, num_rows, first_position, ld,
-                                static_cast<__nv_bfloat16*>(out), pm));
-  else
-    B200_CUDA(launch_overlapped(short_conv_kernel<float>, grid, dim3(64), 0, as_stream(stream), static_cast<const float*>(h),
-                                static_cast<const float*>(conv_w), taps, static_cast<float*>(hist), block_table_row,
-                                num_rows, first_position, ld, static_cast<float*>(out), pm));
-  return 0;
+    return launch_short_conv<__nv_bfloat16>(h, conv_w, taps, hist, block_table_row, num_rows, first_position, ld, out, pm, grid,
+                                            as_stream(stream));
+  return launch_short_conv<float>(h, conv_w, taps, hist, block_table_row, num_rows, first_position, ld, out, pm, grid,
+                                  as_stream(stream));
 }
 
 extern "C" int b200_latent_norm_append(const float* raw, const void* weight, float eps, int num_rows, int rank, int ld,

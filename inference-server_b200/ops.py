@@ -408,11 +408,12 @@ def latent_attn_supported(rank: int, page_size: int, dtype) -> bool:
 
 
 def latent_split_tokens(batch: int, max_ctx: int, num_sms: int = 148) -> int:
-    """Tokens per split of the latent decode kernel (all heads of a row in one CTA): enough CTAs to fill the GPU about
-    twice over, splits no shorter than 256 tokens."""
-    per_row = max(1, -(-2 * num_sms // max(1, batch)))
-    split = -(-max(1, max_ctx) // per_row)
-    return int(min(4096, max(256, -(-split // 64) * 64)))
+    """Tokens per split of the latent decode kernel (all heads of a row in one CTA, two CTAs per SM): few rows are cut so that
+    about 1.3 CTAs per SM exist over their expected tokens, a full batch into pieces of 768 (both measured)."""
+    if batch >= 192:
+        return 768
+    split = -(-max(1, max_ctx // 2) * batch * 10 // (13 * num_sms))
+    return int(min(1408, max(128, -(-split // 64) * 64)))
 
 
 def latent_attn_decode(q, c_pool, block_table, ctx_lens, scale: float, split_tokens: int, workspace, gate=None, out=None):

@@ -8,6 +8,7 @@
                                                                # the denominator for the MoE GEMM's tensor fraction
     python microbench.py prefill         # tiled causal prompt attention: a chunk of 1024 tokens at several
                                                                # depths of one sequence, beside the row-per-token form
+    python microbench.py latent          # decode attention over latents (one vector per token, all heads), 256 sequences
     python microbench.py dense           # the bf16 projections (q/k/v, o, router, lm_head + arg-max) at decode
                                                                # sizes, every K split, beside the library GEMM
     ... attn --small / moe --small                             # few launches on a few hundred MB: sized for a profiler
@@ -126,6 +127,38 @@ def run_attn(args) -> None:
                       "alg_MB": alg / 1e6, "logical_MB": sum(lens) * hkv * d * 4 / 1e6, "GBs": alg / med / 1e3,
                       "frac_of_hbm_peak": alg / med / 1e3 / peak, "peak_GBs": peak, "peak_source": src,
                       "note": "time covers the split kernel and the split reduce"}))
+
+
+def run_latent(args) -> None:
+    H, R = args.heads, args.rank
+    if args.small:
+        batch, lens = 32, [4096] * 32
+    else:
+        batch = args.batch
+        lens = np.random.default_rng(0).integers(args.ctx_min, args.ctx_max + 1, size=batch).tolist()
+    _, pool, _, table, ctx, unique = paged_case(batch, 1, 1, R, lens, 0)
+    pool = pool[:, 0].contiguous()
+    q = torch.randn(batch, H, R, device=DEV).bfloat16()
+    gate = torch.randn(batch, H, device=DEV)
+    out = torch.empty_like(q)
+    alg = unique * PAGE * R * 2 + batch * H * R * 4 + 4 * unique + 4 * batch
+    peak, src = measured_hbm_gbs()
+    for st in [int(x) for x in args.split_tokens.split(",")]:
+        st = st or ops.latent_split_tokens(batch, table.shape[1] * PAGE)
+        ws = ops.paged_attn_workspace(batch, H, R, table.shape[1], PAGE, st, DEV)
+        fn = lambda: ops.latent_attn_decode(q, pool, table, ctx, R ** -0.5, st, ws, gate, out)
+        if args.small:
+            for _ in range(4):
+                fn()
+            torch.cuda.synchronize()
+            ops.read_status(ws, "latent attention")
+            print(json.dumps({"case": "latent --small", "launches": 4, "alg_MB": alg / 1e6, "split_tokens": st}))
+            return
+        med, mn = Timer(args.iters)(fn)
+        ops.read_status(ws, "latent attention")
+        print(json.dumps({"case": "latent", "batch": batch, "heads": H, "rank": R, "mean_ctx": float(np.mean(lens)), "split_tokens": st,
+                          "us_median": med, "us_min": mn, "alg_MB": alg / 1e6, "GBs": alg / med / 1e3,
+                          "frac_of_hbm_peak": alg / med / 1e3 / peak, "peak_source": src}))
 
 
 # ------------------------------------------------------------------------ MoE --
@@ -360,6 +393,13 @@ def main() -> None:
     a.add_argument("--share-group", type=int, default=8)
     a.add_argument("--share-tokens", type=int, default=1024)
     a.add_argument("--split-tokens", type=int, default=0)
+    la = sub.add_parser("latent")
+    la.add_argument("--batch", type=int, default=256)
+    la.add_argument("--heads", type=int, default=16)
+    la.add_argument("--rank", type=int, default=512)
+    la.add_argument("--ctx-min", type=int, default=512)
+    la.add_argument("--ctx-max", type=int, default=4096)
+    la.add_argument("--split-tokens", default="0", help="comma separated; 0 = the default")
     m = sub.add_parser("moe")
     m.add_argument("--tokens", default=MOE_TOKENS_DEFAULT, help="token counts; with --small only the first (default 64)")
     m.add_argument("--tiled", action="store_true", help="weights stored as contiguous 128x128 blocks")
@@ -393,13 +433,13 @@ def main() -> None:
     f.add_argument("--size", type=int, default=8192)
     f.add_argument("--iters", type=int, default=20)
     f.add_argument("--small", action="store_true", help=argparse.SUPPRESS)
-    for p in (a, m, e):
+    for p in (a, la, m, e):
         p.add_argument("--iters", type=int, default=20)
         p.add_argument("--small", action="store_true", help="a few launches on a small case (for a profiler)")
     args = ap.parse_args()
     if not torch.cuda.is_available():
         raise SystemExit("microbench.py needs a CUDA device")
-    {"attn": run_attn, "moe": run_moe, "ep": run_ep, "fp8peak": run_fp8peak, "dense": run_dense, "prefill": run_prefill}[args.case](args)
+    {"attn": run_attn, "latent": run_latent, "moe": run_moe, "ep": run_ep, "fp8peak": run_fp8peak, "dense": run_dense, "prefill": run_prefill}[args.case](args)
 
 
 if __name__ == "__main__":

@@ -60,7 +60,7 @@ def test_embed_sinusoid(ops, dtype, width, ld):
 
 @pytest.mark.parametrize("dtype", [BF, F32])
 @pytest.mark.parametrize("width,ld,groups", [(192, 192, 3), (204, 256, 6), (1024, 1024, 4), (2048, 2048, 1), (70, 128, 10),
-                                              (4096, 4096, 8), (768, 768, 2)])
+                                              (4096, 4096, 8), (768, 768, 2), (8192, 8192, 4), (8100, 8128, 5)])
 def test_group_rmsnorm(ops, dtype, width, ld, groups):
     x, d, w = torch.zeros(9, ld), torch.zeros(9, ld), torch.zeros(ld)
     # one group per row is far larger than the others, so a statistic over the wrong columns shows
@@ -113,9 +113,9 @@ def test_short_conv_in_portions_and_decoded(ops, taps, dtype):
         assert rel_err(torch.cat(got), want) < (2e-2 if dtype == BF else 2e-5), (taps, cuts)
 
 
-def test_decode_convolution_rows_are_independent(ops):
+@pytest.mark.parametrize("ld,taps", [(64, 4), (64, 7), (4160, 3)])
+def test_decode_convolution_rows_are_independent(ops, ld, taps):
     """Rows of one step at their own positions and pages; a position at a sequence's start sees zeros."""
-    ld, taps = 64, 4
     w, g = randn(taps, ld, seed=1).to(DEV), torch.ones(ld, device=DEV)
     hist = torch.zeros(6, taps, ld, device=DEV)
     seqs = [randn(40, ld, seed=10 + i) for i in range(3)]
