@@ -256,6 +256,7 @@ int b200_dense_gemm_grouped(const void* x, const void* w, void* y, void* status_
  *   kind 2  page slots of a pool [num_blocks, heads, page_size, dim] bf16, heads * dim = width: row m goes to
  *           position positions[m] of the sequence whose pages are block_table[m] (positions NULL: position m;
  *           block_table NULL: page p of the sequence is block p)
+ * Segments of kinds 0 and 2 begin and end at even features; page_size a power of two.
  * seg_* are HOST arrays; seg_ptr holds device pointers.  x [num_rows, in_features], w [seg_end[last], in_features].
  */
 int b200_proj_split_gemm(const void* x, const void* w, const float* col_scale, const int32_t* seg_end,

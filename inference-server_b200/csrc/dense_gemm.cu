@@ -115,6 +115,7 @@ struct DenseParams {
   __nv_bfloat16* v_pool;
   float eps;
   int hq, hkv, page, num_blocks, max_pages, max_pos;
+  int page_shift;     // kEpiSplit: page is a power of two
   int* err;
   int M, N, K;
   int m_tiles;        // ceil(M / xbox)
@@ -161,6 +162,15 @@ __device__ __forceinline__ uint32_t float_key(float f) {
 }
 __device__ __forceinline__ float key_float(uint32_t k) {
   return __uint_as_float(k ^ ((k >> 31) ? 0x80000000u : 0xffffffffu));
+}
+
+// Two neighbouring lanes hold two neighbouring features of the same rows.  For the rows i and i + 1 they swap one value, and
+// the even lane ends up with both features of row i, the odd lane with both of row i + 1: one 4-byte store per lane and two
+// rows instead of two 2-byte stores.  The caller stores at row i + (lane & 1), feature t & ~1.
+__device__ __forceinline__ uint32_t pack_row_pair(float row_i, float row_i1, int lane) {
+  const bool odd = (lane & 1) != 0;
+  const float other = __shfl_xor_sync(0xffffffffu, odd ? row_i : row_i1, 1);
+  return odd ? pack_bf16x2(other, row_i1) : pack_bf16x2(row_i, other);
 }
 
 template <int A_TILES, int EPI>
@@ -317,7 +327,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
       }
       // kEpiSplit: where this thread's feature goes, and the page and slot of the rows of this warp's chunks (lane i:
       // row i of the chunk), fetched while the MMAs of the item are still running; page -1 = not written
-      int seg_kind = -1, seg_page_stride = 0, seg_dim = 0, seg_ld = 0, row_page4[4], row_slot4[4];
+      int seg_kind = -1, seg_page_stride = 0, seg_dim = 0, seg_ld = 0, row_at4[4];
       void* seg_ptr = nullptr;
       float seg_scale = 1.f;
       if (EPI == kEpiSplit) {
@@ -347,8 +357,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
         if (p.col_scale != nullptr && n < p.N) seg_scale = p.col_scale[n];
 #pragma unroll
         for (int cc = 0; cc < 4; ++cc) {
-          row_page4[cc] = -1;
-          row_slot4[cc] = 0;
+          row_at4[cc] = -1;
           const int r = (cc * 2 + half) * 32 + lane, m = m0 + r;
           if (pages && r < p.xbox && m < p.M) {
             const int ps = p.positions != nullptr ? p.positions[m] : m;
@@ -360,8 +369,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
               if (id < 0 || id >= p.num_blocks) {
                 set_error(p.err, kErrDevBadBlockId);
               } else {
-                row_page4[cc] = id;
-                row_slot4[cc] = ps - pg * p.page;
+                row_at4[cc] = id * p.page + (ps - pg * p.page);
               }
             }
           }
@@ -382,21 +390,25 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           const int left = p.M - (m0 + c * 32);  // rows of this chunk that exist
 #pragma unroll
           for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * seg_scale);
-          if (__any_sync(0xffffffffu, seg_kind == kSegPages)) {
-            __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(seg_ptr);
+          // Segments begin at even features and are even wide (checked on the host), so a pair of lanes is in one segment.
+          if (__any_sync(0xffffffffu, seg_kind == kSegPages || seg_kind == kSegBf16)) {
+            __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(seg_ptr) - (lane & 1);
 #pragma unroll
-            for (int i = 0; i < 32; ++i) {
-              const int page = __shfl_sync(0xffffffffu, row_page4[cc], i), slot = __shfl_sync(0xffffffffu, row_slot4[cc], i);
-              if (seg_kind == kSegPages && page >= 0 && i < left)
-                dst[static_cast<size_t>(page) * seg_page_stride + slot * seg_dim] = __float2bfloat16(__uint_as_float(v[i]));
+            for (int i = 0; i < 32; i += 2) {
+              const uint32_t two = pack_row_pair(__uint_as_float(v[i]), __uint_as_float(v[i + 1]), lane);
+              const int r = i + (lane & 1);
+              const int at = __shfl_sync(0xffffffffu, row_at4[cc], r);  // page * page size + slot, -1 = not written
+              if (seg_kind == kSegPages) {
+                if (at >= 0 && r < left) {
+                  const int page = at >> p.page_shift, slot = at - (page << p.page_shift);
+                  *reinterpret_cast<uint32_t*>(dst + static_cast<size_t>(page) * seg_page_stride + slot * seg_dim) = two;
+                }
+              } else if (seg_kind == kSegBf16 && r < left) {
+                *reinterpret_cast<uint32_t*>(dst + static_cast<size_t>(m0 + c * 32 + r) * seg_ld) = two;
+              }
             }
           }
-          if (seg_kind == kSegBf16) {
-            __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(seg_ptr) + static_cast<size_t>(m0 + c * 32) * seg_ld;
-#pragma unroll
-            for (int i = 0; i < 32; ++i)
-              if (i < left) dst[static_cast<size_t>(i) * seg_ld] = __float2bfloat16(__uint_as_float(v[i]));
-          } else if (seg_kind == kSegF32) {
+          if (seg_kind == kSegF32) {
             float* dst = static_cast<float*>(seg_ptr) + static_cast<size_t>(m0 + c * 32) * seg_ld;
 #pragma unroll
             for (int i = 0; i < 32; ++i)
@@ -411,14 +423,16 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           tmem_ld32(lane_addr + c * 32, v);
           tmem_ld32(lane_addr + (A_TILES > 1 ? kDenseMaxRows : 0) + c * 32, u);
           tmem_ld_wait();
-          if (n < p.N) {
+          // p.N is a multiple of 128: every lane has a feature
+          const int left = p.M - (m0 + c * 32);
+          __nv_bfloat16* dst = p.y + static_cast<size_t>(m0 + c * 32 + (lane & 1)) * p.ldy + (n & ~1);
 #pragma unroll
-            for (int i = 0; i < 32; ++i) {
-              const int m = m0 + c * 32 + i;
-              if (m < p.M)
-                p.y[static_cast<size_t>(m) * p.ldy + n] = __float2bfloat16(clamped_glu_fast(
-                    __uint_as_float(v[i]), __uint_as_float(u[i]), p.glu_limit, p.glu_alpha));
-            }
+          for (int i = 0; i < 32; ++i)
+            v[i] = __float_as_uint(clamped_glu_fast(__uint_as_float(v[i]), __uint_as_float(u[i]), p.glu_limit, p.glu_alpha));
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) {
+            const uint32_t two = pack_row_pair(__uint_as_float(v[i]), __uint_as_float(v[i + 1]), lane);
+            if (i + (lane & 1) < left) *reinterpret_cast<uint32_t*>(dst + static_cast<size_t>(i) * p.ldy) = two;
           }
         }
       } else
@@ -442,7 +456,15 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
             uint32_t v[32];
             tmem_ld32(t0 + c * 32, v);
             tmem_ld_wait();
-            if (n < p.N) {
+            if (p.y_f32 == nullptr && ((p.N | p.ldy | p.y_step) & 1) == 0) {
+              const int left = p.M - (m0 + c * 32);
+              __nv_bfloat16* dst = p.y + static_cast<size_t>(m0 + c * 32 + (lane & 1)) * p.ldy + g * p.y_step + (n & ~1);
+#pragma unroll
+              for (int i = 0; i < 32; i += 2) {
+                const uint32_t two = pack_row_pair(__uint_as_float(v[i]), __uint_as_float(v[i + 1]), lane);
+                if (n < p.N && i + (lane & 1) < left) *reinterpret_cast<uint32_t*>(dst + static_cast<size_t>(i) * p.ldy) = two;
+              }
+            } else if (n < p.N) {
 #pragma unroll
               for (int i = 0; i < 32; ++i) {
                 const int m = m0 + c * 32 + i;
@@ -949,8 +971,9 @@ extern "C" int b200_dense_gemm_grouped(const void* x, const void* w, void* y, vo
   B200_REQUIRE(x_cols % 8 == 0 && (groups - 1) * x_step + in_features <= x_cols &&
                    (groups - 1) * y_step + out_features <= y_cols,
                "dense_gemm_grouped: the groups do not fit %d input and %d output columns", x_cols, y_cols);
-  B200_REQUIRE(((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0,
-               "dense_gemm_grouped: x and w must be 16-byte aligned");
+  B200_REQUIRE(((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) == 0 &&
+                   (reinterpret_cast<uintptr_t>(y) & 3) == 0,
+               "dense_gemm_grouped: x and w must be 16-byte aligned, y 4-byte aligned");
   int rc = check_device(nullptr);
   if (rc) return rc;
   int sms = 148;
@@ -998,6 +1021,10 @@ extern "C" int b200_proj_split_gemm(const void* x, const void* w, const float* c
       B200_REQUIRE(seg_heads[i] > 0 && seg_dim[i] > 0 && seg_heads[i] * seg_dim[i] == seg_end[i] - begin && page_size > 0 &&
                        num_blocks > 0 && max_pages_per_seq > 0,
                    "proj_split_gemm: page segment %d does not match its pool", i);
+    if (seg_kind[i] != kSegF32)
+      B200_REQUIRE(begin % 2 == 0 && seg_end[i] % 2 == 0 && (seg_kind[i] != kSegPages || seg_dim[i] % 2 == 0) &&
+                       (reinterpret_cast<uintptr_t>(seg_ptr[i]) & 3) == 0,
+                   "proj_split_gemm: bf16 segment %d must begin and end at even features, 4-byte aligned", i);
     p.segs[i] = DenseSeg{seg_end[i], seg_kind[i], seg_heads[i], seg_dim[i], seg_ptr[i]};
     begin = seg_end[i];
   }
@@ -1020,7 +1047,10 @@ extern "C" int b200_proj_split_gemm(const void* x, const void* w, const float* c
   p.col_scale = col_scale;
   p.positions = positions;
   p.block_table = block_table;
+  B200_REQUIRE(page_size > 0 && (page_size & (page_size - 1)) == 0, "proj_split_gemm: page_size %d is not a power of two",
+               page_size);
   p.page = page_size;
+  while ((1 << p.page_shift) < page_size) ++p.page_shift;
   p.num_blocks = num_blocks;
   p.max_pages = max_pages_per_seq;
   CUtensorMap w_map, x_map;
@@ -1036,7 +1066,8 @@ extern "C" int b200_dense_glu_gemm(const void* x, const void* w_interleaved, voi
                                    int inter, int in_features, float limit, float alpha, void* stream) {
   int rc = dense_args_ok(x, w_interleaved, num_rows, 2 * inter, in_features, "dense_glu_gemm");
   if (rc) return rc;
-  B200_REQUIRE(y && inter % 128 == 0, "dense_glu_gemm: %d inner features (a multiple of 128)", inter);
+  B200_REQUIRE(y && inter % 128 == 0 && (reinterpret_cast<uintptr_t>(y) & 3) == 0,
+               "dense_glu_gemm: %d inner features (a multiple of 128)", inter);
   rc = check_device(nullptr);
   if (rc) return rc;
   int sms = 148;
