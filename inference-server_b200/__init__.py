@@ -8,6 +8,10 @@ The directory name contains a hyphen, so import it with
 - ``ops``       operator wrappers on torch CUDA tensors (paged attention, KV
                 append, MoE route/permute/quant/GEMM/combine).
 - ``quant``     load-time e4m3 128x128 block quantisation of expert weights.
+- ``engine``    ``PagedEngine`` (step, graphs, prompt passes) and the Qwen3-MoE
+                ``DecodeEngine`` on it.
+- ``layered``   layer-list decoders (Sulepel) on ``PagedEngine``.
+- ``registry``, ``checkpoint``  which engine serves a model; reading model folders.
 - ``backend``   ``B200Backend``: the reference ``InferenceBackend`` interface on
                 block tables instead of dense caches.
 """
