@@ -250,8 +250,9 @@ int b200_dense_gemm_grouped(const void* x, const void* w, void* y, void* status_
                             int y_cols, void* stream);
 
 /*
- * A projection whose output goes to up to four places, split by ranges of features (segment i = features
- * [seg_end[i-1], seg_end[i])), each feature first multiplied by col_scale[n] in fp32 when col_scale is given:
+ * A projection whose output goes to up to eight places, split by ranges of features (segment i = features
+ * [seg_end[i-1], seg_end[i])).  In fp32, each feature is multiplied by col_scale[n] and col_bias[n] is added (either may be
+ * NULL), then seg_act (NULL: none) applies: 0 nothing, 1 z * sigmoid(z), 2 sigmoid(z).
  *   kind 0  bf16 rows [num_rows, width of the segment]          kind 1  the same in fp32
  *   kind 2  page slots of a pool [num_blocks, heads, page_size, dim] bf16, heads * dim = width: row m goes to
  *           position positions[m] of the sequence whose pages are block_table[m] (positions NULL: position m;
@@ -259,8 +260,9 @@ int b200_dense_gemm_grouped(const void* x, const void* w, void* y, void* status_
  * Segments of kinds 0 and 2 begin and end at even features; page_size a power of two.
  * seg_* are HOST arrays; seg_ptr holds device pointers.  x [num_rows, in_features], w [seg_end[last], in_features].
  */
-int b200_proj_split_gemm(const void* x, const void* w, const float* col_scale, const int32_t* seg_end,
-                         const int32_t* seg_kind, const int32_t* seg_heads, const int32_t* seg_dim,
+int b200_proj_split_gemm(const void* x, const void* w, const float* col_scale, const float* col_bias,
+                         const int32_t* seg_end, const int32_t* seg_kind, const int32_t* seg_act,
+                         const int32_t* seg_heads, const int32_t* seg_dim,
                          void* const* seg_ptr, int num_segs, const int32_t* positions, const int32_t* block_table,
                          void* status_word, int num_rows, int in_features, int page_size, int num_blocks,
                          int max_pages_per_seq, void* stream);
@@ -373,7 +375,7 @@ int b200_add_rmsnorm_route(void* x, const void* delta, const void* norm_weight, 
 /* dtype: the activations' type (B200_DTYPE_*); the residual stream x is always fp32.  No counterparts in the
  * reference. */
 
-/* x[m, i] = embed[tokens[m], i] + sinusoid(positions[m])_i for i < width, 0 for width <= i < ld.  The sinusoid comes from
+/* x[m, i] = embed[tokens[m], i] + sinusoid(positions[m])_i for i < width, 0 for width <= i < ld (lo and hi NULL: no sinusoid).  The sinusoid comes from
  * two fp32 tables by the addition theorem: lo [64, ld] holds (sin, cos) pairs of positions 0..63, hi [n_hi, ld] those of
  * the multiples of 64. */
 int b200_embed_sinusoid(const int64_t* tokens, const int32_t* positions, const void* embed, const float* lo,
@@ -408,15 +410,108 @@ int b200_gather_pages(const void* c_pool, const int32_t* block_table_row, void* 
                       int page_size, int num_blocks, int max_pages_per_seq, void* status_word, int dtype, void* stream);
 
 /* Unfused forms, for fp32: the split store of b200_proj_split_gemm on a finished fp32 product y [num_rows, n] (segment
- * kinds 0 and 2 in dtype), the clamped gated unit on gate/up columns interleaved in blocks of 128, and the arg-max of
- * fp32 logits (ties to the lower index). */
-int b200_split_store(const float* y, const float* col_scale, const int32_t* seg_end, const int32_t* seg_kind,
-                     const int32_t* seg_heads, const int32_t* seg_dim, void* const* seg_ptr, int num_segs,
+ * kinds 0 and 2 in dtype), the clamped gated unit (g sigmoid(alpha g) (u + shift)) on gate/up columns interleaved in
+ * blocks of 128, and the arg-max of fp32 logits (ties to the lower index). */
+int b200_split_store(const float* y, const float* col_scale, const float* col_bias, const int32_t* seg_end,
+                     const int32_t* seg_kind, const int32_t* seg_act, const int32_t* seg_heads, const int32_t* seg_dim, void* const* seg_ptr, int num_segs,
                      const int32_t* positions, const int32_t* block_table, void* status_word, int num_rows,
                      int page_size, int num_blocks, int max_pages_per_seq, int dtype, void* stream);
-int b200_clamped_glu(const void* gate_up, void* out, int num_rows, int inter, float limit, float alpha, int dtype,
-                     void* stream);
+int b200_clamped_glu(const void* gate_up, void* out, int num_rows, int inter, float limit, float alpha, float shift,
+                     int dtype, void* stream);
 int b200_argmax_rows(const float* logits, int64_t* out, int num_rows, int n, void* stream);
+
+/*
+ * x [num_rows, ld] fp32 += (sublayer + bias) * gate in place, then out = (x - mean) / sqrt(variance + eps) * weight over the
+ * first `width` columns (center), or x / sqrt(mean square + eps) * weight.  The sublayer's rows are delta [num_rows, ld], or
+ * the pair_weight-weighted sum of expert_rows[row_of_pair[m, k]], k < top_k (-1: no row), or absent (both NULL: x unchanged).
+ * bias [ld] fp32, gate [num_rows, ld] may be NULL; weight [ld] fp32.  ld a multiple of 8, at most 8192; columns from width on
+ * stay zero.
+ */
+int b200_residual_norm(float* x, const void* delta, const void* expert_rows, const int32_t* row_of_pair,
+                       const float* pair_weight, int top_k, const float* bias, const void* gate, const float* weight,
+                       float eps, int num_rows, int width, int ld, int center, void* out, int dtype, void* stream);
+
+/* ---------------------------- attention with mixed heads, and recurrences -- */
+/* No counterparts in the reference.  dtype: type of activations, pools and rings (B200_DTYPE_*). */
+
+/* out [num_rows, heads, kv_heads, head_dim]: out[m, h, c] = sum over the query heads g of kv head c of mix[h, g] q[m, g];
+ * q [num_rows, heads, head_dim] and mix [heads, heads] fp32; head_dim a multiple of 4. */
+int b200_mix_heads(const float* q, const float* mix, void* out, int num_rows, int heads, int kv_heads, int head_dim,
+                   int dtype, void* stream);
+
+/*
+ * Attention whose scores are mixed over the heads: query head h of a row at position i sees the tokens j with
+ * 0 <= i - j < window, with score q[h] . (keys of all kv heads of token j) - bias[h, i - j], and sums values of its own kv
+ * head; times out_scale.
+ *   q [num_rows, num_q_heads, num_kv_heads * key_dim] (b200_mix_heads); k_pool [num_blocks, num_kv_heads, page_size, key_dim];
+ *   v_pool [num_blocks, num_kv_heads, page_size, value_dim]; block_table rows table_stride apart (0: one row for all);
+ *   positions [num_rows]; bias [num_q_heads, bias_ld] fp32, bias_ld at least min(window, positions of the table);
+ *   out [num_rows, out_ld], head h at column h * value_dim.
+ */
+int b200_mixed_attn(const void* q, const void* k_pool, const void* v_pool, const int32_t* block_table, int table_stride,
+                    const int32_t* positions, const float* bias, int bias_ld, int window, void* out, int out_ld,
+                    float out_scale, void* status_word, int num_rows, int num_q_heads, int num_kv_heads, int key_dim,
+                    int value_dim, int page_size, int num_blocks, int max_pages_per_seq, int dtype, void* stream);
+
+/*
+ * out[m] = z * sigmoid(z), z = sum_j conv_w[j] * in[position - taps + 1 + j] per channel, zeros before the sequence's start.
+ * Earlier inputs come from, and the last ones go to, ring [num_slots, taps, channels] (position p in row p % taps).
+ * chunk: the rows are consecutive positions positions[0].. of one sequence with slot slots[0]; otherwise row m is at
+ * positions[m] of the sequence with slot slots[m].  conv_w [taps, channels]; channels a multiple of 8.
+ */
+int b200_conv_silu(const void* in, const void* conv_w, int taps, void* ring, const int32_t* slots, const int32_t* positions,
+                   int num_rows, int chunk, int channels, int num_slots, void* out, void* status_word, int dtype, void* stream);
+
+/*
+ * A matrix state per head, S [dim, vdim] fp32: S <- g S, S <- S + k u^T, o = S^T q per token.
+ *   decay given: u = v, g = decay[h].  Otherwise (gated delta rule) q and k are divided by sqrt(sum of squares + 1e-6), q
+ *   multiplied by q_scale, u = beta (v - S^T k) with the decayed S, beta = sigmoid(ba[m, h]),
+ *   g = exp(-exp(a_log[h]) softplus(ba[m, heads + h] + dt_bias[h])).
+ * act [num_rows, ld] holds q [qk_heads, dim] at q_off, k at k_off and v [heads, vdim] at v_off; head h uses q/k head
+ * h / (heads / qk_heads).  state [num_slots, 2, heads, dim, vdim]: the state after position p in half p & 1 of the
+ * sequence's slot; position 0 starts from zeros.  slots, positions, chunk as above.  o [num_rows, heads, vdim] fp32.
+ */
+int b200_state_scan(const void* act, int ld, int q_off, int k_off, int v_off, const float* ba, const float* a_log,
+                    const float* dt_bias, const float* decay, float* state, const int32_t* slots, const int32_t* positions,
+                    float* o, void* status_word, int num_rows, int chunk, int heads, int qk_heads, int dim, int vdim,
+                    int num_slots, float q_scale, int dtype, void* stream);
+
+/* out[m, g] = o[m, g] / sqrt(mean square over `size` + eps) * weight * gate[m, g] * scale; o [num_rows, groups, group_ld] fp32,
+ * zero from column `size` of a group on; weight [group_ld] (shared_weight) or [groups, group_ld] fp32; gate
+ * [num_rows, groups, group_ld]; out rows out_ld apart.  group_ld and out_ld multiples of 4. */
+int b200_group_norm_gate(const float* o, const float* weight, const void* gate, float eps, int num_rows, int groups, int size,
+                         int group_ld, int shared_weight, float scale, void* out, int out_ld, int dtype, void* stream);
+
+/* ------------------------------------------------- experts in bf16 / fp32 -- */
+/* No counterparts in the reference. */
+
+/* Routing by s = sigmoid(logit): the top_k largest (equal logits: lower id), weights s / (sum of the chosen s + 1e-20) * scale
+ * (renormalize) or s * scale.  At most 32 of 1024 experts. */
+int b200_moe_route_sigmoid(const void* logits, int logits_dtype, int num_tokens, int num_experts, int top_k, int renormalize,
+                           float scale, int32_t* topk_ids, float* topk_weights, void* stream);
+
+/* The pairs of b200_moe_permute in expert order with the tokens' rows copied along: sorted_rows[row_of_pair[t, k]] = x[t].
+ * tiles (16 bytes each: expert, first row, rows, 0): at most tile_rows rows of one expert; room for
+ * ceil(pairs / tile_rows) + num_experts of them.  row_bytes a multiple of 16.  workspace: b200_moe_permute_workspace_bytes,
+ * its first word the device status. */
+int b200_moe_permute_copy(const int32_t* topk_ids, const void* x, int num_tokens, int num_experts, int top_k, int row_bytes,
+                          int tile_rows, int32_t* row_of_pair, void* tiles, int32_t* num_tiles, void* sorted_rows,
+                          void* workspace, size_t workspace_bytes, void* stream);
+
+/* Products of sorted rows with their experts' weights, tiles as b200_moe_permute_copy makes them (at most max_tiles).
+ * gate_up: h = g sigmoid(alpha g) (u + shift) with g, u clamped as in b200_dense_glu_gemm (limit may be infinite);
+ *   w_interleaved [num_experts, 2*inter, in_features], gate and up rows in alternating blocks of 128.  tile_rows a multiple of
+ *   32 up to 256, the one the tiles were cut with.
+ * down: y [num_rows, out_features], w [num_experts, out_features, in_features].
+ * gemm_f32: the same product in true fp32, tiles of at most 64 rows. */
+int b200_moe_bf16_gate_up(const void* x, const void* w_interleaved, void* h, const void* tiles, const int32_t* num_tiles,
+                          void* status_word, int num_rows, int num_experts, int max_tiles, int tile_rows, int inter,
+                          int in_features, float limit, float alpha, float shift, void* stream);
+int b200_moe_bf16_down(const void* h, const void* w, void* y, const void* tiles, const int32_t* num_tiles, void* status_word,
+                       int num_rows, int num_experts, int max_tiles, int tile_rows, int out_features, int in_features,
+                       void* stream);
+int b200_moe_gemm_f32(const float* x, const float* w, float* y, const void* tiles, const int32_t* num_tiles, int num_rows,
+                      int num_experts, int max_tiles, int out_features, int in_features, void* stream);
 
 /* ------------------------------------------------------------------- MoE -- */
 

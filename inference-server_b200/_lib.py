@@ -38,7 +38,7 @@ SIGNATURES = {
     "b200_dense_gemm_bf16": (c_int, [c_void_p] * 4 + [c_size_t, c_void_p] + [c_int] * 4 + [c_void_p]),
     "b200_dense_gemm_bf16_f32": (c_int, [c_void_p] * 4 + [c_size_t, c_void_p] + [c_int] * 4 + [c_void_p]),
     "b200_dense_gemm_grouped": (c_int, [c_void_p] * 4 + [c_int] * 9 + [c_void_p]),
-    "b200_proj_split_gemm": (c_int, [c_void_p] * 8 + [c_int] + [c_void_p] * 3 + [c_int] * 5 + [c_void_p]),
+    "b200_proj_split_gemm": (c_int, [c_void_p] * 10 + [c_int] + [c_void_p] * 3 + [c_int] * 5 + [c_void_p]),
     "b200_dense_glu_gemm": (c_int, [c_void_p] * 4 + [c_int] * 3 + [c_float] * 2 + [c_void_p]),
     "b200_gemm_f32": (c_int, [c_void_p] * 3 + [c_int] * 9 + [c_void_p]),
     "b200_embed_sinusoid": (c_int, [c_void_p] * 7 + [c_int] * 6 + [c_void_p]),
@@ -49,8 +49,20 @@ SIGNATURES = {
     "b200_latent_norm_append": (c_int, [c_void_p] * 2 + [c_float] + [c_int] * 3 + [c_void_p] * 3 + [c_int] * 3
                                 + [c_void_p, c_int, c_void_p]),
     "b200_gather_pages": (c_int, [c_void_p] * 3 + [c_int] * 5 + [c_void_p, c_int, c_void_p]),
-    "b200_split_store": (c_int, [c_void_p] * 7 + [c_int] + [c_void_p] * 3 + [c_int] * 5 + [c_void_p]),
-    "b200_clamped_glu": (c_int, [c_void_p] * 2 + [c_int] * 2 + [c_float] * 2 + [c_int, c_void_p]),
+    "b200_split_store": (c_int, [c_void_p] * 9 + [c_int] + [c_void_p] * 3 + [c_int] * 5 + [c_void_p]),
+    "b200_clamped_glu": (c_int, [c_void_p] * 2 + [c_int] * 2 + [c_float] * 3 + [c_int, c_void_p]),
+    "b200_moe_gemm_f32": (c_int, [c_void_p] * 5 + [c_int] * 5 + [c_void_p]),
+    "b200_moe_bf16_gate_up": (c_int, [c_void_p] * 6 + [c_int] * 6 + [c_float] * 3 + [c_void_p]),
+    "b200_moe_bf16_down": (c_int, [c_void_p] * 6 + [c_int] * 6 + [c_void_p]),
+    "b200_moe_route_sigmoid": (c_int, [c_void_p] + [c_int] * 5 + [c_float] + [c_void_p] * 3),
+    "b200_moe_permute_copy": (c_int, [c_void_p] * 2 + [c_int] * 5 + [c_void_p] * 5 + [c_size_t, c_void_p]),
+    "b200_residual_norm": (c_int, [c_void_p] * 5 + [c_int] + [c_void_p] * 3 + [c_float] + [c_int] * 4 + [c_void_p, c_int, c_void_p]),
+    "b200_mix_heads": (c_int, [c_void_p] * 3 + [c_int] * 5 + [c_void_p]),
+    "b200_conv_silu": (c_int, [c_void_p] * 2 + [c_int] + [c_void_p] * 3 + [c_int] * 4 + [c_void_p] * 2 + [c_int, c_void_p]),
+    "b200_group_norm_gate": (c_int, [c_void_p] * 3 + [c_float] + [c_int] * 5 + [c_float, c_void_p] + [c_int] * 2 + [c_void_p]),
+    "b200_state_scan": (c_int, [c_void_p] + [c_int] * 4 + [c_void_p] * 9 + [c_int] * 7 + [c_float, c_int, c_void_p]),
+    "b200_mixed_attn": (c_int, [c_void_p] * 4 + [c_int] + [c_void_p] * 2 + [c_int] * 2 + [c_void_p, c_int, c_float, c_void_p]
+                        + [c_int] * 9 + [c_void_p]),
     "b200_argmax_rows": (c_int, [c_void_p] * 2 + [c_int] * 2 + [c_void_p]),
     "b200_qkv_rope_append_supported": (c_int, [c_int, c_int]),
     "b200_qkv_rope_append_gemm": (c_int, [c_void_p] * 12 + [c_int] * 5 + [c_float] + [c_int] * 4 + [c_void_p]),

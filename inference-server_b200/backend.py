@@ -48,12 +48,14 @@ PAGE = 16
 
 @dataclass
 class SeqKV:
-    """KV handle of one sequence: which pages hold it and how many tokens are valid."""
+    """KV handle of one sequence: which pages hold it, how many tokens are valid, and, for models with recurrent layers, the
+    slot of its state."""
 
     block_ids: list[int]
     ctx_len: int
     private_blocks: list = field(default_factory=list)  # allocator handles this row must give back
     reserve_tokens: int = 0
+    slot: int | None = None
 
 
 @dataclass
@@ -91,6 +93,7 @@ class B200Backend:
         self._eos_ids: set[int] = set(eos_ids or ())
         self._lock = threading.Lock()  # the scheduler takes backend._lock (scheduler.py:184)
         self._alloc = _FreeListAllocator(engine.num_blocks) if engine is not None else None
+        self._slots = _FreeListAllocator(getattr(engine, "num_slots", 0))
         self.max_new_tokens = max_new_tokens
         self._table_cpu = None
         self._lens_cpu = None
@@ -150,6 +153,7 @@ class B200Backend:
             self.engine = self._engine_from_model(model, num_blocks, max_batch, max_pages_per_seq)
             del model
         self._alloc = _FreeListAllocator(self.engine.num_blocks)
+        self._slots = _FreeListAllocator(getattr(self.engine, "num_slots", 0))
         self._table_cpu = self._lens_cpu = self._synced_batch = None
         if self.cache_adapter is not None:
             self.set_cache_adapter(self.cache_adapter)
@@ -258,6 +262,29 @@ class B200Backend:
         else:
             self.cache_adapter.block_manager.free(handles)
 
+    # A sequence of a model with recurrent layers holds one state slot beside its pages, from its first prompt pass until its
+    # row goes.  Models that keep everything in pages have no slots and their handles carry None.
+    def _take_slot(self) -> int | None:
+        if not getattr(self.engine, "num_slots", 0):
+            return None
+        if not self._slots.free:
+            raise MemoryError(f"all {self.engine.num_slots} state slots are taken")
+        return self._slots.allocate(1)[0]
+
+    def _give_back_slot(self, slot: int | None) -> None:
+        if slot is not None:
+            self._slots.release([slot])
+
+    def _release_row(self, row: SeqKV) -> None:
+        self._give_back(row.private_blocks)
+        row.private_blocks = []
+        self._give_back_slot(row.slot)
+        row.slot = None
+
+    @staticmethod
+    def _slot_arg(slot: int | None) -> dict:
+        return {} if slot is None else {"slot": slot}
+
     # -------------------------------------------------------------- prefill
     def _lookup(self, token_ids: list[int], session_id: str):
         """Prefix lookup as TorchBackend does (torch_backend.py:113-119).
@@ -321,18 +348,20 @@ class B200Backend:
                              f"the block table is {self.engine.max_pages} wide")
         matched, shared_ids, tail, held = self._lookup(token_ids, session_id)
         self.last_cache_hit_tokens = matched
-        handles = []
+        handles, slot = [], None
         try:
             ids, handles = self._take_pages(total_pages - len(shared_ids))
-            kv = SeqKV(block_ids=shared_ids + ids, ctx_len=n, private_blocks=handles)
+            slot = self._take_slot()
+            kv = SeqKV(block_ids=shared_ids + ids, ctx_len=n, private_blocks=handles, slot=slot)
             tail_blocks, held = held, []
             self._adopt_tail(kv, len(shared_ids) * PAGE, tail, tail_blocks)
-            first, _ = self.engine.prefill(token_ids, kv.block_ids, cached_tokens=matched)
+            first, _ = self.engine.prefill(token_ids, kv.block_ids, cached_tokens=matched, **self._slot_arg(slot))
             self._check_status("prefill")
         except BaseException:
             for blk in held:
                 blk.release()
             self._give_back(handles)
+            self._give_back_slot(slot)
             self._release_shared(shared_ids)
             raise
         self._store(token_ids, kv, matched, session_id)
@@ -384,15 +413,22 @@ class B200Backend:
             raise ValueError(f"{new_len} tokens plus {self.max_new_tokens} reserved need {total_pages} pages; "
                              f"the block table is {self.engine.max_pages} wide")
         ids, handles = self._take_pages(total_pages - len(kv.block_ids))
+        slot = kv.slot
         try:
+            if partial_kv is None:
+                slot = self._take_slot()
             # only the tokens past `cached_tokens` are embedded; the earlier ones are already pages
             tokens = [0] * kv.ctx_len + list(chunk_token_ids)
             asked = {} if want is None else {"want": [kv.ctx_len + w for w in want]}
-            last, self.last_logits = self.engine.prefill(tokens, kv.block_ids + ids, cached_tokens=kv.ctx_len, **asked)
+            last, self.last_logits = self.engine.prefill(tokens, kv.block_ids + ids, cached_tokens=kv.ctx_len, **asked,
+                                                             **self._slot_arg(slot))
             self._check_status("prefill_chunk")
         except BaseException:
             self._give_back(handles)
+            if partial_kv is None:
+                self._give_back_slot(slot)
             raise
+        kv.slot = slot
         kv.block_ids += ids
         kv.private_blocks += handles
         kv.ctx_len = new_len
@@ -404,8 +440,7 @@ class B200Backend:
     # --------------------------------------------------------------- batching
     def _reclaim_rows(self, rows: list) -> None:
         for row in rows:
-            self._give_back(row.private_blocks)
-            row.private_blocks = []
+            self._release_row(row)
         rows.clear()
 
     def splice_into_batched(self, batched_kv, new_kv, new_kv_len: int):
@@ -429,8 +464,7 @@ class B200Backend:
 
     def remove_row_from_cache(self, batched_kv, row_idx: int):
         row = batched_kv.rows.pop(row_idx)
-        self._give_back(row.private_blocks)
-        row.private_blocks = []
+        self._release_row(row)
         batched_kv.dirty = True
         return batched_kv
 
@@ -446,14 +480,18 @@ class B200Backend:
                 pin = torch.cuda.is_available()
                 self._table_cpu = torch.zeros(eng.max_batch, eng.max_pages, dtype=torch.int32, pin_memory=pin)
                 self._lens_cpu = torch.zeros(eng.max_batch, dtype=torch.int32, pin_memory=pin)
+                self._slots_cpu = torch.zeros(eng.max_batch, dtype=torch.int32, pin_memory=pin)
             self._table_cpu.zero_()
             for i, row in enumerate(batch.rows):
                 if len(row.block_ids) > eng.max_pages:
                     raise ValueError("sequence needs more pages than the block table is wide")
                 self._table_cpu[i, : len(row.block_ids)] = torch.tensor(row.block_ids, dtype=torch.int32)
                 self._lens_cpu[i] = row.ctx_len
+                self._slots_cpu[i] = row.slot or 0
             eng.block_table.copy_(self._table_cpu, non_blocking=True)
             eng.ctx_lens.copy_(self._lens_cpu, non_blocking=True)
+            if getattr(eng, "num_slots", 0):
+                eng.state_slots.copy_(self._slots_cpu, non_blocking=True)
             batch.dirty = False
             self._synced_batch = weakref.ref(batch)  # weak: a dropped batch must still give its pages back
         return B
@@ -514,19 +552,25 @@ class B200Backend:
                 row.private_blocks += handles
                 batch.dirty = True
         ids, handles = self._take_pages(total_pages - len(kv.block_ids))
+        slot = kv.slot
         try:
+            if partial_kv is None:
+                slot = self._take_slot()
             B = self._sync_table(batch)
             tok = current_tokens.reshape(-1).to(torch.int64)
             eng.tokens[:B].copy_(tok, non_blocking=True)
-            nxt, last, _ = eng.mixed_step(B, list(chunk_token_ids), kv.block_ids + ids, kv.ctx_len)
+            nxt, last, _ = eng.mixed_step(B, list(chunk_token_ids), kv.block_ids + ids, kv.ctx_len, **self._slot_arg(slot))
             out = nxt.to("cpu")
             self._check_status("decode_step_with_prefill_chunk")
         except BaseException:
             self._give_back(handles)
+            if partial_kv is None:
+                self._give_back_slot(slot)
             batch.dirty = True  # the device lengths may have moved; re-upload them from the rows next time
             raise
         for row in batch.rows:
             row.ctx_len += 1
+        kv.slot = slot
         kv.block_ids += ids
         kv.private_blocks += handles
         kv.ctx_len = new_len

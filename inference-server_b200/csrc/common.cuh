@@ -255,17 +255,20 @@ __device__ __forceinline__ int first_visible(int L, int chunk) {
 __device__ __forceinline__ float head_gate(const float* gate, size_t i) {
   return gate == nullptr ? 1.f : 1.f / (1.f + expf(-gate[i]));
 }
-// Clamped gated unit: g * sigmoid(alpha g) * (u + 1) with g capped at `limit` and u held to +-limit.
-__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float alpha) {
+// Clamped gated unit: g * sigmoid(alpha g) * (u + shift) with g capped at `limit` and u held to +-limit; an infinite limit,
+// alpha 1 and shift 0 make it silu(g) * u.
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float alpha, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+  return g / (1.f + expf(-alpha * g)) * (u + shift);
 }
-__device__ __forceinline__ float clamped_glu_fast(float g, float u, float limit, float alpha) {
+__device__ __forceinline__ float clamped_glu_fast(float g, float u, float limit, float alpha, float shift) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
-  return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);
+  return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + shift);
 }
+__device__ __forceinline__ float silu_of(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + expf(-z)); }
 template <typename T>
 __device__ __forceinline__ float to_f32(T v);
 template <>

@@ -70,10 +70,11 @@ constexpr int kDenseMaxRows = 256;                // rows of X per MMA (its N)
 
 enum : int { kEpiStore = 0, kEpiArgmax = 1, kEpiQkvRope = 2, kEpiSplit = 3, kEpiGlu = 4 };
 enum : int { kSegBf16 = 0, kSegF32 = 1, kSegPages = 2 };
-constexpr int kMaxSegs = 4;
+enum : int { kActNone = 0, kActSilu = 1, kActSigmoid = 2 };
+constexpr int kMaxSegs = 8;
 // kEpiSplit: features [end of the segment before, end) go to `ptr`.
 struct DenseSeg {
-  int end, kind;
+  int end, kind, act;  // act: what the feature goes through before it is stored (kAct*)
   int heads, dim;  // kSegPages: pool [num_blocks, heads, page, dim]
   void* ptr;       // kSegBf16 / kSegF32: [M, end - begin]
 };
@@ -97,8 +98,14 @@ struct DenseParams {
   // kEpiSplit (positions, block_table, page, num_blocks, max_pages below serve its page segments; positions NULL =
   // row m is position m, block_table NULL = page p of the sequence is block p)
   const float* col_scale;  // [N] or NULL
+  const float* col_bias;   // [N] or NULL, added after the scale
   DenseSeg segs[kMaxSegs];
-  float glu_limit, glu_alpha;  // kEpiGlu
+  float glu_limit, glu_alpha, glu_shift;  // kEpiGlu
+  // products of experts: X's rows are sorted by expert and cut into tiles of at most xbox rows of one expert; an item is
+  // (tile, W tile of that expert) instead of (group, W tile, rows of X).  M bounds the tiles' rows.
+  const MoeTile* tiles;
+  const int* num_tiles;
+  int num_experts, max_tiles;
   float* part_val;    // kEpiArgmax: [grid * 4, 256] candidates per TMEM lane quarter
   int* part_idx;
   float* exchange;    // kEpiStore, split K: [tile][finishing CTA][source CTA][rows_per][128] fp32
@@ -173,6 +180,33 @@ __device__ __forceinline__ uint32_t pack_row_pair(float row_i, float row_i1, int
   return odd ? pack_bf16x2(other, row_i1) : pack_bf16x2(row_i, other);
 }
 
+// Which weight rows and which rows of X an item multiplies: W tile nt of group (or expert) g, rows [m0, m_end).
+struct DenseItem {
+  int g, nt, m0, m_end;
+};
+__device__ __forceinline__ DenseItem dense_item(const DenseParams& p, int tile) {
+  DenseItem it;
+  if (p.tiles != nullptr) {
+    const int t = tile / p.n_tiles;
+    it.nt = tile - t * p.n_tiles;
+    MoeTile mt = p.tiles[t];
+    if (mt.expert < 0 || mt.expert >= p.num_experts || mt.row0 < 0 || mt.rows < 0 || mt.rows > p.xbox || mt.row0 + mt.rows > p.M) {
+      set_error(p.err, kErrDevBadExpert);
+      mt.expert = mt.row0 = mt.rows = 0;  // computed on the first rows, nothing stored
+    }
+    it.g = mt.expert;
+    it.m0 = mt.row0;
+    it.m_end = mt.row0 + mt.rows;
+  } else {
+    const int gn = tile / p.m_tiles, mt = tile - gn * p.m_tiles;
+    it.g = gn / p.n_tiles;
+    it.nt = gn - it.g * p.n_tiles;
+    it.m0 = mt * p.xbox;
+    it.m_end = p.M;
+  }
+  return it;
+}
+
 template <int A_TILES, int EPI>
 __global__ void __launch_bounds__(kDenseThreads, 1)
 dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map,
@@ -221,7 +255,15 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
 
   const int ks = p.ksplit;
   const int kb_per = (p.K + kDenseBlockK - 1) / kDenseBlockK / ks;  // K blocks of one work item
-  const int total = p.groups * p.n_tiles * p.m_tiles * ks;
+  int listed = p.groups * p.m_tiles;
+  if (p.tiles != nullptr) {
+    listed = *p.num_tiles;
+    if (listed < 0 || listed > p.max_tiles) {
+      if (threadIdx.x == 0) set_error(p.err, kErrDevBadExpert);
+      listed = 0;
+    }
+  }
+  const int total = listed * p.n_tiles * ks;
   const uint32_t stage_tx = A_TILES * kDenseWBytes + static_cast<uint32_t>(p.xbox) * 128u;
 
   if (warp == 0) {
@@ -231,8 +273,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
       bool alive = true;
       for (int w = blockIdx.x; w < total && alive; w += gridDim.x) {
         const int tile = w / ks, kidx = w - tile * ks;
-        const int gn = tile / p.m_tiles, mt = tile - gn * p.m_tiles;
-        const int g = gn / p.n_tiles, nt = gn - g * p.n_tiles;
+        const DenseItem item = dense_item(p, tile);
+        const int g = item.g, nt = item.nt;
         for (int kb = 0; kb < kb_per; ++kb, ++it) {
           const uint32_t slot = it % kStages, phase = (it / kStages) & 1;
           alive = mbar_wait(bar_empty + 8 * slot, phase ^ 1, p.err);
@@ -244,7 +286,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           for (int a = 0; a < A_TILES; ++a)
             tma_load_2d(sw + a * kDenseWBytes, &w_map, bar_full + 8 * slot, kx,
                         g * p.w_step + (nt * A_TILES + a) * 128);
-          tma_load_2d(sx, &x_map, bar_full + 8 * slot, g * p.x_step + kx, mt * p.xbox);
+          tma_load_2d(sx, &x_map, bar_full + 8 * slot, g * p.x_step + kx, item.m0);
         }
       }
     }
@@ -301,11 +343,10 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
     uint32_t item = 0;
     bool alive = true;
     for (int w = blockIdx.x; w < total && alive; w += gridDim.x, ++item) {
-      const int tile = w / ks;
-      const int gn = tile / p.m_tiles, mt = tile - gn * p.m_tiles;
-      const int g = gn / p.n_tiles, nt = gn - g * p.n_tiles;
+      const DenseItem di = dense_item(p, w / ks);
+      const int g = di.g, nt = di.nt;
       const uint32_t buf = item % kBufs, aphase = (item / kBufs) & 1;
-      const int m0 = mt * p.xbox;
+      const int m0 = di.m0, m_end = di.m_end;
       // kEpiQkvRope: position and page of the rows this warp will finish (lane i: row (warp - 2) + 8 i of the
       // tile), fetched while the MMAs of the item are still running; -1 = not a row, or reported as bad
       int row_pos = -1, row_page = -1;
@@ -329,7 +370,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
       // row i of the chunk), fetched while the MMAs of the item are still running; page -1 = not written
       int seg_kind = -1, seg_page_stride = 0, seg_dim = 0, seg_ld = 0, row_at4[4];
       void* seg_ptr = nullptr;
-      float seg_scale = 1.f;
+      float seg_scale = 1.f, seg_bias = 0.f;
+      int seg_act = kActNone;
       if (EPI == kEpiSplit) {
         const int n = nt * 128 + t;
         int begin = 0;
@@ -341,6 +383,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           if (n >= begin && n < sg.end) {
             const int local = n - begin;
             seg_kind = sg.kind;
+            seg_act = sg.act;
             if (sg.kind == kSegPages) {
               const int head = local / sg.dim;
               seg_dim = sg.dim;
@@ -355,6 +398,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           begin = max(begin, sg.end);
         }
         if (p.col_scale != nullptr && n < p.N) seg_scale = p.col_scale[n];
+        if (p.col_bias != nullptr && n < p.N) seg_bias = p.col_bias[n];
 #pragma unroll
         for (int cc = 0; cc < 4; ++cc) {
           row_at4[cc] = -1;
@@ -389,7 +433,14 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           tmem_ld_wait();
           const int left = p.M - (m0 + c * 32);  // rows of this chunk that exist
 #pragma unroll
-          for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * seg_scale);
+          for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(fmaf(__uint_as_float(v[i]), seg_scale, seg_bias));
+          if (seg_act != kActNone) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const float z = __uint_as_float(v[i]);
+              v[i] = __float_as_uint(__fdividef(seg_act == kActSilu ? z : 1.f, 1.f + __expf(-z)));
+            }
+          }
           // Segments begin at even features and are even wide (checked on the host), so a pair of lanes is in one segment.
           if (__any_sync(0xffffffffu, seg_kind == kSegPages || seg_kind == kSegBf16)) {
             __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(seg_ptr) - (lane & 1);
@@ -424,11 +475,11 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
           tmem_ld32(lane_addr + (A_TILES > 1 ? kDenseMaxRows : 0) + c * 32, u);
           tmem_ld_wait();
           // p.N is a multiple of 128: every lane has a feature
-          const int left = p.M - (m0 + c * 32);
+          const int left = m_end - (m0 + c * 32);
           __nv_bfloat16* dst = p.y + static_cast<size_t>(m0 + c * 32 + (lane & 1)) * p.ldy + (n & ~1);
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            v[i] = __float_as_uint(clamped_glu_fast(__uint_as_float(v[i]), __uint_as_float(u[i]), p.glu_limit, p.glu_alpha));
+            v[i] = __float_as_uint(clamped_glu_fast(__uint_as_float(v[i]), __uint_as_float(u[i]), p.glu_limit, p.glu_alpha, p.glu_shift));
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
             const uint32_t two = pack_row_pair(__uint_as_float(v[i]), __uint_as_float(v[i + 1]), lane);
@@ -457,7 +508,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
             tmem_ld32(t0 + c * 32, v);
             tmem_ld_wait();
             if (p.y_f32 == nullptr && ((p.N | p.ldy | p.y_step) & 1) == 0) {
-              const int left = p.M - (m0 + c * 32);
+              const int left = m_end - (m0 + c * 32);
               __nv_bfloat16* dst = p.y + static_cast<size_t>(m0 + c * 32 + (lane & 1)) * p.ldy + g * p.y_step + (n & ~1);
 #pragma unroll
               for (int i = 0; i < 32; i += 2) {
@@ -469,7 +520,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_consta
               for (int i = 0; i < 32; ++i) {
                 const int m = m0 + c * 32 + i;
                 const size_t at = static_cast<size_t>(m) * p.ldy + g * p.y_step + n;
-                if (m < p.M) {
+                if (m < m_end) {
                   if (p.y_f32 != nullptr) p.y_f32[at] = __uint_as_float(v[i]);
                   else p.y[at] = __float2bfloat16(__uint_as_float(v[i]));
                 }
@@ -1003,8 +1054,9 @@ extern "C" int b200_dense_gemm_grouped(const void* x, const void* w, void* y, vo
   return launch_dense<1, kEpiStore>(w_map, x_map, p, items < sms ? items : sms, as_stream(stream));
 }
 
-extern "C" int b200_proj_split_gemm(const void* x, const void* w, const float* col_scale, const int32_t* seg_end,
-                                    const int32_t* seg_kind, const int32_t* seg_heads, const int32_t* seg_dim,
+extern "C" int b200_proj_split_gemm(const void* x, const void* w, const float* col_scale, const float* col_bias,
+                                    const int32_t* seg_end, const int32_t* seg_kind, const int32_t* seg_act,
+                                    const int32_t* seg_heads, const int32_t* seg_dim,
                                     void* const* seg_ptr, int num_segs, const int32_t* positions,
                                     const int32_t* block_table, void* status_word, int num_rows, int in_features,
                                     int page_size, int num_blocks, int max_pages_per_seq, void* stream) {
@@ -1025,7 +1077,9 @@ extern "C" int b200_proj_split_gemm(const void* x, const void* w, const float* c
       B200_REQUIRE(begin % 2 == 0 && seg_end[i] % 2 == 0 && (seg_kind[i] != kSegPages || seg_dim[i] % 2 == 0) &&
                        (reinterpret_cast<uintptr_t>(seg_ptr[i]) & 3) == 0,
                    "proj_split_gemm: bf16 segment %d must begin and end at even features, 4-byte aligned", i);
-    p.segs[i] = DenseSeg{seg_end[i], seg_kind[i], seg_heads[i], seg_dim[i], seg_ptr[i]};
+    const int act = seg_act ? seg_act[i] : 0;
+    B200_REQUIRE(act >= kActNone && act <= kActSigmoid, "proj_split_gemm: segment activation %d", act);
+    p.segs[i] = DenseSeg{seg_end[i], seg_kind[i], act, seg_heads[i], seg_dim[i], seg_ptr[i]};
     begin = seg_end[i];
   }
   int rc = dense_args_ok(x, w, num_rows, begin, in_features, "proj_split_gemm");
@@ -1045,6 +1099,7 @@ extern "C" int b200_proj_split_gemm(const void* x, const void* w, const float* c
   p.xbox = pick_xbox_waves(num_rows, p.n_tiles, 128, sms);
   p.m_tiles = (num_rows + p.xbox - 1) / p.xbox;
   p.col_scale = col_scale;
+  p.col_bias = col_bias;
   p.positions = positions;
   p.block_table = block_table;
   B200_REQUIRE(page_size > 0 && (page_size & (page_size - 1)) == 0, "proj_split_gemm: page_size %d is not a power of two",
@@ -1087,6 +1142,7 @@ extern "C" int b200_dense_glu_gemm(const void* x, const void* w_interleaved, voi
   p.m_tiles = (num_rows + p.xbox - 1) / p.xbox;
   p.glu_limit = limit;
   p.glu_alpha = alpha;
+  p.glu_shift = 1.f;
   CUtensorMap w_map, x_map;
   rc = get_tensor_map_2d(w_interleaved, static_cast<uint64_t>(2) * inter, in_features, 2, 128, 64, &w_map);
   if (rc) return rc;
@@ -1094,6 +1150,85 @@ extern "C" int b200_dense_glu_gemm(const void* x, const void* w_interleaved, voi
   if (rc) return rc;
   const int items = p.n_tiles * p.m_tiles;
   return launch_dense<2, kEpiGlu>(w_map, x_map, p, items < sms ? items : sms, as_stream(stream));
+}
+
+namespace b200 {
+
+// What the two products of an expert layer share: rows sorted by expert, cut into tiles.
+static int expert_params(const void* x, const void* w, void* y, const void* tiles, const int32_t* num_tiles, void* status_word,
+                         int num_rows, int num_experts, int max_tiles, int tile_rows, int w_rows, int in_features,
+                         const char* who, DenseParams* p) {
+  int rc = dense_args_ok(x, w, num_rows, w_rows, in_features, who);
+  if (rc) return rc;
+  B200_REQUIRE(y && tiles && num_tiles && num_experts > 0 && max_tiles > 0 && (reinterpret_cast<uintptr_t>(y) & 3) == 0,
+               "%s: null pointer, or no experts", who);
+  B200_REQUIRE(tile_rows >= 32 && tile_rows <= kDenseMaxRows && tile_rows % 32 == 0, "%s: tiles of %d rows", who, tile_rows);
+  rc = check_device(nullptr);
+  if (rc) return rc;
+  p->y = static_cast<__nv_bfloat16*>(y);
+  p->groups = 1;
+  p->err = static_cast<int*>(status_word);
+  p->M = num_rows;
+  p->K = in_features;
+  p->ksplit = 1;
+  p->xbox = tile_rows;
+  p->m_tiles = 1;
+  p->tiles = static_cast<const MoeTile*>(tiles);
+  p->num_tiles = num_tiles;
+  p->num_experts = num_experts;
+  p->max_tiles = max_tiles;
+  return 0;
+}
+
+}  // namespace b200
+
+extern "C" int b200_moe_bf16_gate_up(const void* x, const void* w_interleaved, void* h, const void* tiles,
+                                     const int32_t* num_tiles, void* status_word, int num_rows, int num_experts, int max_tiles,
+                                     int tile_rows, int inter, int in_features, float limit, float alpha, float shift,
+                                     void* stream) {
+  DenseParams p{};
+  int rc = expert_params(x, w_interleaved, h, tiles, num_tiles, status_word, num_rows, num_experts, max_tiles, tile_rows,
+                         2 * inter, in_features, "moe_bf16_gate_up", &p);
+  if (rc) return rc;
+  B200_REQUIRE(inter % 128 == 0, "moe_bf16_gate_up: %d inner features (a multiple of 128)", inter);
+  p.ldy = inter;
+  p.N = inter;
+  p.n_tiles = inter / 128;
+  p.w_step = 2 * inter;
+  p.glu_limit = limit;
+  p.glu_alpha = alpha;
+  p.glu_shift = shift;
+  int sms = 148;
+  rc = device_sm_count(&sms);
+  if (rc) return rc;
+  CUtensorMap w_map, x_map;
+  rc = get_tensor_map_2d(w_interleaved, static_cast<uint64_t>(num_experts) * 2 * inter, in_features, 2, 128, 64, &w_map);
+  if (rc) return rc;
+  rc = get_tensor_map_2d(x, num_rows, in_features, 2, tile_rows, 64, &x_map);
+  if (rc) return rc;
+  return launch_dense<2, kEpiGlu>(w_map, x_map, p, sms, as_stream(stream));
+}
+
+extern "C" int b200_moe_bf16_down(const void* h, const void* w, void* y, const void* tiles, const int32_t* num_tiles,
+                                  void* status_word, int num_rows, int num_experts, int max_tiles, int tile_rows,
+                                  int out_features, int in_features, void* stream) {
+  DenseParams p{};
+  int rc = expert_params(h, w, y, tiles, num_tiles, status_word, num_rows, num_experts, max_tiles, tile_rows, out_features,
+                         in_features, "moe_bf16_down", &p);
+  if (rc) return rc;
+  p.ldy = out_features;
+  p.N = out_features;
+  p.n_tiles = (out_features + 127) / 128;
+  p.w_step = out_features;
+  int sms = 148;
+  rc = device_sm_count(&sms);
+  if (rc) return rc;
+  CUtensorMap w_map, x_map;
+  rc = get_tensor_map_2d(w, static_cast<uint64_t>(num_experts) * out_features, in_features, 2, 128, 64, &w_map);
+  if (rc) return rc;
+  rc = get_tensor_map_2d(h, num_rows, in_features, 2, tile_rows, 64, &x_map);
+  if (rc) return rc;
+  return launch_dense<1, kEpiStore>(w_map, x_map, p, sms, as_stream(stream));
 }
 
 extern "C" int b200_qkv_rope_append_supported(int head_dim, int in_features) {

@@ -10,103 +10,12 @@
 // that p itself reads (a CUDA graph's warm-up runs the same step several times).
 // A sequence's state is taken, moved and given back with its pages, and there is no slot to manage.
 
-#include <initializer_list>
-
-#include "common.cuh"
-#include "host.h"
+#include "glue.cuh"
 
 namespace b200 {
 
-constexpr int kGlueMaxSegs = 4;
+constexpr int kGlueMaxSegs = 8;
 constexpr int kFastTaps = 5;  // convolutions of up to this many taps keep their rows in registers
-
-template <typename T>
-__device__ __forceinline__ void load8(const T* p, float (&f)[8]);
-template <>
-__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&f)[8]) {
-  const uint4 raw = *reinterpret_cast<const uint4*>(p);
-  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    const float2 v = __bfloat1622float2(h[j]);
-    f[2 * j] = v.x;
-    f[2 * j + 1] = v.y;
-  }
-}
-template <>
-__device__ __forceinline__ void load8<float>(const float* p, float (&f)[8]) {
-  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
-  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-}
-template <typename T>
-__device__ __forceinline__ void store8(T* p, const float (&f)[8]);
-template <>
-__device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&f)[8]) {
-  uint4 raw;
-  raw.x = pack_bf16x2(f[0], f[1]);
-  raw.y = pack_bf16x2(f[2], f[3]);
-  raw.z = pack_bf16x2(f[4], f[5]);
-  raw.w = pack_bf16x2(f[6], f[7]);
-  *reinterpret_cast<uint4*>(p) = raw;
-}
-template <>
-__device__ __forceinline__ void store8<float>(float* p, const float (&f)[8]) {
-  reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
-  reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
-}
-template <typename T>
-__device__ __forceinline__ float round_to(float v) { return to_f32<T>(from_f32<T>(v)); }
-
-// Eight columns as they lie in memory, so that several rows can be asked for before the first is used.
-template <typename T>
-struct Raw8;
-template <>
-struct Raw8<__nv_bfloat16> {
-  uint4 v;
-  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint4*>(p); }
-  __device__ __forceinline__ void zero() { v = make_uint4(0u, 0u, 0u, 0u); }
-  __device__ __forceinline__ void get(float (&f)[8]) const {
-    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float2 t = __bfloat1622float2(h[j]);
-      f[2 * j] = t.x;
-      f[2 * j + 1] = t.y;
-    }
-  }
-};
-template <>
-struct Raw8<float> {
-  float4 a, b;
-  __device__ __forceinline__ void load(const float* p) {
-    a = reinterpret_cast<const float4*>(p)[0];
-    b = reinterpret_cast<const float4*>(p)[1];
-  }
-  __device__ __forceinline__ void zero() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
-  __device__ __forceinline__ void get(float (&f)[8]) const {
-    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
-    f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-  }
-};
-
-// Where the pages of a row or sequence are; -1 and a status code for anything outside.
-struct PageMap {
-  int page, num_blocks, max_pages;
-  int* err;
-};
-__device__ __forceinline__ int page_of(const PageMap& pm, const int* table_row, int pos) {
-  if (pos < 0 || pos >= pm.max_pages * pm.page) {
-    set_error(pm.err, kErrDevBadCtxLen);
-    return -1;
-  }
-  const int id = table_row[pos / pm.page];
-  if (id < 0 || id >= pm.num_blocks) {
-    set_error(pm.err, kErrDevBadBlockId);
-    return -1;
-  }
-  return id;
-}
 
 template <typename T>
 __global__ void embed_sinusoid_kernel(const long long* __restrict__ tokens, const int* __restrict__ positions,
@@ -124,9 +33,14 @@ __global__ void embed_sinusoid_kernel(const long long* __restrict__ tokens, cons
     pos = 0;
   }
   const T* e = embed + static_cast<size_t>(tok) * ld;
+  float* o = x + static_cast<size_t>(m) * ld;
+  if (lo == nullptr) {  // no sinusoid
+    for (int c = threadIdx.x * 2; c < ld; c += blockDim.x * 2)
+      *reinterpret_cast<float2*>(o + c) = make_float2(c < width ? to_f32<T>(e[c]) : 0.f, c + 1 < width ? to_f32<T>(e[c + 1]) : 0.f);
+    return;
+  }
   const float* l = lo + static_cast<size_t>(pos & 63) * ld;
   const float* h = hi + static_cast<size_t>(pos >> 6) * ld;
-  float* o = x + static_cast<size_t>(m) * ld;
   for (int c = threadIdx.x * 2; c < ld; c += blockDim.x * 2) {
     const float2 a = *reinterpret_cast<const float2*>(h + c), b = *reinterpret_cast<const float2*>(l + c);
     float2 r;  // sin(a + b), cos(a + b)
@@ -388,13 +302,14 @@ __global__ void gather_pages_kernel(const uint4* __restrict__ pool, const int* _
 }
 
 struct GlueSegs {
-  int end[kGlueMaxSegs], kind[kGlueMaxSegs], heads[kGlueMaxSegs], dim[kGlueMaxSegs];
+  int end[kGlueMaxSegs], kind[kGlueMaxSegs], act[kGlueMaxSegs], heads[kGlueMaxSegs], dim[kGlueMaxSegs];
   void* ptr[kGlueMaxSegs];
   int count;
 };
 
 template <typename T>
-__global__ void split_store_kernel(const float* __restrict__ y, const float* __restrict__ col_scale, GlueSegs segs,
+__global__ void split_store_kernel(const float* __restrict__ y, const float* __restrict__ col_scale,
+                                   const float* __restrict__ col_bias, GlueSegs segs,
                                    const int* __restrict__ positions, const int* __restrict__ block_table, PageMap pm) {
   const int m = blockIdx.x, total = segs.end[segs.count - 1];
   const int pos = positions != nullptr ? positions[m] : m;
@@ -402,8 +317,11 @@ __global__ void split_store_kernel(const float* __restrict__ y, const float* __r
   for (int n = threadIdx.x; n < total; n += blockDim.x) {
     float v = y[static_cast<size_t>(m) * total + n];
     if (col_scale != nullptr) v *= col_scale[n];
+    if (col_bias != nullptr) v += col_bias[n];
     int s = 0, begin = 0;
     while (n >= segs.end[s]) begin = segs.end[s++];
+    if (segs.act[s] == 1) v = silu_of(v);
+    else if (segs.act[s] == 2) v = sigmoid_of(v);
     const int local = n - begin, wd = segs.end[s] - begin;
     if (segs.kind[s] == 0) {
       static_cast<T*>(segs.ptr[s])[static_cast<size_t>(m) * wd + local] = from_f32<T>(v);
@@ -425,13 +343,13 @@ __global__ void split_store_kernel(const float* __restrict__ y, const float* __r
 // gate_up [rows, 2 * inter], gate and up columns in alternating blocks of 128.
 template <typename T>
 __global__ void clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ out, long long total, int inter, float limit,
-                                   float alpha) {
+                                   float alpha, float shift) {
   const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= total) return;
   const long long m = i / inter;
   const int n = static_cast<int>(i - m * inter);
   const T* row = gu + m * 2 * inter + (n / 128) * 256 + n % 128;
-  out[i] = from_f32<T>(clamped_glu(to_f32<T>(row[0]), to_f32<T>(row[128]), limit, alpha));
+  out[i] = from_f32<T>(clamped_glu(to_f32<T>(row[0]), to_f32<T>(row[128]), limit, alpha, shift));
 }
 
 __global__ void __launch_bounds__(256)
@@ -477,10 +395,20 @@ argmax_rows_kernel(const float* __restrict__ logits, long long* __restrict__ out
 // Every element is summed over k in the same order whatever the shape.
 __global__ void __launch_bounds__(256)
 gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, float* __restrict__ y, int M, int N, int K,
-                int x_step, int w_step, int y_step, int ldx, int ldy) {
+                int x_step, int w_step, int y_step, int ldx, int ldy, const MoeTile* __restrict__ tiles,
+                const int* __restrict__ num_tiles, int num_experts) {
   __shared__ float xs[16][64 + 4], ws[16][64 + 4];
-  const int g = blockIdx.z;
-  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  int g = blockIdx.z, m0 = blockIdx.y * 64;
+  const int n0 = blockIdx.x * 64;
+  if (tiles != nullptr) {  // rows sorted by expert: blockIdx.y counts tiles of at most 64 rows of one expert
+    if (static_cast<int>(blockIdx.y) >= *num_tiles) return;
+    const MoeTile t = tiles[blockIdx.y];
+    if (t.expert < 0 || t.expert >= num_experts || t.row0 < 0 || t.rows < 0 || t.rows > 64 || t.row0 + t.rows > M) return;
+    g = t.expert;
+    m0 = t.row0;
+    M = t.row0 + t.rows;
+    x_step = y_step = 0;
+  }
   const int tid = threadIdx.x, r = tid >> 2, kq = (tid & 3) * 4;
   const int ty = tid >> 4, tx = tid & 15;
   float acc[4][4];
@@ -519,12 +447,6 @@ gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, float*
       if (n < N) y[static_cast<size_t>(m) * ldy + g * y_step + n] = acc[i][j];
     }
   }
-}
-
-static bool aligned16(std::initializer_list<const void*> ps) {
-  uintptr_t all = 0;
-  for (const void* p : ps) all |= reinterpret_cast<uintptr_t>(p);
-  return (all & 15) == 0;
 }
 
 template <typename T>
@@ -572,17 +494,10 @@ static int launch_short_conv(const void* h, const void* conv_w, int taps, void* 
 
 using namespace b200;
 
-#define B200_GLUE_DTYPE(name)                                                                        \
-  B200_REQUIRE(dtype == 0 || dtype == 1, name ": dtype %d is neither 0 (bf16) nor 1 (f32)", dtype);  \
-  {                                                                                                  \
-    int rc__ = check_device(nullptr);                                                                \
-    if (rc__) return rc__;                                                                           \
-  }
-
 extern "C" int b200_embed_sinusoid(const int64_t* tokens, const int32_t* positions, const void* embed, const float* lo,
                                    const float* hi, float* x, void* status_word, int num_rows, int width, int ld,
                                    int vocab, int n_hi, int dtype, void* stream) {
-  B200_REQUIRE(tokens && positions && embed && lo && hi && x, "embed_sinusoid: null pointer");
+  B200_REQUIRE(tokens && positions && embed && (lo != nullptr) == (hi != nullptr) && x, "embed_sinusoid: null pointer");
   B200_REQUIRE(num_rows >= 0 && width > 0 && ld >= width && ld % 8 == 0 && vocab > 0 && n_hi > 0,
                "embed_sinusoid: rows %d, width %d, pitch %d", num_rows, width, ld);
   B200_REQUIRE(aligned16({lo, hi, x}), "embed_sinusoid: tables and x must be 16-byte aligned");
@@ -685,8 +600,8 @@ extern "C" int b200_gather_pages(const void* c_pool, const int32_t* block_table_
   return 0;
 }
 
-extern "C" int b200_split_store(const float* y, const float* col_scale, const int32_t* seg_end, const int32_t* seg_kind,
-                                const int32_t* seg_heads, const int32_t* seg_dim, void* const* seg_ptr, int num_segs,
+extern "C" int b200_split_store(const float* y, const float* col_scale, const float* col_bias, const int32_t* seg_end,
+                                const int32_t* seg_kind, const int32_t* seg_act, const int32_t* seg_heads, const int32_t* seg_dim, void* const* seg_ptr, int num_segs,
                                 const int32_t* positions, const int32_t* block_table, void* status_word, int num_rows,
                                 int page_size, int num_blocks, int max_pages_per_seq, int dtype, void* stream) {
   B200_REQUIRE(y && seg_end && seg_kind && seg_heads && seg_dim && seg_ptr && num_segs >= 1 && num_segs <= kGlueMaxSegs,
@@ -702,6 +617,7 @@ extern "C" int b200_split_store(const float* y, const float* col_scale, const in
                    "split_store: page segment %d does not match its pool", i);
     s.end[i] = seg_end[i];
     s.kind[i] = seg_kind[i];
+    s.act[i] = seg_act ? seg_act[i] : 0;
     s.heads[i] = seg_heads[i];
     s.dim[i] = seg_dim[i];
     s.ptr[i] = seg_ptr[i];
@@ -711,15 +627,15 @@ extern "C" int b200_split_store(const float* y, const float* col_scale, const in
   if (num_rows <= 0) return 0;
   const PageMap pm{page_size, num_blocks, max_pages_per_seq, static_cast<int*>(status_word)};
   if (dtype == 0)
-    split_store_kernel<__nv_bfloat16><<<num_rows, 256, 0, as_stream(stream)>>>(y, col_scale, s, positions, block_table, pm);
+    split_store_kernel<__nv_bfloat16><<<num_rows, 256, 0, as_stream(stream)>>>(y, col_scale, col_bias, s, positions, block_table, pm);
   else
-    split_store_kernel<float><<<num_rows, 256, 0, as_stream(stream)>>>(y, col_scale, s, positions, block_table, pm);
+    split_store_kernel<float><<<num_rows, 256, 0, as_stream(stream)>>>(y, col_scale, col_bias, s, positions, block_table, pm);
   B200_CUDA(cudaGetLastError());
   return 0;
 }
 
-extern "C" int b200_clamped_glu(const void* gate_up, void* out, int num_rows, int inter, float limit, float alpha, int dtype,
-                                void* stream) {
+extern "C" int b200_clamped_glu(const void* gate_up, void* out, int num_rows, int inter, float limit, float alpha, float shift,
+                                int dtype, void* stream) {
   B200_REQUIRE(gate_up && out && num_rows >= 0 && inter > 0 && inter % 128 == 0,
                "clamped_glu: %d rows of %d inner features (a multiple of 128)", num_rows, inter);
   B200_GLUE_DTYPE("clamped_glu");
@@ -728,10 +644,10 @@ extern "C" int b200_clamped_glu(const void* gate_up, void* out, int num_rows, in
   const unsigned blocks = static_cast<unsigned>((total + 255) / 256);
   if (dtype == 0)
     clamped_glu_kernel<__nv_bfloat16><<<blocks, 256, 0, as_stream(stream)>>>(
-        static_cast<const __nv_bfloat16*>(gate_up), static_cast<__nv_bfloat16*>(out), total, inter, limit, alpha);
+        static_cast<const __nv_bfloat16*>(gate_up), static_cast<__nv_bfloat16*>(out), total, inter, limit, alpha, shift);
   else
     clamped_glu_kernel<float><<<blocks, 256, 0, as_stream(stream)>>>(static_cast<const float*>(gate_up),
-                                                                     static_cast<float*>(out), total, inter, limit, alpha);
+                                                                     static_cast<float*>(out), total, inter, limit, alpha, shift);
   B200_CUDA(cudaGetLastError());
   return 0;
 }
@@ -762,7 +678,25 @@ extern "C" int b200_gemm_f32(const float* x, const float* w, float* y, int num_r
   B200_REQUIRE((num_rows + 63) / 64 <= 65535, "gemm_f32: too many rows");
   const dim3 grid((out_features + 63) / 64, (num_rows + 63) / 64, groups);
   gemm_f32_kernel<<<grid, 256, 0, as_stream(stream)>>>(x, w, y, num_rows, out_features, in_features, x_step, w_step, y_step,
-                                                       x_cols, y_cols);
+                                                       x_cols, y_cols, nullptr, nullptr, 0);
+  B200_CUDA(cudaGetLastError());
+  return 0;
+}
+
+extern "C" int b200_moe_gemm_f32(const float* x, const float* w, float* y, const void* tiles, const int32_t* num_tiles,
+                                 int num_rows, int num_experts, int max_tiles, int out_features, int in_features, void* stream) {
+  B200_REQUIRE(x && w && y && tiles && num_tiles, "moe_gemm_f32: null pointer");
+  B200_REQUIRE(num_rows >= 0 && num_experts > 0 && max_tiles > 0 && max_tiles <= 65535 && out_features > 0 && in_features > 0 &&
+                   in_features % 4 == 0,
+               "moe_gemm_f32: %d rows, %d experts, at most %d tiles, N %d, K %d", num_rows, num_experts, max_tiles, out_features,
+               in_features);
+  B200_REQUIRE(aligned16({x, w}), "moe_gemm_f32: x and w must be 16-byte aligned");
+  int rc = check_device(nullptr);
+  if (rc) return rc;
+  if (num_rows == 0) return 0;
+  gemm_f32_kernel<<<dim3((out_features + 63) / 64, max_tiles), 256, 0, as_stream(stream)>>>(
+      x, w, y, num_rows, out_features, in_features, 0, out_features, 0, in_features, out_features,
+      static_cast<const MoeTile*>(tiles), num_tiles, num_experts);
   B200_CUDA(cudaGetLastError());
   return 0;
 }

@@ -98,6 +98,60 @@ moe_route_kernel(const LT* __restrict__ logits, int T, int E, int K, int renorm,
   }
 }
 
+// Routing by scores s = sigmoid(logit): the K largest, value descending, equal logits by lower expert id; weights s / (sum of
+// the chosen + 1e-20) * scale, or s * scale without `renorm`.  A warp per token, PER logits per lane.
+template <typename LT, int PER>
+__global__ void __launch_bounds__(kRouteWarps * 32)
+moe_route_sigmoid_kernel(const LT* __restrict__ logits, int T, int E, int K, int renorm, float scale,
+                         int* __restrict__ topk_ids, float* __restrict__ topk_w) {
+  grid_dep_wait();
+  grid_dep_launch();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * kRouteWarps + warp;
+  if (t >= T) return;
+  float v[PER];
+#pragma unroll
+  for (int j = 0; j < PER; ++j) {
+    const int e = lane + 32 * j;
+    v[j] = e < E ? logit_f32(logits, static_cast<size_t>(t) * E + e) : -INFINITY;
+  }
+  unsigned taken = 0;
+  float sum = 0.f, my_s = 0.f;
+  int my_id = 0;
+  for (int k = 0; k < K; ++k) {
+    float bv = -INFINITY;
+    int be = 0x7fffffff;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+      const int e = lane + 32 * j;
+      if (e < E && !((taken >> j) & 1u) && (be == 0x7fffffff || v[j] > bv)) {
+        bv = v[j];
+        be = e;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+      if (oe != 0x7fffffff && (be == 0x7fffffff || ov > bv || (ov == bv && oe < be))) {
+        bv = ov;
+        be = oe;
+      }
+    }
+    if ((be & 31) == lane) taken |= 1u << (be >> 5);
+    const float s = 1.f / (1.f + expf(-bv));
+    sum += s;
+    if (lane == k) {
+      my_s = s;
+      my_id = be;
+    }
+  }
+  if (lane < K) {
+    topk_ids[static_cast<size_t>(t) * K + lane] = my_id;
+    topk_w[static_cast<size_t>(t) * K + lane] = (renorm ? my_s / (sum + 1e-20f) : my_s) * scale;
+  }
+}
+
 // ---------------------------------------------------------------- permute ---
 constexpr int kRankThreads = 256;
 
@@ -336,6 +390,59 @@ __device__ __forceinline__ void block_exclusive_scan(const int* v, int* out, int
   }
   if (tid == 0) out[n] = carry;
   __syncthreads();
+}
+
+// Scatter + row copy in one pass: one CTA per token places the token's pairs and copies its row (`vec` 16-byte pieces) to
+// their sorted rows.  CTA 0 also publishes the offsets and the row tiles.
+__global__ void __launch_bounds__(256)
+moe_scatter_copy_kernel(const uint4* __restrict__ x, const int* __restrict__ topk_ids, const int* __restrict__ rank,
+                        const int* __restrict__ counts, int E, int K, int vec, int tile_rows, int* __restrict__ row_of_pair,
+                        MoeTile* __restrict__ tiles, int* __restrict__ num_tiles, uint4* __restrict__ dst_rows,
+                        int* __restrict__ err) {
+  extern __shared__ int sm[];  // cnt[E], off[E+1], ntile[E], toff[E+1], warp_tot[32], dst[K]
+  grid_dep_wait();
+  grid_dep_launch();
+  int* cnt = sm;
+  int* off = cnt + E;
+  int* ntile = off + E + 1;
+  int* toff = ntile + E;
+  int* warp_tot = toff + E + 1;
+  int* dst = warp_tot + 32;
+  const int t = blockIdx.x, tid = threadIdx.x;
+  // the token's row and its pairs travel while the counts are scanned
+  uint4 piece = make_uint4(0u, 0u, 0u, 0u);
+  if (tid < vec) piece = x[static_cast<size_t>(t) * vec + tid];
+  int my_e = -1, pair_rank = 0;
+  if (tid < K) {
+    my_e = topk_ids[t * K + tid];
+    pair_rank = rank[t * K + tid];
+  }
+  for (int e = tid; e < E; e += blockDim.x) {
+    cnt[e] = counts[e];
+    ntile[e] = (cnt[e] + tile_rows - 1) / tile_rows;
+  }
+  __syncthreads();
+  block_exclusive_scan(cnt, off, E, warp_tot);
+  if (t == 0) {
+    block_exclusive_scan(ntile, toff, E, warp_tot);
+    for (int e = tid; e < E; e += blockDim.x)
+      for (int j = 0; j < ntile[e]; ++j)
+        tiles[toff[e] + j] = MoeTile{e, off[e] + j * tile_rows, min(tile_rows, cnt[e] - j * tile_rows), 0};
+    if (tid == 0) *num_tiles = toff[E];
+  }
+  if (tid < K) {
+    int d = -1;
+    if (my_e >= 0 && my_e < E) d = off[my_e] + pair_rank;
+    else if (my_e != -1) set_error(err, kErrDevBadExpert);  // -1 is "no expert": the pair is left out
+    row_of_pair[t * K + tid] = d;
+    dst[tid] = d;
+  }
+  __syncthreads();
+  for (int c = tid; c < vec; c += blockDim.x) {
+    if (c != tid) piece = x[static_cast<size_t>(t) * vec + c];
+    for (int k = 0; k < K; ++k)
+      if (dst[k] >= 0) dst_rows[static_cast<size_t>(dst[k]) * vec + c] = piece;
+  }
 }
 
 // Scatter + activation quantisation in one pass.  One CTA per token, 8 columns per
@@ -690,6 +797,69 @@ static int permute_quant_impl(const int32_t* topk_ids, const void* x, int num_to
                               128, sorted_pair_ids, row_of_pair, expert_offsets, static_cast<MoeTile*>(tiles),
                               num_tiles, static_cast<uint8_t*>(xq), x_scale, err, ep_world, ep_capacity, slot_of_pair,
                               expert_of_slot, overflow, peers));
+  return 0;
+}
+
+extern "C" int b200_moe_route_sigmoid(const void* logits, int logits_dtype, int num_tokens, int num_experts, int top_k,
+                                      int renormalize, float scale, int32_t* topk_ids, float* topk_weights, void* stream) {
+  B200_REQUIRE(logits && topk_ids && topk_weights, "moe_route_sigmoid: null pointer");
+  B200_REQUIRE(logits_dtype == 0 || logits_dtype == 1, "moe_route_sigmoid: logits dtype %d is neither 0 (bf16) nor 1 (f32)",
+               logits_dtype);
+  B200_REQUIRE(num_tokens >= 0 && num_experts > 0 && num_experts <= 1024 && top_k > 0 && top_k <= 32 && top_k <= num_experts,
+               "moe_route_sigmoid: top %d of %d experts (at most 32 of 1024)", top_k, num_experts);
+  int rc = check_device(nullptr);
+  if (rc) return rc;
+  if (num_tokens == 0) return 0;
+  const dim3 grid((num_tokens + kRouteWarps - 1) / kRouteWarps), block(kRouteWarps * 32);
+#define B200_ROUTE(LT, PER)                                                                                              \
+  B200_CUDA(launch_overlapped(moe_route_sigmoid_kernel<LT, PER>, grid, block, 0, as_stream(stream),                      \
+                              static_cast<const LT*>(logits), num_tokens, num_experts, top_k, renormalize, scale, topk_ids, \
+                              topk_weights))
+  if (logits_dtype == 1) {
+    if (num_experts <= 256) B200_ROUTE(float, 8);
+    else B200_ROUTE(float, 32);
+  } else {
+    if (num_experts <= 256) B200_ROUTE(__nv_bfloat16, 8);
+    else B200_ROUTE(__nv_bfloat16, 32);
+  }
+#undef B200_ROUTE
+  return 0;
+}
+
+extern "C" int b200_moe_permute_copy(const int32_t* topk_ids, const void* x, int num_tokens, int num_experts, int top_k,
+                                     int row_bytes, int tile_rows, int32_t* row_of_pair, void* tiles, int32_t* num_tiles,
+                                     void* sorted_rows, void* workspace, size_t workspace_bytes, void* stream) {
+  B200_REQUIRE(topk_ids && x && row_of_pair && tiles && num_tiles && sorted_rows && workspace, "moe_permute_copy: null pointer");
+  B200_REQUIRE(num_tokens >= 0 && num_experts > 0 && num_experts <= 1024 && top_k > 0 && top_k <= 32 && tile_rows > 0 &&
+                   row_bytes > 0 && row_bytes % 16 == 0,
+               "moe_permute_copy: %d tokens, top %d of %d experts, rows of %d bytes, tiles of %d", num_tokens, top_k, num_experts,
+               row_bytes, tile_rows);
+  B200_REQUIRE(((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(sorted_rows)) & 15) == 0,
+               "moe_permute_copy: rows must be 16-byte aligned");
+  const size_t need = b200_moe_permute_workspace_bytes(num_tokens, num_experts, top_k);
+  if (workspace_bytes < need) {
+    set_detail("moe_permute_copy: workspace %zu < required %zu", workspace_bytes, need);
+    return -kErrWorkspace;
+  }
+  int rc = check_device(nullptr);
+  if (rc) return rc;
+  cudaStream_t st = as_stream(stream);
+  if (num_tokens == 0) {
+    B200_CUDA(cudaMemsetAsync(num_tiles, 0, sizeof(int32_t), st));
+    return 0;
+  }
+  uint8_t* p = static_cast<uint8_t*>(workspace);
+  int* counts = reinterpret_cast<int*>(p + 256);
+  int* rank = reinterpret_cast<int*>(p + 256 + ((static_cast<size_t>(num_experts) * 4 + 255) & ~size_t(255)));
+  B200_CUDA(launch_overlapped(moe_rank_kernel, dim3(num_experts), dim3(kRankThreads), 0, st, topk_ids, num_tokens * top_k, rank,
+                              counts));
+  const int vec = row_bytes / 16;
+  const int threads = vec >= 256 ? 256 : (vec + 31) / 32 * 32;
+  const size_t smem = (4 * static_cast<size_t>(num_experts) + 2 + 32 + top_k) * sizeof(int);
+  B200_CUDA(launch_overlapped(moe_scatter_copy_kernel, dim3(num_tokens), dim3(threads), smem, st, static_cast<const uint4*>(x),
+                              topk_ids, rank, counts, num_experts, top_k, vec, tile_rows, row_of_pair,
+                              static_cast<MoeTile*>(tiles), num_tiles, static_cast<uint4*>(sorted_rows),
+                              reinterpret_cast<int*>(p)));
   return 0;
 }
 

@@ -142,9 +142,15 @@ class PagedEngine:
 
       _decode_hidden(B)                        final normed hidden rows of one decode step of rows [0, B)
       _begin_prompt(chunk) -> chunk            buffers for prompt passes of up to `chunk` tokens
-      _prompt_hidden(token_ids, row, lo, chunk)     hidden rows of one chunk at positions lo.. of the sequence with table `row`
-      _mixed_hidden(tokens, pos, table, first_pos, n, B)   rows of a chunk (first n) and of a decode step (the rest)
+      _prompt_hidden(token_ids, row, lo, chunk, slot)     hidden rows of one chunk at positions lo.. of the sequence with table
+                                               `row` (and state slot `slot`)
+      _mixed_hidden(tokens, pos, table, first_pos, n, B, slot)   rows of a chunk (first n) and of a decode step (the rest)
       _pick(h, out) / _logits(h)               next tokens (arg-max) / logits of hidden rows
+
+    A model with recurrent layers also keeps a state per sequence, in slots: `num_slots` of them for sequences and one more
+    for padding rows.  `state_slots[i]` names the slot of row i (row i itself unless the caller says otherwise), a prompt
+    pass is told its sequence's.  The state after position p must survive running position p's decode step again
+    (`_build_graph` does), and a sequence that starts at position 0 must not depend on what its slot holds.
     """
 
     prompt_chunk = 1024       # tokens of a prompt pass unless the caller says otherwise
@@ -152,6 +158,8 @@ class PagedEngine:
     round_hook = None
     takes_reference_pools = False  # whether a reference BlockManager's K/V pools can stand in for the engine's own
     logits_dtype = torch.bfloat16
+    num_slots = 0             # state slots for sequences; 0: the model keeps everything in pages
+    state_slots = None
 
     def _init_step_state(self, num_blocks: int, max_batch: int, max_pages_per_seq: int, device, use_graphs: bool,
                          keep_logits: bool, scratch_page: bool) -> None:
@@ -174,6 +182,8 @@ class PagedEngine:
         self.ctx_lens = torch.zeros(max_batch, dtype=torch.int32, device=self.device)
         self.block_table = torch.zeros(max_batch, max_pages_per_seq, dtype=torch.int32, device=self.device)
         self.next_tokens = torch.zeros(max_batch, dtype=torch.int64, device=self.device)
+        if self.num_slots:
+            self.state_slots = torch.arange(max_batch, dtype=torch.int32, device=self.device)
         self._graphs: dict[int, torch.cuda.CUDAGraph] = {}
         self._graph_logits: dict[int, torch.Tensor] = {}
 
@@ -210,6 +220,8 @@ class PagedEngine:
             self.tokens[lo:hi] = 0
             self.ctx_lens[lo:hi] = 0
             self.block_table[lo:hi, 0] = self.scratch_block
+            if self.num_slots:
+                self.state_slots[lo:hi] = self.num_slots
 
     def _build_graph(self, B: int, pad_from: int | None = None) -> torch.cuda.CUDAGraph:
         """Capture the step for B rows (two eager warm-up runs, then the capture).  `pad_from`: rows from
@@ -268,6 +280,10 @@ class PagedEngine:
             self.last_logits = self._graph_logits[B]  # the buffer this graph writes
         return self.next_tokens[:real]
 
+    def _check_slot(self, slot: int) -> None:
+        if self.num_slots and not 0 <= slot < self.num_slots:
+            raise ValueError(f"state slot {slot} outside [0, {self.num_slots})")
+
     def idle_pass(self) -> None:
         """Expert parallelism: take part in one exchange round without any rows of one's own."""
         self.step(0, joined=True)
@@ -275,7 +291,7 @@ class PagedEngine:
     # --------------------------------------------------------------- prefill
     @torch.no_grad()
     def prefill(self, token_ids: list[int], block_ids: list[int], cached_tokens: int = 0,
-                chunk: int | None = None, want: list[int] | None = None) -> tuple[int, torch.Tensor]:
+                chunk: int | None = None, want: list[int] | None = None, slot: int = 0) -> tuple[int, torch.Tensor]:
         """Prompt pass for one sequence; writes K/V of tokens [cached_tokens, n) into `block_ids` pages.
 
         Runs in chunks of `chunk` prompt tokens through the same projection, glue and MoE kernels as decode
@@ -289,6 +305,8 @@ class PagedEngine:
         Under expert parallelism a chunk is one exchange round like a decode step: it is padded to the
         exchange's fixed shape (the engine's full batch) with rows that route nowhere, and the other ranks spend
         the round on a decode step, a chunk of their own or an idle pass.
+        `slot`: the sequence's state slot, for models with recurrent layers; it must hold the state after position
+        cached_tokens - 1.
         Returns (first generated token, logits): the last position's, None unless the engine was built with keep_logits;
         or, with `want`, a [len(want), vocab] tensor of the logits at those positions (at or after cached_tokens)."""
         n = len(token_ids)
@@ -298,6 +316,7 @@ class PagedEngine:
             raise ValueError("not enough pages for the prompt")
         if len(block_ids) > self.max_pages:
             raise ValueError("sequence needs more pages than the block table is wide")
+        self._check_slot(slot)
         chunk = self._begin_prompt(chunk or self.prompt_chunk)
         row = torch.zeros(self.max_pages, dtype=torch.int32)
         row[: len(block_ids)] = torch.tensor(block_ids, dtype=torch.int32)
@@ -308,7 +327,7 @@ class PagedEngine:
         wanted = None if want is None else torch.empty(len(want), self.vocab_size, dtype=self.logits_dtype, device=self.device)
         for lo in range(cached_tokens, n, chunk):
             hi = min(n, lo + chunk)
-            h = self._prompt_hidden(token_ids[lo:hi], row, lo, chunk)
+            h = self._prompt_hidden(token_ids[lo:hi], row, lo, chunk, slot)
             here = [i for i, p in enumerate(want or ()) if lo <= p < hi]
             if here:
                 logits = self._logits(h[torch.tensor([want[i] - lo for i in here], device=self.device)])
@@ -322,7 +341,7 @@ class PagedEngine:
 
     @torch.no_grad()
     def mixed_step(self, B: int, chunk_token_ids: list[int], block_ids: list[int], first_pos: int,
-                   want_first: bool = True) -> tuple[torch.Tensor, int | None, torch.Tensor | None]:
+                   want_first: bool = True, slot: int = 0) -> tuple[torch.Tensor, int | None, torch.Tensor | None]:
         """One pass that is a decode step for rows [0, B) of the static state AND a prompt chunk of one other
         sequence: its tokens `chunk_token_ids` sit at positions first_pos.. of the sequence whose pages are
         `block_ids` (earlier positions already written).  The reference runs the two as separate forwards
@@ -342,13 +361,14 @@ class PagedEngine:
             raise ValueError(f"mixed pass needs a chunk and 1..{self.max_batch} decode rows (got {n} and {B})")
         if len(block_ids) * PAGE < first_pos + n or len(block_ids) > self.max_pages:
             raise ValueError("the chunk's sequence needs more pages than it was given or than the block table is wide")
+        self._check_slot(slot)
         row = torch.zeros(self.max_pages, dtype=torch.int32)
         row[: len(block_ids)] = torch.tensor(block_ids, dtype=torch.int32)
         row = row.to(self.device)
         tokens = torch.cat([torch.tensor(chunk_token_ids, device=self.device), self.tokens[:B]])
         pos = torch.cat([torch.arange(first_pos, first_pos + n, device=self.device, dtype=torch.int32), self.ctx_lens[:B]])
         table = torch.cat([row.unsqueeze(0).expand(n, -1), self.block_table[:B]])
-        h = self._mixed_hidden(tokens, pos, table, first_pos, n, B)
+        h = self._mixed_hidden(tokens, pos, table, first_pos, n, B, slot)
         first = logits = None
         if want_first:
             # the chunk's last row and the decode rows are neighbours: lm_head is streamed once for both
@@ -618,7 +638,7 @@ class DecodeEngine(PagedEngine):
         self._prefill_pairs = not tiled and ops.paged_attn_pairs_supported(cfg.q_heads, cfg.kv_heads, cfg.head_dim, PAGE, torch.bfloat16)
         return chunk
 
-    def _prompt_hidden(self, token_ids: list[int], row: torch.Tensor, lo: int, chunk: int) -> torch.Tensor:
+    def _prompt_hidden(self, token_ids: list[int], row: torch.Tensor, lo: int, chunk: int, slot: int) -> torch.Tensor:
         hi = lo + len(token_ids)
         ep = self.ep_state is not None
         tokens = torch.tensor(token_ids, device=self.device)
@@ -638,7 +658,7 @@ class DecodeEngine(PagedEngine):
         return self._forward(tokens, pos, table, self._prefill_attn_ws, self._prefill_moe_ws, self._prefill_split,
                           ep, pairs=self._prefill_pairs, chunk_of=(lo, hi - lo) if self._prefill_tiled else None)
 
-    def _mixed_hidden(self, tokens, pos, table, first_pos: int, n: int, B: int) -> torch.Tensor:
+    def _mixed_hidden(self, tokens, pos, table, first_pos: int, n: int, B: int, slot: int) -> torch.Tensor:
         cfg = self.cfg
         if not ops.paged_attn_prefill_supported(cfg.q_heads, cfg.kv_heads, cfg.head_dim, PAGE, torch.bfloat16):
             raise ValueError("mixed passes need the tiled prompt-attention kernel, which is not built for this head shape")

@@ -1,10 +1,11 @@
-"""Layer-list decoders: models whose config.json lists their layers one by one (design: Sulepel).
+"""Layer-list decoders: models whose config.json lists their layers one by one.  Two designs: Sulepel, described here, and
+Sefalorn, whose mechanisms are in ``gated.py``; the engine, its step and its pass over the layers are the same.
 
     x_p = embed[token_p] + sinusoid(p)
     per layer   x += mixer(short_conv(norm1 x));   x += ff(norm2 x)        (a layer may have no ff)
     logits      = head norm(x)
 
-with a grouped RMSNorm, a short causal convolution in front of every mixer, mixers of two kinds in any order and of any
+(Sulepel) with a grouped RMSNorm, a short causal convolution in front of every mixer, mixers of two kinds in any order and of any
 sizes - grouped-query attention over the position's own chunk, and latent attention whose cache is one vector per
 token -, a sigmoid gate per head on either, and a dense feed-forward with a clamped gated unit.
 
@@ -32,7 +33,7 @@ from dataclasses import dataclass
 
 import torch
 
-from . import ops
+from . import gated, ops
 from .engine import PAGE, PagedEngine
 
 GLU_ALPHA = 1.702          # of the design's gated unit
@@ -72,8 +73,8 @@ class GluSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec | LatentSpec
-    mlp: GluSpec | None
+    mixer: AttentionSpec | LatentSpec | gated.ParallelSpec | gated.LightningSpec
+    mlp: GluSpec | gated.MoeSpec | None
 
 
 @dataclass(frozen=True)
@@ -83,8 +84,10 @@ class LayeredConfig:
     width: int
     norm_groups: int
     norm_eps: float
-    taps: int
+    taps: int                   # of the convolution ahead of every mixer
     layer_list: tuple[LayerSpec, ...]
+    gated: bool = False         # Sefalorn: layer norm, gated residual, no convolution ahead of a mixer, no positions added
+    logit_scale: float = 1.0
 
     @property
     def hidden(self) -> int:
@@ -96,6 +99,12 @@ class LayeredConfig:
 
     @staticmethod
     def from_json(c: dict) -> "LayeredConfig":
+        if c["architecture"] == "Sefalorn":
+            layers = tuple(LayerSpec(gated.mixer_from_json(e["type"], e["mixer"]), gated.mlp_from_json(e.get("mlp")))
+                           for e in c["layers"])
+            return LayeredConfig(c["architecture"], c["vocab"], c["width"], 1, float(c["norm"]["eps"]), 1, layers, gated=True,
+                                 logit_scale=float(c["logit_scale"]))
+
         def mixer(kind: str, m: dict):
             if kind == "attention":
                 mask = m.get("mask")
@@ -130,6 +139,9 @@ class LayeredConfig:
         out = {"embed": (self.vocab_size, W), "final.norm": (W,), "head": (self.vocab_size, W)}
         for i, layer in enumerate(self.layer_list):
             m, p = layer.mixer, f"l{i}."
+            if self.gated:
+                out.update({p + name: shape for name, shape in gated.layer_shapes(layer, W).items()})
+                continue
             out[p + "norm1"] = (W,)
             out[p + "canon1"] = (W, self.taps)
             out[p + "mix.q"] = (m.heads * m.dim, W)
@@ -162,10 +174,26 @@ def uniform_config(name: str, vocab: int, width: int, groups: int, taps: int, pa
                          tuple(LayerSpec(a if ch == "a" else lat, glu) for ch in pattern))
 
 
+def gated_config(name: str, vocab: int, width: int, pattern: str, heads: int, kv_heads: int, dim: int, window: int,
+                 state_heads: int, state_dim: int, taps: int, experts: int, top: int, inner: int) -> LayeredConfig:
+    """A built-in Sefalorn shape: `pattern` has a letter per layer, p = parallel, l = lightning."""
+    par = gated.ParallelSpec(gated.WindowAttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, window),
+                             gated.DeltaSpec(state_heads, state_heads, state_dim, state_dim, taps), 1.0, 1.0)
+    light = gated.LightningSpec(state_heads, state_dim, state_dim,
+                                tuple(1.0 - 2.0 ** -(2 + 8 * i / max(1, state_heads - 1)) for i in range(state_heads)))
+    moe = gated.MoeSpec(experts, top, inner, 1.0)
+    return LayeredConfig(name, vocab, width, 1, 1e-6, 1, tuple(LayerSpec(par if ch == "p" else light, moe) for ch in pattern),
+                         gated=True)
+
+
 # Shapes for benchmarks with random weights.
 CONFIGS = {
     # the width, heads and vocabulary of qwen3-30b-a3b, 12 layers
     "sulepel-2048": uniform_config("sulepel-2048", 151936, 2048, 4, 4, "aaal" * 3, 32, 4, 128, 2048, 16, 512, 6144, 7.0),
+    # the width, attention heads, experts and vocabulary of qwen3-30b-a3b, 8 layers
+    "sefalorn-2048": gated_config("sefalorn-2048", 151936, 2048, "plpl" * 2, 32, 4, 128, 1024, 16, 128, 4, 128, 8, 768),
+    # the width, attention heads and experts of qwen3-235b-a22b, 4 layers
+    "sefalorn-4096": gated_config("sefalorn-4096", 151936, 4096, "plpl", 64, 4, 128, 2048, 32, 128, 4, 128, 8, 1536),
     # the width and heads of qwen3-235b-a22b, 8 layers
     "sulepel-4096": uniform_config("sulepel-4096", 151936, 4096, 8, 4, "aaal" * 2, 64, 4, 128, 4096, 32, 512, 12288, 7.0),
 }
@@ -294,7 +322,7 @@ def sinusoid_tables(width: int, ld: int, max_pos: int, device) -> tuple[torch.Te
 # --------------------------------------------------------------------- engine
 
 
-class LayeredEngine(PagedEngine):
+class LayeredEngine(gated.GatedMechanisms, PagedEngine):
     """A layer-list decoder on the paged step: weights, pools and one pass over the layers."""
 
     logits_dtype = torch.float32
@@ -302,8 +330,12 @@ class LayeredEngine(PagedEngine):
 
     def __init__(self, cfg: LayeredConfig, num_blocks: int, max_batch: int, max_pages_per_seq: int, device="cuda", seed: int = 0,
                  tensors: dict[str, torch.Tensor] | None = None, dtype: torch.dtype = torch.bfloat16, use_graphs: bool = True,
-                 graph_buckets: bool = True, keep_logits: bool = False, split_tokens: int | None = None):
-        """`tensors`: a checkpoint's tensors (any device); random weights from `seed` without."""
+                 graph_buckets: bool = True, keep_logits: bool = False, split_tokens: int | None = None,
+                 num_slots: int | None = None):
+        """`tensors`: a checkpoint's tensors (any device); random weights from `seed` without.  `num_slots`: sequences that may
+        hold a recurrent state at a time, max_batch and a few whose prompts are under way unless given."""
+        if cfg.gated:
+            self.num_slots = max(max_batch, num_slots or max_batch + 4)
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError(f"dtype {dtype}: bfloat16 or float32")
         self._init_step_state(num_blocks, max_batch, max_pages_per_seq, device, use_graphs, keep_logits, graph_buckets)
@@ -327,14 +359,23 @@ class LayeredEngine(PagedEngine):
         self.layers = []
         for i, spec in enumerate(cfg.layer_list):
             p = f"l{i}."
-            self.layers.append(LayeredWeights(spec, {n[len(p):]: fetch(n) for n in shapes if n.startswith(p)}, cfg, self.device,
-                                              dtype))
+            t = {n[len(p):]: fetch(n) for n in shapes if n.startswith(p)}
+            if cfg.gated:
+                self.layers.append(gated.GatedWeights(spec, t, cfg.width, self.W, max_pages_per_seq * PAGE, self.device, dtype))
+            else:
+                self.layers.append(LayeredWeights(spec, t, cfg, self.device, dtype))
 
         def table(name):
             return _cols(fetch(name).to(self.device), self.W).to(dtype).contiguous()
 
-        self.embed, self.lm_head, self.final_norm = table("embed"), table("head"), table("final.norm")
-        self.sinusoid = sinusoid_tables(cfg.width, self.W, max_pages_per_seq * PAGE, self.device)
+        self.embed, self.lm_head = table("embed"), table("head")
+        if cfg.gated:
+            # the logits' factor goes with the norm's fp32 weight
+            self.final_norm = (_cols(fetch("final.norm").to(self.device).float(), self.W) * cfg.logit_scale).contiguous()
+            self.sinusoid = _up(max_pages_per_seq * PAGE, 64)
+        else:
+            self.final_norm = table("final.norm")
+            self.sinusoid = sinusoid_tables(cfg.width, self.W, max_pages_per_seq * PAGE, self.device)
 
         nb = num_blocks + (1 if self.scratch_block is not None else 0)
 
@@ -343,12 +384,19 @@ class LayeredEngine(PagedEngine):
 
         self.k_pools, self.v_pools, self.c_pools, self.hist = [], [], [], []
         for spec, w in zip(cfg.layer_list, self.layers):
+            if cfg.gated:
+                a = getattr(spec.mixer, "left", None)
+                self.k_pools.append(pool(a.kv_heads, PAGE, w.Dk) if a else None)
+                self.v_pools.append(pool(a.kv_heads, PAGE, w.Dv) if a else None)
+                continue
             attn = isinstance(spec.mixer, AttentionSpec)
             self.k_pools.append(pool(spec.mixer.kv_heads, PAGE, w.D) if attn else None)
             self.v_pools.append(pool(spec.mixer.kv_heads, PAGE, w.D) if attn else None)
             self.c_pools.append(None if attn else pool(PAGE, w.R))
             self.hist.append(pool(min(cfg.taps, PAGE), self.W) if cfg.taps > 1 else None)
 
+        if cfg.gated:
+            self._init_states(self.num_slots)
         self._fixed_split = split_tokens
         self.status = torch.zeros(64, dtype=torch.int32, device=self.device)  # glue kernels, projections
         widest = max([self.W] + [w.wproj.shape[0] for w in self.layers])
@@ -356,6 +404,9 @@ class LayeredEngine(PagedEngine):
         self.argmax_ws = ops.lm_head_argmax_workspace(self.device) if dtype == torch.bfloat16 else None
         self._row_ws: dict[int, tuple[dict, torch.Tensor]] = {}
         self._kv_scratch: dict[tuple[int, int], tuple] = {}
+        if cfg.gated:
+            self.kernel_launches_per_step = 4 + sum(gated.launches(s) for s in cfg.layer_list)
+            return
         # kernels of one decode step: embedding, final norm, lm_head arg-max and its fold; per layer norm + convolution,
         # projection, attention, its fold, output projection (+ latents' norm, two maps per head), norm, two products
         self.kernel_launches_per_step = 4 + sum(
@@ -481,11 +532,21 @@ class LayeredEngine(PagedEngine):
                               plan if plan is not None and n else self._attn_for(R - n), out[n:])
         return self._linear(out.view(R, m.heads * D), w.wo)
 
-    def _forward(self, tokens, pos, table, chunk_of: tuple[int, int] | None = None, plan=None) -> torch.Tensor:
-        """One pass: row i is token `tokens[i]` at position `pos[i]` of the sequence with pages `table[i]`.  With `chunk_of` =
-        (first position, n) the first n rows are consecutive tokens of one sequence; the others are decode rows of other
-        sequences, with attention `plan` (see _attn_for).  Returns the final normed rows."""
+    def _forward(self, tokens, pos, table, chunk_of: tuple[int, int] | None = None, plan=None, slots=None) -> torch.Tensor:
+        """One pass: row i is token `tokens[i]` at position `pos[i]` of the sequence with pages `table[i]` (and state slot
+        `slots[i]`).  With `chunk_of` = (first position, n) the first n rows are consecutive tokens of one sequence; the others
+        are decode rows of other sequences, with attention `plan` (see _attn_for).  Returns the final normed rows."""
         c = self.cfg
+        if c.gated:
+            rows = gated.Rows(pos, table, slots, *(chunk_of or (0, 0)))
+            x, pending = ops.embed_sinusoid(tokens, pos, self.embed, self.sinusoid, c.width, self.status), None
+            for li, (spec, w) in enumerate(zip(c.layer_list, self.layers)):
+                h = self._add_norm(x, pending, w.norm1)
+                mixer = self._parallel if isinstance(spec.mixer, gated.ParallelSpec) else self._lightning
+                pending = mixer(h, li, spec.mixer, w, rows)
+                if spec.mlp is not None:
+                    pending = self._experts(self._add_norm(x, pending, w.norm2), spec.mlp, w)
+            return self._add_norm(x, pending, self.final_norm)
         new_len = pos + 1
         x = ops.embed_sinusoid(tokens, pos, self.embed, self.sinusoid, c.width, self.status)
         delta = None
@@ -501,18 +562,25 @@ class LayeredEngine(PagedEngine):
 
     # ----------------------------------------------------------------- hooks
     def _decode_hidden(self, B: int) -> torch.Tensor:
+        if self.cfg.gated:
+            return self._forward(self.tokens[:B], self.ctx_lens[:B], self.block_table[:B], slots=self.state_slots[:B])
         return self._forward(self.tokens[:B], self.ctx_lens[:B], self.block_table[:B], None, self._attn_for(B))
 
     def _begin_prompt(self, chunk: int) -> int:
         return chunk
 
-    def _prompt_hidden(self, token_ids: list[int], row: torch.Tensor, lo: int, chunk: int) -> torch.Tensor:
+    def _prompt_hidden(self, token_ids: list[int], row: torch.Tensor, lo: int, chunk: int, slot: int) -> torch.Tensor:
         n = len(token_ids)
         tokens = torch.tensor(token_ids, device=self.device)
         pos = torch.arange(lo, lo + n, device=self.device, dtype=torch.int32)
-        return self._forward(tokens, pos, row.unsqueeze(0).expand(n, -1).contiguous(), (lo, n))
+        return self._forward(tokens, pos, row.unsqueeze(0).expand(n, -1).contiguous(), (lo, n), slots=self._slots_of(slot, n))
 
-    def _mixed_hidden(self, tokens, pos, table, first_pos: int, n: int, B: int) -> torch.Tensor:
+    def _slots_of(self, slot: int, n: int):
+        return torch.full((n,), slot, dtype=torch.int32, device=self.device) if self.num_slots else None
+
+    def _mixed_hidden(self, tokens, pos, table, first_pos: int, n: int, B: int, slot: int) -> torch.Tensor:
+        if self.cfg.gated:
+            return self._forward(tokens, pos, table, (first_pos, n), slots=torch.cat([self._slots_of(slot, n), self.state_slots[:B]]))
         return self._forward(tokens, pos, table, (first_pos, n), self._attn_for(B))
 
     def _pick(self, h, out=None) -> torch.Tensor:
@@ -530,6 +598,8 @@ class LayeredEngine(PagedEngine):
         ops.read_status(self.status, where)
         for rows, (_, ws) in self._row_ws.items():
             ops.read_status(ws, f"{where}: attention ({rows} rows)")
+        for ws in getattr(self, "_moe_ws", ()):
+            ops.read_status(ws, f"{where}: experts")
 
     # ------------------------------------------------------------ accounting
     def kv_bytes_per_token(self) -> int:
@@ -537,6 +607,17 @@ class LayeredEngine(PagedEngine):
         size = torch.empty(0, dtype=self.dtype).element_size()
         total = 0
         for spec, w in zip(self.cfg.layer_list, self.layers):
+            if self.cfg.gated:
+                a = getattr(spec.mixer, "left", None)
+                total += a.kv_heads * (w.Dk + w.Dv) if a else 0
+                continue
             total += 2 * spec.mixer.kv_heads * w.D if isinstance(spec.mixer, AttentionSpec) else w.R
             total += min(self.cfg.taps, PAGE) * self.W // PAGE if self.cfg.taps > 1 else 0
         return total * size
+
+    def state_bytes_per_sequence(self) -> int:
+        """Bytes a sequence holds whatever its length (recurrent states, both halves, and convolution inputs)."""
+        if not self.cfg.gated:
+            return 0
+        per = [t[0] for t in self.states + self.rings if t is not None]
+        return sum(t.numel() * t.element_size() for t in per)

@@ -347,6 +347,7 @@ def qk_norm_rope_append(qkv, q_norm_w, k_norm_w, cos, sin, positions, block_tabl
 # ------------------------------------------- layer-list decoders (layered.py)
 
 SEG_ROWS, SEG_F32, SEG_PAGES = 0, 1, 2
+ACT_NONE, ACT_SILU, ACT_SIGMOID = 0, 1, 2
 
 
 def paged_attn_decode_chunked(q, k_pool, v_pool, block_table, ctx_lens, scale: float, split_tokens: int, workspace, chunk: int = 0,
@@ -498,10 +499,10 @@ def gemm_f32(x, w, out=None):
 
 
 def _segments(segs):
-    """segs: (kind, target) or (SEG_PAGES, pool, heads, dim) in feature order -> ctypes arrays."""
+    """segs: (kind, target) or (kind, target, activation) in feature order -> ctypes arrays."""
     import ctypes
     n = len(segs)
-    end, kind, heads, dim = ((ctypes.c_int32 * n)() for _ in range(4))
+    end, kind, act, heads, dim = ((ctypes.c_int32 * n)() for _ in range(5))
     ptr = (ctypes.c_void_p * n)()
     at = 0
     for i, s in enumerate(segs):
@@ -515,7 +516,8 @@ def _segments(segs):
             width = t[0].numel() if t.shape[0] else 0
         at += width
         end[i], kind[i], ptr[i] = at, s[0], t.data_ptr()
-    return end, kind, heads, dim, ptr, n, at
+        act[i] = s[2] if len(s) > 2 else ACT_NONE
+    return (end, kind, act, heads, dim, ptr, n), at
 
 
 def _segment_pages(segs):
@@ -525,21 +527,25 @@ def _segment_pages(segs):
     return 1, 1
 
 
-def proj_split(x, w, segs, col_scale=None, positions=None, block_table=None, status=None, max_pages: int | None = None):
+def proj_split(x, w, segs, col_scale=None, positions=None, block_table=None, status=None, max_pages: int | None = None,
+               col_bias=None):
     """x w^T with consecutive ranges of output features sent to different places: segs lists (SEG_ROWS, bf16/fp32 tensor
     [M, ...] of x's dtype), (SEG_F32, fp32 tensor [M, ...]) and (SEG_PAGES, pool [blocks, heads, page, dim], written at
-    positions[m] of the sequence block_table[m]; both None: row m of page-contiguous scratch).  `col_scale` multiplies the
-    features in fp32.  One kernel in bf16; in fp32 a product and a store kernel."""
+    positions[m] of the sequence block_table[m]; both None: row m of page-contiguous scratch), each with an optional
+    activation (ACT_*) as a third entry.  `col_scale` multiplies the features and `col_bias` is added to them, in fp32.  One kernel in bf16; in fp32 a product and a store kernel."""
     _need(x, "x")
     _need(w, "w", x.dtype)
     M, K = x.shape
     if M == 0:
         return
-    end, kind, heads, dim, ptr, n, total = _segments(segs)
+    (end, kind, act, heads, dim, ptr, n), total = _segments(segs)
     if w.shape != (total, K):
         raise ValueError(f"w is {tuple(w.shape)}, the segments need {(total, K)}")
-    if col_scale is not None:
-        _need(col_scale, "col_scale", torch.float32)
+    for name, t in (("col_scale", col_scale), ("col_bias", col_bias)):
+        if t is not None:
+            _need(t, name, torch.float32)
+            if t.numel() != total:
+                raise ValueError(f"{name} has {t.numel()} entries for {total} features")
     page, nb = _segment_pages(segs)
     if positions is not None:
         _need(positions, "positions", torch.int32)
@@ -550,24 +556,24 @@ def proj_split(x, w, segs, col_scale=None, positions=None, block_table=None, sta
         max_pages = nb
     lib = _lib.load()
     if x.dtype == torch.bfloat16:
-        rc = lib.b200_proj_split_gemm(_ptr(x), _ptr(w), _ptr(col_scale), end, kind, heads, dim, ptr, n, _ptr(positions),
+        rc = lib.b200_proj_split_gemm(_ptr(x), _ptr(w), _ptr(col_scale), _ptr(col_bias), end, kind, act, heads, dim, ptr, n, _ptr(positions),
                                       _ptr(block_table), _ptr(status), M, K, page, nb, max_pages, _stream())
         check(rc, "b200_proj_split_gemm")
     else:
-        split_store(gemm_f32(x, w), segs, col_scale, positions, block_table, status, torch.float32, max_pages)
+        split_store(gemm_f32(x, w), segs, col_scale, positions, block_table, status, torch.float32, max_pages, col_bias)
 
 
 def split_store(y, segs, col_scale=None, positions=None, block_table=None, status=None, dtype=torch.float32,
-                max_pages: int | None = None):
+                max_pages: int | None = None, col_bias=None):
     """The store of `proj_split` on a finished fp32 product y [M, N]."""
     _need(y, "y", torch.float32)
-    end, kind, heads, dim, ptr, n, total = _segments(segs)
+    (end, kind, act, heads, dim, ptr, n), total = _segments(segs)
     if y.shape[1] != total:
         raise ValueError(f"y has {y.shape[1]} columns, the segments {total}")
     page, nb = _segment_pages(segs)
     if block_table is not None:
         max_pages = block_table.shape[1]
-    rc = _lib.load().b200_split_store(_ptr(y), _ptr(col_scale), end, kind, heads, dim, ptr, n, _ptr(positions),
+    rc = _lib.load().b200_split_store(_ptr(y), _ptr(col_scale), _ptr(col_bias), end, kind, act, heads, dim, ptr, n, _ptr(positions),
                                       _ptr(block_table), _ptr(status), y.shape[0], page, nb, max_pages or nb, DTYPE_CODE[dtype],
                                       _stream())
     check(rc, "b200_split_store")
@@ -594,27 +600,29 @@ def glu_proj(x, w_interleaved, limit: float, alpha: float, status=None, out=None
     return clamped_glu(gemm_f32(x, w_interleaved), limit, alpha, out)
 
 
-def clamped_glu(gate_up, limit: float, alpha: float, out=None):
+def clamped_glu(gate_up, limit: float, alpha: float, out=None, shift: float = 1.0):
     """The gated unit alone on gate/up columns interleaved in blocks of 128."""
     _need(gate_up, "gate_up")
     M, F = gate_up.shape[0], gate_up.shape[1] // 2
     if out is None:
         out = torch.empty(M, F, dtype=gate_up.dtype, device=gate_up.device)
-    check(_lib.load().b200_clamped_glu(_ptr(gate_up), _ptr(out), M, F, float(limit), float(alpha), DTYPE_CODE[gate_up.dtype],
-                                       _stream()), "b200_clamped_glu")
+    check(_lib.load().b200_clamped_glu(_ptr(gate_up), _ptr(out), M, F, float(limit), float(alpha), float(shift),
+                                       DTYPE_CODE[gate_up.dtype], _stream()), "b200_clamped_glu")
     return out
 
 
 def embed_sinusoid(tokens, positions, embed, tables, width: int, status=None):
-    """fp32 residual rows embed[token] + sinusoid(position); tables = (lo, hi) as `layered.sinusoid_tables` makes them."""
+    """fp32 residual rows embed[token] + sinusoid(position); tables = (lo, hi) as `layered.sinusoid_tables` makes them, or the
+    number of positions (a multiple of 64): no sinusoid."""
     _need(tokens, "tokens", torch.int64)
     _need(positions, "positions", torch.int32)
     _need(embed, "embed")
-    lo, hi = tables
+    lo, hi = (None, None) if isinstance(tables, int) else tables
+    n_hi = tables // 64 if hi is None else hi.shape[0]
     M, ld = tokens.shape[0], embed.shape[1]
     x = torch.empty(M, ld, dtype=torch.float32, device=embed.device)
     rc = _lib.load().b200_embed_sinusoid(_ptr(tokens), _ptr(positions), _ptr(embed), _ptr(lo), _ptr(hi), _ptr(x), _ptr(status), M,
-                                         int(width), ld, embed.shape[0], hi.shape[0], DTYPE_CODE[embed.dtype], _stream())
+                                         int(width), ld, embed.shape[0], n_hi, DTYPE_CODE[embed.dtype], _stream())
     check(rc, "b200_embed_sinusoid")
     return x
 
@@ -690,6 +698,218 @@ def argmax_rows(logits, out=None):
     _need(out, "out", torch.int64)
     check(_lib.load().b200_argmax_rows(_ptr(logits), _ptr(out), logits.shape[0], logits.shape[1], _stream()), "b200_argmax_rows")
     return out
+
+
+# --------------------------------------- gated layer-list decoders (gated.py)
+
+
+def residual_norm(x, pending, weight, eps: float, width: int, center: bool = True, out=None, dtype=torch.bfloat16):
+    """x (fp32) += (sublayer + bias) * gate in place (`pending`: gated.Pending or None); returns layer norm (center) or RMS norm
+    of x over its first `width` columns times weight (fp32)."""
+    _need(x, "x", torch.float32)
+    _need(weight, "weight", torch.float32)
+    M, ld = x.shape
+    if out is None:
+        out = torch.empty(M, ld, dtype=dtype, device=x.device)
+    _need(out, "out", dtype)
+    dense = rows = pairs = pw = bias = gate = None
+    top = 0
+    if pending is not None:
+        dense, rows, pairs, pw, bias, gate = (pending.dense, pending.expert_rows, pending.row_of_pair, pending.pair_weight,
+                                              pending.bias, pending.gate)
+        for name, t, want in (("dense", dense, dtype), ("expert_rows", rows, dtype), ("row_of_pair", pairs, torch.int32),
+                              ("pair_weight", pw, torch.float32), ("bias", bias, torch.float32), ("gate", gate, dtype)):
+            if t is not None:
+                _need(t, name, want)
+        if (dense is not None and dense.shape != x.shape) or (gate is not None and gate.shape != x.shape) or (
+                rows is not None and rows.shape[1] != ld):
+            raise ValueError("sublayer or gate does not match x")
+        if pw is not None:
+            top = pw.shape[1]
+    rc = _lib.load().b200_residual_norm(_ptr(x), _ptr(dense), _ptr(rows), _ptr(pairs), _ptr(pw), top, _ptr(bias), _ptr(gate),
+                                        _ptr(weight), float(eps), M, int(width), ld, int(center), _ptr(out), DTYPE_CODE[dtype],
+                                        _stream())
+    check(rc, "b200_residual_norm")
+    return out
+
+
+def mix_heads(q, mix, kv_heads: int, dtype):
+    """[M, H, D] fp32 -> [M, H, kv_heads * D]: per kv head the mix-weighted sum of its query heads."""
+    _need(q, "q", torch.float32)
+    _need(mix, "mix", torch.float32)
+    M, H, D = q.shape
+    out = torch.empty(M, H, kv_heads * D, dtype=dtype, device=q.device)
+    check(_lib.load().b200_mix_heads(_ptr(q), _ptr(mix), _ptr(out), M, H, kv_heads, D, DTYPE_CODE[dtype], _stream()),
+          "b200_mix_heads")
+    return out
+
+
+def mixed_attn(q, k_pool, v_pool, block_table, positions, bias, window: int, out, out_scale: float, status=None):
+    """Windowed attention of mixed queries [M, H, G * Dk] over pages; writes columns [0, H * Dv) of out [M, ld]."""
+    _need(q, "q")
+    _need(k_pool, "k_pool", q.dtype)
+    _need(v_pool, "v_pool", q.dtype)
+    _need(block_table, "block_table", torch.int32)
+    _need(positions, "positions", torch.int32)
+    _need(bias, "bias", torch.float32)
+    M, H, K = q.shape
+    nb, G, page, Dk = k_pool.shape
+    Dv = v_pool.shape[3]
+    if K != G * Dk or v_pool.shape[:3] != k_pool.shape[:3] or block_table.shape[0] != M or out.shape[0] != M or bias.shape[0] != H:
+        raise ValueError("pools, block table, bias or output do not match q")
+    if out.dtype != q.dtype or out.stride(1) != 1:
+        raise ValueError("out must be rows of q's dtype")
+    mp = block_table.shape[1]
+    rc = _lib.load().b200_mixed_attn(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), mp, _ptr(positions), _ptr(bias),
+                                     bias.shape[1], int(window), out.data_ptr(), out.stride(0), float(out_scale), _ptr(status), M,
+                                     H, G, Dk, Dv, page, nb, mp, DTYPE_CODE[q.dtype], _stream())
+    check(rc, "b200_mixed_attn")
+
+
+def conv_silu(x, conv_w, ring, slots, positions, chunk: bool, status=None, out=None):
+    """Causal convolution per channel, then SiLU; earlier inputs from, last inputs to, the slots' rings."""
+    _need(x, "x")
+    _need(conv_w, "conv_w", x.dtype)
+    _need(slots, "slots", torch.int32)
+    _need(positions, "positions", torch.int32)
+    M, C = x.shape
+    taps = conv_w.shape[0]
+    if conv_w.shape[1] != C or (ring is not None and tuple(ring.shape[1:]) != (taps, C)):
+        raise ValueError("weights or ring do not match x")
+    if out is None:
+        out = torch.empty_like(x)
+    rc = _lib.load().b200_conv_silu(_ptr(x), _ptr(conv_w), taps, _ptr(ring), _ptr(slots), _ptr(positions), M, int(chunk), C,
+                                    2**31 - 1 if ring is None else ring.shape[0], _ptr(out), _ptr(status), DTYPE_CODE[x.dtype],
+                                    _stream())
+    check(rc, "b200_conv_silu")
+    return out
+
+
+def state_scan(act, w, state, slots, positions, o, chunk: bool, status=None, ba=None, q_scale: float = 1.0):
+    """Recurrence over [slots, 2, H, d, dv] states from activated rows (q heads, k heads, v heads side by side): the gated
+    delta rule with `ba` (and w.a_log, w.dt_bias), else decays w.decay; o [M, H, dv] fp32."""
+    _need(act, "act")
+    _need(state, "state", torch.float32)
+    _need(slots, "slots", torch.int32)
+    _need(positions, "positions", torch.int32)
+    _need(o, "o", torch.float32)
+    M, ld = act.shape
+    n, _, H, d, dv = state.shape
+    G = w.qk_heads
+    if ld != 2 * G * d + H * dv or o.shape != (M, H, dv):
+        raise ValueError("rows or output do not match the state")
+    delta = ba is not None
+    if delta:
+        _need(ba, "ba", torch.float32)
+    rc = _lib.load().b200_state_scan(_ptr(act), ld, 0, G * d, 2 * G * d, _ptr(ba), _ptr(w.a_log) if delta else None,
+                                     _ptr(w.dt_bias) if delta else None, None if delta else _ptr(w.decay), _ptr(state), _ptr(slots),
+                                     _ptr(positions), _ptr(o), _ptr(status), M, int(chunk), H, G, d, dv, n, float(q_scale),
+                                     DTYPE_CODE[act.dtype], _stream())
+    check(rc, "b200_state_scan")
+
+
+def group_norm_gate(o, weight, gate, eps: float, size: int, shared_weight: bool, scale: float, out):
+    """RMS norm of fp32 groups [M, G, ld] over their first `size` columns, times weight, gate and scale, into rows of `out`."""
+    _need(o, "o", torch.float32)
+    _need(weight, "weight", torch.float32)
+    _need(gate, "gate", out.dtype)
+    M, G, ld = o.shape
+    if gate.numel() != o.numel() or weight.numel() != (ld if shared_weight else G * ld) or out.shape[0] != M or out.shape[1] < G * ld:
+        raise ValueError("weight, gate or out do not match o")
+    rc = _lib.load().b200_group_norm_gate(_ptr(o), _ptr(weight), _ptr(gate), float(eps), M, G, int(size), ld, int(shared_weight),
+                                          float(scale), out.data_ptr(), out.stride(0), DTYPE_CODE[out.dtype], _stream())
+    check(rc, "b200_group_norm_gate")
+
+
+def moe_route_sigmoid(logits, top_k: int, scale: float, renormalize: bool = True):
+    """(ids, weights): the top_k experts by sigmoid(logit), weights normalised over them and times scale."""
+    _need(logits, "logits")
+    T, E = logits.shape
+    ids = torch.empty(T, top_k, dtype=torch.int32, device=logits.device)
+    w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
+    check(_lib.load().b200_moe_route_sigmoid(_ptr(logits), DTYPE_CODE[logits.dtype], T, E, top_k, int(renormalize), float(scale),
+                                             _ptr(ids), _ptr(w), _stream()), "b200_moe_route_sigmoid")
+    return ids, w
+
+
+def moe_permute_workspace_bytes(num_tokens: int, num_experts: int, top_k: int) -> int:
+    return _lib.load().b200_moe_permute_workspace_bytes(num_tokens, num_experts, top_k)
+
+
+class SortedRows:
+    """Token rows copied into expert order, and the tiles the products of experts run over."""
+
+    __slots__ = ("rows", "row_of_pair", "tiles", "num_tiles", "max_tiles", "tile_rows", "experts")
+
+
+def moe_tile_rows(num_pairs: int, num_experts: int, dtype) -> int:
+    """Rows of a tile: what an expert gets on average, in steps the products are built for."""
+    if dtype == torch.float32:
+        return 64
+    mean = num_pairs / num_experts
+    return 32 if mean <= 32 else 64 if mean <= 64 else 128
+
+
+def moe_permute_copy(ids, x, num_experts: int, workspace, tile_rows: int | None = None) -> SortedRows:
+    _need(ids, "ids", torch.int32)
+    _need(x, "x")
+    T, K = ids.shape
+    p = SortedRows()
+    p.experts = num_experts
+    p.tile_rows = tile_rows or moe_tile_rows(T * K, num_experts, x.dtype)
+    p.max_tiles = min(T * K, -(-T * K // p.tile_rows) + num_experts)
+    p.rows = torch.empty(T * K, x.shape[1], dtype=x.dtype, device=x.device)
+    p.row_of_pair = torch.empty(T, K, dtype=torch.int32, device=x.device)
+    p.tiles = torch.empty(p.max_tiles, 4, dtype=torch.int32, device=x.device)
+    p.num_tiles = torch.empty(1, dtype=torch.int32, device=x.device)
+    rc = _lib.load().b200_moe_permute_copy(_ptr(ids), _ptr(x), T, num_experts, K, x.shape[1] * x.element_size(), p.tile_rows,
+                                           _ptr(p.row_of_pair), _ptr(p.tiles), _ptr(p.num_tiles), _ptr(p.rows), _ptr(workspace),
+                                           workspace.numel(), _stream())
+    check(rc, "b200_moe_permute_copy")
+    return p
+
+
+def moe_gate_up(p: SortedRows, w, status=None, limit: float = float("inf"), alpha: float = 1.0, shift: float = 0.0):
+    """Gate and up products of every sorted row with its expert (w [E, 2F, K], gate and up rows in alternating blocks of 128)
+    and the gated unit between them: [rows, F]."""
+    x = p.rows
+    _need(w, "w", x.dtype)
+    n, K = x.shape
+    E, F2, K2 = w.shape
+    if K2 != K or E != p.experts:
+        raise ValueError("weights do not match the rows")
+    if x.dtype == torch.float32:
+        return clamped_glu(_moe_gemm_f32(p, x, w), limit, alpha, shift=shift)
+    h = torch.empty(n, F2 // 2, dtype=x.dtype, device=x.device)
+    rc = _lib.load().b200_moe_bf16_gate_up(_ptr(x), _ptr(w), _ptr(h), _ptr(p.tiles), _ptr(p.num_tiles), _ptr(status), n, E,
+                                           p.max_tiles, p.tile_rows, F2 // 2, K, float(limit), float(alpha), float(shift), _stream())
+    check(rc, "b200_moe_bf16_gate_up")
+    return h
+
+
+def moe_down(p: SortedRows, h, w, status=None):
+    """[rows, N]: every sorted row of h with its expert's w [E, N, K]."""
+    _need(h, "h")
+    _need(w, "w", h.dtype)
+    n, K = h.shape
+    E, N, K2 = w.shape
+    if K2 != K or E != p.experts or n != p.rows.shape[0]:
+        raise ValueError("weights do not match the rows")
+    if h.dtype == torch.float32:
+        return _moe_gemm_f32(p, h, w)
+    y = torch.empty(n, N, dtype=h.dtype, device=h.device)
+    rc = _lib.load().b200_moe_bf16_down(_ptr(h), _ptr(w), _ptr(y), _ptr(p.tiles), _ptr(p.num_tiles), _ptr(status), n, E, p.max_tiles,
+                                        p.tile_rows, N, K, _stream())
+    check(rc, "b200_moe_bf16_down")
+    return y
+
+
+def _moe_gemm_f32(p: SortedRows, x, w):
+    y = torch.empty(x.shape[0], w.shape[1], dtype=torch.float32, device=x.device)
+    rc = _lib.load().b200_moe_gemm_f32(_ptr(x), _ptr(w), _ptr(y), _ptr(p.tiles), _ptr(p.num_tiles), x.shape[0], p.experts, p.max_tiles,
+                                       w.shape[1], w.shape[2], _stream())
+    check(rc, "b200_moe_gemm_f32")
+    return y
 
 
 # ------------------------------------------------------------------------ MoE

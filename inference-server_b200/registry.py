@@ -29,7 +29,12 @@ def _layered_from_folder(folder: str, config: dict, **kw):
 
 def _layered_shapes():
     from . import layered
-    return layered.CONFIGS
+    return {k: c for k, c in layered.CONFIGS.items() if not c.gated}
+
+
+def _gated_shapes():
+    from . import layered
+    return {k: c for k, c in layered.CONFIGS.items() if c.gated}
 
 
 def _layered_from_shape(cfg, **kw):
@@ -49,14 +54,15 @@ def _qwen_from_shape(cfg, **kw):
 
 QWEN3_MOE = Family(None, _qwen_shapes, _qwen_from_shape)
 LAYERED = Family("layered", _layered_shapes, _layered_from_shape, _layered_from_folder)
+GATED = Family("gated", _gated_shapes, _layered_from_shape, _layered_from_folder)
 
 # config.json `architecture` -> family
-ARCHITECTURES: dict[str, Family] = {"Sulepel": LAYERED}
+ARCHITECTURES: dict[str, Family] = {"Sulepel": LAYERED, "Sefalorn": GATED}
 
 
 def shape_family(name: str) -> tuple[Family, object] | None:
     """(family, shape) of a built-in shape name."""
-    for family in (QWEN3_MOE, LAYERED):
+    for family in (QWEN3_MOE, LAYERED, GATED):
         shapes = family.shapes()
         if name in shapes:
             return family, shapes[name]
