@@ -766,6 +766,10 @@ def mixed_attn(q, k_pool, v_pool, block_table, positions, bias, window: int, out
     check(rc, "b200_mixed_attn")
 
 
+def mixed_attn_prefill_supported(num_q_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, dtype) -> bool:
+    return False
+
+
 def conv_silu(x, conv_w, ring, slots, positions, chunk: bool, status=None, out=None):
     """Causal convolution per channel, then SiLU; earlier inputs from, last inputs to, the slots' rings."""
     _need(x, "x")
