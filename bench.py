@@ -510,7 +510,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--model", default="qwen3-30b-a3b",
-                    help="a built-in shape; a layer-list shape (sulepel-2048, sulepel-4096) measures decode, prefill and "
+                    help="a built-in shape; a layer-list shape (sulepel-2048, sulepel-4096, sefalorn-2048, sefalorn-4096) measures decode, prefill and "
                          "every kernel beside Qwen3-MoE of the same size (bench_layered.py)")
     ap.add_argument("--batch", type=int, default=256, help="concurrent sequences per GPU")
     ap.add_argument("--gen-tokens", type=int, default=256)

@@ -1,4 +1,4 @@
-"""`bench.py --model sulepel-...`: decode and prefill throughput of a layer-list decoder with random weights, its kernels one by
+"""`bench.py --model sulepel-...` or `sefalorn-...`: decode and prefill throughput of a layer-list decoder with random weights, its kernels one by
 one against their rooflines, and beside them the like kernels and the throughput of the framework's closest other model
 (Qwen3-MoE) at the same width, head counts, number of layers, batch and context lengths.
 
@@ -298,9 +298,10 @@ def throughput(eng, args, table, lens, prompt_tokens: int, prompt_blocks: int, c
     out = {"decode_ms": events(step, args.steps)}
     out["decode_tok_s"] = B / out["decode_ms"] * 1e3
     be = backend_mod.B200Backend(eng)
-    be._alloc.free = []
+    be._alloc.free, be._slots.free = [], []
     now = eng.ctx_lens[:B].cpu().tolist()
-    rows = [backend_mod.SeqKV(block_ids=table[b][: -(-(lens[b] + args.gen_tokens) // PAGE)].tolist(), ctx_len=now[b]) for b in range(B)]
+    rows = [backend_mod.SeqKV(block_ids=table[b][: -(-(lens[b] + args.gen_tokens) // PAGE)].tolist(), ctx_len=now[b],
+                              slot=b if getattr(eng, "num_slots", 0) else None) for b in range(B)]
     batch = backend_mod.PagedBatch(rows=rows)
     tok = torch.randint(0, V, (B, 1)).pin_memory()
     for _ in range(3):
@@ -316,8 +317,10 @@ def throughput(eng, args, table, lens, prompt_tokens: int, prompt_blocks: int, c
     prompts = [torch.randint(0, V, (prompt_tokens,), generator=g).tolist() for _ in range(4)]
     blocks = list(range(prompt_blocks, prompt_blocks + -(-prompt_tokens // PAGE)))
 
+    spare_slot = max(0, getattr(eng, "num_slots", 0) - 1)
+
     def prefill(i):
-        eng.prefill(prompts[i % 4], blocks)
+        eng.prefill(prompts[i % 4], blocks, slot=spare_slot)
 
     for i in range(3):
         prefill(i)
@@ -344,15 +347,22 @@ def run(args, build_workload, ClockSampler) -> None:
     gen = torch.Generator(device=dev).manual_seed(5)
     sizes = dict(num_blocks=blocks, max_batch=args.batch, max_pages_per_seq=max_pages, device=dev)
     chunk_first, chunk_n = max(0, args.prompt_tokens - 2048), min(2048, args.prompt_tokens)
-    att = next(s.mixer for s in cfg.layer_list if isinstance(s.mixer, lay.AttentionSpec))
+    att = next(s.mixer.left for s in cfg.layer_list if hasattr(s.mixer, "left")) if cfg.gated else \
+        next(s.mixer for s in cfg.layer_list if isinstance(s.mixer, lay.AttentionSpec))
 
     eng = lay.LayeredEngine(cfg, **sizes)
     fill(eng, gen)
     with ClockSampler(0) as clocks:
         mine = throughput(eng, args, table, lens, args.prompt_tokens, spare, clocks)
     clock_info = clocks.summary()
-    mine["decode_kernels"] = decode_kernels(eng, args.batch, lens_np)
-    mine["prompt_kernels"] = prompt_kernels(eng, chunk_first, chunk_n)
+    if cfg.gated:
+        import bench_gated
+        mine["decode_kernels"] = bench_gated.decode_kernels(eng, args.batch, lens_np)
+        mine["prompt_kernels"] = bench_gated.prompt_kernels(eng, chunk_first, chunk_n)
+        mine["state_bytes_per_sequence"] = eng.state_bytes_per_sequence()
+    else:
+        mine["decode_kernels"] = decode_kernels(eng, args.batch, lens_np)
+        mine["prompt_kernels"] = prompt_kernels(eng, chunk_first, chunk_n)
     launches, kv = eng.kernel_launches_per_step, eng.kv_bytes_per_token()
     del eng
     torch.cuda.empty_cache()

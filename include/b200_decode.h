@@ -447,11 +447,24 @@ int b200_mix_heads(const float* q, const float* mix, void* out, int num_rows, in
  *   v_pool [num_blocks, num_kv_heads, page_size, value_dim]; block_table rows table_stride apart (0: one row for all);
  *   positions [num_rows]; bias [num_q_heads, bias_ld] fp32, bias_ld at least min(window, positions of the table);
  *   out [num_rows, out_ld], head h at column h * value_dim.
+ * bf16 pools with pages of 16 and sizes in multiples of 64 run on the tensor cores, a row's window in splits of split_tokens (a
+ * multiple of 32) whose partials go through the workspace; split_tokens 0 and every other shape take the generic kernel.
  */
+size_t b200_mixed_attn_workspace_bytes(int num_rows, int num_q_heads, int num_kv_heads, int key_dim, int value_dim, int window,
+                                       int max_pages_per_seq, int split_tokens);
 int b200_mixed_attn(const void* q, const void* k_pool, const void* v_pool, const int32_t* block_table, int table_stride,
                     const int32_t* positions, const float* bias, int bias_ld, int window, void* out, int out_ld,
-                    float out_scale, void* status_word, int num_rows, int num_q_heads, int num_kv_heads, int key_dim,
-                    int value_dim, int page_size, int num_blocks, int max_pages_per_seq, int dtype, void* stream);
+                    float out_scale, void* workspace, size_t workspace_bytes, void* status_word, int num_rows, int num_q_heads,
+                    int num_kv_heads, int key_dim, int value_dim, int page_size, int num_blocks, int max_pages_per_seq,
+                    int split_tokens, int dtype, void* stream);
+
+/* The same for a chunk of consecutive prompt tokens of one sequence, positions first_position.. (their K/V already in the
+ * pages), on the tcgen05 tensor cores; bf16, pages of 16.  _supported: whether it is built for these sizes. */
+int b200_mixed_attn_prefill_supported(int num_q_heads, int num_kv_heads, int key_dim, int value_dim);
+int b200_mixed_attn_prefill(const void* q, const void* k_pool, const void* v_pool, const int32_t* block_table_row,
+                            const float* bias, int bias_ld, int window, void* out, int out_ld, float out_scale,
+                            void* status_word, int num_tokens, int first_position, int num_q_heads, int num_kv_heads,
+                            int key_dim, int value_dim, int page_size, int num_blocks, int max_pages_per_seq, void* stream);
 
 /*
  * out[m] = z * sigmoid(z), z = sum_j conv_w[j] * in[position - taps + 1 + j] per channel, zeros before the sequence's start.

@@ -8,7 +8,17 @@
 // B[h][d] = sum_g T[h, g] r1_g ln(1 + r2_g d) is a table over the window's distances.  Every query head then meets the whole
 // of a token's keys, and the values of its own kv head.
 //
-// Generic kernel (here): any sizes, bf16 or fp32, fp32 arithmetic, one CTA per (row, query head).
+// Decode kernel: bf16, key and value sizes multiples of 64.  grid (rows, splits); a CTA owns up to `split_tokens` consecutive
+// tokens of one row, for all heads, and streams their pages (a producer warp, one TMA box of 16 tokens x 128 B per kv head and
+// 64 columns, mbarrier ring of pages).  Eight consumer warps take two pages (32 tokens) at a time:
+//   scores   an item is (page, half of its tokens, 16 query heads): mma.sync m16n8k16 over the keys of all kv heads, queries
+//            from shared memory; times log2 e, less the distance table, masked, into a score tile in shared memory
+//   values   a unit is (kv head, 16 of its query heads, 64 value columns): online softmax over the tile's 32 tokens in the A
+//            operand's registers, O += P V
+// with one 256-thread barrier per two pages (the score tile is double-buffered).  Rows of one split are written as they are,
+// others as fp32 partials that a second kernel folds in split order.
+//
+// Generic kernel: any sizes, bf16 or fp32, fp32 arithmetic, one CTA per (row, query head).
 
 #include "glue.cuh"
 
@@ -105,6 +115,355 @@ mixed_attn_generic_kernel(const MixedAttnParams p) {
   }
 }
 
+constexpr int kMdPage = 16;
+constexpr int kMdWarps = 8;                    // consumers
+constexpr int kMdThreads = (kMdWarps + 1) * 32;
+constexpr int kMdScoreLd = 40;                 // floats per head of a score tile (32 tokens): float2 reads of 8 heads hit all banks
+constexpr float kMdLog2e = 1.4426950408889634f;
+
+struct MixedDecodeParams {
+  MixedAttnParams a;
+  float* part_o;    // [rows, heads, max_splits, dv]
+  float2* part_ml;
+  int split_tokens, max_splits, stages;
+};
+
+// UNITS: units (see above) a warp may own.
+template <int UNITS>
+__global__ void __launch_bounds__(kMdThreads, 1)
+mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const MixedDecodeParams pp) {
+#ifdef B200_DEVICE_OK
+  const MixedAttnParams& p = pp.a;
+  extern __shared__ uint8_t smem_raw[];
+  grid_dep_wait();
+  grid_dep_launch();
+  const int row = blockIdx.x, split = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int pos = p.positions[row];
+  if (pos < 0 || pos >= p.max_pages * kMdPage) {
+    if (threadIdx.x == 0) set_error(p.err, kErrDevBadCtxLen);
+    pos = 0;
+  }
+  const int lo = max(0, pos - p.window + 1);
+  const int range0 = lo & ~(kMdPage - 1);
+  const int start = range0 + split * pp.split_tokens;
+  if (start > pos) return;  // uniform for the whole CTA
+  const int nsplits = (pos + 1 - range0 + pp.split_tokens - 1) / pp.split_tokens;
+  const int end = min(pos + 1, start + pp.split_tokens);
+  const int npages = (end - start + kMdPage - 1) / kMdPage, first_page = start / kMdPage;
+
+  const uint32_t ring = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* ring_ptr = smem_raw + (ring - smem_u32(smem_raw));
+  const int kc = p.kv_heads * (p.dk / 64), vc = p.kv_heads * (p.dv / 64);  // 2 KiB boxes of a page
+  const uint32_t stage_bytes = static_cast<uint32_t>(kc + vc) * 2048u;
+  uint8_t* after = ring_ptr + static_cast<size_t>(pp.stages) * stage_bytes;
+  const uint32_t bars = ring + pp.stages * stage_bytes;  // full[stages], empty[stages]: up to 16 of each
+  float* sc = reinterpret_cast<float*>(after + 256);     // [2][heads16][kMdScoreLd]
+  const int mt = (p.heads + 15) / 16, K = p.kv_heads * p.dk, q_ld = K + 8;
+  __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(sc + 2 * mt * 16 * kMdScoreLd);  // [mt * 16][q_ld]
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < pp.stages; ++s) {
+      mbar_init(bars + 8 * s, 1);
+      mbar_init(bars + 8 * (pp.stages + s), kMdWarps);
+    }
+    fence_mbar_init();
+    fence_proxy_async();
+  }
+  __syncthreads();
+
+  if (warp == kMdWarps) {
+    // ------------------------------------------------------------ producer --
+    if (lane == 0) {
+      tma_prefetch_desc(&k_map);
+      tma_prefetch_desc(&v_map);
+    }
+    const int* table = p.table + static_cast<size_t>(row) * p.table_stride + first_page;
+    int ids = 0;
+    for (int i = 0; i < npages; ++i) {
+      if ((i & 31) == 0) {
+        ids = i + lane < npages ? table[i + lane] : 0;
+        if (ids < 0 || ids >= p.num_blocks) {
+          set_error(p.err, kErrDevBadBlockId);
+          ids = 0;
+        }
+      }
+      const int id = __shfl_sync(0xffffffffu, ids, i & 31);
+      const int slot = i % pp.stages;
+      if (!__all_sync(0xffffffffu, mbar_wait(bars + 8 * (pp.stages + slot), ((i / pp.stages) & 1) ^ 1, p.err))) break;
+      if (lane == 0) mbar_arrive_expect_tx(bars + 8 * slot, stage_bytes);
+      __syncwarp();
+      for (int b = lane; b < kc + vc; b += 32) {
+        const bool is_v = b >= kc;
+        const int bb = is_v ? b - kc : b, n = is_v ? p.dv / 64 : p.dk / 64;
+        const int head = bb / n;
+        tma_load_2d(ring + slot * stage_bytes + b * 2048u, is_v ? &v_map : &k_map, bars + 8 * slot, (bb - head * n) * 64,
+                    (id * p.kv_heads + head) * kMdPage);
+      }
+    }
+    return;
+  }
+
+  // ------------------------------------------------------------- consumers --
+  {  // the row's mixed queries, zero rows after the last head
+    const uint4* src = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) + static_cast<size_t>(row) * p.heads * K);
+    const int per_row = K / 8;
+    for (int i = threadIdx.x; i < mt * 16 * per_row; i += kMdWarps * 32) {
+      const int h = i / per_row, c = i - h * per_row;
+      *reinterpret_cast<uint4*>(q_sm + static_cast<size_t>(h) * q_ld + c * 8) = h < p.heads ? src[i] : make_uint4(0u, 0u, 0u, 0u);
+    }
+  }
+  const int per = p.heads / p.kv_heads, sub = (per + 15) / 16, dvc = p.dv / 64;
+  const int units = p.kv_heads * sub * dvc;
+  float o[UNITS][8][4], m_run[UNITS][2], l_run[UNITS][2];
+#pragma unroll
+  for (int u = 0; u < UNITS; ++u) {
+#pragma unroll
+    for (int n = 0; n < 8; ++n) o[u][n][0] = o[u][n][1] = o[u][n][2] = o[u][n][3] = 0.f;
+    m_run[u][0] = m_run[u][1] = -INFINITY;
+    l_run[u][0] = l_run[u][1] = 0.f;
+  }
+  const int gq = lane >> 2, tq = lane & 3;
+  const int lj = lane >> 3, lr = lane & 7;
+  const uint32_t q_base = smem_u32(q_sm);
+  asm volatile("bar.sync 1, 256;" ::: "memory");  // queries in place
+
+  bool alive = true;
+  const int tiles = (npages + 1) / 2;
+#pragma unroll 1
+  for (int tile = 0; tile < tiles; ++tile) {
+    const int pages_here = min(2, npages - tile * 2);
+    float* score = sc + (tile & 1) * mt * 16 * kMdScoreLd;
+    for (int pg = 0; pg < pages_here && alive; ++pg) {
+      const int i = tile * 2 + pg;
+      alive = mbar_wait(bars + 8 * (i % pp.stages), (i / pp.stages) & 1, p.err);
+    }
+    // ---- scores
+    for (int item = warp; item < pages_here * 2 * mt; item += kMdWarps) {
+      const int pg = item % pages_here, rest = item / pages_here, th = rest & 1, mi = rest >> 1;
+      const int i = tile * 2 + pg;
+      const uint32_t kbase = ring + (i % pp.stages) * stage_bytes;
+      const int tok0 = start + i * kMdPage + th * 8 + 2 * tq;  // token of c0, c2; c1, c3 are the next one
+      // the distance table's entries travel while the products run
+      float bias[2][2];
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int h = mi * 16 + gq + hh * 8, d = pos - tok0 - e;
+          bias[hh][e] = h < p.heads && d >= 0 && d < p.window ? __ldg(p.bias + static_cast<size_t>(h) * p.bias_ld + d) * kMdLog2e : INFINITY;
+        }
+      float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+      const uint32_t a_addr = q_base + ((mi * 16 + (lj & 1) * 8 + lr) * q_ld + (lj >> 1) * 8) * 2;
+      for (int c = 0; c < kc; ++c) {  // 64 of the key columns
+        const uint32_t box = kbase + c * 2048u;
+#pragma unroll
+        for (int k2 = 0; k2 < 2; ++k2) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4(box + swz128(th * 8 + lr, k2 * 4 + lj), b0, b1, b2, b3);
+          uint32_t a0[4], a1[4];
+          ldmatrix_x4(a_addr + (c * 64 + k2 * 32) * 2, a0[0], a0[1], a0[2], a0[3]);
+          ldmatrix_x4(a_addr + (c * 64 + k2 * 32 + 16) * 2, a1[0], a1[1], a1[2], a1[3]);
+          mma_bf16_16816(acc[0], a0, b0, b1);
+          mma_bf16_16816(acc[1], a1, b2, b3);
+        }
+      }
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh) {
+        const float2 v = make_float2(fmaf(acc[0][2 * hh] + acc[1][2 * hh], kMdLog2e, -bias[hh][0]),
+                                     fmaf(acc[0][2 * hh + 1] + acc[1][2 * hh + 1], kMdLog2e, -bias[hh][1]));
+        *reinterpret_cast<float2*>(score + (mi * 16 + gq + hh * 8) * kMdScoreLd + pg * 16 + th * 8 + 2 * tq) = v;
+      }
+    }
+    asm volatile("bar.sync 1, 256;" ::: "memory");  // the score tile is complete; the other one has been read by everybody
+    // ---- values
+#pragma unroll
+    for (int u = 0; u < UNITS; ++u) {
+      const int unit = warp + u * kMdWarps;
+      if (unit >= units) break;
+      const int vcol = unit % dvc, hs = unit / dvc, c = hs / sub, ms = hs - c * sub;
+      const int h0 = ms * 16 + gq;  // head inside the kv group of fragment rows 0-7; +8 for the others
+      const float* s0 = score + (c * per + min(h0, per - 1)) * kMdScoreLd;
+      const float* s1 = score + (c * per + min(h0 + 8, per - 1)) * kMdScoreLd;
+      float s[2][2][4];  // [page][row half][k 2tq, 2tq+1, 2tq+8, 2tq+9]
+      float mx0 = -INFINITY, mx1 = -INFINITY;
+#pragma unroll
+      for (int pg = 0; pg < 2; ++pg) {
+        if (pg < pages_here) {
+          const float2 a = *reinterpret_cast<const float2*>(s0 + pg * 16 + 2 * tq), b = *reinterpret_cast<const float2*>(s0 + pg * 16 + 8 + 2 * tq);
+          const float2 x = *reinterpret_cast<const float2*>(s1 + pg * 16 + 2 * tq), y = *reinterpret_cast<const float2*>(s1 + pg * 16 + 8 + 2 * tq);
+          s[pg][0][0] = a.x; s[pg][0][1] = a.y; s[pg][0][2] = b.x; s[pg][0][3] = b.y;
+          s[pg][1][0] = x.x; s[pg][1][1] = x.y; s[pg][1][2] = y.x; s[pg][1][3] = y.y;
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[pg][0][e] = s[pg][1][e] = -INFINITY;
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          mx0 = fmaxf(mx0, s[pg][0][e]);
+          mx1 = fmaxf(mx1, s[pg][1][e]);
+        }
+      }
+      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+      const float n0 = fmaxf(m_run[u][0], mx0), n1 = fmaxf(m_run[u][1], mx1);
+      const float r0 = n0 == -INFINITY ? 0.f : n0, r1 = n1 == -INFINITY ? 0.f : n1;  // nothing seen yet: all weights come out 0
+      const float al0 = exp2f(m_run[u][0] - r0), al1 = exp2f(m_run[u][1] - r1);
+      m_run[u][0] = n0;
+      m_run[u][1] = n1;
+      uint32_t pa[2][4];
+      float sum0 = 0.f, sum1 = 0.f;
+#pragma unroll
+      for (int pg = 0; pg < 2; ++pg) {
+        float e0[4], e1[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          e0[e] = exp2f(s[pg][0][e] - r0);
+          e1[e] = exp2f(s[pg][1][e] - r1);
+          sum0 += e0[e];
+          sum1 += e1[e];
+        }
+        pa[pg][0] = pack_bf16x2(e0[0], e0[1]);
+        pa[pg][1] = pack_bf16x2(e1[0], e1[1]);
+        pa[pg][2] = pack_bf16x2(e0[2], e0[3]);
+        pa[pg][3] = pack_bf16x2(e1[2], e1[3]);
+      }
+      l_run[u][0] = l_run[u][0] * al0 + sum0;
+      l_run[u][1] = l_run[u][1] * al1 + sum1;
+      if (__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) {
+#pragma unroll
+        for (int n = 0; n < 8; ++n) {
+          o[u][n][0] *= al0;
+          o[u][n][1] *= al0;
+          o[u][n][2] *= al1;
+          o[u][n][3] *= al1;
+        }
+      }
+#pragma unroll
+      for (int pg = 0; pg < 2; ++pg) {
+        if (pg >= pages_here) break;
+        const uint32_t vbase = ring + ((tile * 2 + pg) % pp.stages) * stage_bytes + (kc + c * dvc + vcol) * 2048u;
+#pragma unroll
+        for (int np = 0; np < 4; ++np) {
+          uint32_t v0, v1, v2, v3;
+          ldmatrix_x4_trans(vbase + swz128((lj & 1) * 8 + lr, np * 2 + (lj >> 1)), v0, v1, v2, v3);
+          mma_bf16_16816(o[u][2 * np], pa[pg], v0, v1);
+          mma_bf16_16816(o[u][2 * np + 1], pa[pg], v2, v3);
+        }
+      }
+    }
+    __syncwarp();
+    if (lane == 0)
+      for (int pg = 0; pg < pages_here; ++pg) mbar_arrive(bars + 8 * (pp.stages + (tile * 2 + pg) % pp.stages));
+  }
+
+#pragma unroll
+  for (int u = 0; u < UNITS; ++u) {
+    const int unit = warp + u * kMdWarps;
+    if (unit >= units) break;
+    const int vcol = unit % dvc, hs = unit / dvc, c = hs / sub, ms = hs - c * sub;
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      float l = l_run[u][hh];
+      l += __shfl_xor_sync(0xffffffffu, l, 1);
+      l += __shfl_xor_sync(0xffffffffu, l, 2);
+      const int hl = ms * 16 + gq + hh * 8;
+      if (hl >= per) continue;
+      const int h = c * per + hl;
+      if (nsplits == 1) {
+        const float inv = p.out_scale / l;
+        __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + static_cast<size_t>(row) * p.out_ld + static_cast<size_t>(h) * p.dv + vcol * 64;
+#pragma unroll
+        for (int n = 0; n < 8; ++n)
+          *reinterpret_cast<uint32_t*>(dst + n * 8 + 2 * tq) = pack_bf16x2(o[u][n][2 * hh] * inv, o[u][n][2 * hh + 1] * inv);
+      } else {
+        const size_t at = (static_cast<size_t>(row) * p.heads + h) * pp.max_splits + split;
+#pragma unroll
+        for (int n = 0; n < 8; ++n)
+          *reinterpret_cast<float2*>(pp.part_o + at * p.dv + vcol * 64 + n * 8 + 2 * tq) = make_float2(o[u][n][2 * hh], o[u][n][2 * hh + 1]);
+        if (vcol == 0 && tq == 0) pp.part_ml[at] = make_float2(m_run[u][hh], l);
+      }
+    }
+  }
+#endif
+}
+
+// Folds the partials of one (row, head) in split order; rows of one split are already written.  A warp per (row, head).
+__global__ void __launch_bounds__(128)
+mixed_reduce_kernel(const MixedDecodeParams pp) {
+  const MixedAttnParams& p = pp.a;
+  grid_dep_wait();
+  grid_dep_launch();
+  const int item = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (item >= p.rows * p.heads) return;
+  const int row = item / p.heads, h = item - row * p.heads;
+  int pos = p.positions[row];
+  if (pos < 0 || pos >= p.max_pages * kMdPage) pos = 0;
+  const int range0 = max(0, pos - p.window + 1) & ~(kMdPage - 1);
+  const int n = (pos + 1 - range0 + pp.split_tokens - 1) / pp.split_tokens;
+  if (n <= 1) return;
+  const size_t base = static_cast<size_t>(item) * pp.max_splits;
+  float m = -INFINITY;
+  for (int s = lane; s < n; s += 32) m = fmaxf(m, pp.part_ml[base + s].x);
+  m = warp_max(m);
+  float den = 0.f;
+  for (int s = lane; s < n; s += 32) {
+    const float2 ml = pp.part_ml[base + s];
+    den += exp2f(ml.x - m) * ml.y;
+  }
+  const float inv = p.out_scale / warp_sum(den);
+  __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + static_cast<size_t>(row) * p.out_ld + static_cast<size_t>(h) * p.dv;
+  for (int d = lane * 2; d < p.dv; d += 64) {
+    float a = 0.f, b = 0.f;
+#pragma unroll 4
+    for (int s = 0; s < n; ++s) {
+      const float w = exp2f(pp.part_ml[base + s].x - m);
+      const float2 v = *reinterpret_cast<const float2*>(pp.part_o + (base + s) * p.dv + d);
+      a = fmaf(w, v.x, a);
+      b = fmaf(w, v.y, b);
+    }
+    *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16x2(a * inv, b * inv);
+  }
+}
+
+// Splits of the longest window.
+static int mixed_max_splits(int window, int max_pages, int split_tokens) {
+  const long long all = static_cast<long long>(max_pages) * kMdPage;
+  long long seen = (static_cast<long long>(window) + kMdPage - 1) / kMdPage * kMdPage + kMdPage;
+  if (seen > all) seen = all;
+  return static_cast<int>((seen + split_tokens - 1) / split_tokens);
+}
+
+// Pages in flight and shared memory of the decode kernel; 0: not built for this shape.
+static int mixed_decode_stages(int heads, int kv_heads, int dk, int dv, size_t* smem_out) {
+  if (heads % kv_heads || dk % 64 || dv % 64) return 0;
+  const int per = heads / kv_heads, units = kv_heads * ((per + 15) / 16) * (dv / 64);
+  if (units > 4 * kMdWarps) return 0;
+  const size_t mt = (heads + 15) / 16, K = static_cast<size_t>(kv_heads) * dk;
+  const size_t fixed = 1024 + 256 + 2 * mt * 16 * kMdScoreLd * 4 + mt * 16 * (K + 8) * 2;
+  const size_t stage = static_cast<size_t>(kv_heads) * (dk + dv) / 64 * 2048, room = 227 * 1024;
+  if (fixed + 4 * stage > room) return 0;
+  size_t stages = (room - fixed) / stage;
+  // small pages: leave room for a second CTA on the multiprocessor once 64 KiB are in flight
+  const size_t enough = (64 * 1024 + stage - 1) / stage + 2;
+  if (stages > enough && fixed + enough * stage <= room / 2) stages = enough;
+  if (stages > 16) stages = 16;
+  if (smem_out) *smem_out = fixed + stages * stage;
+  return static_cast<int>(stages);
+}
+
+template <int UNITS>
+static int launch_mixed_decode(const CUtensorMap& km, const CUtensorMap& vm, const MixedDecodeParams& pp, size_t smem, cudaStream_t st) {
+  int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mixed_decode_kernel<UNITS>), 227 * 1024);
+  if (rc) return rc;
+  B200_CUDA(launch_overlapped(mixed_decode_kernel<UNITS>, dim3(pp.a.rows, pp.max_splits), dim3(kMdThreads), smem, st, km, vm, pp));
+  if (pp.max_splits > 1)
+    B200_CUDA(launch_overlapped(mixed_reduce_kernel, dim3((pp.a.rows * pp.a.heads + 3) / 4), dim3(128), 0, st, pp));
+  return 0;
+}
+
 template <typename T>
 static int launch_mixed_generic(const MixedAttnParams& p, cudaStream_t st) {
   const size_t smem = (static_cast<size_t>(p.kv_heads) * p.dk + static_cast<size_t>(kMixWarps) * p.dv) * 4;
@@ -125,11 +484,19 @@ static int launch_mixed_generic(const MixedAttnParams& p, cudaStream_t st) {
 
 using namespace b200;
 
+extern "C" size_t b200_mixed_attn_workspace_bytes(int num_rows, int num_q_heads, int num_kv_heads, int key_dim, int value_dim,
+                                                  int window, int max_pages_per_seq, int split_tokens) {
+  if (num_rows <= 0 || num_q_heads <= 0 || num_kv_heads <= 0 || key_dim <= 0 || value_dim <= 0 || window <= 0 ||
+      max_pages_per_seq <= 0 || split_tokens <= 0 || mixed_decode_stages(num_q_heads, num_kv_heads, key_dim, value_dim, nullptr) == 0)
+    return 256;
+  return carve(nullptr, num_rows, num_q_heads, value_dim, mixed_max_splits(window, max_pages_per_seq, split_tokens)).bytes;
+}
+
 extern "C" int b200_mixed_attn(const void* q, const void* k_pool, const void* v_pool, const int32_t* block_table,
                                int table_stride, const int32_t* positions, const float* bias, int bias_ld, int window,
-                               void* out, int out_ld, float out_scale, void* status_word, int num_rows, int num_q_heads,
-                               int num_kv_heads, int key_dim, int value_dim, int page_size, int num_blocks,
-                               int max_pages_per_seq, int dtype, void* stream) {
+                               void* out, int out_ld, float out_scale, void* workspace, size_t workspace_bytes,
+                               void* status_word, int num_rows, int num_q_heads, int num_kv_heads, int key_dim, int value_dim,
+                               int page_size, int num_blocks, int max_pages_per_seq, int split_tokens, int dtype, void* stream) {
   B200_REQUIRE(q && k_pool && v_pool && block_table && positions && bias && out, "mixed_attn: null pointer");
   B200_REQUIRE(num_rows >= 0 && num_rows <= 65535 && num_q_heads > 0 && num_kv_heads > 0 && num_q_heads % num_kv_heads == 0 &&
                    key_dim > 0 && value_dim > 0 && value_dim <= 1024 && page_size > 0 && num_blocks > 0 &&
@@ -144,5 +511,33 @@ extern "C" int b200_mixed_attn(const void* q, const void* k_pool, const void* v_
   const MixedAttnParams p{q, k_pool, v_pool, block_table, table_stride, positions, bias, bias_ld, window, out, out_ld,
                           out_scale, static_cast<int*>(status_word), num_rows, num_q_heads, num_kv_heads, key_dim, value_dim,
                           page_size, num_blocks, max_pages_per_seq};
+  size_t smem = 0;
+  const int stages = dtype == 0 && page_size == kMdPage && split_tokens > 0
+                         ? mixed_decode_stages(num_q_heads, num_kv_heads, key_dim, value_dim, &smem) : 0;
+  if (stages > 0) {
+    B200_REQUIRE(split_tokens % 32 == 0 && out_ld % 2 == 0, "mixed_attn: split_tokens %d is no multiple of 32", split_tokens);
+    B200_REQUIRE(aligned16({q, k_pool, v_pool}) && (reinterpret_cast<uintptr_t>(out) & 3) == 0, "mixed_attn: buffers must be aligned");
+    MixedDecodeParams pp{p, nullptr, nullptr, split_tokens, mixed_max_splits(window, max_pages_per_seq, split_tokens), stages};
+    B200_REQUIRE(pp.max_splits <= 65535, "mixed_attn: grid too large");
+    if (pp.max_splits > 1) {
+      const AttnWorkspace w = carve(workspace, num_rows, num_q_heads, value_dim, pp.max_splits);
+      if (workspace == nullptr || workspace_bytes < w.bytes) {
+        set_detail("mixed_attn: workspace %zu < required %zu", workspace_bytes, w.bytes);
+        return -kErrWorkspace;
+      }
+      pp.part_o = w.o;
+      pp.part_ml = w.ml;
+    }
+    CUtensorMap km, vm;
+    const uint64_t pool_rows = static_cast<uint64_t>(num_blocks) * num_kv_heads * kMdPage;
+    int rc = get_tensor_map_2d(k_pool, pool_rows, key_dim, 2, kMdPage, 64, &km);
+    if (rc) return rc;
+    rc = get_tensor_map_2d(v_pool, pool_rows, value_dim, 2, kMdPage, 64, &vm);
+    if (rc) return rc;
+    const int per = num_q_heads / num_kv_heads, units = num_kv_heads * ((per + 15) / 16) * (value_dim / 64);
+    if (units <= kMdWarps) return launch_mixed_decode<1>(km, vm, pp, smem, as_stream(stream));
+    if (units <= 2 * kMdWarps) return launch_mixed_decode<2>(km, vm, pp, smem, as_stream(stream));
+    return launch_mixed_decode<4>(km, vm, pp, smem, as_stream(stream));
+  }
   return dtype == 0 ? launch_mixed_generic<__nv_bfloat16>(p, as_stream(stream)) : launch_mixed_generic<float>(p, as_stream(stream));
 }

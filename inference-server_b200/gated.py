@@ -301,6 +301,7 @@ class GatedMechanisms:
             taps = spec.mixer.right.taps if isinstance(spec.mixer, ParallelSpec) else 1
             self.rings.append(torch.zeros(num_slots + 1, taps, w.channels, dtype=self.dtype, device=self.device) if taps > 1 else None)
         self._moe_ws: list[torch.Tensor] = []
+        self._mixed_ws: dict[tuple, tuple[int, torch.Tensor]] = {}
 
     def _add_norm(self, x, pending: Pending | None, weight, out=None):
         return ops.residual_norm(x, pending, weight, self.cfg.norm_eps, self.cfg.width, out=out, dtype=self.dtype)
@@ -339,7 +340,26 @@ class GatedMechanisms:
 
     def _window_attention(self, q, kp, vp, a: WindowAttentionSpec, w: GatedWeights, rows: Rows, scale: float, out) -> None:
         qm = ops.mix_heads(q, w.mix, a.kv_heads, self.dtype)
-        ops.mixed_attn(qm, kp, vp, rows.table, rows.pos, w.bias, a.window, out, scale, self.status)
+        tiled = ops.mixed_attn_prefill_supported(a.heads, a.kv_heads, w.Dk, w.Dv, self.dtype)
+        for lo, hi, chunk in rows.parts():
+            if chunk and tiled:
+                ops.mixed_attn_prefill(qm[lo:hi], kp, vp, rows.table[0], rows.first, w.bias, a.window, out[lo:hi], scale, self.status)
+            else:
+                split, ws = (None, None) if chunk and self.dtype == torch.bfloat16 else self._mixed_plan(hi - lo, a, w)
+                ops.mixed_attn(qm[lo:hi], kp, vp, rows.table[lo:hi], rows.pos[lo:hi], w.bias, a.window, out[lo:hi], scale, self.status,
+                               split, ws)
+
+    def _mixed_plan(self, rows: int, a: WindowAttentionSpec, w: GatedWeights):
+        """(tokens per split, workspace) of the decode attention kernel; one workspace per shape and number of rows, kept for the
+        graphs that use it."""
+        if self.dtype != torch.bfloat16:
+            return 0, None
+        key = (rows, a, w.Dk, w.Dv)
+        if key not in self._mixed_ws:
+            split = self._fixed_split or ops.mixed_split_tokens(rows, a.window, self.max_pages * PAGE)
+            self._mixed_ws[key] = (split, ops.mixed_attn_workspace(rows, a.heads, a.kv_heads, w.Dk, w.Dv, a.window, self.max_pages, split,
+                                                                   self.device))
+        return self._mixed_ws[key]
 
     def _lightning(self, h, li: int, m: LightningSpec, w: GatedWeights, rows: Rows) -> Pending:
         R = h.shape[0]

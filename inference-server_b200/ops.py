@@ -744,30 +744,66 @@ def mix_heads(q, mix, kv_heads: int, dtype):
     return out
 
 
-def mixed_attn(q, k_pool, v_pool, block_table, positions, bias, window: int, out, out_scale: float, status=None):
-    """Windowed attention of mixed queries [M, H, G * Dk] over pages; writes columns [0, H * Dv) of out [M, ld]."""
+def mixed_split_tokens(rows: int, window: int, max_ctx: int, num_sms: int = 148) -> int:
+    """Tokens per split of the decode kernel (all heads of a row in one CTA, one CTA per SM for large pages): about four CTAs per
+    SM over the rows' windows, at least 128 tokens each."""
+    seen = min(window, max_ctx) + 15
+    split = -(-seen * rows // (4 * num_sms))
+    return int(min(-(-seen // 32) * 32, max(128, -(-split // 32) * 32)))
+
+
+def mixed_attn_workspace(rows, num_q_heads, num_kv_heads, key_dim, value_dim, window, max_pages, split_tokens, device):
+    n = _lib.load().b200_mixed_attn_workspace_bytes(rows, num_q_heads, num_kv_heads, key_dim, value_dim, window, max_pages, split_tokens)
+    return torch.zeros(n, dtype=torch.uint8, device=device)
+
+
+def _mixed_shapes(q, k_pool, v_pool, bias, out):
     _need(q, "q")
     _need(k_pool, "k_pool", q.dtype)
     _need(v_pool, "v_pool", q.dtype)
-    _need(block_table, "block_table", torch.int32)
-    _need(positions, "positions", torch.int32)
     _need(bias, "bias", torch.float32)
     M, H, K = q.shape
     nb, G, page, Dk = k_pool.shape
-    Dv = v_pool.shape[3]
-    if K != G * Dk or v_pool.shape[:3] != k_pool.shape[:3] or block_table.shape[0] != M or out.shape[0] != M or bias.shape[0] != H:
-        raise ValueError("pools, block table, bias or output do not match q")
-    if out.dtype != q.dtype or out.stride(1) != 1:
+    if K != G * Dk or v_pool.shape[:3] != k_pool.shape[:3] or bias.shape[0] != H:
+        raise ValueError("pools or bias do not match q")
+    if out.dtype != q.dtype or out.stride(1) != 1 or out.shape[0] != M:
         raise ValueError("out must be rows of q's dtype")
+    return M, H, G, Dk, v_pool.shape[3], page, nb
+
+
+def mixed_attn(q, k_pool, v_pool, block_table, positions, bias, window: int, out, out_scale: float, status=None,
+               split_tokens: int | None = None, workspace=None):
+    """Windowed attention of mixed queries [M, H, G * Dk] over pages; writes columns [0, H * Dv) of out [M, ld].  `split_tokens`
+    0: the generic kernel."""
+    M, H, G, Dk, Dv, page, nb = _mixed_shapes(q, k_pool, v_pool, bias, out)
+    _need(block_table, "block_table", torch.int32)
+    _need(positions, "positions", torch.int32)
+    if block_table.shape[0] != M or positions.shape[0] != M:
+        raise ValueError("block table or positions do not match q")
     mp = block_table.shape[1]
+    if split_tokens is None:
+        split_tokens = mixed_split_tokens(M, window, mp * page)
+    if workspace is None and split_tokens:
+        workspace = mixed_attn_workspace(M, H, G, Dk, Dv, window, mp, split_tokens, q.device)
     rc = _lib.load().b200_mixed_attn(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), mp, _ptr(positions), _ptr(bias),
-                                     bias.shape[1], int(window), out.data_ptr(), out.stride(0), float(out_scale), _ptr(status), M,
-                                     H, G, Dk, Dv, page, nb, mp, DTYPE_CODE[q.dtype], _stream())
+                                     bias.shape[1], int(window), out.data_ptr(), out.stride(0), float(out_scale), _ptr(workspace),
+                                     0 if workspace is None else workspace.numel(), _ptr(status), M, H, G, Dk, Dv, page, nb, mp,
+                                     int(split_tokens), DTYPE_CODE[q.dtype], _stream())
     check(rc, "b200_mixed_attn")
 
 
 def mixed_attn_prefill_supported(num_q_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, dtype) -> bool:
-    return False
+    return dtype == torch.bfloat16 and bool(_lib.load().b200_mixed_attn_prefill_supported(num_q_heads, num_kv_heads, key_dim, value_dim))
+
+
+def mixed_attn_prefill(q, k_pool, v_pool, table_row, first_pos: int, bias, window: int, out, out_scale: float, status=None):
+    """`mixed_attn` for consecutive tokens of one sequence, positions first_pos.., on the tensor cores."""
+    M, H, G, Dk, Dv, page, nb = _mixed_shapes(q, k_pool, v_pool, bias, out)
+    _need(table_row, "table_row", torch.int32)
+    rc = _lib.load().b200_mixed_attn_prefill(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(table_row), _ptr(bias), bias.shape[1], int(window),
+                                             out.data_ptr(), out.stride(0), float(out_scale), _ptr(status), M, int(first_pos), H, G, Dk,
+                                             Dv, page, nb, table_row.numel(), _stream())
+    check(rc, "b200_mixed_attn_prefill")
 
 
 def conv_silu(x, conv_w, ring, slots, positions, chunk: bool, status=None, out=None):
