@@ -445,7 +445,8 @@ int b200_mix_heads(const float* q, const float* mix, void* out, int num_rows, in
  * head; times out_scale.
  *   q [num_rows, num_q_heads, num_kv_heads * key_dim] (b200_mix_heads); k_pool [num_blocks, num_kv_heads, page_size, key_dim];
  *   v_pool [num_blocks, num_kv_heads, page_size, value_dim]; block_table rows table_stride apart (0: one row for all);
- *   positions [num_rows]; bias [num_q_heads, bias_ld] fp32, bias_ld at least min(window, positions of the table);
+ *   positions [num_rows]; bias [num_q_heads, bias_ld] fp32 in log2 units: distance d at entry 256 + d, +inf in the 256 entries
+ *   before distance 0 and in at least 264 after the last of min(window, positions of the table); bias_ld a multiple of 4;
  *   out [num_rows, out_ld], head h at column h * value_dim.
  * bf16 pools with pages of 16 and sizes in multiples of 64 run on the tensor cores, a row's window in splits of split_tokens (a
  * multiple of 32) whose partials go through the workspace; split_tokens 0 and every other shape take the generic kernel.

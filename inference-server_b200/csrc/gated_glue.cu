@@ -7,6 +7,18 @@
 
 namespace b200 {
 
+template <typename T>
+__device__ __forceinline__ void store4(T* dst, const float4& v) {
+  if constexpr (sizeof(T) == 2) {
+    uint2 two;
+    two.x = pack_bf16x2(v.x, v.y);
+    two.y = pack_bf16x2(v.z, v.w);
+    *reinterpret_cast<uint2*>(dst) = two;
+  } else {
+    *reinterpret_cast<float4*>(dst) = v;
+  }
+}
+
 // What a sublayer left for the residual stream: rows of its own, or the experts' rows that the token's pairs point to.
 template <typename T>
 struct Pending {
@@ -115,35 +127,73 @@ residual_norm_kernel(float* __restrict__ x, const Pending<T> p, const float* __r
 }
 
 // out[m, h, c * D + d] = sum over the query heads g of kv head c of mix[h, g] * q[m, g, d]: with it, scores mixed over the
-// heads are plain products with the keys of all kv heads side by side.  One CTA per (row, kv head); a thread makes four
-// columns of four heads.
+// heads are plain products with the keys of all kv heads side by side.  One CTA per (`rows_per` rows, kv head); a thread makes
+// four columns of four heads.
 template <typename T>
 __global__ void __launch_bounds__(256)
-mix_heads_kernel(const float* __restrict__ q, const float* __restrict__ mix, T* __restrict__ out, int heads, int kv_heads,
-                 int D) {
+mix_heads_kernel(const float* __restrict__ q, const float* __restrict__ mix, T* __restrict__ out, int num_rows, int rows_per,
+                 int heads, int kv_heads, int D) {
   grid_dep_wait();
   grid_dep_launch();
   extern __shared__ float mh_sm[];
-  const int m = blockIdx.x, c = blockIdx.y, per = heads / kv_heads;
-  float* qs = mh_sm;                  // [per, D]
-  float* ms = mh_sm + per * D;        // [per, heads rounded up to 4]
-  const int hp = (heads + 3) & ~3;
-  const float* src = q + (static_cast<size_t>(m) * heads + c * per) * D;
-  for (int i = threadIdx.x * 4; i < per * D; i += blockDim.x * 4)
-    *reinterpret_cast<float4*>(qs + i) = *reinterpret_cast<const float4*>(src + i);
+  const int c = blockIdx.y, per = heads / kv_heads;
+  const int m0 = blockIdx.x * rows_per, rows = min(rows_per, num_rows - m0);
+  const int hp = (heads + 3) & ~3, row_q = per * D;
+  float* ms = mh_sm;             // [per, heads rounded up to 4]
+  float* qs = mh_sm + per * hp;  // [rows, per, D]
   for (int i = threadIdx.x; i < per * hp; i += blockDim.x) {
     const int g = i / hp, h = i - g * hp;
     ms[i] = h < heads ? mix[static_cast<size_t>(h) * heads + c * per + g] : 0.f;
   }
+  for (int i = threadIdx.x * 4; i < rows * row_q; i += blockDim.x * 4) {
+    const int r = i / row_q, x = i - r * row_q;
+    *reinterpret_cast<float4*>(qs + i) = *reinterpret_cast<const float4*>(q + (static_cast<size_t>(m0 + r) * heads + c * per) * D + x);
+  }
   __syncthreads();
-  const int d4 = D / 4, items = (hp / 4) * d4;
+  const int d4 = D / 4, per_row = (hp / 4) * d4, items = rows * per_row;
+  if (per <= 8) {  // a thread's mixing factors stay in registers over the rows
+    for (int rest = threadIdx.x; rest < per_row; rest += blockDim.x) {
+      const int h0 = rest / d4 * 4, d = (rest % d4) * 4;
+      float4 a[8];
+#pragma unroll
+      for (int g = 0; g < 8; ++g)
+        a[g] = g < per ? *reinterpret_cast<const float4*>(ms + g * hp + h0) : make_float4(0.f, 0.f, 0.f, 0.f);
+      T* dst = out + ((static_cast<size_t>(m0) * heads + h0) * kv_heads + c) * D + d;
+#pragma unroll 2
+      for (int r = 0; r < rows; ++r) {
+        float4 acc[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) acc[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int g = 0; g < 8; ++g) {
+          if (g >= per) break;
+          const float4 v = *reinterpret_cast<const float4*>(qs + r * row_q + g * D + d);
+          const float aa[4] = {a[g].x, a[g].y, a[g].z, a[g].w};
+#pragma unroll
+          for (int u = 0; u < 4; ++u) {
+            acc[u].x = fmaf(aa[u], v.x, acc[u].x);
+            acc[u].y = fmaf(aa[u], v.y, acc[u].y);
+            acc[u].z = fmaf(aa[u], v.z, acc[u].z);
+            acc[u].w = fmaf(aa[u], v.w, acc[u].w);
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+          if (h0 + u < heads) store4(dst + (static_cast<size_t>(r) * heads + u) * kv_heads * D, acc[u]);
+      }
+    }
+    return;
+  }
   for (int it = threadIdx.x; it < items; it += blockDim.x) {
-    const int h0 = it / d4 * 4, d = (it % d4) * 4;
+    const int r = it / per_row, rest = it - r * per_row;
+    const int h0 = rest / d4 * 4, d = (rest % d4) * 4;
+    const float* qr = qs + r * row_q + d;
     float4 acc[4];
 #pragma unroll
     for (int u = 0; u < 4; ++u) acc[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
     for (int g = 0; g < per; ++g) {
-      const float4 v = *reinterpret_cast<const float4*>(qs + g * D + d);
+      const float4 v = *reinterpret_cast<const float4*>(qr + g * D);
       const float4 a = *reinterpret_cast<const float4*>(ms + g * hp + h0);
       const float aa[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
@@ -157,15 +207,7 @@ mix_heads_kernel(const float* __restrict__ q, const float* __restrict__ mix, T* 
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       if (h0 + u >= heads) break;
-      T* dst = out + ((static_cast<size_t>(m) * heads + h0 + u) * kv_heads + c) * D + d;
-      if constexpr (sizeof(T) == 2) {
-        uint2 two;
-        two.x = pack_bf16x2(acc[u].x, acc[u].y);
-        two.y = pack_bf16x2(acc[u].z, acc[u].w);
-        *reinterpret_cast<uint2*>(dst) = two;
-      } else {
-        *reinterpret_cast<float4*>(dst) = acc[u];
-      }
+      store4(out + ((static_cast<size_t>(m0 + r) * heads + h0 + u) * kv_heads + c) * D + d, acc[u]);
     }
   }
 }
@@ -253,14 +295,7 @@ group_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w,
     const float4 v = *reinterpret_cast<const float4*>(src + c), a = *reinterpret_cast<const float4*>(wg + c);
     const float g0 = to_f32<T>(gt[c]), g1 = to_f32<T>(gt[c + 1]), g2 = to_f32<T>(gt[c + 2]), g3 = to_f32<T>(gt[c + 3]);
     const float r[4] = {v.x * inv * a.x * g0, v.y * inv * a.y * g1, v.z * inv * a.z * g2, v.w * inv * a.w * g3};
-    if constexpr (sizeof(T) == 2) {
-      uint2 two;
-      two.x = pack_bf16x2(r[0], r[1]);
-      two.y = pack_bf16x2(r[2], r[3]);
-      *reinterpret_cast<uint2*>(dst + c) = two;
-    } else {
-      *reinterpret_cast<float4*>(dst + c) = make_float4(r[0], r[1], r[2], r[3]);
-    }
+    store4(dst + c, make_float4(r[0], r[1], r[2], r[3]));
   }
 }
 
@@ -316,21 +351,24 @@ extern "C" int b200_mix_heads(const float* q, const float* mix, void* out, int n
                "mix_heads: %d heads over %d kv heads of %d", heads, kv_heads, head_dim);
   B200_REQUIRE(aligned16({q, out}), "mix_heads: buffers must be 16-byte aligned");
   const int per = heads / kv_heads;
-  const size_t smem = (static_cast<size_t>(per) * head_dim + static_cast<size_t>(per) * ((heads + 3) & ~3)) * 4;
+  const size_t mix_bytes = static_cast<size_t>(per) * ((heads + 3) & ~3) * 4, row_bytes = static_cast<size_t>(per) * head_dim * 4;
+  int rows_per = num_rows * kv_heads >= 4096 ? 8 : 1;  // many rows: the mixing matrix is fetched once for several
+  while (rows_per > 1 && mix_bytes + rows_per * row_bytes > 64 * 1024) rows_per >>= 1;
+  const size_t smem = mix_bytes + rows_per * row_bytes;
   B200_REQUIRE(smem <= 200 * 1024, "mix_heads: %d heads of %d per kv head do not fit", per, head_dim);
   B200_GLUE_DTYPE("mix_heads");
   if (num_rows == 0) return 0;
-  const dim3 grid(num_rows, kv_heads);
+  const dim3 grid((num_rows + rows_per - 1) / rows_per, kv_heads);
   if (dtype == 0) {
     int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mix_heads_kernel<__nv_bfloat16>), 200 * 1024);
     if (rc) return rc;
     B200_CUDA(launch_overlapped(mix_heads_kernel<__nv_bfloat16>, grid, dim3(256), smem, as_stream(stream), q, mix,
-                                static_cast<__nv_bfloat16*>(out), heads, kv_heads, head_dim));
+                                static_cast<__nv_bfloat16*>(out), num_rows, rows_per, heads, kv_heads, head_dim));
   } else {
     int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mix_heads_kernel<float>), 200 * 1024);
     if (rc) return rc;
     B200_CUDA(launch_overlapped(mix_heads_kernel<float>, grid, dim3(256), smem, as_stream(stream), q, mix,
-                                static_cast<float*>(out), heads, kv_heads, head_dim));
+                                static_cast<float*>(out), num_rows, rows_per, heads, kv_heads, head_dim));
   }
   return 0;
 }

@@ -5,17 +5,18 @@
 //
 // Mixing is linear, so it is taken out of the score loop: score_h = Q'_h . K_j - B[h][i - j], where K_j are the keys of all kv
 // heads side by side, Q'_h[c] = sum over the heads g of kv head c of T[h, g] scale q_g (mix_heads_kernel), and
-// B[h][d] = sum_g T[h, g] r1_g ln(1 + r2_g d) is a table over the window's distances.  Every query head then meets the whole
+// B[h][d] = sum_g T[h, g] r1_g ln(1 + r2_g d) is a table over the window's distances, kept in log2 units and padded with +inf on
+// both sides (kDistPad, kDistTail): outside the window, and for later tokens, it masks.  Every query head then meets the whole
 // of a token's keys, and the values of its own kv head.
 //
 // Decode kernel: bf16, key and value sizes multiples of 64.  grid (rows, splits); a CTA owns up to `split_tokens` consecutive
 // tokens of one row, for all heads, and streams their pages (a producer warp, one TMA box of 16 tokens x 128 B per kv head and
-// 64 columns, mbarrier ring of pages).  Eight consumer warps take two pages (32 tokens) at a time:
+// 64 columns, mbarrier ring of pages).  Groups of eight consumer warps take two pages (32 tokens) at a time:
 //   scores   an item is (page, half of its tokens, 16 query heads): mma.sync m16n8k16 over the keys of all kv heads, queries
 //            from shared memory; times log2 e, less the distance table, masked, into a score tile in shared memory
 //   values   a unit is (kv head, 16 of its query heads, 64 value columns): online softmax over the tile's 32 tokens in the A
 //            operand's registers, O += P V
-// with one 256-thread barrier per two pages (the score tile is double-buffered).  Rows of one split are written as they are,
+// with one barrier of the group per two pages (the score tile is double-buffered).  Rows of one split are written as they are,
 // others as fp32 partials that a second kernel folds in split order.
 //
 // Generic kernel: any sizes, bf16 or fp32, fp32 arithmetic, one CTA per (row, query head).
@@ -25,6 +26,7 @@
 namespace b200 {
 
 constexpr int kMixWarps = 4;
+constexpr float kMixLog2e = 1.4426950408889634f;
 
 struct MixedAttnParams {
   const void* q;            // [rows, heads, kv_heads * dk]
@@ -33,7 +35,7 @@ struct MixedAttnParams {
   const int* table;         // [rows, max_pages], or one row for all (table_stride 0)
   int table_stride;
   const int* positions;     // [rows]: position of the row's token
-  const float* bias;        // [heads, bias_ld]
+  const float* bias;        // [heads, bias_ld], distance d at kDistPad + d
   int bias_ld, window;
   void* out;                // [rows, out_ld], head h at column h * dv
   int out_ld;
@@ -78,9 +80,9 @@ mixed_attn_generic_kernel(const MixedAttnParams p) {
       const T* kr = kp + ((static_cast<size_t>(id) * p.kv_heads + c) * p.page + slot) * p.dk;
       for (int d = lane; d < p.dk; d += 32) dot = fmaf(mg_sm[c * p.dk + d], to_f32<T>(kr[d]), dot);
     }
-    dot = warp_sum(dot) - bias[min(pos - tok, p.bias_ld - 1)];
+    dot = fmaf(warp_sum(dot), kMixLog2e, -bias[kDistPad + pos - tok]);
     const float mn = fmaxf(m, dot);
-    const float a = expf(m - mn), w = expf(dot - mn);
+    const float a = exp2f(m - mn), w = exp2f(dot - mn);
     m = mn;
     l = l * a + w;
     const T* vr = vp + ((static_cast<size_t>(id) * p.kv_heads + kvh) * p.page + slot) * p.dv;
@@ -106,7 +108,7 @@ mixed_attn_generic_kernel(const MixedAttnParams p) {
   for (int d = threadIdx.x; d < p.dv; d += blockDim.x) {
     float num = 0.f, den = 0.f;
     for (int w = 0; w < kMixWarps; ++w) {
-      const float wgt = m_sm[w] == -INFINITY ? 0.f : expf(m_sm[w] - mmax);
+      const float wgt = m_sm[w] == -INFINITY ? 0.f : exp2f(m_sm[w] - mmax);
       num += wgt * o_sm[w * p.dv + d];
       den += wgt * l_sm[w];
     }
@@ -116,10 +118,9 @@ mixed_attn_generic_kernel(const MixedAttnParams p) {
 }
 
 constexpr int kMdPage = 16;
-constexpr int kMdWarps = 8;                    // consumers
-constexpr int kMdThreads = (kMdWarps + 1) * 32;
+constexpr int kMdWarps = 8;                    // consumers of a group
 constexpr int kMdScoreLd = 40;                 // floats per head of a score tile (32 tokens): float2 reads of 8 heads hit all banks
-constexpr float kMdLog2e = 1.4426950408889634f;
+constexpr int kMdMergeFloats = 8 * 32 * 36;    // what the second group hands to the first
 
 struct MixedDecodeParams {
   MixedAttnParams a;
@@ -128,9 +129,10 @@ struct MixedDecodeParams {
   int split_tokens, max_splits, stages;
 };
 
-// UNITS: units (see above) a warp may own.
-template <int UNITS>
-__global__ void __launch_bounds__(kMdThreads, 1)
+// UNITS: units (see above) a warp may own.  GROUPS: groups of eight consumer warps; two of them take the tiles in turn, each with
+// a softmax of its own, and are merged at the end.
+template <int UNITS, int GROUPS>
+__global__ void __launch_bounds__((GROUPS * kMdWarps + 1) * 32, 1)
 mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map, const MixedDecodeParams pp) {
 #ifdef B200_DEVICE_OK
   const MixedAttnParams& p = pp.a;
@@ -156,30 +158,34 @@ mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
   uint8_t* ring_ptr = smem_raw + (ring - smem_u32(smem_raw));
   const int kc = p.kv_heads * (p.dk / 64), vc = p.kv_heads * (p.dv / 64);  // 2 KiB boxes of a page
   const uint32_t stage_bytes = static_cast<uint32_t>(kc + vc) * 2048u;
-  uint8_t* after = ring_ptr + static_cast<size_t>(pp.stages) * stage_bytes;
-  const uint32_t bars = ring + pp.stages * stage_bytes;  // full[stages], empty[stages]: up to 16 of each
-  float* sc = reinterpret_cast<float*>(after + 256);     // [2][heads16][kMdScoreLd]
+  const int stages = pp.stages;
+  uint8_t* after = ring_ptr + static_cast<size_t>(stages) * stage_bytes;
+  const uint32_t bar_full = ring + stages * stage_bytes, bar_empty = bar_full + 8 * stages;  // up to 16 of each
   const int mt = (p.heads + 15) / 16, K = p.kv_heads * p.dk, q_ld = K + 8;
-  __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(sc + 2 * mt * 16 * kMdScoreLd);  // [mt * 16][q_ld]
+  const int score_floats = mt * 16 * kMdScoreLd;
+  float* sc = reinterpret_cast<float*>(after + 256);     // [GROUPS][2][mt * 16][kMdScoreLd]
+  __nv_bfloat16* q_sm = reinterpret_cast<__nv_bfloat16*>(sc + GROUPS * 2 * score_floats);  // [mt * 16][q_ld]
 
   if (threadIdx.x == 0) {
-    for (int s = 0; s < pp.stages; ++s) {
-      mbar_init(bars + 8 * s, 1);
-      mbar_init(bars + 8 * (pp.stages + s), kMdWarps);
+    for (int s = 0; s < stages; ++s) {
+      mbar_init(bar_full + 8 * s, 1);
+      mbar_init(bar_empty + 8 * s, kMdWarps);
     }
     fence_mbar_init();
     fence_proxy_async();
   }
   __syncthreads();
 
-  if (warp == kMdWarps) {
+  if (warp == GROUPS * kMdWarps) {
     // ------------------------------------------------------------ producer --
     if (lane == 0) {
       tma_prefetch_desc(&k_map);
       tma_prefetch_desc(&v_map);
     }
     const int* table = p.table + static_cast<size_t>(row) * p.table_stride + first_page;
-    int ids = 0;
+    const int kn = p.dk / 64, vn = p.dv / 64;
+    int ids = 0, slot = 0;
+    uint32_t phase = 1;
     for (int i = 0; i < npages; ++i) {
       if ((i & 31) == 0) {
         ids = i + lane < npages ? table[i + lane] : 0;
@@ -189,150 +195,156 @@ mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
         }
       }
       const int id = __shfl_sync(0xffffffffu, ids, i & 31);
-      const int slot = i % pp.stages;
-      if (!__all_sync(0xffffffffu, mbar_wait(bars + 8 * (pp.stages + slot), ((i / pp.stages) & 1) ^ 1, p.err))) break;
-      if (lane == 0) mbar_arrive_expect_tx(bars + 8 * slot, stage_bytes);
+      if (!__all_sync(0xffffffffu, mbar_wait(bar_empty + 8 * slot, phase, p.err))) break;
+      if (lane == 0) mbar_arrive_expect_tx(bar_full + 8 * slot, stage_bytes);
       __syncwarp();
       for (int b = lane; b < kc + vc; b += 32) {
         const bool is_v = b >= kc;
-        const int bb = is_v ? b - kc : b, n = is_v ? p.dv / 64 : p.dk / 64;
+        const int bb = is_v ? b - kc : b, n = is_v ? vn : kn;
         const int head = bb / n;
-        tma_load_2d(ring + slot * stage_bytes + b * 2048u, is_v ? &v_map : &k_map, bars + 8 * slot, (bb - head * n) * 64,
+        tma_load_2d(ring + slot * stage_bytes + b * 2048u, is_v ? &v_map : &k_map, bar_full + 8 * slot, (bb - head * n) * 64,
                     (id * p.kv_heads + head) * kMdPage);
       }
+      if (++slot == stages) {
+        slot = 0;
+        phase ^= 1;
+      }
     }
+    if (GROUPS > 1) asm volatile("bar.sync 3, %0;" ::"n"((GROUPS * kMdWarps + 1) * 32) : "memory");
     return;
   }
 
   // ------------------------------------------------------------- consumers --
+  const int group = GROUPS > 1 ? warp / kMdWarps : 0, w = warp - group * kMdWarps;
   {  // the row's mixed queries, zero rows after the last head
     const uint4* src = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) + static_cast<size_t>(row) * p.heads * K);
     const int per_row = K / 8;
-    for (int i = threadIdx.x; i < mt * 16 * per_row; i += kMdWarps * 32) {
+    for (int i = threadIdx.x; i < mt * 16 * per_row; i += GROUPS * kMdWarps * 32) {
       const int h = i / per_row, c = i - h * per_row;
       *reinterpret_cast<uint4*>(q_sm + static_cast<size_t>(h) * q_ld + c * 8) = h < p.heads ? src[i] : make_uint4(0u, 0u, 0u, 0u);
     }
   }
   const int per = p.heads / p.kv_heads, sub = (per + 15) / 16, dvc = p.dv / 64;
   const int units = p.kv_heads * sub * dvc;
+  const int gq = lane >> 2, tq = lane & 3;
+  const int lj = lane >> 3, lr = lane & 7;
   float o[UNITS][8][4], m_run[UNITS][2], l_run[UNITS][2];
+  int s_off[UNITS][2], v_off[UNITS];  // score rows and value boxes of this warp's units; v_off < 0: no such unit
 #pragma unroll
   for (int u = 0; u < UNITS; ++u) {
 #pragma unroll
     for (int n = 0; n < 8; ++n) o[u][n][0] = o[u][n][1] = o[u][n][2] = o[u][n][3] = 0.f;
     m_run[u][0] = m_run[u][1] = -INFINITY;
     l_run[u][0] = l_run[u][1] = 0.f;
+    const int unit = w + u * kMdWarps, hs = unit / dvc, c = hs / sub, h0 = (hs - c * sub) * 16 + gq;
+    const bool is = unit < units;
+    s_off[u][0] = is ? (c * per + min(h0, per - 1)) * kMdScoreLd + 2 * tq : 0;  // a row past the last head repeats it and is not kept
+    s_off[u][1] = is ? (c * per + min(h0 + 8, per - 1)) * kMdScoreLd + 2 * tq : 0;
+    v_off[u] = is ? (kc + c * dvc + (unit - hs * dvc)) * 2048 : -1;
   }
-  const int gq = lane >> 2, tq = lane & 3;
-  const int lj = lane >> 3, lr = lane & 7;
-  const uint32_t q_base = smem_u32(q_sm);
-  asm volatile("bar.sync 1, 256;" ::: "memory");  // queries in place
+  const uint32_t v_sw = swz128((lj & 1) * 8 + lr, lj >> 1);  // value columns 16 further: ^ 32, ^ 64, ^ 96
+  // All 16 warps: queries in place.
+  if (GROUPS > 1) asm volatile("bar.sync 4, %0;" ::"n"(GROUPS * kMdWarps * 32) : "memory");
+  else asm volatile("bar.sync 4, %0;" ::"n"(kMdWarps * 32) : "memory");
+  const uint32_t a_base = smem_u32(q_sm) + (((lj & 1) * 8 + lr) * q_ld + (lj >> 1) * 8) * 2;
 
   bool alive = true;
   const int tiles = (npages + 1) / 2;
+  // this group's first page in the ring, and its parity
+  int slot = group * 2;
+  uint32_t phase = 0;
+  while (slot >= stages) {
+    slot -= stages;
+    phase ^= 1;
+  }
 #pragma unroll 1
-  for (int tile = 0; tile < tiles; ++tile) {
+  for (int tile = group, turn = 0; tile < tiles; tile += GROUPS, ++turn) {
     const int pages_here = min(2, npages - tile * 2);
-    float* score = sc + (tile & 1) * mt * 16 * kMdScoreLd;
-    for (int pg = 0; pg < pages_here && alive; ++pg) {
-      const int i = tile * 2 + pg;
-      alive = mbar_wait(bars + 8 * (i % pp.stages), (i / pp.stages) & 1, p.err);
+    int slot1 = slot + 1;
+    uint32_t phase1 = phase;
+    if (slot1 == stages) {
+      slot1 = 0;
+      phase1 ^= 1;
     }
-    // ---- scores
-    for (int item = warp; item < pages_here * 2 * mt; item += kMdWarps) {
-      const int pg = item % pages_here, rest = item / pages_here, th = rest & 1, mi = rest >> 1;
-      const int i = tile * 2 + pg;
-      const uint32_t kbase = ring + (i % pp.stages) * stage_bytes;
-      const int tok0 = start + i * kMdPage + th * 8 + 2 * tq;  // token of c0, c2; c1, c3 are the next one
+    float* score = sc + (group * 2 + (turn & 1)) * score_floats;
+    const int tok_tile = start + tile * 2 * kMdPage;
+    if (alive) alive = mbar_wait(bar_full + 8 * slot, phase, p.err);
+    if (pages_here > 1 && alive) alive = mbar_wait(bar_full + 8 * slot1, phase1, p.err);
+    // ---- scores: items count up by (page, token half), then by 16 heads
+    const int items = mt * 4;
+#pragma unroll 1
+    for (int item = w; item < items; item += kMdWarps) {
+      const int pg = item & 1, th = (item >> 1) & 1, mi = item >> 2;
+      if (pg >= pages_here) continue;
       // the distance table's entries travel while the products run
-      float bias[2][2];
-#pragma unroll
-      for (int hh = 0; hh < 2; ++hh)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int h = mi * 16 + gq + hh * 8, d = pos - tok0 - e;
-          bias[hh][e] = h < p.heads && d >= 0 && d < p.window ? __ldg(p.bias + static_cast<size_t>(h) * p.bias_ld + d) * kMdLog2e : INFINITY;
-        }
-      float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-      const uint32_t a_addr = q_base + ((mi * 16 + (lj & 1) * 8 + lr) * q_ld + (lj >> 1) * 8) * 2;
+      const float* bt = p.bias + static_cast<size_t>(mi * 16 + gq) * p.bias_ld + (kDistPad + pos - tok_tile - pg * 16 - th * 8 - 2 * tq);
+      const bool h_lo = mi * 16 + gq < p.heads, h_hi = mi * 16 + gq + 8 < p.heads;
+      const size_t b_hi = static_cast<size_t>(8) * p.bias_ld;
+      const float b00 = h_lo ? __ldg(bt) : 0.f, b01 = h_lo ? __ldg(bt - 1) : 0.f;
+      const float b10 = h_hi ? __ldg(bt + b_hi) : 0.f, b11 = h_hi ? __ldg(bt + b_hi - 1) : 0.f;
+      float acc0[4] = {0.f, 0.f, 0.f, 0.f}, acc1[4] = {0.f, 0.f, 0.f, 0.f};
+      uint32_t a_addr = a_base + mi * 16 * q_ld * 2;
+      uint32_t k_lo = ring + (pg ? slot1 : slot) * stage_bytes + swz128(th * 8 + lr, lj);
+#pragma unroll 4
       for (int c = 0; c < kc; ++c) {  // 64 of the key columns
-        const uint32_t box = kbase + c * 2048u;
-#pragma unroll
-        for (int k2 = 0; k2 < 2; ++k2) {
-          uint32_t b0, b1, b2, b3;
-          ldmatrix_x4(box + swz128(th * 8 + lr, k2 * 4 + lj), b0, b1, b2, b3);
-          uint32_t a0[4], a1[4];
-          ldmatrix_x4(a_addr + (c * 64 + k2 * 32) * 2, a0[0], a0[1], a0[2], a0[3]);
-          ldmatrix_x4(a_addr + (c * 64 + k2 * 32 + 16) * 2, a1[0], a1[1], a1[2], a1[3]);
-          mma_bf16_16816(acc[0], a0, b0, b1);
-          mma_bf16_16816(acc[1], a1, b2, b3);
-        }
+        uint32_t b0, b1, b2, b3, b4, b5, b6, b7, a0[4], a1[4], a2[4], a3[4];
+        ldmatrix_x4(k_lo, b0, b1, b2, b3);
+        ldmatrix_x4(k_lo ^ 64u, b4, b5, b6, b7);
+        ldmatrix_x4(a_addr, a0[0], a0[1], a0[2], a0[3]);
+        ldmatrix_x4(a_addr + 32, a1[0], a1[1], a1[2], a1[3]);
+        ldmatrix_x4(a_addr + 64, a2[0], a2[1], a2[2], a2[3]);
+        ldmatrix_x4(a_addr + 96, a3[0], a3[1], a3[2], a3[3]);
+        mma_bf16_16816(acc0, a0, b0, b1);
+        mma_bf16_16816(acc1, a1, b2, b3);
+        mma_bf16_16816(acc0, a2, b4, b5);
+        mma_bf16_16816(acc1, a3, b6, b7);
+        k_lo += 2048u;
+        a_addr += 128u;
       }
-#pragma unroll
-      for (int hh = 0; hh < 2; ++hh) {
-        const float2 v = make_float2(fmaf(acc[0][2 * hh] + acc[1][2 * hh], kMdLog2e, -bias[hh][0]),
-                                     fmaf(acc[0][2 * hh + 1] + acc[1][2 * hh + 1], kMdLog2e, -bias[hh][1]));
-        *reinterpret_cast<float2*>(score + (mi * 16 + gq + hh * 8) * kMdScoreLd + pg * 16 + th * 8 + 2 * tq) = v;
-      }
+      float* dst = score + (mi * 16 + gq) * kMdScoreLd + pg * 16 + th * 8 + 2 * tq;
+      *reinterpret_cast<float2*>(dst) = make_float2(fmaf(acc0[0] + acc1[0], kMixLog2e, -b00), fmaf(acc0[1] + acc1[1], kMixLog2e, -b01));
+      *reinterpret_cast<float2*>(dst + 8 * kMdScoreLd) =
+          make_float2(fmaf(acc0[2] + acc1[2], kMixLog2e, -b10), fmaf(acc0[3] + acc1[3], kMixLog2e, -b11));
     }
-    asm volatile("bar.sync 1, 256;" ::: "memory");  // the score tile is complete; the other one has been read by everybody
+    // the group's score tile is complete, and its other one has been read by all its warps
+    asm volatile("bar.sync %0, %1;" ::"r"(1 + group), "n"(kMdWarps * 32) : "memory");
     // ---- values
 #pragma unroll
     for (int u = 0; u < UNITS; ++u) {
-      const int unit = warp + u * kMdWarps;
-      if (unit >= units) break;
-      const int vcol = unit % dvc, hs = unit / dvc, c = hs / sub, ms = hs - c * sub;
-      const int h0 = ms * 16 + gq;  // head inside the kv group of fragment rows 0-7; +8 for the others
-      const float* s0 = score + (c * per + min(h0, per - 1)) * kMdScoreLd;
-      const float* s1 = score + (c * per + min(h0 + 8, per - 1)) * kMdScoreLd;
+      if (v_off[u] < 0) break;
+      const float* s0 = score + s_off[u][0];
+      const float* s1 = score + s_off[u][1];
       float s[2][2][4];  // [page][row half][k 2tq, 2tq+1, 2tq+8, 2tq+9]
-      float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
       for (int pg = 0; pg < 2; ++pg) {
-        if (pg < pages_here) {
-          const float2 a = *reinterpret_cast<const float2*>(s0 + pg * 16 + 2 * tq), b = *reinterpret_cast<const float2*>(s0 + pg * 16 + 8 + 2 * tq);
-          const float2 x = *reinterpret_cast<const float2*>(s1 + pg * 16 + 2 * tq), y = *reinterpret_cast<const float2*>(s1 + pg * 16 + 8 + 2 * tq);
+        if (pg == 0 || pages_here > 1) {
+          const float2 a = *reinterpret_cast<const float2*>(s0 + pg * 16), b = *reinterpret_cast<const float2*>(s0 + pg * 16 + 8);
+          const float2 x = *reinterpret_cast<const float2*>(s1 + pg * 16), y = *reinterpret_cast<const float2*>(s1 + pg * 16 + 8);
           s[pg][0][0] = a.x; s[pg][0][1] = a.y; s[pg][0][2] = b.x; s[pg][0][3] = b.y;
           s[pg][1][0] = x.x; s[pg][1][1] = x.y; s[pg][1][2] = y.x; s[pg][1][3] = y.y;
         } else {
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[pg][0][e] = s[pg][1][e] = -INFINITY;
         }
+      }
+      float mx0 = s[0][0][0], mx1 = s[0][1][0];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          mx0 = fmaxf(mx0, s[pg][0][e]);
-          mx1 = fmaxf(mx1, s[pg][1][e]);
-        }
+      for (int e = 1; e < 8; ++e) {
+        mx0 = fmaxf(mx0, s[e >> 2][0][e & 3]);
+        mx1 = fmaxf(mx1, s[e >> 2][1][e & 3]);
       }
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
-      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
       const float n0 = fmaxf(m_run[u][0], mx0), n1 = fmaxf(m_run[u][1], mx1);
       const float r0 = n0 == -INFINITY ? 0.f : n0, r1 = n1 == -INFINITY ? 0.f : n1;  // nothing seen yet: all weights come out 0
-      const float al0 = exp2f(m_run[u][0] - r0), al1 = exp2f(m_run[u][1] - r1);
-      m_run[u][0] = n0;
-      m_run[u][1] = n1;
-      uint32_t pa[2][4];
-      float sum0 = 0.f, sum1 = 0.f;
-#pragma unroll
-      for (int pg = 0; pg < 2; ++pg) {
-        float e0[4], e1[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          e0[e] = exp2f(s[pg][0][e] - r0);
-          e1[e] = exp2f(s[pg][1][e] - r1);
-          sum0 += e0[e];
-          sum1 += e1[e];
-        }
-        pa[pg][0] = pack_bf16x2(e0[0], e0[1]);
-        pa[pg][1] = pack_bf16x2(e1[0], e1[1]);
-        pa[pg][2] = pack_bf16x2(e0[2], e0[3]);
-        pa[pg][3] = pack_bf16x2(e1[2], e1[3]);
-      }
-      l_run[u][0] = l_run[u][0] * al0 + sum0;
-      l_run[u][1] = l_run[u][1] * al1 + sum1;
-      if (__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) {
+      if (__any_sync(0xffffffffu, n0 != m_run[u][0] || n1 != m_run[u][1])) {
+        const float al0 = fast_ex2(m_run[u][0] - r0), al1 = fast_ex2(m_run[u][1] - r1);
+        m_run[u][0] = n0;
+        m_run[u][1] = n1;
+        l_run[u][0] *= al0;
+        l_run[u][1] *= al1;
 #pragma unroll
         for (int n = 0; n < 8; ++n) {
           o[u][n][0] *= al0;
@@ -341,39 +353,97 @@ mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
           o[u][n][3] *= al1;
         }
       }
+      uint32_t pa[2][4];
 #pragma unroll
       for (int pg = 0; pg < 2; ++pg) {
-        if (pg >= pages_here) break;
-        const uint32_t vbase = ring + ((tile * 2 + pg) % pp.stages) * stage_bytes + (kc + c * dvc + vcol) * 2048u;
+        float e0[4], e1[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          e0[e] = fast_ex2(s[pg][0][e] - r0);
+          e1[e] = fast_ex2(s[pg][1][e] - r1);
+        }
+        l_run[u][0] += (e0[0] + e0[1]) + (e0[2] + e0[3]);
+        l_run[u][1] += (e1[0] + e1[1]) + (e1[2] + e1[3]);
+        pa[pg][0] = pack_bf16x2(e0[0], e0[1]);
+        pa[pg][1] = pack_bf16x2(e1[0], e1[1]);
+        pa[pg][2] = pack_bf16x2(e0[2], e0[3]);
+        pa[pg][3] = pack_bf16x2(e1[2], e1[3]);
+      }
+#pragma unroll
+      for (int pg = 0; pg < 2; ++pg) {
+        if (pg > 0 && pages_here < 2) break;
+        const uint32_t vbase = ring + (pg ? slot1 : slot) * stage_bytes + v_off[u] + v_sw;
 #pragma unroll
         for (int np = 0; np < 4; ++np) {
           uint32_t v0, v1, v2, v3;
-          ldmatrix_x4_trans(vbase + swz128((lj & 1) * 8 + lr, np * 2 + (lj >> 1)), v0, v1, v2, v3);
+          ldmatrix_x4_trans(vbase ^ (np * 32u), v0, v1, v2, v3);
           mma_bf16_16816(o[u][2 * np], pa[pg], v0, v1);
           mma_bf16_16816(o[u][2 * np + 1], pa[pg], v2, v3);
         }
       }
     }
     __syncwarp();
-    if (lane == 0)
-      for (int pg = 0; pg < pages_here; ++pg) mbar_arrive(bars + 8 * (pp.stages + (tile * 2 + pg) % pp.stages));
+    if (lane == 0) {
+      mbar_arrive(bar_empty + 8 * slot);
+      if (pages_here > 1) mbar_arrive(bar_empty + 8 * slot1);
+    }
+    slot += 2 * GROUPS;
+    while (slot >= stages) {
+      slot -= stages;
+      phase ^= 1;
+    }
+  }
+
+#pragma unroll
+  for (int u = 0; u < UNITS; ++u)
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      l_run[u][hh] += __shfl_xor_sync(0xffffffffu, l_run[u][hh], 1);
+      l_run[u][hh] += __shfl_xor_sync(0xffffffffu, l_run[u][hh], 2);
+    }
+  if (GROUPS > 1) {  // every page has been read: the second group's results go through the ring
+    float* mg = reinterpret_cast<float*>(ring_ptr) + (w * 36) * 32 + lane;
+    // all copies have landed and been read (the producer has issued its last one before it comes here)
+    asm volatile("bar.sync 3, %0;" ::"n"((GROUPS * kMdWarps + 1) * 32) : "memory");
+    if (group == 1) {
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) mg[(n * 4 + e) * 32] = o[0][n][e];
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh) {
+        mg[(32 + hh) * 32] = m_run[0][hh];
+        mg[(34 + hh) * 32] = l_run[0][hh];
+      }
+    }
+    asm volatile("bar.sync 4, %0;" ::"n"(GROUPS * kMdWarps * 32) : "memory");
+    if (group == 1) return;
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      const float m1 = mg[(32 + hh) * 32], l1 = mg[(34 + hh) * 32], m0 = m_run[0][hh];
+      const float m = fmaxf(m0, m1), r = m == -INFINITY ? 0.f : m;
+      const float c0 = fast_ex2(m0 - r), c1 = fast_ex2(m1 - r);
+      m_run[0][hh] = m;
+      l_run[0][hh] = l_run[0][hh] * c0 + l1 * c1;
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int e = 2 * hh; e < 2 * hh + 2; ++e) o[0][n][e] = o[0][n][e] * c0 + mg[(n * 4 + e) * 32] * c1;
+    }
   }
 
 #pragma unroll
   for (int u = 0; u < UNITS; ++u) {
-    const int unit = warp + u * kMdWarps;
+    const int unit = w + u * kMdWarps;
     if (unit >= units) break;
     const int vcol = unit % dvc, hs = unit / dvc, c = hs / sub, ms = hs - c * sub;
 #pragma unroll
     for (int hh = 0; hh < 2; ++hh) {
-      float l = l_run[u][hh];
-      l += __shfl_xor_sync(0xffffffffu, l, 1);
-      l += __shfl_xor_sync(0xffffffffu, l, 2);
       const int hl = ms * 16 + gq + hh * 8;
       if (hl >= per) continue;
       const int h = c * per + hl;
       if (nsplits == 1) {
-        const float inv = p.out_scale / l;
+        const float inv = p.out_scale / l_run[u][hh];
         __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + static_cast<size_t>(row) * p.out_ld + static_cast<size_t>(h) * p.dv + vcol * 64;
 #pragma unroll
         for (int n = 0; n < 8; ++n)
@@ -383,7 +453,7 @@ mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
 #pragma unroll
         for (int n = 0; n < 8; ++n)
           *reinterpret_cast<float2*>(pp.part_o + at * p.dv + vcol * 64 + n * 8 + 2 * tq) = make_float2(o[u][n][2 * hh], o[u][n][2 * hh + 1]);
-        if (vcol == 0 && tq == 0) pp.part_ml[at] = make_float2(m_run[u][hh], l);
+        if (vcol == 0 && tq == 0) pp.part_ml[at] = make_float2(m_run[u][hh], l_run[u][hh]);
       }
     }
   }
@@ -436,29 +506,29 @@ static int mixed_max_splits(int window, int max_pages, int split_tokens) {
   return static_cast<int>((seen + split_tokens - 1) / split_tokens);
 }
 
-// Pages in flight and shared memory of the decode kernel; 0: not built for this shape.
-static int mixed_decode_stages(int heads, int kv_heads, int dk, int dv, size_t* smem_out) {
+// Pages in flight, groups of consumer warps and shared memory of the decode kernel; 0: not built for this shape.
+static int mixed_decode_stages(int heads, int kv_heads, int dk, int dv, size_t* smem_out, int* groups_out) {
   if (heads % kv_heads || dk % 64 || dv % 64) return 0;
   const int per = heads / kv_heads, units = kv_heads * ((per + 15) / 16) * (dv / 64);
   if (units > 4 * kMdWarps) return 0;
   const size_t mt = (heads + 15) / 16, K = static_cast<size_t>(kv_heads) * dk;
-  const size_t fixed = 1024 + 256 + 2 * mt * 16 * kMdScoreLd * 4 + mt * 16 * (K + 8) * 2;
   const size_t stage = static_cast<size_t>(kv_heads) * (dk + dv) / 64 * 2048, room = 227 * 1024;
-  if (fixed + 4 * stage > room) return 0;
-  size_t stages = (room - fixed) / stage;
-  // small pages: leave room for a second CTA on the multiprocessor once 64 KiB are in flight
-  const size_t enough = (64 * 1024 + stage - 1) / stage + 2;
-  if (stages > enough && fixed + enough * stage <= room / 2) stages = enough;
+  const auto fixed = [&](int groups) { return 1024 + 256 + groups * 2 * mt * 16 * kMdScoreLd * 4 + mt * 16 * (K + 8) * 2; };
+  // two groups where their accumulators fit the registers and five pages the shared memory
+  int groups = units <= kMdWarps && fixed(2) + 5 * stage <= room && 5 * stage >= kMdMergeFloats * 4 ? 2 : 1;
+  if (fixed(groups) + 3 * stage > room) return 0;
+  size_t stages = (room - fixed(groups)) / stage;
   if (stages > 16) stages = 16;
-  if (smem_out) *smem_out = fixed + stages * stage;
+  if (smem_out) *smem_out = fixed(groups) + stages * stage;
+  if (groups_out) *groups_out = groups;
   return static_cast<int>(stages);
 }
 
-template <int UNITS>
+template <int UNITS, int GROUPS>
 static int launch_mixed_decode(const CUtensorMap& km, const CUtensorMap& vm, const MixedDecodeParams& pp, size_t smem, cudaStream_t st) {
-  int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mixed_decode_kernel<UNITS>), 227 * 1024);
+  int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mixed_decode_kernel<UNITS, GROUPS>), 227 * 1024);
   if (rc) return rc;
-  B200_CUDA(launch_overlapped(mixed_decode_kernel<UNITS>, dim3(pp.a.rows, pp.max_splits), dim3(kMdThreads), smem, st, km, vm, pp));
+  B200_CUDA(launch_overlapped(mixed_decode_kernel<UNITS, GROUPS>, dim3(pp.a.rows, pp.max_splits), dim3((GROUPS * kMdWarps + 1) * 32), smem, st, km, vm, pp));
   if (pp.max_splits > 1)
     B200_CUDA(launch_overlapped(mixed_reduce_kernel, dim3((pp.a.rows * pp.a.heads + 3) / 4), dim3(128), 0, st, pp));
   return 0;
@@ -487,7 +557,7 @@ using namespace b200;
 extern "C" size_t b200_mixed_attn_workspace_bytes(int num_rows, int num_q_heads, int num_kv_heads, int key_dim, int value_dim,
                                                   int window, int max_pages_per_seq, int split_tokens) {
   if (num_rows <= 0 || num_q_heads <= 0 || num_kv_heads <= 0 || key_dim <= 0 || value_dim <= 0 || window <= 0 ||
-      max_pages_per_seq <= 0 || split_tokens <= 0 || mixed_decode_stages(num_q_heads, num_kv_heads, key_dim, value_dim, nullptr) == 0)
+      max_pages_per_seq <= 0 || split_tokens <= 0 || mixed_decode_stages(num_q_heads, num_kv_heads, key_dim, value_dim, nullptr, nullptr) == 0)
     return 256;
   return carve(nullptr, num_rows, num_q_heads, value_dim, mixed_max_splits(window, max_pages_per_seq, split_tokens)).bytes;
 }
@@ -504,7 +574,7 @@ extern "C" int b200_mixed_attn(const void* q, const void* k_pool, const void* v_
                "mixed_attn: %d rows, %d query heads over %d, key size %d, value size %d, window %d", num_rows, num_q_heads,
                num_kv_heads, key_dim, value_dim, window);
   const long long all = static_cast<long long>(max_pages_per_seq) * page_size;
-  B200_REQUIRE(bias_ld >= (window < all ? window : all) && out_ld >= num_q_heads * value_dim,
+  B200_REQUIRE(bias_ld >= kDistPad + (window < all ? window : all) + kDistTail && out_ld >= num_q_heads * value_dim,
                "mixed_attn: bias rows of %d for a window of %d, output rows of %d", bias_ld, window, out_ld);
   B200_GLUE_DTYPE("mixed_attn");
   if (num_rows == 0) return 0;
@@ -512,8 +582,9 @@ extern "C" int b200_mixed_attn(const void* q, const void* k_pool, const void* v_
                           out_scale, static_cast<int*>(status_word), num_rows, num_q_heads, num_kv_heads, key_dim, value_dim,
                           page_size, num_blocks, max_pages_per_seq};
   size_t smem = 0;
+  int groups = 1;
   const int stages = dtype == 0 && page_size == kMdPage && split_tokens > 0
-                         ? mixed_decode_stages(num_q_heads, num_kv_heads, key_dim, value_dim, &smem) : 0;
+                         ? mixed_decode_stages(num_q_heads, num_kv_heads, key_dim, value_dim, &smem, &groups) : 0;
   if (stages > 0) {
     B200_REQUIRE(split_tokens % 32 == 0 && out_ld % 2 == 0, "mixed_attn: split_tokens %d is no multiple of 32", split_tokens);
     B200_REQUIRE(aligned16({q, k_pool, v_pool}) && (reinterpret_cast<uintptr_t>(out) & 3) == 0, "mixed_attn: buffers must be aligned");
@@ -535,9 +606,10 @@ extern "C" int b200_mixed_attn(const void* q, const void* k_pool, const void* v_
     rc = get_tensor_map_2d(v_pool, pool_rows, value_dim, 2, kMdPage, 64, &vm);
     if (rc) return rc;
     const int per = num_q_heads / num_kv_heads, units = num_kv_heads * ((per + 15) / 16) * (value_dim / 64);
-    if (units <= kMdWarps) return launch_mixed_decode<1>(km, vm, pp, smem, as_stream(stream));
-    if (units <= 2 * kMdWarps) return launch_mixed_decode<2>(km, vm, pp, smem, as_stream(stream));
-    return launch_mixed_decode<4>(km, vm, pp, smem, as_stream(stream));
+    if (groups == 2) return launch_mixed_decode<1, 2>(km, vm, pp, smem, as_stream(stream));
+    if (units <= kMdWarps) return launch_mixed_decode<1, 1>(km, vm, pp, smem, as_stream(stream));
+    if (units <= 2 * kMdWarps) return launch_mixed_decode<2, 1>(km, vm, pp, smem, as_stream(stream));
+    return launch_mixed_decode<4, 1>(km, vm, pp, smem, as_stream(stream));
   }
   return dtype == 0 ? launch_mixed_generic<__nv_bfloat16>(p, as_stream(stream)) : launch_mixed_generic<float>(p, as_stream(stream));
 }

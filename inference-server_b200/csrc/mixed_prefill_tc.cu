@@ -5,19 +5,23 @@
 //            its kv head, and walks the key tiles (128 keys = 8 pages) from the one that holds the first key its first row
 //            sees to the one of its last position.
 //   warp 0   K producer: a tile's keys of ALL kv heads, 64 columns (16 KiB: 8 boxes of 16 tokens x 128 B) at a time, into a
-//            ring.  Before that the mixed queries of the tile, once, if its boxes fit the swizzle (per a multiple of 8).
-//   warp 1   issuer (one thread): S(0), then S(j + 1) and O += P(j) V(j) for every tile j.  S = Q' K^T is 4 x tcgen05.mma
-//            M128 N128 K16 per 64 columns into one of two S accumulators in TMEM; P (bf16) is an A operand in TMEM, V an
-//            MN-major B operand straight from its page layout.  While the softmax of tile j runs, S(j + 1) is in the tensor pipe.
-//   warp 2   the distance table: per tile the slice of B[h][.] that the tile's rows and keys meet, as +inf where a distance is
-//            negative (a later token) or outside the window, so the mask costs nothing of its own.
+//            ring.
+//   warp 1   issuer (one elected lane): S(0), then S(j + 1) and O += P(j) V(j) for every tile j.  S = Q' K^T is 4 x tcgen05.mma
+//            M128 N128 K16 per 64 columns; V is an MN-major B operand straight from its page layout.  While the softmax of
+//            tile j runs, S(j + 1) is in the tensor pipe.
+//   warp 2   the distance table (log2 units): per tile a bulk copy of the slice of B[h][.] that the tile's rows and keys meet.
+//            It is +inf where a distance is negative (a later token) or outside the window, so the mask costs nothing.
 //   warp 3   V producer: the values of the CTA's kv head, one tile at a time.
 //   warps 4-11  softmax: a thread owns a score row and 64 of the tile's 128 keys (TMEM lanes are bound to warp_id % 4; the two
 //            warps with the same rows meet on a named barrier for the row maximum).  s = score * log2 e - B from the slice in
-//            shared memory, lazy rescale of O as in paged_prefill_tc.cu, P = exp2(s - m) stored to TMEM.
+//            shared memory, lazy rescale of O as in paged_prefill_tc.cu, P = exp2(s - m) as bf16.
 //
-// TMEM: S0 columns 0-127, S1 128-255, O from 256 on, P in the last 64 columns; with value size 256, where none are left, P(j)
-// lies over S(j), and the issuer then waits for the product with P(j) before it writes that S accumulator again.
+// The queries meet the keys of all kv heads, so they are kv_heads times as wide as a head, and so is a tile of keys: what a CTA
+// can have in flight decides its speed.  Two forms (QTMEM):
+//   true   Q' is an A operand in TMEM (columns / 2 of it), beside O and one or two S accumulators; P goes through shared memory,
+//          which is left to the ring.  Whenever those fit the 512 columns.
+//   false  Q' in shared memory; S0 columns 0-127, S1 128-255, O from 256 on, P in the last 64 columns; with value size 256, where
+//          none are left, P(j) lies over S(j), and the issuer waits for the product with P(j) before it writes that S again.
 // Every mbarrier wait is bounded; one that runs out records kErrDevWaitTimeout, and the thread stops waiting but keeps the loop
 // structure (the named barriers between partner warps are still met), so the kernel ends.
 
@@ -30,7 +34,8 @@ constexpr int kMpRows = 128, kMpKeys = 128;
 constexpr int kMpChunk = 128 * 128;  // 128 rows x 64 bf16
 constexpr int kMpSoftmaxWarps = 8;
 constexpr int kMpThreads = (4 + kMpSoftmaxWarps) * 32;
-constexpr int kMpMaxStages = 8;
+constexpr int kMpMaxStages = 12;
+constexpr int kMpBarBytes = 384;  // barriers, tmem base
 constexpr float kMpRescaleLog2 = 8.f;
 constexpr float kMpLog2e = 1.4426950408889634f;
 
@@ -45,27 +50,42 @@ struct MixedPrefillParams {
   int num_tokens, first_pos, heads, kv_heads, num_blocks;
   int k_chunks;            // 64-wide pieces of a mixed query (all kv heads)
   int dk_chunks;           // of one kv head's keys
-  int stages, q_tma;
+  int stages, s_bufs;
   int bias_stride;         // floats per head of a slice
 };
 
 __host__ __device__ constexpr uint32_t mp_idesc(uint32_t n, uint32_t b_mn) {
   return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn << 16) | ((n >> 3) << 17) | ((128u >> 4) << 24);
 }
+// Issued by a converged warp: one elected lane sends the instruction, and the descriptors, the same in all lanes, can stay in
+// uniform registers (a branch on the lane number around the loop costs more than the instructions themselves).
 __device__ __forceinline__ void mp_mma_ss(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t acc) {
   asm volatile(
-      "{\n\t.reg .pred p;\n\t"
+      "{\n\t.reg .pred p, e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
       "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}" ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(acc)
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}" ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(acc)
       : "memory");
 }
 // A from TMEM: lane = row, a 32-bit column = two neighbouring K elements.
 __device__ __forceinline__ void mp_mma_ts(uint32_t d, uint32_t a, uint64_t b, uint32_t idesc, uint32_t acc) {
   asm volatile(
-      "{\n\t.reg .pred p;\n\t"
+      "{\n\t.reg .pred p, e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
       "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}" ::"r"(d), "r"(a), "l"(b), "r"(idesc), "r"(acc)
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}" ::"r"(d), "r"(a), "l"(b), "r"(idesc), "r"(acc)
       : "memory");
+}
+__device__ __forceinline__ void mp_commit(uint32_t bar) {
+  asm volatile(
+      "{\n\t.reg .pred e;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\t"
+      "@e tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}" ::"r"(bar)
+      : "memory");
+}
+// A wait of a whole warp, true if it has not run out for any lane.
+__device__ __forceinline__ bool mp_wait_all(uint32_t bar, uint32_t parity, int* err) {
+  return __all_sync(0xffffffffu, mbar_wait(bar, parity, err));
 }
 __device__ __forceinline__ uint64_t mp_desc_mn(uint32_t addr) {  // MN-major, 128-byte swizzle, next 64 columns kMpChunk further
   uint64_t d = 0;
@@ -88,11 +108,6 @@ __device__ __forceinline__ void mp_tmem_st32(uint32_t taddr, const uint32_t (&r)
       : "memory");
 }
 __device__ __forceinline__ void mp_tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ float mp_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 __device__ __forceinline__ void mp_pair_barrier(int quarter) {
   switch (quarter) {
     case 0: asm volatile("bar.sync 1, 64;" ::: "memory"); break;
@@ -102,38 +117,39 @@ __device__ __forceinline__ void mp_pair_barrier(int quarter) {
   }
 }
 
-template <int DV>
+template <int DV, bool QTMEM>
 __global__ void __launch_bounds__(kMpThreads, 1)
-mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
-                        const __grid_constant__ CUtensorMap v_map, const MixedPrefillParams p) {
+mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
+                        const MixedPrefillParams p) {
 #ifdef B200_DEVICE_OK
   constexpr int kVChunks = DV / 64;
-  constexpr bool kAlias = DV > 192;  // P over S
+  constexpr bool kAlias = !QTMEM && DV > 192;  // P over S
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* base_ptr = smem_raw + (base - smem_u32(smem_raw));
-  const uint32_t q_sm = base, v_sm = q_sm + p.k_chunks * kMpChunk, k_sm = v_sm + kVChunks * kMpChunk;
-  uint8_t* extra = base_ptr + (p.k_chunks + kVChunks + p.stages) * kMpChunk;
+  // Q' or P (two halves of 64 keys), V, the ring of keys
+  const int first_chunks = QTMEM ? 2 : p.k_chunks;
+  const uint32_t q_sm = base, v_sm = q_sm + first_chunks * kMpChunk, k_sm = v_sm + kVChunks * kMpChunk;
+  uint8_t* extra = base_ptr + (first_chunks + kVChunks + p.stages) * kMpChunk;
   const uint32_t bars = k_sm + p.stages * kMpChunk;
   const uint32_t bar_q = bars, bar_vfull = bars + 8, bar_vempty = bars + 16;
   const uint32_t bar_sfull = bars + 24, bar_sempty = bars + 40;  // [2] each
   const uint32_t bar_pfull = bars + 56, bar_odone = bars + 64;
   const uint32_t bar_bfull = bars + 72, bar_bempty = bars + 88;  // [2] each: slice of the distance table
   const uint32_t bar_kfull = bars + 104, bar_kempty = bar_kfull + 8 * kMpMaxStages;
-  uint32_t* tmem_base_sm = reinterpret_cast<uint32_t*>(extra + 240);
-  float* mx_sm = reinterpret_cast<float*>(extra + 256);  // [2 tiles][2 halves][128 rows]
+  uint32_t* tmem_base_sm = reinterpret_cast<uint32_t*>(extra + kMpBarBytes - 16);
+  float* mx_sm = reinterpret_cast<float*>(extra + kMpBarBytes);  // [2 tiles][2 halves][128 rows]
   float* l_sm = mx_sm + 2 * 2 * kMpRows;                 // [2 halves][128 rows]
   float* b_sm = l_sm + 2 * kMpRows;                      // [2][per][bias_stride]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int per = p.heads / p.kv_heads, QT = kMpRows / per;
   if (threadIdx.x == 32) {
-    tma_prefetch_desc(&q_map);
     tma_prefetch_desc(&k_map);
     tma_prefetch_desc(&v_map);
   }
   if (threadIdx.x == 0) {
-    mbar_init(bar_q, p.q_tma ? 1 : kMpSoftmaxWarps);
+    mbar_init(bar_q, kMpSoftmaxWarps);
     mbar_init(bar_vfull, 1);
     mbar_init(bar_vempty, 1);
     mbar_init(bar_pfull, kMpSoftmaxWarps);
@@ -156,6 +172,9 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_base_sm;
+  // columns: QTMEM  O, Q', S buffers;  else  S0, S1, O, P
+  const uint32_t o_col = QTMEM ? 0u : 256u, q_col = DV, s_col = QTMEM ? DV + p.k_chunks * 32u : 0u;
+  const int s_bufs = QTMEM ? p.s_bufs : 2;
   grid_dep_wait();
   grid_dep_launch();
 
@@ -169,16 +188,8 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
 
   if (warp == 0 || warp == 3) {
     // -------------------------------------------------------- K / V producers ------
-    if (warp == 0 && p.q_tma) {
-      if (lane == 0) mbar_arrive_expect_tx(bar_q, p.k_chunks * kMpChunk);
-      __syncwarp();
-      for (int i = lane; i < p.k_chunks * QT; i += 32) {
-        const int tl = i / p.k_chunks, c = i - tl * p.k_chunks;
-        tma_load_2d(q_sm + c * kMpChunk + tl * per * 128, &q_map, bar_q, c * 64, (t0 + tl) * p.heads + g * per);
-      }
-    }
     bool alive = true;
-    uint32_t it = 0;
+    uint32_t slot = 0, kphase = 1;
 #pragma unroll 1
     for (int j = 0; j < n_tiles && alive; ++j) {
       // lanes 0-7 own a page each; pages past the last position stand in for by it: their keys are masked, their values meet
@@ -194,21 +205,23 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
       const int row0 = page * p.kv_heads * kMpPage;
       if (warp == 0) {
 #pragma unroll 1
-        for (int c = 0; c < p.k_chunks && alive; ++c, ++it) {
-          const uint32_t st = it % p.stages, ph = (it / p.stages) & 1;
-          alive = mbar_wait(bar_kempty + 8 * st, ph ^ 1, p.err);
-          alive = __all_sync(0xffffffffu, alive);
-          if (!alive) break;
-          if (lane == 0) mbar_arrive_expect_tx(bar_kfull + 8 * st, kMpChunk);
-          __syncwarp();
-          const int head = c / p.dk_chunks;
-          if (lane < 8)
-            tma_load_2d(k_sm + st * kMpChunk + lane * (kMpPage * 128), &k_map, bar_kfull + 8 * st, (c - head * p.dk_chunks) * 64,
-                        row0 + head * kMpPage);
+        for (int head = 0; head < p.kv_heads && alive; ++head) {
+#pragma unroll 1
+          for (int c = 0; c < p.dk_chunks; ++c) {
+            alive = mp_wait_all(bar_kempty + 8 * slot, kphase, p.err);
+            if (!alive) break;
+            if (lane == 0) mbar_arrive_expect_tx(bar_kfull + 8 * slot, kMpChunk);
+            __syncwarp();
+            if (lane < 8)
+              tma_load_2d(k_sm + slot * kMpChunk + lane * (kMpPage * 128), &k_map, bar_kfull + 8 * slot, c * 64, row0 + head * kMpPage);
+            if (++slot == static_cast<uint32_t>(p.stages)) {
+              slot = 0;
+              kphase ^= 1;
+            }
+          }
         }
       } else {
-        alive = mbar_wait(bar_vempty, (j & 1) ^ 1, p.err);
-        alive = __all_sync(0xffffffffu, alive);
+        alive = mp_wait_all(bar_vempty, (j & 1) ^ 1, p.err);
         if (!alive) break;
         if (lane == 0) mbar_arrive_expect_tx(bar_vfull, kVChunks * kMpChunk);
         __syncwarp();
@@ -220,78 +233,99 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
     }
   } else if (warp == 1) {
     // ---------------------------------------------------------------- issuer ------
-    if (lane == 0) {
-      constexpr uint32_t idesc_s = mp_idesc(kMpKeys, 0), idesc_o = mp_idesc(DV, 1);
-      const uint32_t tmem_o = tmem_base + 256;
-      bool alive = mbar_wait(bar_q, 0, p.err);
-      uint32_t it = 0;
-      auto scores = [&](int t) {
-        const int sb = t & 1;
-        const uint32_t ph = (t >> 1) & 1;
-        if (alive) alive = mbar_wait(bar_sempty + 8 * sb, ph ^ 1, p.err);
-        if (kAlias && t >= 2 && alive) alive = mbar_wait(bar_odone, (t - 2) & 1, p.err);  // P(t - 2) lies there
+    constexpr uint32_t idesc_s = mp_idesc(kMpKeys, 0), idesc_o = mp_idesc(DV, 1);
+    const uint32_t tmem_o = tmem_base + o_col;
+    bool alive = mp_wait_all(bar_q, 0, p.err);
+    uint32_t slot = 0, kphase = 0;
+    const uint64_t q_desc = umma_desc_k128(q_sm), k_desc = umma_desc_k128(k_sm), v_desc = mp_desc_mn(v_sm);
+    auto scores = [&](int t) {
+      const int sb = s_bufs == 2 ? t & 1 : 0;
+      const uint32_t ph = (s_bufs == 2 ? t >> 1 : t) & 1, s_acc = tmem_base + s_col + sb * kMpKeys;
+      if (alive) alive = mp_wait_all(bar_sempty + 8 * sb, ph ^ 1, p.err);
+      if (kAlias && t >= 2 && alive) alive = mp_wait_all(bar_odone, (t - 2) & 1, p.err);  // P(t - 2) lies there
 #pragma unroll 1
-        for (int c = 0; c < p.k_chunks && alive; ++c, ++it) {
-          const uint32_t st = it % p.stages;
-          alive = mbar_wait(bar_kfull + 8 * st, (it / p.stages) & 1, p.err);
-          if (!alive) break;
-          tc_fence_after();
-          const uint64_t a0 = umma_desc_k128(q_sm + c * kMpChunk), b0 = umma_desc_k128(k_sm + st * kMpChunk);
-#pragma unroll
-          for (int k = 0; k < 4; ++k)
-            mp_mma_ss(tmem_base + sb * kMpKeys, a0 + 2 * k, b0 + 2 * k, idesc_s, (c > 0 || k > 0) ? 1u : 0u);
-          tc_commit(bar_kempty + 8 * st);
-        }
-        if (alive) tc_commit(bar_sfull + 8 * sb);
-      };
-      scores(0);
-#pragma unroll 1
-      for (int j = 0; j < n_tiles && alive; ++j) {
-        if (j + 1 < n_tiles) scores(j + 1);
-        if (alive) alive = mbar_wait(bar_vfull, j & 1, p.err);
-        if (alive) alive = mbar_wait(bar_pfull, j & 1, p.err);
+      for (int c = 0; c < p.k_chunks && alive; ++c) {
+        alive = mp_wait_all(bar_kfull + 8 * slot, kphase, p.err);
         if (!alive) break;
         tc_fence_after();
-        const uint32_t pa = tmem_base + (kAlias ? static_cast<uint32_t>((j & 1) * kMpKeys) : 448u);
+        const uint64_t a0 = q_desc + static_cast<uint32_t>(c) * (kMpChunk >> 4), b0 = k_desc + slot * (kMpChunk >> 4);
 #pragma unroll
-        for (int kk = 0; kk < 8; ++kk)
-          mp_mma_ts(tmem_o, pa + kk * 8, mp_desc_mn(v_sm + kk * (16 * 128)), idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
-        tc_commit(bar_odone);
-        tc_commit(bar_vempty);
+        for (int k = 0; k < 4; ++k) {
+          if (QTMEM) mp_mma_ts(s_acc, tmem_base + q_col + c * 32 + k * 8, b0 + 2 * k, idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+          else mp_mma_ss(s_acc, a0 + 2 * k, b0 + 2 * k, idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+        }
+        mp_commit(bar_kempty + 8 * slot);
+        if (++slot == static_cast<uint32_t>(p.stages)) {
+          slot = 0;
+          kphase ^= 1;
+        }
       }
+      if (alive) mp_commit(bar_sfull + 8 * sb);
+    };
+    scores(0);
+#pragma unroll 1
+    for (int j = 0; j < n_tiles && alive; ++j) {
+      if (j + 1 < n_tiles) scores(j + 1);
+      if (alive) alive = mp_wait_all(bar_vfull, j & 1, p.err);
+      if (alive) alive = mp_wait_all(bar_pfull, j & 1, p.err);
+      if (!alive) break;
+      tc_fence_after();
+      const uint32_t pa = tmem_base + (kAlias ? static_cast<uint32_t>((j & 1) * kMpKeys) : 448u);
+#pragma unroll
+      for (int kk = 0; kk < 8; ++kk) {
+        const uint64_t b = v_desc + kk * ((16 * 128) >> 4);
+        if (QTMEM) mp_mma_ss(tmem_o, q_desc + (kk >> 2) * (kMpChunk >> 4) + 2 * (kk & 3), b, idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
+        else mp_mma_ts(tmem_o, pa + kk * 8, b, idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
+      }
+      mp_commit(bar_odone);
+      mp_commit(bar_vempty);
     }
   } else if (warp == 2) {
     // ------------------------------------------- slices of the distance table ------
-    // entry x of a head: distance p0 - (first key of the tile) - 127 + x
+    // entry x of a head: distance p0 - (first key of the tile) - 127 + x, after up to 3 entries that make the copy's start a
+    // multiple of 16 bytes
     bool alive = true;
     const int span = kMpKeys + QT - 1;
 #pragma unroll 1
     for (int j = 0; j < n_tiles && alive; ++j) {
-      alive = mbar_wait(bar_bempty + 8 * (j & 1), ((j >> 1) & 1) ^ 1, p.err);
-      alive = __all_sync(0xffffffffu, alive);
+      alive = mp_wait_all(bar_bempty + 8 * (j & 1), ((j >> 1) & 1) ^ 1, p.err);
       if (!alive) break;
-      const int d0 = p0 - (kt0 + j) * kMpKeys - (kMpKeys - 1);
-      float* dst = b_sm + (j & 1) * per * p.bias_stride;
-      for (int hh = 0; hh < per; ++hh) {
-        const float* src = p.bias + static_cast<size_t>(g * per + hh) * p.bias_ld;
-#pragma unroll 4
-        for (int x = lane; x < span; x += 32) {
-          const int d = d0 + x;
-          dst[hh * p.bias_stride + x] = d >= 0 && d < p.window && d < p.bias_ld ? __ldg(src + d) * kMpLog2e : INFINITY;
-        }
-      }
+      const int at = kDistPad + p0 - (kt0 + j) * kMpKeys - (kMpKeys - 1);
+      const uint32_t bytes = static_cast<uint32_t>(((at & 3) + span + 3) & ~3) * 4u;
+      if (lane == 0) mbar_arrive_expect_tx(bar_bfull + 8 * (j & 1), bytes * per);
       __syncwarp();
-      if (lane == 0) mbar_arrive(bar_bfull + 8 * (j & 1));
+      const uint32_t dst = smem_u32(b_sm) + static_cast<uint32_t>((j & 1) * per * p.bias_stride) * 4u;
+      for (int hh = lane; hh < per; hh += 32)
+        bulk_load(dst + static_cast<uint32_t>(hh * p.bias_stride) * 4u,
+                  p.bias + static_cast<size_t>(g * per + hh) * p.bias_ld + (at & ~3), bytes, bar_bfull + 8 * (j & 1));
     }
   } else {
     // --------------------------------------------------------------- softmax ------
     const int sw = warp - 4, hf = sw >> 2, quarter = warp & 3;
     const int r = quarter * 32 + lane;
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16);
-    const uint32_t tmem_o = lane_addr + 256 + hf * (DV / 2);
+    const uint32_t tmem_o = lane_addr + o_col + hf * (DV / 2);
     const int tl = r / per, head = r - tl * per;
     const bool real = tl < QT && t0 + tl < p.num_tokens;
-    if (!p.q_tma) {  // copy the Q' tile: neighbouring threads take neighbouring 16-byte pieces of a row
+    // the tile's mixed queries; zero rows past its last position
+    if (QTMEM) {  // 64 columns of this thread's row at a time: one half of them per thread of the row
+      const uint4* src = reinterpret_cast<const uint4*>(p.q + (static_cast<size_t>(t0 + tl) * p.heads + g * per + head) * (p.k_chunks * 64));
+#pragma unroll 2
+      for (int c = hf; c < p.k_chunks; c += 2) {
+        uint32_t v[32];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const uint4 x = real ? __ldg(src + c * 8 + e) : make_uint4(0u, 0u, 0u, 0u);
+          v[4 * e] = x.x;
+          v[4 * e + 1] = x.y;
+          v[4 * e + 2] = x.z;
+          v[4 * e + 3] = x.w;
+        }
+        mp_tmem_st32(lane_addr + q_col + c * 32, v);
+      }
+      mp_tmem_st_wait();
+      tc_fence_before();
+    } else {  // neighbouring threads take neighbouring 16-byte pieces of a row
       const int pieces = p.k_chunks * 8;
       for (int i = sw * 32 + lane; i < kMpRows * pieces; i += kMpSoftmaxWarps * 32) {
         const int qr = i / pieces, ch = i - qr * pieces, qtl = qr / per;
@@ -302,26 +336,27 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
         *reinterpret_cast<uint4*>(base_ptr + (ch >> 3) * kMpChunk + swz128(qr, ch & 7)) = v;
       }
       fence_proxy_async();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(bar_q);
     }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(bar_q);
     // slice entry of this row and key column c: distance (p0 + tl) - (tile key) - c
-    const float* b_row = b_sm + min(head, per - 1) * p.bias_stride + min(tl, QT - 1) + (kMpKeys - 1) - hf * 64;
+    const float* b_row = b_sm + head * p.bias_stride + min(tl, QT - 1) + (kMpKeys - 1) - hf * 64 +
+                         ((kDistPad + p0 - (kMpKeys - 1)) & 3);  // a tile's first key is a multiple of 128
     float m_run = -INFINITY, l_run = 0.f;
     bool alive = true;
 #pragma unroll 1
     for (int j = 0; j < n_tiles; ++j) {
-      const int buf = j & 1;
+      const int buf = j & 1, sb = s_bufs == 2 ? buf : 0;
       const float* bt = b_row + buf * per * p.bias_stride;
       if (alive) alive = mbar_wait(bar_bfull + 8 * buf, (j >> 1) & 1, p.err);
-      if (alive) alive = mbar_wait(bar_sfull + 8 * buf, (j >> 1) & 1, p.err);
+      if (alive) alive = mbar_wait(bar_sfull + 8 * sb, (s_bufs == 2 ? j >> 1 : j) & 1, p.err);
       tc_fence_after();
       float s[64];
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         uint32_t raw[32];
-        tmem_ld32(lane_addr + buf * kMpKeys + hf * 64 + half * 32, raw);
+        tmem_ld32(lane_addr + s_col + sb * kMpKeys + hf * 64 + half * 32, raw);
         tmem_ld_wait();
 #pragma unroll
         for (int c = 0; c < 32; ++c) {
@@ -334,7 +369,7 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
       __syncwarp();
       if (lane == 0) {
         mbar_arrive(bar_bempty + 8 * buf);
-        if (!kAlias) mbar_arrive(bar_sempty + 8 * buf);  // this S accumulator may be overwritten
+        if (!kAlias) mbar_arrive(bar_sempty + 8 * sb);  // this S accumulator may be overwritten
       }
       const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       float* mxb = mx_sm + buf * 2 * kMpRows;
@@ -347,7 +382,7 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
       tc_fence_after();
       if (__any_sync(0xffffffffu, need)) {
         if (j > 0) {
-          const float alpha = m_new == -INFINITY ? 1.f : mp_exp2(m_run - m_new);
+          const float alpha = m_new == -INFINITY ? 1.f : fast_ex2(m_run - m_new);
           l_run *= alpha;
 #pragma unroll
           for (int c0 = 0; c0 < DV / 2; c0 += 32) {
@@ -366,13 +401,22 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
       uint32_t pw[32];
 #pragma unroll
       for (int c = 0; c < 32; ++c) {
-        const float e0 = mp_exp2(s[2 * c] - mb), e1 = mp_exp2(s[2 * c + 1] - mb);
+        const float e0 = fast_ex2(s[2 * c] - mb), e1 = fast_ex2(s[2 * c + 1] - mb);
         sum4[c & 3] += e0 + e1;
         pw[c] = pack_bf16x2(e0, e1);
       }
       l_run += (sum4[0] + sum4[1]) + (sum4[2] + sum4[3]);
-      mp_tmem_st32(lane_addr + (kAlias ? buf * kMpKeys : 448) + hf * 32, pw);
-      mp_tmem_st_wait();
+      if (QTMEM) {
+        uint8_t* p_half = base_ptr + hf * kMpChunk;
+#pragma unroll
+        for (int ch = 0; ch < 8; ++ch)
+          *reinterpret_cast<uint4*>(p_half + swz128(r, ch)) = make_uint4(pw[4 * ch], pw[4 * ch + 1], pw[4 * ch + 2], pw[4 * ch + 3]);
+        mp_tmem_st_wait();    // a rescaled O
+        fence_proxy_async();  // the tensor core reads P through the async proxy
+      } else {
+        mp_tmem_st32(lane_addr + (kAlias ? buf * kMpKeys : 448) + hf * 32, pw);
+        mp_tmem_st_wait();
+      }
       tc_fence_before();
       __syncwarp();
       if (lane == 0) {
@@ -414,38 +458,47 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
 #endif
 }
 
-// Floats per head of a slice: a step of 32 / per (per a power of two up to 32) puts the 32 rows of a warp into 32 banks.
+// Floats per head of a slice (rows of 16 bytes): a step of 32 / per (per a power of two up to 8) puts the 32 rows of a warp into
+// 32 banks.
 static int mixed_bias_stride(int per) {
-  const int need = kMpKeys + kMpRows / per;
-  int step = 1;
+  const int need = kMpKeys + kMpRows / per + 6;
+  int step = 4;
   while (step * per < 32) step <<= 1;
   int s = (need + 31) / 32 * 32 + step;
   if (s - 32 >= need) s -= 32;
   return s;
 }
 
-// Stages of the K ring that fit beside the queries, the values and the slices; below 2 the kernel is not used.
-static int mixed_prefill_stages(int heads, int kv_heads, int key_dim, int value_dim, size_t* smem_out) {
-  if (heads % kv_heads || heads / kv_heads > kMpRows || key_dim % 64 || value_dim % 64 || value_dim > 256) return 0;
-  const int per = heads / kv_heads, chunks = kv_heads * key_dim / 64;
-  const size_t fixed = 1024 + 256 + (4 + 2) * kMpRows * 4 + static_cast<size_t>(2) * per * mixed_bias_stride(per) * 4 +
-                       static_cast<size_t>(chunks + value_dim / 64) * kMpChunk;
+// How the kernel runs for a shape: stages of the ring (below 2: not built for it), whether Q' lies in TMEM, S accumulators.
+struct MixedPrefillPlan {
+  int stages, q_tmem, s_bufs;
+  size_t smem;
+};
+static MixedPrefillPlan mixed_prefill_plan(int heads, int kv_heads, int key_dim, int value_dim) {
+  MixedPrefillPlan pl{0, 0, 2, 0};
+  if (heads % kv_heads || heads / kv_heads > kMpRows || key_dim % 64 || value_dim % 64 || value_dim > 256) return pl;
+  const int per = heads / kv_heads, chunks = kv_heads * key_dim / 64, columns = value_dim + chunks * 32;
+  if (columns + kMpKeys <= 512) {
+    pl.q_tmem = 1;
+    pl.s_bufs = columns + 2 * kMpKeys <= 512 ? 2 : 1;
+  }
+  const size_t fixed = 1024 + kMpBarBytes + (4 + 2) * kMpRows * 4 + static_cast<size_t>(2) * per * mixed_bias_stride(per) * 4 +
+                       static_cast<size_t>((pl.q_tmem ? 2 : chunks) + value_dim / 64) * kMpChunk;
   const size_t room = 227 * 1024;
-  if (fixed >= room) return 0;
-  int stages = static_cast<int>((room - fixed) / kMpChunk);
-  if (stages > kMpMaxStages) stages = kMpMaxStages;
-  if (smem_out) *smem_out = fixed + static_cast<size_t>(stages) * kMpChunk;
-  return stages;
+  if (fixed >= room) return pl;
+  pl.stages = static_cast<int>((room - fixed) / kMpChunk);
+  if (pl.stages > kMpMaxStages) pl.stages = kMpMaxStages;
+  pl.smem = fixed + static_cast<size_t>(pl.stages) * kMpChunk;
+  return pl;
 }
 
-template <int DV>
-static int launch_mixed_prefill(const CUtensorMap& qm, const CUtensorMap& km, const CUtensorMap& vm, const MixedPrefillParams& p,
-                                size_t smem, cudaStream_t st) {
-  int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mixed_prefill_tc_kernel<DV>), 227 * 1024);
+template <int DV, bool QTMEM>
+static int launch_mixed_prefill(const CUtensorMap& km, const CUtensorMap& vm, const MixedPrefillParams& p, size_t smem, cudaStream_t st) {
+  int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mixed_prefill_tc_kernel<DV, QTMEM>), 227 * 1024);
   if (rc) return rc;
   const int qt = kMpRows / (p.heads / p.kv_heads);
-  B200_CUDA(launch_overlapped(mixed_prefill_tc_kernel<DV>, dim3((p.num_tokens + qt - 1) / qt, p.kv_heads), dim3(kMpThreads), smem, st,
-                              qm, km, vm, p));
+  B200_CUDA(launch_overlapped(mixed_prefill_tc_kernel<DV, QTMEM>, dim3((p.num_tokens + qt - 1) / qt, p.kv_heads), dim3(kMpThreads),
+                              smem, st, km, vm, p));
   return 0;
 }
 
@@ -455,7 +508,7 @@ using namespace b200;
 
 extern "C" int b200_mixed_attn_prefill_supported(int num_q_heads, int num_kv_heads, int key_dim, int value_dim) {
   if (num_q_heads <= 0 || num_kv_heads <= 0 || key_dim <= 0 || value_dim <= 0 || num_kv_heads > 65535) return 0;
-  return mixed_prefill_stages(num_q_heads, num_kv_heads, key_dim, value_dim, nullptr) >= 2;
+  return mixed_prefill_plan(num_q_heads, num_kv_heads, key_dim, value_dim).stages >= 2;
 }
 
 extern "C" int b200_mixed_attn_prefill(const void* q, const void* k_pool, const void* v_pool, const int32_t* block_table_row,
@@ -467,18 +520,16 @@ extern "C" int b200_mixed_attn_prefill(const void* q, const void* k_pool, const 
   B200_REQUIRE(num_tokens > 0 && first_position >= 0 && page_size == kMpPage && num_blocks > 0 && window > 0 &&
                    first_position + num_tokens <= static_cast<long long>(max_pages_per_seq) * page_size,
                "mixed_attn_prefill: %d tokens from %d, pages of %d, window %d", num_tokens, first_position, page_size, window);
-  size_t smem = 0;
-  const int stages = b200_mixed_attn_prefill_supported(num_q_heads, num_kv_heads, key_dim, value_dim)
-                         ? mixed_prefill_stages(num_q_heads, num_kv_heads, key_dim, value_dim, &smem) : 0;
-  B200_REQUIRE(stages >= 2, "mixed_attn_prefill: not built for %d query heads over %d, key size %d, value size %d", num_q_heads,
+  B200_REQUIRE(b200_mixed_attn_prefill_supported(num_q_heads, num_kv_heads, key_dim, value_dim), "mixed_attn_prefill: not built for %d query heads over %d, key size %d, value size %d", num_q_heads,
                num_kv_heads, key_dim, value_dim);
   const long long seen = first_position + num_tokens < window ? first_position + num_tokens : window;
-  B200_REQUIRE(bias_ld >= seen && out_ld >= num_q_heads * value_dim && out_ld % 8 == 0,
+  B200_REQUIRE(bias_ld >= kDistPad + seen + kDistTail && bias_ld % 4 == 0 && out_ld >= num_q_heads * value_dim && out_ld % 8 == 0,
                "mixed_attn_prefill: bias rows of %d, output rows of %d", bias_ld, out_ld);
-  B200_REQUIRE(aligned16({q, k_pool, v_pool, out}), "mixed_attn_prefill: buffers must be 16-byte aligned");
+  B200_REQUIRE(aligned16({q, k_pool, v_pool, out, bias}), "mixed_attn_prefill: buffers must be 16-byte aligned");
   int rc = check_device(nullptr);
   if (rc) return rc;
   const int per = num_q_heads / num_kv_heads;
+  const MixedPrefillPlan plan = mixed_prefill_plan(num_q_heads, num_kv_heads, key_dim, value_dim);
   MixedPrefillParams p{};
   p.table_row = block_table_row;
   p.q = static_cast<const __nv_bfloat16*>(q);
@@ -496,25 +547,24 @@ extern "C" int b200_mixed_attn_prefill(const void* q, const void* k_pool, const 
   p.num_blocks = num_blocks;
   p.dk_chunks = key_dim / 64;
   p.k_chunks = num_kv_heads * p.dk_chunks;
-  p.stages = stages;
-  p.q_tma = per % 8 == 0 && 128 % per == 0;
+  p.stages = plan.stages;
+  p.s_bufs = plan.s_bufs;
   p.bias_stride = mixed_bias_stride(per);
-  CUtensorMap qm, km, vm;
+  CUtensorMap km, vm;
   const uint64_t rows = static_cast<uint64_t>(num_blocks) * num_kv_heads * kMpPage;
   rc = get_tensor_map_2d(k_pool, rows, key_dim, 2, kMpPage, 64, &km);
   if (rc) return rc;
   rc = get_tensor_map_2d(v_pool, rows, value_dim, 2, kMpPage, 64, &vm);
   if (rc) return rc;
-  qm = km;
-  if (p.q_tma) {
-    rc = get_tensor_map_2d(q, static_cast<uint64_t>(num_tokens) * num_q_heads, static_cast<uint64_t>(p.k_chunks) * 64, 2, per, 64, &qm);
-    if (rc) return rc;
-  }
   cudaStream_t st = as_stream(stream);
+#define B200_MIXED_PREFILL(DV)                                                             \
+  return plan.q_tmem ? launch_mixed_prefill<DV, true>(km, vm, p, plan.smem, st)            \
+                     : launch_mixed_prefill<DV, false>(km, vm, p, plan.smem, st)
   switch (value_dim) {
-    case 64: return launch_mixed_prefill<64>(qm, km, vm, p, smem, st);
-    case 128: return launch_mixed_prefill<128>(qm, km, vm, p, smem, st);
-    case 192: return launch_mixed_prefill<192>(qm, km, vm, p, smem, st);
-    default: return launch_mixed_prefill<256>(qm, km, vm, p, smem, st);
+    case 64: B200_MIXED_PREFILL(64);
+    case 128: B200_MIXED_PREFILL(128);
+    case 192: B200_MIXED_PREFILL(192);
+    default: B200_MIXED_PREFILL(256);
   }
+#undef B200_MIXED_PREFILL
 }

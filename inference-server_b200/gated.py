@@ -158,10 +158,11 @@ def _pad(t: torch.Tensor, dim: int, to: int) -> torch.Tensor:
 
 
 def distance_table(talk: torch.Tensor, r1: torch.Tensor, r2: torch.Tensor, distances: int) -> torch.Tensor:
-    """[heads, distances] fp32: what the mixed score of a head loses at each distance, sum_g talk[h, g] r1_g ln(1 + r2_g d)."""
+    """What the mixed score of a head loses at each distance, sum_g talk[h, g] r1_g ln(1 + r2_g d), d < distances, as the
+    attention kernels take it (`ops.pad_distances`)."""
     d = torch.arange(distances, dtype=torch.float64, device=talk.device)
     own = r1.double()[:, None] * torch.log1p(r2.double()[:, None] * d[None])
-    return (talk.double() @ own).float().contiguous()
+    return ops.pad_distances(talk.double() @ own)
 
 
 class Projection:

@@ -744,6 +744,17 @@ def mix_heads(q, mix, kv_heads: int, dtype):
     return out
 
 
+DIST_PAD, DIST_TAIL = 256, 264
+
+
+def pad_distances(table):
+    """[heads, distances] -> fp32 rows in log2 units with +inf (a mask) before distance 0, at entry DIST_PAD, and after the last."""
+    H, n = table.shape
+    out = torch.full((H, -(-(DIST_PAD + n + DIST_TAIL) // 4) * 4), float("inf"), dtype=torch.float32, device=table.device)
+    out[:, DIST_PAD:DIST_PAD + n] = (table.double() * 1.4426950408889634).float()
+    return out
+
+
 def mixed_split_tokens(rows: int, window: int, max_ctx: int, num_sms: int = 148) -> int:
     """Tokens per split of the decode kernel (all heads of a row in one CTA, one CTA per SM for large pages): about four CTAs per
     SM over the rows' windows, at least 128 tokens each."""
@@ -773,8 +784,8 @@ def _mixed_shapes(q, k_pool, v_pool, bias, out):
 
 def mixed_attn(q, k_pool, v_pool, block_table, positions, bias, window: int, out, out_scale: float, status=None,
                split_tokens: int | None = None, workspace=None):
-    """Windowed attention of mixed queries [M, H, G * Dk] over pages; writes columns [0, H * Dv) of out [M, ld].  `split_tokens`
-    0: the generic kernel."""
+    """Windowed attention of mixed queries [M, H, G * Dk] over pages; writes columns [0, H * Dv) of out [M, ld].  bias: see
+    `pad_distances`.  `split_tokens` 0: the generic kernel."""
     M, H, G, Dk, Dv, page, nb = _mixed_shapes(q, k_pool, v_pool, bias, out)
     _need(block_table, "block_table", torch.int32)
     _need(positions, "positions", torch.int32)

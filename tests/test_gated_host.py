@@ -76,11 +76,12 @@ def test_run_time_weights_compute_the_same_layer(name):
                                  for c in range(a.kv_heads)], 2)
             s = torch.einsum("mhcd,ncd->hmn", mixed, k)
             n = min(a.window, 400)
-            assert w.bias.shape == (a.heads, n)
+            bias = w.bias[:, 256:256 + n] / 1.4426950408889634  # kept in log2 units, +inf around it
+            assert w.bias.shape[1] % 4 == 0 and bool(w.bias[:, :256].isinf().all()) and bool(w.bias[:, 256 + n:].isinf().all())
             dist = (torch.arange(5)[:, None] - torch.arange(5)[None]).clamp(0, n - 1)
             want = ref.talking_scores(q, k, a.scale, f["mix.left.r1"], f["mix.left.r2"], f["mix.left.talk"])
             seen = ref.window_mask(5, a.window)
-            assert torch.allclose((s - w.bias[:, dist])[:, seen], want[:, seen], atol=2e-4)
+            assert torch.allclose((s - bias[:, dist])[:, seen], want[:, seen], atol=2e-4)
             oa, orr = torch.randn(5, a.heads, a.vdim, generator=gen), torch.randn(5, r.heads, r.vdim, generator=gen)
             out = torch.zeros(5, w.out_ld)
             out[:, : a.heads * w.Dv].view(5, a.heads, w.Dv)[..., : a.vdim] = oa * m.left_scale

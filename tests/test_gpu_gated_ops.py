@@ -164,7 +164,7 @@ def test_mixed_attention(ops, H, G, dk, dv, window, dtype):
             if j >= 0:
                 k[j] = (qm[i, (i + j) % H].view(G, dk).float() * 8 / qm[i, (i + j) % H].float().pow(2).sum()).to(dtype)
                 kp[order[j // 16], :, j % 16] = k[j]
-    dev = [t.to(DEV) for t in (qm, kp, vp, bias, order)]
+    dev = [t.to(DEV) for t in (qm, kp, vp, ops.pad_distances(bias), order)]
     Q, KP, VP, B, O = dev
     rows = [0, 1, 15, 16, 17, 31, 32, 40, 47, 48, 96, 99, 100, 150, 169]
     pos = torch.tensor(rows, dtype=torch.int32, device=DEV)
@@ -188,7 +188,7 @@ def test_mixed_attention(ops, H, G, dk, dv, window, dtype):
 
 def test_mixed_attention_reports_bad_pages_and_positions(ops):
     qm, k, v, bias, kp, vp, order = attention_case(40, 8, 2, 64, 64, 32, BF, 1)
-    Q, KP, VP, B, O = (t.to(DEV) for t in (qm, kp, vp, bias, order))
+    Q, KP, VP, B, O = (t.to(DEV) for t in (qm, kp, vp, ops.pad_distances(bias), order))
     out = torch.empty(1, 512, dtype=BF, device=DEV)
     for table, pos in ((torch.full((1, 3), 99, dtype=torch.int32, device=DEV), i32(20)), (O[None].contiguous(), i32(48))):
         st = status()
