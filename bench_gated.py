@@ -56,10 +56,12 @@ def kernels(eng, rows, positions, ids: dict, decode: bool) -> dict:
             t.add("windowed attention with mixed heads (all its kernels)",
                   [lambda i=i: eng._window_attention(q, eng.k_pools[i], eng.v_pools[i], a, eng.layers[i], rows, 1.0, out) for i in li],
                   read + n * a.heads * (w0.Dk * 4 + w0.Dv * 2), 2 * seen * a.heads * (w0.Dk + w0.Dv))
-            parts = rows.parts()
-            t.add("convolution + SiLU", [lambda i=i: [ops.conv_silu(pre[lo:hi], eng.layers[i].conv, eng.rings[i], rows.slots[lo:hi], rows.pos[lo:hi], c, eng.status, act[lo:hi])
-                                                       for lo, hi, c in parts] for i in li], n * w0.channels * (4 + (2 * r.taps if decode else 0)), 0)
-            act.normal_()
+            pre.normal_()
+            if not decode:
+                t.add("convolution + SiLU", [lambda i=i: ops.conv_silu(pre, eng.layers[i].conv, eng.rings[i], rows.slots, rows.pos, True,
+                                                                       eng.status, act) for i in li], n * w0.channels * 4, 0)
+                act.normal_()
+            ba.normal_()
         else:
             ba = None
 
@@ -70,18 +72,25 @@ def kernels(eng, rows, positions, ids: dict, decode: bool) -> dict:
 
             t.add("lightning projection", [lambda i=i: proj(i) for i in li], N * W * 2 + n * (W + N) * 2, 2 * n * N * W)
             act.normal_()
-        name = "gated delta rule" if kind == "parallel" else "lightning recurrence"
         moved = n * H * S * 8 if decode else H * S * 8
-        t.add(f"{name} ({'decode' if decode else 'prompt'} form)", [lambda i=i: eng._recurrence(act, i, eng.layers[i], rows, ba, 0.1) for i in li],
-              moved + n * (w0.channels * 2 + H * w0.dv * 4), (6 if kind == "parallel" else 4) * n * H * S)
+        flops = (6 if kind == "parallel" else 4) * n * H * S
+        if kind == "parallel" and decode:
+            t.add("gated delta rule with convolution, head norm and gate", [
+                lambda i=i: eng._delta(pre, ba, gt, i, m.right, eng.layers[i], rows, 1.0, out[:, m.left.heads * w0.Dv:]) for i in li],
+                moved + n * (w0.channels * (2 + 2 * m.right.taps) + H * w0.dv * 4), flops)
+        else:
+            t.add("gated delta rule" if kind == "parallel" else "lightning recurrence",
+                  [lambda i=i: eng._recurrence(act, i, eng.layers[i], rows, 0, n, not decode, o, ba, 0.1) for i in li],
+                  moved + n * (w0.channels * 2 + H * w0.dv * 4), flops)
         if kind == "parallel":
             args = (m.right.vdim, True, 1.0, out[:, m.left.heads * w0.Dv:])
             og = o.normal_()
         else:
             args = (H * m.vdim, False, 1.0, out)
             og = o.normal_().view(n, 1, -1)
-        t.add(f"{kind}: head norm and gate", [lambda i=i: ops.group_norm_gate(og, eng.layers[i].head_norm, gt, cfg.norm_eps, *args) for i in li],
-              n * H * w0.dv * 8, 0)
+        if not (kind == "parallel" and decode):
+            t.add(f"{kind}: head norm and gate", [lambda i=i: ops.group_norm_gate(og, eng.layers[i].head_norm, gt, cfg.norm_eps, *args) for i in li],
+                  n * H * w0.dv * 8, 0)
         t.add(f"{kind} output projection", [lambda i=i: ops.dense_gemm(out, eng.layers[i].wo, out=y, status=eng.status, workspace=eng.gemm_ws)
                                             for i in li], W * w0.out_ld * 2 + n * (W + w0.out_ld) * 2, 2 * n * W * w0.out_ld)
     moe = [i for i, s in enumerate(cfg.layer_list) if s.mlp is not None]

@@ -490,6 +490,27 @@ int b200_state_scan(const void* act, int ld, int q_off, int k_off, int v_off, co
                     float* o, void* status_word, int num_rows, int chunk, int heads, int qk_heads, int dim, int vdim,
                     int num_slots, float q_scale, int dtype, void* stream);
 
+/* The same for a chunk of one sequence (bf16 activations, dim and vdim multiples of 16, dim at most 128), in blocks of 64 tokens
+ * on the tensor cores, every fp32 operand as the sum of two bf16 numbers.  Decays at least 0. */
+size_t b200_state_chunk_workspace_bytes(int num_rows, int heads, int delta);
+int b200_state_chunk(const void* act, int ld, int q_off, int k_off, int v_off, const float* ba, const float* a_log,
+                     const float* dt_bias, const float* decay, float* state, const int32_t* slots, const int32_t* positions,
+                     float* o, void* workspace, size_t workspace_bytes, void* status_word, int num_rows, int heads, int qk_heads,
+                     int dim, int vdim, int num_slots, float q_scale, void* stream);
+
+/*
+ * One decode step: every row is a sequence of its own.  decay given: act is activated, o [num_rows, heads, vdim] gets the
+ * result.  Otherwise act holds the inputs of the convolution (conv_w, taps and ring as in b200_conv_silu over the rows' ld
+ * channels), and out[m, h] = o / sqrt(mean square over norm_size + eps) * norm * gate[m, h] * out_scale, rows out_ld apart.
+ * _supported: dim and vdim multiples of 4 that fit a CTA's registers.
+ */
+int b200_state_step_supported(int dim, int vdim);
+int b200_state_step(const void* act, int ld, int q_off, int k_off, int v_off, const void* conv_w, void* ring, int taps,
+                    const float* ba, const float* a_log, const float* dt_bias, const float* decay, float* state,
+                    const int32_t* slots, const int32_t* positions, float* o, const void* gate, const float* norm, void* out,
+                    int out_ld, int norm_size, float eps, float out_scale, void* status_word, int num_rows, int heads,
+                    int qk_heads, int dim, int vdim, int num_slots, float q_scale, int dtype, void* stream);
+
 /* out[m, g] = o[m, g] / sqrt(mean square over `size` + eps) * weight * gate[m, g] * scale; o [num_rows, groups, group_ld] fp32,
  * zero from column `size` of a group on; weight [group_ld] (shared_weight) or [groups, group_ld] fp32; gate
  * [num_rows, groups, group_ld]; out rows out_ld apart.  group_ld and out_ld multiples of 4. */

@@ -61,6 +61,11 @@ SIGNATURES = {
     "b200_conv_silu": (c_int, [c_void_p] * 2 + [c_int] + [c_void_p] * 3 + [c_int] * 4 + [c_void_p] * 2 + [c_int, c_void_p]),
     "b200_group_norm_gate": (c_int, [c_void_p] * 3 + [c_float] + [c_int] * 5 + [c_float, c_void_p] + [c_int] * 2 + [c_void_p]),
     "b200_state_scan": (c_int, [c_void_p] + [c_int] * 4 + [c_void_p] * 9 + [c_int] * 7 + [c_float, c_int, c_void_p]),
+    "b200_state_chunk_workspace_bytes": (c_size_t, [c_int] * 3),
+    "b200_state_chunk": (c_int, [c_void_p] + [c_int] * 4 + [c_void_p] * 9 + [c_size_t, c_void_p] + [c_int] * 6 + [c_float, c_void_p]),
+    "b200_state_step_supported": (c_int, [c_int] * 2),
+    "b200_state_step": (c_int, [c_void_p] + [c_int] * 4 + [c_void_p] * 2 + [c_int] + [c_void_p] * 11 + [c_int] * 2 + [c_float] * 2
+                        + [c_void_p] + [c_int] * 6 + [c_float, c_int, c_void_p]),
     "b200_mixed_attn_workspace_bytes": (c_size_t, [c_int] * 8),
     "b200_mixed_attn": (c_int, [c_void_p] * 4 + [c_int] + [c_void_p] * 2 + [c_int] * 2
                         + [c_void_p, c_int, c_float, c_void_p, c_size_t, c_void_p] + [c_int] * 10 + [c_void_p]),

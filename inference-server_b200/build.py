@@ -18,14 +18,14 @@ INCLUDE = os.path.join(ROOT_DIR, "include")
 LIB_PATH = os.path.join(PKG_DIR, "libb200decode.so")
 SOURCES = ["host.cu", "paged_attn.cu", "paged_prefill.cu", "paged_prefill_tc.cu", "decode_glue.cu", "dense_gemm.cu", "router_fused.cu", "moe_route.cu", "moe_gemm.cu",
            "moe_layer.cu", "ep_p2p.cu", "latent_attn.cu", "layer_glue.cu", "gated_glue.cu", "state_scan.cu", "mixed_attn.cu",
-           "mixed_prefill_tc.cu"]
+           "mixed_prefill_tc.cu", "state_step.cu", "state_chunk.cu"]
 # Parts of the library that are enough for some model families, each with a library file of its own, for a process that
 # has to build before it can run and needs no more than that.
 SUBSETS = {
     "layered": ["host.cu", "paged_attn.cu", "paged_prefill.cu", "paged_prefill_tc.cu", "dense_gemm.cu", "latent_attn.cu",
                 "layer_glue.cu"],
     "gated": ["host.cu", "dense_gemm.cu", "moe_route.cu", "layer_glue.cu", "gated_glue.cu", "state_scan.cu", "mixed_attn.cu",
-              "mixed_prefill_tc.cu"],
+              "mixed_prefill_tc.cu", "state_step.cu", "state_chunk.cu"],
 }
 HEADERS = ["common.cuh", "glue.cuh", "host.h"]
 NVCC_FLAGS = [

@@ -26,6 +26,8 @@ import torch
 from . import ops
 
 PAGE = 16
+# Prompt chunks of fewer tokens than this run a recurrence token by token; longer ones in blocks of 64 on the tensor cores.
+BLOCKED_ROWS = 32
 SILU_GLU = dict(limit=float("inf"), alpha=1.0, shift=0.0)  # the clamped gated unit as silu(g) * u
 
 
@@ -222,7 +224,7 @@ class GatedWeights:
             wo = torch.cat([_heads(get("mix.left.o").t(), a.heads, a.vdim, self.Dv),
                             _heads(get("mix.right.o").t(), r.heads, r.vdim, self.dv)])
             self.o_bias = vec(get("mix.left.o.b").float() * m.left_scale, W)
-            self.heads, self.qk_heads = r.heads, r.kv_heads
+            self.heads, self.qk_heads, self.blocked = r.heads, r.kv_heads, True
         else:
             self.d, self.dv = _up(m.dim, 16), _up(m.vdim, 16)
             for name, size, to in (("q", m.dim, self.d), ("k", m.dim, self.d), ("v", m.vdim, self.dv), ("g", m.vdim, self.dv)):
@@ -233,6 +235,7 @@ class GatedWeights:
             self.head_norm = vec(_heads(get("mix.norm"), m.heads, m.vdim, self.dv))
             wo = _heads(get("mix.o").t(), m.heads, m.vdim, self.dv)
             self.heads = self.qk_heads = m.heads
+            self.blocked = min(m.decay) >= 0.0  # products of decays are summed logarithms there
         self.wproj, self.proj_bias = proj.finish(dtype)
         self.out_cols, self.out_ld = wo.shape[0], _up(wo.shape[0], 64)
         self.wo = _pad(_pad(wo, 0, self.out_ld), 1, W).t().to(dtype).contiguous()
@@ -254,9 +257,9 @@ class GatedWeights:
 
 
 def launches(spec) -> int:
-    """Kernels of one layer in a decode step: norm, projection, output projection; mixed queries, attention, convolution,
-    recurrence, head norm; norm, projection, routing, ranks, scatter, two products of the experts."""
-    return 3 + (5 if isinstance(spec.mixer, ParallelSpec) else 2) + (7 if spec.mlp is not None else 0)
+    """Kernels of one layer in a decode step: norm, projection, output projection; mixed queries, attention, its fold, gated delta
+    rule, or recurrence and head norm; norm, projection, routing, ranks, scatter, two products of the experts."""
+    return 3 + (4 if isinstance(spec.mixer, ParallelSpec) else 2) + (7 if spec.mlp is not None else 0)
 
 
 # --------------------------------------------------------------------- passes
@@ -310,13 +313,32 @@ class GatedMechanisms:
     def _act(self, *shape, dtype=None):
         return torch.empty(*shape, dtype=dtype or self.dtype, device=self.device)
 
-    def _recurrence(self, act, li: int, w: GatedWeights, rows: Rows, ba=None, q_scale: float = 1.0):
-        """[rows, heads, dv] fp32 from activated q, k, v."""
-        o = self._act(act.shape[0], w.heads, w.dv, dtype=torch.float32)
+    def _recurrence(self, act, li: int, w: GatedWeights, rows: Rows, lo: int, hi: int, chunk: bool, o, ba=None, q_scale: float = 1.0):
+        """Rows [lo, hi) of o [rows, heads, dv] fp32 from activated q, k, v: blocks of tokens on the tensor cores for a long enough
+        chunk, token by token otherwise."""
+        args = (act[lo:hi], w, self.states[li], rows.slots[lo:hi], rows.pos[lo:hi], o[lo:hi])
+        more = dict(ba=None if ba is None else ba[lo:hi], q_scale=q_scale)
+        if chunk and hi - lo >= BLOCKED_ROWS and w.blocked and ops.state_chunk_supported(w.d, w.dv, self.dtype):
+            ops.state_chunk(*args, self.status, **more)
+        elif not chunk and ba is None and ops.state_step_supported(w.d, w.dv):
+            ops.state_step(*args, self.status)
+        else:
+            ops.state_scan(*args, chunk, self.status, **more)
+
+    def _delta(self, pre, ba, g, li: int, r: DeltaSpec, w: GatedWeights, rows: Rows, scale: float, out) -> None:
+        """Gated delta rule with its convolution in front and its head norm and gate behind: one kernel for decode rows."""
+        q_scale, eps = r.dim ** -0.5, self.cfg.norm_eps
         for lo, hi, chunk in rows.parts():
-            ops.state_scan(act[lo:hi], w, self.states[li], rows.slots[lo:hi], rows.pos[lo:hi], o[lo:hi], chunk, self.status,
-                           ba=None if ba is None else ba[lo:hi], q_scale=q_scale)
-        return o
+            at = (rows.slots[lo:hi], rows.pos[lo:hi])
+            if not chunk and ops.state_step_supported(w.d, w.dv):
+                ops.state_step(pre[lo:hi], w, self.states[li], *at, None, self.status, ba=ba[lo:hi], q_scale=q_scale, ring=self.rings[li],
+                               gate=g[lo:hi], eps=eps, size=r.vdim, scale=scale, out=out[lo:hi])
+                continue
+            act = ops.conv_silu(pre[lo:hi], w.conv, self.rings[li], *at, chunk, self.status)
+            o = self._act(hi - lo, w.heads, w.dv, dtype=torch.float32)
+            part = Rows(rows.pos[lo:hi], rows.table[lo:hi], rows.slots[lo:hi], rows.first, hi - lo if chunk else 0)
+            self._recurrence(act, li, w, part, 0, hi - lo, chunk, o, ba[lo:hi], q_scale)
+            ops.group_norm_gate(o, w.head_norm, g[lo:hi], eps, r.vdim, True, scale, out[lo:hi])
 
     def _parallel(self, h, li: int, m: ParallelSpec, w: GatedWeights, rows: Rows) -> Pending:
         a, r, R = m.left, m.right, h.shape[0]
@@ -332,11 +354,7 @@ class GatedMechanisms:
         if w.out_ld != w.out_cols:
             out[:, w.out_cols:].zero_()
         self._window_attention(q, kp, vp, a, w, rows, m.left_scale, out)
-        act = torch.empty_like(pre)
-        for lo, hi, chunk in rows.parts():
-            ops.conv_silu(pre[lo:hi], w.conv, self.rings[li], rows.slots[lo:hi], rows.pos[lo:hi], chunk, self.status, act[lo:hi])
-        o = self._recurrence(act, li, w, rows, ba, r.dim ** -0.5)
-        ops.group_norm_gate(o, w.head_norm, g, self.cfg.norm_eps, r.vdim, True, m.right_scale, out[:, a.heads * w.Dv:])
+        self._delta(pre, ba, g, li, r, w, rows, m.right_scale, out[:, a.heads * w.Dv:])
         return Pending(gate, dense=self._linear(out, w.wo), bias=w.o_bias)
 
     def _window_attention(self, q, kp, vp, a: WindowAttentionSpec, w: GatedWeights, rows: Rows, scale: float, out) -> None:
@@ -367,7 +385,9 @@ class GatedMechanisms:
         act, g, gate = self._act(R, w.channels), self._act(R, m.heads * w.dv), self._act(R, self.W)
         ops.proj_split(h, w.wproj, [(ops.SEG_ROWS, act, ops.ACT_SILU), (ops.SEG_ROWS, g, ops.ACT_SIGMOID),
                                     (ops.SEG_ROWS, gate, ops.ACT_SIGMOID)], status=self.status, col_bias=w.proj_bias)
-        o = self._recurrence(act, li, w, rows)
+        o = self._act(R, m.heads, w.dv, dtype=torch.float32)
+        for lo, hi, chunk in rows.parts():
+            self._recurrence(act, li, w, rows, lo, hi, chunk, o)
         out = self._act(R, w.out_ld)
         if w.out_ld != w.out_cols:
             out[:, w.out_cols:].zero_()

@@ -859,6 +859,71 @@ def state_scan(act, w, state, slots, positions, o, chunk: bool, status=None, ba=
     check(rc, "b200_state_scan")
 
 
+def _state_args(act, w, state, slots, positions, ba):
+    _need(act, "act")
+    _need(state, "state", torch.float32)
+    _need(slots, "slots", torch.int32)
+    _need(positions, "positions", torch.int32)
+    M, ld = act.shape
+    n, _, H, d, dv = state.shape
+    G = w.qk_heads
+    if ld != 2 * G * d + H * dv or slots.shape[0] != M or positions.shape[0] != M:
+        raise ValueError("rows do not match the state")
+    if ba is not None:
+        _need(ba, "ba", torch.float32)
+        if ba.shape != (M, 2 * H):
+            raise ValueError("ba does not match the rows")
+    return M, ld, n, H, G, d, dv
+
+
+def state_chunk_supported(dim: int, vdim: int, dtype) -> bool:
+    return dtype == torch.bfloat16 and dim <= 128 and dim % 16 == 0 and vdim % 16 == 0
+
+
+def state_chunk(act, w, state, slots, positions, o, status=None, ba=None, q_scale: float = 1.0):
+    """`state_scan` for a chunk of one sequence in blocks of 64 tokens on the tensor cores."""
+    M, ld, n, H, G, d, dv = _state_args(act, w, state, slots, positions, ba)
+    _need(act, "act", torch.bfloat16)
+    _need(o, "o", torch.float32)
+    if o.shape != (M, H, dv):
+        raise ValueError("output does not match the state")
+    lib, delta = _lib.load(), ba is not None
+    ws = torch.empty(lib.b200_state_chunk_workspace_bytes(M, H, int(delta)), dtype=torch.uint8, device=act.device)
+    rc = lib.b200_state_chunk(_ptr(act), ld, 0, G * d, 2 * G * d, _ptr(ba), _ptr(w.a_log) if delta else None,
+                              _ptr(w.dt_bias) if delta else None, None if delta else _ptr(w.decay), _ptr(state), _ptr(slots),
+                              _ptr(positions), _ptr(o), _ptr(ws), ws.numel(), _ptr(status), M, H, G, d, dv, n, float(q_scale), _stream())
+    check(rc, "b200_state_chunk")
+
+
+def state_step_supported(dim: int, vdim: int) -> bool:
+    return bool(_lib.load().b200_state_step_supported(int(dim), int(vdim)))
+
+
+def state_step(act, w, state, slots, positions, o, status=None, ba=None, q_scale: float = 1.0, ring=None, gate=None, eps: float = 0.0,
+               size: int = 0, scale: float = 1.0, out=None):
+    """One decode step of the recurrence per row.  Without `ba`: `act` is activated, o [M, H, dv] fp32 gets the result.  With it
+    (gated delta rule): `act` is the input of the convolution w.conv over `ring`, and the result, normed per head over its first
+    `size` columns, times w.head_norm, gate and scale, goes to rows of `out`."""
+    M, ld, n, H, G, d, dv = _state_args(act, w, state, slots, positions, ba)
+    delta = ba is not None
+    if delta:
+        _need(w.conv, "conv", act.dtype)
+        _need(gate, "gate", act.dtype)
+        taps = w.conv.shape[0]
+        if w.conv.shape[1] != ld or gate.numel() != M * H * dv or out.dtype != act.dtype or out.shape[0] != M or (
+                taps > 1 and tuple(ring.shape) != (n, taps, ld)):
+            raise ValueError("convolution, ring, gate or out do not match the rows")
+    else:
+        _need(o, "o", torch.float32)
+        taps = 1
+    rc = _lib.load().b200_state_step(
+        _ptr(act), ld, 0, G * d, 2 * G * d, _ptr(w.conv) if delta else None, _ptr(ring), taps, _ptr(ba), _ptr(w.a_log) if delta else None,
+        _ptr(w.dt_bias) if delta else None, None if delta else _ptr(w.decay), _ptr(state), _ptr(slots), _ptr(positions), _ptr(o),
+        _ptr(gate), _ptr(w.head_norm) if delta else None, out.data_ptr() if delta else None, out.stride(0) if delta else 0, int(size),
+        float(eps), float(scale), _ptr(status), M, H, G, d, dv, n, float(q_scale), DTYPE_CODE[act.dtype], _stream())
+    check(rc, "b200_state_step")
+
+
 def group_norm_gate(o, weight, gate, eps: float, size: int, shared_weight: bool, scale: float, out):
     """RMS norm of fp32 groups [M, G, ld] over their first `size` columns, times weight, gate and scale, into rows of `out`."""
     _need(o, "o", torch.float32)

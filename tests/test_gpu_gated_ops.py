@@ -222,34 +222,118 @@ def recurrence_case(T, H, G, d, dv, delta, dtype, seed):
     return act, ba, w, want
 
 
+def run_recurrence(ops, A, BA, w, state, at, n, d, dv, H, delta, how, st):
+    """n tokens of the sequence in slot 1 from position `at` on, by the kernel `how`."""
+    o = torch.empty(n, H, dv, device=DEV)
+    slots, pos = torch.full((n,), 1, dtype=torch.int32, device=DEV), torch.arange(at, at + n, dtype=torch.int32, device=DEV)
+    ba, q_scale = None if BA is None else BA[at:at + n], d ** -0.5 if delta else 1.0
+    if how == "chunk":
+        ops.state_chunk(A[at:at + n], w, state, slots, pos, o, st, ba=ba, q_scale=q_scale)
+    elif how == "step":
+        ops.state_step(A[at:at + n], w, state, slots, pos, o, st)
+    else:
+        ops.state_scan(A[at:at + n], w, state, slots, pos, o, n > 1, st, ba=ba, q_scale=q_scale)
+    return o.cpu().double()
+
+
 @pytest.mark.parametrize("dtype", [BF, F32])
 @pytest.mark.parametrize("delta", [True, False])
 @pytest.mark.parametrize("H,G,d,dv", [(4, 4, 64, 64), (4, 2, 128, 128), (3, 3, 16, 48), (6, 2, 48, 32), (2, 1, 32, 144), (2, 2, 208, 64),
-                                      (1, 1, 304, 16), (2, 2, 64, 256)])
+                                      (1, 1, 304, 16), (2, 2, 64, 256), (2, 2, 112, 16)])
 def test_recurrence_in_portions_and_decoded(ops, H, G, d, dv, delta, dtype):
-    """Any cut of a sequence gives the whole sequence's recurrence: portions from two tokens on, over and at the borders of
-    the kernels' inner blocks, decode rows in between (each run twice); other slots keep their states."""
+    """Any cut of a sequence gives the whole sequence's recurrence, by every kernel that takes the portion: portions from two
+    tokens on, over and at the borders of the kernels' inner blocks, decode rows in between (each run twice); other slots keep
+    their states."""
     if not delta and H != G:
         pytest.skip("one query/key head per head")
     T = 200
     act, ba, w, want = recurrence_case(T, H, G, d, dv, delta, dtype, seed=H + d)
     A, BA = act.to(DEV), None if ba is None else ba.to(DEV)
     scale = want.abs().amax(0, keepdim=True).clamp_min(1e-6)
-    for cuts in ([T], [2, 3, 1, 15, 17, 2, 64, 1, 1, 94], [64, 64, 72], [1] * 20 + [130, 50], [33, 65, 2, 100]):
-        state = torch.full((3, 2, H, d, dv), 9.0, device=DEV)
-        st, got, at = status(), [], 0
-        for n in cuts:
-            for _ in range(2 if n == 1 else 1):
-                o = torch.empty(n, H, dv, device=DEV)
-                ops.state_scan(A[at:at + n], w, state, torch.full((n,), 1, dtype=torch.int32, device=DEV),
-                               torch.arange(at, at + n, dtype=torch.int32, device=DEV), o, n > 1, st,
-                               ba=None if BA is None else BA[at:at + n], q_scale=d ** -0.5 if delta else 1.0)
-            got.append(o.cpu().double())
-            at += n
+    blocked = ops.state_chunk_supported(d, dv, dtype)
+    for cuts in ([T], [2, 3, 1, 15, 17, 2, 64, 1, 1, 94], [64, 64, 72], [1] * 20 + [130, 50], [33, 65, 2, 100], [63, 1, 128, 8]):
+        for how in ("scan", "chunk") if blocked else ("scan",):
+            state = torch.full((3, 2, H, d, dv), 9.0, device=DEV)
+            st, got, at = status(), [], 0
+            for n in cuts:
+                kernel = how if n > 1 else "step" if not delta and how == "chunk" and ops.state_step_supported(d, dv) else "scan"
+                for _ in range(2 if n == 1 else 1):
+                    o = run_recurrence(ops, A, BA, w, state, at, n, d, dv, H, delta, kernel, st)
+                got.append(o)
+                at += n
+            ops.read_status(st, "recurrence")
+            err = float(((torch.cat(got) - want) / scale).abs().max())
+            assert err < (2e-4 if dtype == BF else 2e-5), (how, cuts, err)
+            assert bool((state[[0, 2]] == 9.0).all())
+
+
+def test_recurrence_with_extreme_decays(ops):
+    """Decays of 0 and 1 and step sizes near 0 and 1 in the blocked kernel; keys that repeat (the inverse is far from 1)."""
+    H, d, dv, T = 4, 64, 32, 150
+    for delta in (True, False):
+        act, ba, w, want = recurrence_case(T, H, H, d, dv, delta, BF, seed=9)
+        if delta:
+            act[20:140, H * d:2 * H * d] = act[20:21, H * d:2 * H * d]
+            ba[:, :H] = torch.tensor([8.0, 8.0, -8.0, 0.0])
+            ba[:, H:] = torch.tensor([-20.0, 40.0, -20.0, 1.0])
+            ba[100] = -ba[100]
+            a_log, dt = w.a_log.cpu().double(), w.dt_bias.cpu().double()
+            q, k, v = (
+                act[:, :H * d].double().view(T, H, d), act[:, H * d:2 * H * d].double().view(T, H, d), act[:, 2 * H * d:].double().view(T, H, dv))
+            g = torch.exp(-torch.exp(a_log) * torch.nn.functional.softplus(ba[:, H:].double() + dt))
+            want = torch.stack([ref.delta_rule(ref.unit(q[:, h]) * d ** -0.5, ref.unit(k[:, h]), v[:, h], torch.sigmoid(ba[:, h].double()), g[:, h])
+                                for h in range(H)], 1)
+        else:
+            w.decay = torch.tensor([0.0, 1.0, 1e-6, 0.5], device=DEV)
+            q, k, v = act[:, :H * d].double().view(T, H, d), act[:, H * d:2 * H * d].double().view(T, H, d), act[:, 2 * H * d:].double().view(T, H, dv)
+            want = torch.stack([ref.decay_attention(q[:, h], k[:, h], v[:, h], float(w.decay[h])) for h in range(H)], 1)
+        state, st = torch.full((3, 2, H, d, dv), 9.0, device=DEV), status()
+        got = run_recurrence(ops, act.to(DEV), None if ba is None else ba.to(DEV), w, state, 0, T, d, dv, H, delta, "chunk", st)
+        assert float(((got - want) / want.abs().amax(0, keepdim=True)).abs().max()) < 3e-4, delta
         ops.read_status(st, "recurrence")
-        err = float(((torch.cat(got) - want) / scale).abs().max())
-        assert err < (2e-3 if dtype == BF else 2e-5), (cuts, err)
-        assert bool((state[[0, 2]] == 9.0).all())
+
+
+@pytest.mark.parametrize("dtype", [BF, F32])
+@pytest.mark.parametrize("H,G,d,dv,taps,size", [(4, 4, 64, 64, 4, 64), (6, 2, 48, 32, 1, 20), (4, 1, 128, 128, 3, 128), (2, 2, 16, 272, 7, 260)])
+def test_decode_step_of_the_gated_delta_rule(ops, H, G, d, dv, taps, size, dtype):
+    """The one-kernel decode step (convolution, recurrence, head norm, gate) against the same in separate kernels, on top of a
+    prompt chunk and of other decode steps; every step run twice."""
+    T, C = 40, 2 * G * d + H * dv
+    pre, conv = randn(T, C, seed=1, dtype=dtype), randn(taps, C, seed=2, dtype=dtype)
+    pre.view(T, C)[:, 2 * G * d:].view(T, H, dv)[..., size:] = 0
+    _, ba, w, _ = recurrence_case(T, H, G, d, dv, True, dtype, seed=3)
+    w.conv, w.head_norm = conv.to(DEV), (1 + 0.3 * randn(dv, seed=4)).to(DEV)
+    g = randn(T, H * dv, seed=5, dtype=dtype).to(DEV)
+    P, BA, q_scale = pre.to(DEV), ba.to(DEV), d ** -0.5
+    rings = [torch.full((3, taps, C), 7.0, dtype=dtype, device=DEV) if taps > 1 else None for _ in range(2)]
+    states, st = [torch.full((3, 2, H, d, dv), 9.0, device=DEV) for _ in range(2)], status()
+    for at, n in [(0, 11)] + [(i, 1) for i in range(11, T)]:
+        slots, pos = torch.full((n,), 2, dtype=torch.int32, device=DEV), torch.arange(at, at + n, dtype=torch.int32, device=DEV)
+        outs = []
+        for which in range(2 if n == 1 else 1):
+            out = torch.full((n, H * dv + 16), 5.0, dtype=dtype, device=DEV)
+            for _ in range(2):
+                if which == 1:
+                    ops.state_step(P[at:at + n], w, states[1], slots, pos, None, st, ba=BA[at:at + n], q_scale=q_scale, ring=rings[1],
+                                   gate=g[at:at + n], eps=1e-5, size=size, scale=1.4, out=out)
+                    continue
+                a = ops.conv_silu(P[at:at + n], w.conv, rings[0], slots, pos, n > 1, st)
+                o = torch.empty(n, H, dv, device=DEV)
+                ops.state_scan(a, w, states[0], slots, pos, o, n > 1, st, ba=BA[at:at + n], q_scale=q_scale)
+                ops.group_norm_gate(o, w.head_norm, g[at:at + n], 1e-5, size, True, 1.4, out)
+                if n > 1:
+                    break
+            outs.append(out)
+        if n > 1:  # the prompt chunk goes to both
+            states[1].copy_(states[0])
+            if taps > 1:
+                rings[1].copy_(rings[0])
+        else:
+            assert rel_err(outs[1][:, : H * dv], outs[0][:, : H * dv]) < (1e-2 if dtype == BF else 2e-5) and bool((outs[1][:, H * dv:] == 5.0).all())
+            assert rel_err(states[1], states[0]) < 1e-5
+            if taps > 1:
+                assert torch.equal(rings[1], rings[0])
+    ops.read_status(st, "delta step")
 
 
 def test_recurrence_rows_are_independent_sequences(ops):
