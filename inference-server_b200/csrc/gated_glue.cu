@@ -218,7 +218,8 @@ mix_heads_kernel(const float* __restrict__ q, const float* __restrict__ mix, T* 
 // chunk: the rows are consecutive positions of one sequence, positions[0] on, with slot slots[0]; a CTA takes
 // `rows_per` of them, the first CTA alone reads the ring (rows_per >= taps - 1) and, each column by the thread that has
 // read it, writes it.  Otherwise every row is a sequence of its own.
-template <typename T>
+// TAPS > 0: that many, weights and the window's rows in registers; 0: `taps`, every row read again for every tap.
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(64)
 conv_silu_kernel(const T* __restrict__ in, const T* __restrict__ w, int taps, T* __restrict__ ring,
                  const int* __restrict__ slots, const int* __restrict__ positions, int num_rows, int chunk, int rows_per,
@@ -237,6 +238,41 @@ conv_silu_kernel(const T* __restrict__ in, const T* __restrict__ w, int taps, T*
     return;
   }
   T* hist = taps > 1 ? ring + static_cast<size_t>(slot) * taps * C + col : nullptr;
+  if (TAPS > 1) {
+    float w_r[TAPS > 1 ? TAPS : 1][8];
+    Raw8<T> win[TAPS > 1 ? TAPS - 1 : 1];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load8<T>(w + static_cast<size_t>(j) * C + col, w_r[j]);
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j) {
+      const int r = lo - (TAPS - 1 - j), pos = first + (r - base);
+      if (pos < 0) win[j].zero();
+      else if (r >= base) win[j].load(in + static_cast<size_t>(r) * C + col);
+      else win[j].load(hist + static_cast<size_t>(pos % TAPS) * C);
+    }
+#pragma unroll 4
+    for (int r = lo; r < hi; ++r) {
+      Raw8<T> x;
+      x.load(in + static_cast<size_t>(r) * C + col);
+      float acc[8], f[8];
+      x.get(f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j) {
+        float a[8];
+        win[j].get(a);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] = fmaf(w_r[j][e], a[e], acc[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[e] = silu_of(fmaf(w_r[TAPS > 0 ? TAPS - 1 : 0][e], f[e], acc[e]));
+#pragma unroll
+      for (int j = 0; j + 2 < TAPS; ++j) win[j] = win[j + 1];
+      win[TAPS > 1 ? TAPS - 2 : 0] = x;
+      store8<T>(out + static_cast<size_t>(r) * C + col, acc);
+    }
+  } else
 #pragma unroll 2
   for (int r = lo; r < hi; ++r) {
     const int pos = first + (r - base);
@@ -385,15 +421,19 @@ extern "C" int b200_conv_silu(const void* in, const void* conv_w, int taps, void
   const int rows_per = chunk ? (taps - 1 > 16 ? taps - 1 : 16) : 1;
   const dim3 grid((num_rows + rows_per - 1) / rows_per, (channels / 8 + 63) / 64);
   int* err = static_cast<int*>(status_word);
-  if (dtype == 0)
-    B200_CUDA(launch_overlapped(conv_silu_kernel<__nv_bfloat16>, grid, dim3(64), 0, as_stream(stream),
-                                static_cast<const __nv_bfloat16*>(in), static_cast<const __nv_bfloat16*>(conv_w), taps,
-                                static_cast<__nv_bfloat16*>(ring), slots, positions, num_rows, chunk, rows_per, channels,
-                                num_slots, static_cast<__nv_bfloat16*>(out), err));
-  else
-    B200_CUDA(launch_overlapped(conv_silu_kernel<float>, grid, dim3(64), 0, as_stream(stream), static_cast<const float*>(in),
-                                static_cast<const float*>(conv_w), taps, static_cast<float*>(ring), slots, positions,
-                                num_rows, chunk, rows_per, channels, num_slots, static_cast<float*>(out), err));
+#define B200_CONV(T, TAPS)                                                                                                     \
+  B200_CUDA(launch_overlapped(conv_silu_kernel<T, TAPS>, grid, dim3(64), 0, as_stream(stream), static_cast<const T*>(in),      \
+                              static_cast<const T*>(conv_w), taps, static_cast<T*>(ring), slots, positions, num_rows, chunk,   \
+                              rows_per, channels, num_slots, static_cast<T*>(out), err))
+  if (dtype == 0) {
+    if (taps == 2) B200_CONV(__nv_bfloat16, 2);
+    else if (taps == 3) B200_CONV(__nv_bfloat16, 3);
+    else if (taps == 4) B200_CONV(__nv_bfloat16, 4);
+    else B200_CONV(__nv_bfloat16, 0);
+  } else {
+    B200_CONV(float, 0);
+  }
+#undef B200_CONV
   return 0;
 }
 

@@ -6,9 +6,8 @@
 //     P[t, s] = iq_t ik_s G_t / G_s (q_t . k_s),  s <= t            A[t, s] = beta_t ik_t ik_s G_t / G_s (k_t . k_s),  s < t
 //     U = (I + A)^-1 diag(beta) (V - diag(G ik) K S)    (gated delta rule; otherwise U = V)
 //     O = diag(G iq) Q S + P U                           S' = G_64 S + K^T diag(G_64 / G ik) U
-// The prepare kernel makes P and T = (I + A)^-1 for all blocks and heads side by side (the inverse by forward substitution, a
-// column per thread); the block kernel walks the blocks in order, a CTA per head and 16 columns of the state, which stay in
-// registers as accumulators.
+// The prepare kernel makes P and T = (I + A)^-1 for all blocks and heads side by side; the block kernel walks the blocks in
+// order, a CTA per head and 16 columns of the state, which stay in registers as accumulators.
 //
 // fp32 where the recurrence is: q, k and v enter as the bf16 numbers they are, all factors are applied to fp32 values, and every
 // other operand of a product - S, U, P, T and the residuals - is split into the bf16 number next to it and the bf16 number next
@@ -58,12 +57,68 @@ __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool h
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(have ? 16 : 0) : "memory");
 }
 
-// A 64-row tile of q or k into shared memory, rows of dim + 8, zero rows past the last token.
-__device__ __forceinline__ void load_tile(uint32_t dst, const __nv_bfloat16* src, int ld, int cnt, int dim) {
-  const int pieces = dim / 8;
-  for (int i = threadIdx.x; i < kBlk * pieces; i += kChunkThreads) {
-    const int r = i / pieces, c = i - r * pieces;
-    cp_async16(dst + (r * (dim + 8) + c * 8) * 2, src + static_cast<size_t>(r < cnt ? r : 0) * ld + c * 8, r < cnt);
+// Room for the two tiles of the prepare kernel.
+__host__ __device__ __forceinline__ int prep_k_bytes(int dim) {
+  const int t = kBlk * (dim + 8) * 2;
+  return t > 32 * 68 * 4 ? t : 32 * 68 * 4;
+}
+__host__ __device__ __forceinline__ int prep_q_bytes(int dim, bool delta) {
+  const int t = kBlk * (dim + 8) * 2;
+  return !delta || t > kBlk * 68 * 4 ? t : kBlk * 68 * 4;
+}
+
+// 64-row tiles of k and q into shared memory (k, then q `tile_bytes` further), rows of dim + 8, zero rows past the last token.  A
+// thread keeps its 16-byte column; row and column are worked out once.
+struct TileLoader {
+  uint32_t dst;
+  int row, step, col, ld;
+  __device__ __forceinline__ TileLoader(int dim, int ld_, int t, int threads) {
+    const int pieces = dim / 8;
+    step = threads / pieces;
+    row = t / pieces;
+    col = (t - row * pieces) * 8;
+    if (row >= step) row = kBlk;  // left over
+    ld = ld_;
+    dst = (row * (dim + 8) + col) * 2;
+  }
+  __device__ __forceinline__ void load(uint32_t sm, int tile_bytes, const __nv_bfloat16* k, const __nv_bfloat16* q, int cnt, int ldk) const {
+    uint32_t d = sm + dst;
+    const __nv_bfloat16* kp = k + static_cast<size_t>(row) * ld + col;
+    const __nv_bfloat16* qp = q + static_cast<size_t>(row) * ld + col;
+    const size_t hop = static_cast<size_t>(step) * ld;
+    for (int r = row; r < kBlk; r += step) {
+      const bool have = r < cnt;
+      cp_async16(d, have ? kp : k, have);
+      cp_async16(d + tile_bytes, have ? qp : q, have);
+      d += step * ldk * 2;
+      kp += hop;
+      qp += hop;
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+};
+
+// C[r][c] (+)= sign * sum over k < n of a[r][k] b[k][c] for an n x n tile (n 16 or 32) of fp32 rows of 68; a thread takes four
+// columns of one row.  `threads` of them, numbered from 0.
+template <int N>
+__device__ __forceinline__ void small_product(const float* a, const float* b, float* c, float sign, int t, int threads) {
+  for (int i = t; i < N * N / 4; i += threads) {
+    const int r = i / (N / 4), c4 = (i - r * (N / 4)) * 4;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int k = 0; k < N; k += 4) {
+      const float4 x = *reinterpret_cast<const float4*>(a + r * 68 + k);
+      const float xs[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float4 y = *reinterpret_cast<const float4*>(b + (k + e) * 68 + c4);
+        acc.x = fmaf(xs[e], y.x, acc.x);
+        acc.y = fmaf(xs[e], y.y, acc.y);
+        acc.z = fmaf(xs[e], y.z, acc.z);
+        acc.w = fmaf(xs[e], y.w, acc.w);
+      }
+    }
+    *reinterpret_cast<float4*>(c + r * 68 + c4) = make_float4(sign * acc.x, sign * acc.y, sign * acc.z, sign * acc.w);
   }
 }
 
@@ -78,13 +133,16 @@ chunk_prepare_kernel(const ChunkParams p) {
   const int gq = lane >> 2, tq = lane & 3, lj = lane >> 3, lr = lane & 7;
   const int t0 = blk * kBlk, cnt = min(kBlk, p.rows - t0);
   const int qh = h / (p.heads / p.qk_heads), ldk = p.dim + 8;
-  const uint32_t k_sm = smem_u32(cp_sm), q_sm = k_sm + kBlk * ldk * 2;
-  float* A = reinterpret_cast<float*>(cp_sm + 2 * kBlk * ldk * 2);  // [64][68]
-  float* Ti = A + kBlk * 68;
-  load_tile(k_sm, p.act + static_cast<size_t>(t0) * p.ld + p.k_off + qh * p.dim, p.ld, cnt, p.dim);
-  load_tile(q_sm, p.act + static_cast<size_t>(t0) * p.ld + p.q_off + qh * p.dim, p.ld, cnt, p.dim);
-  asm volatile("cp.async.commit_group;" ::: "memory");
-  if (tid < kBlk) {  // decays, summed up in the log domain; a decay of 0 becomes e^-1000
+  // k (later a scratch tile), q (later the inverse), A: fp32 tiles have rows of 68
+  const int k_room = prep_k_bytes(p.dim), q_room = prep_q_bytes(p.dim, DELTA);
+  const uint32_t k_sm = smem_u32(cp_sm), q_sm = k_sm + k_room;
+  float* A = reinterpret_cast<float*>(cp_sm + k_room + q_room);
+  float* Ti = reinterpret_cast<float*>(cp_sm + k_room);
+  {
+    const __nv_bfloat16* src = p.act + static_cast<size_t>(t0) * p.ld + qh * p.dim;
+    TileLoader(p.dim, p.ld, tid, kChunkThreads).load(k_sm, q_sm - k_sm, src + p.k_off, src + p.q_off, cnt, ldk);
+  }
+  if (tid < kBlk) {  // decays, their logarithms (base 2) summed up; a decay of 0 becomes 2^-1000
     float lg = 0.f, beta = 0.f;
     if (tid < cnt) {
       if (DELTA) {
@@ -94,7 +152,7 @@ chunk_prepare_kernel(const ChunkParams p) {
       } else {
         lg = logf(p.decay[h]);
       }
-      lg = fmaxf(lg, -1000.f);
+      lg = fmaxf(lg * 1.4426950408889634f, -1000.f);
     }
 #pragma unroll
     for (int s = 1; s < 32; s <<= 1) {
@@ -108,20 +166,26 @@ chunk_prepare_kernel(const ChunkParams p) {
   __syncthreads();
   const float carry = L[31];
   if (DELTA) {
-    const __nv_bfloat16* kp = reinterpret_cast<const __nv_bfloat16*>(cp_sm);
-    for (int r = warp * 16; r < warp * 16 + 16; ++r) {
-      float kk = 0.f, qq = 0.f;
-      for (int c = lane; c < p.dim; c += 32) {
-        const float a = __bfloat162float(kp[r * ldk + c]), b = __bfloat162float(kp[(kBlk + r) * ldk + c]);
-        kk = fmaf(a, a, kk);
-        qq = fmaf(b, b, qq);
+    // two threads per row
+    const int r = tid >> 1;
+    const uint8_t* kr = cp_sm + r * ldk * 2;
+    const uint8_t* qr = cp_sm + k_room + r * ldk * 2;
+    float kk = 0.f, qq = 0.f;
+    for (int c = tid & 1; c < p.dim / 8; c += 2) {
+      float a[8], b[8];
+      load8<__nv_bfloat16>(reinterpret_cast<const __nv_bfloat16*>(kr) + c * 8, a);
+      load8<__nv_bfloat16>(reinterpret_cast<const __nv_bfloat16*>(qr) + c * 8, b);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        kk = fmaf(a[e], a[e], kk);
+        qq = fmaf(b[e], b[e], qq);
       }
-      kk = warp_sum(kk);
-      qq = warp_sum(qq);
-      if (lane == 0) {
-        ikv[r] = 1.f / sqrtf(kk + 1e-6f);
-        iqv[r] = p.q_scale / sqrtf(qq + 1e-6f);
-      }
+    }
+    kk += __shfl_xor_sync(0xffffffffu, kk, 1);
+    qq += __shfl_xor_sync(0xffffffffu, qq, 1);
+    if ((tid & 1) == 0) {
+      ikv[r] = 1.f / sqrtf(kk + 1e-6f);
+      iqv[r] = p.q_scale / sqrtf(qq + 1e-6f);
     }
   } else if (tid < kBlk) {
     ikv[tid] = 1.f;
@@ -135,13 +199,13 @@ chunk_prepare_kernel(const ChunkParams p) {
     float* f = p.factors + bh * kFactors * kBlk;
     const float last = L[kBlk - 1];
     if (tid < kBlk) {
-      const float G = expf(L[tid]);
+      const float G = exp2f(L[tid]);
       f[tid] = G * iqv[tid];
       f[kBlk + tid] = G * ikv[tid];
       f[2 * kBlk + tid] = bt[tid];
-      f[3 * kBlk + tid] = expf(last - L[tid]) * ikv[tid];
+      f[3 * kBlk + tid] = exp2f(last - L[tid]) * ikv[tid];
     }
-    if (tid == 0) p.factors[static_cast<size_t>(p.blocks) * p.heads * kFactors * kBlk + bh] = expf(last);
+    if (tid == 0) p.factors[static_cast<size_t>(p.blocks) * p.heads * kFactors * kBlk + bh] = exp2f(last);
   }
   // rows 16 warp.. of Q K^T and K K^T, columns up to the diagonal
   float sq[8][4], sk[8][4];
@@ -174,7 +238,7 @@ chunk_prepare_kernel(const ChunkParams p) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int t = e < 2 ? r0 : r1, s = n * 8 + 2 * tq + (e & 1);
-      const float w = s <= t ? expf(L[t] - L[s]) * ikv[s] : 0.f;
+      const float w = s <= t ? fast_ex2(L[t] - L[s]) * ikv[s] : 0.f;
       sq[n][e] *= w * iqv[t];
       if (DELTA) A[t * 68 + s] = s < t ? sk[n][e] * w * ikv[t] * bt[t] : 0.f;
     }
@@ -193,23 +257,42 @@ chunk_prepare_kernel(const ChunkParams p) {
   }
   if (!DELTA) return;
   __syncthreads();
-  if (tid < kBlk) {  // column tid of the inverse
-    float x[kBlk];
+  // (I + A)^-1: a warp inverts its 16 x 16 block on the diagonal, a column per lane; then twice [[X, 0], [-Y A' X, Y]] joins
+  // neighbours of 16 and of 32.  Zeros above the diagonal are written where the joins read them.
+  {
+    const float* Ad = A + warp * 16 * 68 + warp * 16;
+    float* Td = Ti + warp * 16 * 68 + warp * 16;
+    if (lane < 16) {
+      float x[16];
 #pragma unroll
-    for (int i = 0; i < kBlk; ++i) {
-      float a0 = i == tid ? 1.f : 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+      for (int i = 0; i < 16; ++i) {
+        float a0 = i == lane ? 1.f : 0.f, a1 = 0.f;
 #pragma unroll
-      for (int s = 0; s < i; s += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(A + i * 68 + s);
-        a0 = fmaf(-a.x, x[s], a0);
-        if (s + 1 < i) a1 = fmaf(-a.y, x[s + 1], a1);
-        if (s + 2 < i) a2 = fmaf(-a.z, x[s + 2], a2);
-        if (s + 3 < i) a3 = fmaf(-a.w, x[s + 3], a3);
+        for (int s = 0; s < i; s += 2) {
+          const float2 a = *reinterpret_cast<const float2*>(Ad + i * 68 + s);
+          a0 = fmaf(-a.x, x[s], a0);
+          if (s + 1 < i) a1 = fmaf(-a.y, x[s + 1], a1);
+        }
+        x[i] = a0 + a1;
+        Td[i * 68 + lane] = x[i];
       }
-      x[i] = (a0 + a1) + (a2 + a3);
-      Ti[i * 68 + tid] = x[i];
+    } else if (warp < 3) {  // the 16 columns to the right
+      for (int i = 0; i < 16; ++i) Td[i * 68 + lane] = 0.f;
     }
   }
+  float* tmp = reinterpret_cast<float*>(cp_sm);  // [32][68]
+  __syncthreads();
+  {
+    const int pair = warp >> 1, at = pair * 32, t = tid & 63;
+    float* tp = tmp + pair * 16 * 68;
+    small_product<16>(A + (at + 16) * 68 + at, Ti + at * 68 + at, tp, 1.f, t, 64);
+    __syncthreads();
+    small_product<16>(Ti + (at + 16) * 68 + at + 16, tp, Ti + (at + 16) * 68 + at, -1.f, t, 64);
+  }
+  __syncthreads();
+  small_product<32>(A + 32 * 68, Ti, tmp, 1.f, tid, kChunkThreads);
+  __syncthreads();
+  small_product<32>(Ti + 32 * 68 + 32, tmp, Ti + 32 * 68, -1.f, tid, kChunkThreads);
   __syncthreads();
   uint4* tf = p.t_frags + bh * kFragsPerBlock + warp * (4 * 2 * 32) + lane;
 #pragma unroll
@@ -245,9 +328,13 @@ __device__ __forceinline__ void get4(const uint4& v, uint32_t (&a)[4]) {
   a[3] = v.w;
 }
 
-// MT: 16-row tiles of the state per warp.
+constexpr int kScanThreads = 9 * 32;
+
+// Warps 0-3 carry the state (16 tokens each of K S, the residuals and U; MT 16-row tiles each of the state), warps 4-7 make the
+// output (16 tokens each) while the state moves on, warp 8 fetches the next block's k and q.  All meet at two or three barriers
+// per block: state and tiles in place, residuals in place, U in place.
 template <int MT, bool DELTA>
-__global__ void __launch_bounds__(kChunkThreads)
+__global__ void __launch_bounds__(kScanThreads)
 chunk_scan_kernel(const ChunkParams p) {
   extern __shared__ __align__(16) uint8_t cs_sm[];
   grid_dep_wait();
@@ -263,13 +350,104 @@ chunk_scan_kernel(const ChunkParams p) {
   const uint32_t kq_sm = smem_u32(cs_sm);               // [2 buffers][k, q][64][ldk]
   const uint32_t s_sm = kq_sm + 4 * tile_bytes;         // state: [high, low][dim][kSmLd]
   const uint32_t s_lo = p.dim * kSmLd * 2;
-  const uint32_t u_sm = s_sm + 2 * s_lo;                // residuals / U / scaled U: [3][high, low][64][kSmLd]
+  const uint32_t u_sm = s_sm + 2 * s_lo;                // residuals, U, scaled U: [3][high, low][64][kSmLd]
   constexpr uint32_t kURows = kBlk * kSmLd * 2;
-  uint8_t* u_ptr = cs_sm + 4 * tile_bytes + 2 * s_lo;
   uint8_t* s_ptr = cs_sm + 4 * tile_bytes;
+  uint8_t* u_ptr = s_ptr + 2 * s_lo;
+  const size_t fac_total = static_cast<size_t>(p.blocks) * p.heads * kFactors * kBlk;
+
+  if (warp == 8) {
+    // --------------------------------------------------------------- loader --
+    const TileLoader loader(p.dim, p.ld, lane, 32);
+    const __nv_bfloat16* src = p.act + qh * p.dim;
+    for (int blk = 0; blk <= p.blocks; ++blk) {
+      if (blk < p.blocks) {
+        const size_t at = static_cast<size_t>(blk) * kBlk * p.ld;
+        loader.load(kq_sm + (blk & 1) * 2 * tile_bytes, tile_bytes, src + p.k_off + at, src + p.q_off + at, min(kBlk, p.rows - blk * kBlk), ldk);
+      }
+      if (blk > 0) {
+        if (DELTA) __syncthreads();  // residuals in place
+        __syncthreads();             // U in place
+      }
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+      if (blk < p.blocks) __syncthreads();  // state and tiles in place; everybody is through with the other tiles
+    }
+    return;
+  }
+  const int w4 = warp & 3, r0 = w4 * 16 + gq, r1 = r0 + 8;
+  const uint32_t a_off = ((w4 * 16 + (lj & 1) * 8 + lr) * ldk + (lj >> 1) * 8) * 2;
+
+  if (warp >= 4) {
+    // --------------------------------------------------------------- output --
+#pragma unroll 1
+    for (int blk = 0; blk < p.blocks; ++blk) {
+      const int t0 = blk * kBlk, cnt = min(kBlk, p.rows - t0);
+      const size_t bh = static_cast<size_t>(blk) * p.heads + h;
+      const float* fac = p.factors + bh * kFactors * kBlk;
+      const float gq0 = fac[r0], gq1 = fac[r1];
+      const uint4* pf = p.p_frags + bh * kFragsPerBlock + w4 * (4 * 2 * 32) + lane;
+      uint4 pfr[4][2];
+#pragma unroll
+      for (int ks = 0; ks < 4; ++ks)
+        if (ks <= w4) {
+          pfr[ks][0] = __ldg(pf + ks * 64);
+          pfr[ks][1] = __ldg(pf + ks * 64 + 32);
+        }
+      float Q[2][2][4];  // from the state's high and low parts
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) Q[0][n][e] = Q[1][n][e] = 0.f;
+      __syncthreads();  // state and tiles in place
+      const uint32_t q_sm = kq_sm + (blk & 1) * 2 * tile_bytes + tile_bytes;
+#pragma unroll 4
+      for (int ks = 0; ks < mtiles; ++ks) {
+        uint32_t bh4[4], bl4[4], a[4];
+        load_b16(s_sm, ks * 16, lane, bh4);
+        load_b16(s_sm + s_lo, ks * 16, lane, bl4);
+        ldmatrix_x4(q_sm + a_off + ks * 32, a[0], a[1], a[2], a[3]);
+        mma_2(Q[0], a, bh4);
+        mma_2(Q[1], a, bl4);
+      }
+      if (DELTA) __syncthreads();  // residuals in place
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          Q[0][n][e] = (Q[0][n][e] + Q[1][n][e]) * (e < 2 ? gq0 : gq1);
+          Q[1][n][e] = 0.f;
+        }
+      __syncthreads();  // U in place
+#pragma unroll
+      for (int ks = 0; ks < 4; ++ks) {
+        if (ks > w4) break;
+        uint32_t bh4[4], bl4[4], a[4], al[4];
+        load_b16(u_sm + 2 * kURows, ks * 16, lane, bh4);
+        get4(pfr[ks][0], a);
+        get4(pfr[ks][1], al);
+        mma_2(Q[0], a, bh4);
+        mma_2(Q[1], al, bh4);
+        if (DELTA) {  // v is exactly bf16
+          load_b16(u_sm + 3 * kURows, ks * 16, lane, bl4);
+          mma_2(Q[0], a, bl4);
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int r = e == 0 ? r0 : r1;
+          if (r < cnt)
+            *reinterpret_cast<float2*>(p.o + (static_cast<size_t>(t0 + r) * p.heads + h) * p.vdim + c0 + n * 8 + 2 * tq) =
+                make_float2(Q[0][n][e] + Q[1][n][e], Q[0][n][e + 1] + Q[1][n][e + 1]);
+        }
+    }
+    return;
+  }
+
+  // ------------------------------------------------------------------ state --
   const size_t half = static_cast<size_t>(p.heads) * p.dim * p.vdim;
   float* st = p.state + static_cast<size_t>(slot) * 2 * half + static_cast<size_t>(h) * p.dim * p.vdim + c0;
-
   float S[MT][2][4];
   {
     const float* src = st + ((first - 1) & 1) * half;
@@ -286,48 +464,8 @@ chunk_scan_kernel(const ChunkParams p) {
           S[i][n][e + 1] = v.y;
         }
   }
-  auto fetch = [&](int blk) {
-    const int t0 = blk * kBlk, cnt = min(kBlk, p.rows - t0);
-    const uint32_t dst = kq_sm + (blk & 1) * 2 * tile_bytes;
-    const __nv_bfloat16* src = p.act + static_cast<size_t>(t0) * p.ld + qh * p.dim;
-    load_tile(dst, src + p.k_off, p.ld, cnt, p.dim);
-    load_tile(dst + tile_bytes, src + p.q_off, p.ld, cnt, p.dim);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  fetch(0);
-  const int r0 = warp * 16 + gq, r1 = r0 + 8;
 #pragma unroll 1
   for (int blk = 0; blk < p.blocks; ++blk) {
-    const int t0 = blk * kBlk, cnt = min(kBlk, p.rows - t0);
-    const size_t bh = static_cast<size_t>(blk) * p.heads + h;
-    // this block's inputs that go to registers
-    const float* fac = p.factors + bh * kFactors * kBlk;
-    const float gq0 = fac[r0], gq1 = fac[r1], gk0 = fac[kBlk + r0], gk1 = fac[kBlk + r1];
-    const float be0 = fac[2 * kBlk + r0], be1 = fac[2 * kBlk + r1], uk0 = fac[3 * kBlk + r0], uk1 = fac[3 * kBlk + r1];
-    const float g_all = p.factors[static_cast<size_t>(p.blocks) * p.heads * kFactors * kBlk + bh];
-    float v[2][4];
-#pragma unroll
-    for (int n = 0; n < 2; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        const int r = e == 0 ? r0 : r1;
-        float2 f = make_float2(0.f, 0.f);
-        if (r < cnt)
-          f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.act + static_cast<size_t>(t0 + r) * p.ld + p.v_off + h * p.vdim + c0 + n * 8 + 2 * tq));
-        v[n][e] = f.x;
-        v[n][e + 1] = f.y;
-      }
-    const uint4* pf = p.p_frags + bh * kFragsPerBlock + warp * (4 * 2 * 32) + lane;
-    const uint4* tf = p.t_frags + bh * kFragsPerBlock + warp * (4 * 2 * 32) + lane;
-    uint4 tfr[4][2];
-    if (DELTA) {
-#pragma unroll
-      for (int ks = 0; ks < 4; ++ks)
-        if (ks <= warp) {
-          tfr[ks][0] = __ldg(tf + ks * 64);
-          tfr[ks][1] = __ldg(tf + ks * 64 + 32);
-        }
-    }
     // the state as an operand
 #pragma unroll
     for (int i = 0; i < MT; ++i) {
@@ -344,50 +482,67 @@ chunk_scan_kernel(const ChunkParams p) {
           *reinterpret_cast<uint32_t*>(s_ptr + s_lo + at) = lo;
         }
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();  // state and this block's tiles in place; everybody is through with the other tiles
-    if (blk + 1 < p.blocks) fetch(blk + 1);
-    const uint32_t k_sm = kq_sm + (blk & 1) * 2 * tile_bytes, q_sm = k_sm + tile_bytes;
-    float KS[2][4], QS[2][4];
+    const int t0 = blk * kBlk, cnt = min(kBlk, p.rows - t0);
+    const size_t bh = static_cast<size_t>(blk) * p.heads + h;
+    // inputs that go to registers
+    const float* fac = p.factors + bh * kFactors * kBlk;
+    const float uk0 = fac[3 * kBlk + r0], uk1 = fac[3 * kBlk + r1];
+    const float g_all = p.factors[fac_total + bh];
+    float v[2][4], gk0 = 0.f, gk1 = 0.f, be0 = 0.f, be1 = 0.f;
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) KS[n][e] = QS[n][e] = 0.f;
-    const uint32_t a_off = ((warp * 16 + (lj & 1) * 8 + lr) * ldk + (lj >> 1) * 8) * 2;
-#pragma unroll 4
-    for (int ks = 0; ks < mtiles; ++ks) {
-      uint32_t bh4[4], bl4[4], a[4];
-      load_b16(s_sm, ks * 16, lane, bh4);
-      load_b16(s_sm + s_lo, ks * 16, lane, bl4);
-      if (DELTA) {
-        ldmatrix_x4(k_sm + a_off + ks * 32, a[0], a[1], a[2], a[3]);
-        mma_2(KS, a, bh4);
-        mma_2(KS, a, bl4);
+      for (int e = 0; e < 4; e += 2) {
+        const int r = e == 0 ? r0 : r1;
+        float2 f = make_float2(0.f, 0.f);
+        if (r < cnt)
+          f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.act + static_cast<size_t>(t0 + r) * p.ld + p.v_off + h * p.vdim + c0 + n * 8 + 2 * tq));
+        v[n][e] = f.x;
+        v[n][e + 1] = f.y;
       }
-      ldmatrix_x4(q_sm + a_off + ks * 32, a[0], a[1], a[2], a[3]);
-      mma_2(QS, a, bh4);
-      mma_2(QS, a, bl4);
-    }
-    uint4 pfr[4][2];
+    uint4 tfr[4][2];
+    if (DELTA) {
+      gk0 = fac[kBlk + r0];
+      gk1 = fac[kBlk + r1];
+      be0 = fac[2 * kBlk + r0];
+      be1 = fac[2 * kBlk + r1];
+      const uint4* tf = p.t_frags + bh * kFragsPerBlock + warp * (4 * 2 * 32) + lane;
 #pragma unroll
-    for (int ks = 0; ks < 4; ++ks)
-      if (ks <= warp) {
-        pfr[ks][0] = __ldg(pf + ks * 64);
-        pfr[ks][1] = __ldg(pf + ks * 64 + 32);
-      }
+      for (int ks = 0; ks < 4; ++ks)
+        if (ks <= warp) {
+          tfr[ks][0] = __ldg(tf + ks * 64);
+          tfr[ks][1] = __ldg(tf + ks * 64 + 32);
+        }
+    }
+    __syncthreads();  // state and tiles in place
+    const uint32_t k_sm = kq_sm + (blk & 1) * 2 * tile_bytes;
     float U[2][4];
     if (DELTA) {
+      float K[2][2][4];
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) K[0][n][e] = K[1][n][e] = 0.f;
+#pragma unroll 4
+      for (int ks = 0; ks < mtiles; ++ks) {
+        uint32_t bh4[4], bl4[4], a[4];
+        load_b16(s_sm, ks * 16, lane, bh4);
+        load_b16(s_sm + s_lo, ks * 16, lane, bl4);
+        ldmatrix_x4(k_sm + a_off + ks * 32, a[0], a[1], a[2], a[3]);
+        mma_2(K[0], a, bh4);
+        mma_2(K[1], a, bl4);
+      }
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 4; e += 2) {
           const float be = e == 0 ? be0 : be1, gk = e == 0 ? gk0 : gk1;
           uint32_t hi, lo;
-          split2(be * (v[n][e] - gk * KS[n][e]), be * (v[n][e + 1] - gk * KS[n][e + 1]), hi, lo);
+          split2(be * (v[n][e] - gk * (K[0][n][e] + K[1][n][e])), be * (v[n][e + 1] - gk * (K[0][n][e + 1] + K[1][n][e + 1])), hi, lo);
           const uint32_t at = ((e == 0 ? r0 : r1) * kSmLd + n * 8 + 2 * tq) * 2;
           *reinterpret_cast<uint32_t*>(u_ptr + at) = hi;
           *reinterpret_cast<uint32_t*>(u_ptr + kURows + at) = lo;
-          U[n][e] = U[n][e + 1] = 0.f;
+          K[0][n][e] = K[0][n][e + 1] = K[1][n][e] = K[1][n][e + 1] = 0.f;
         }
       __syncthreads();  // residuals in place
 #pragma unroll
@@ -398,10 +553,14 @@ chunk_scan_kernel(const ChunkParams p) {
         load_b16(u_sm + kURows, ks * 16, lane, bl4);
         get4(tfr[ks][0], a);
         get4(tfr[ks][1], al);
-        mma_2(U, a, bh4);
-        mma_2(U, a, bl4);
-        mma_2(U, al, bh4);
+        mma_2(K[0], a, bh4);
+        mma_2(K[1], a, bl4);
+        mma_2(K[1], al, bh4);
       }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) U[n][e] = K[0][n][e] + K[1][n][e];
     } else {
 #pragma unroll
       for (int n = 0; n < 2; ++n)
@@ -417,19 +576,23 @@ chunk_scan_kernel(const ChunkParams p) {
         const uint32_t at = ((e == 0 ? r0 : r1) * kSmLd + n * 8 + 2 * tq) * 2;
         split2(U[n][e], U[n][e + 1], hi, lo);
         *reinterpret_cast<uint32_t*>(u_ptr + 2 * kURows + at) = hi;
-        *reinterpret_cast<uint32_t*>(u_ptr + 3 * kURows + at) = lo;
+        if (DELTA) *reinterpret_cast<uint32_t*>(u_ptr + 3 * kURows + at) = lo;
         split2(U[n][e] * uk, U[n][e + 1] * uk, hi, lo);
         *reinterpret_cast<uint32_t*>(u_ptr + 4 * kURows + at) = hi;
         *reinterpret_cast<uint32_t*>(u_ptr + 5 * kURows + at) = lo;
       }
     __syncthreads();  // U in place
-    // state: rows of this warp's tiles
+    // the state moves on
+    float D[MT][2][4];  // from U's low part
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) S[i][n][e] *= g_all;
+        for (int e = 0; e < 4; ++e) {
+          S[i][n][e] *= g_all;
+          D[i][n][e] = 0.f;
+        }
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks) {
       uint32_t bh4[4], bl4[4];
@@ -442,40 +605,15 @@ chunk_scan_kernel(const ChunkParams p) {
         uint32_t a[4];  // K^T: rows = state rows, columns = tokens
         ldmatrix_x4_trans(k_sm + ((ks * 16 + lr + (lj >> 1) * 8) * ldk + mt * 16 + (lj & 1) * 8) * 2, a[0], a[1], a[2], a[3]);
         mma_2(S[i], a, bh4);
-        mma_2(S[i], a, bl4);
-      }
-    }
-    // output
-#pragma unroll
-    for (int n = 0; n < 2; ++n) {
-      QS[n][0] *= gq0;
-      QS[n][1] *= gq0;
-      QS[n][2] *= gq1;
-      QS[n][3] *= gq1;
-    }
-#pragma unroll
-    for (int ks = 0; ks < 4; ++ks) {
-      if (ks > warp) break;
-      uint32_t bh4[4], bl4[4], a[4], al[4];
-      load_b16(u_sm + 2 * kURows, ks * 16, lane, bh4);
-      get4(pfr[ks][0], a);
-      get4(pfr[ks][1], al);
-      mma_2(QS, a, bh4);
-      mma_2(QS, al, bh4);
-      if (DELTA) {  // v is exactly bf16
-        load_b16(u_sm + 3 * kURows, ks * 16, lane, bl4);
-        mma_2(QS, a, bl4);
+        mma_2(D[i], a, bl4);
       }
     }
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+    for (int i = 0; i < MT; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        const int r = e == 0 ? r0 : r1;
-        if (r < cnt)
-          *reinterpret_cast<float2*>(p.o + (static_cast<size_t>(t0 + r) * p.heads + h) * p.vdim + c0 + n * 8 + 2 * tq) =
-              make_float2(QS[n][e], QS[n][e + 1]);
-      }
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[i][n][e] += D[i][n][e];
   }
   float* dst = st + ((first + p.rows - 1) & 1) * half;
 #pragma unroll
@@ -506,7 +644,7 @@ static ChunkWorkspace chunk_carve(int rows, int heads, bool delta) {
 template <bool DELTA>
 static int launch_chunks(const ChunkParams& p, cudaStream_t st) {
   const size_t tile = static_cast<size_t>(kBlk) * (p.dim + 8) * 2;
-  const size_t prep = 2 * tile + (DELTA ? 2 * kBlk * 68 * 4 : 0), scan = 4 * tile + 2 * static_cast<size_t>(p.dim) * kSmLd * 2 + 6 * kBlk * kSmLd * 2;
+  const size_t prep = prep_k_bytes(p.dim) + prep_q_bytes(p.dim, DELTA) + (DELTA ? kBlk * 68 * 4 : 0), scan = 4 * tile + 2 * static_cast<size_t>(p.dim) * kSmLd * 2 + 6 * kBlk * kSmLd * 2;
   int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&chunk_prepare_kernel<DELTA>), 128 * 1024);
   if (rc) return rc;
   B200_CUDA(launch_overlapped(chunk_prepare_kernel<DELTA>, dim3(p.blocks, p.heads), dim3(kChunkThreads), prep, st, p));
@@ -515,7 +653,7 @@ static int launch_chunks(const ChunkParams& p, cudaStream_t st) {
   do {                                                                                                           \
     rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&chunk_scan_kernel<MT, DELTA>), 128 * 1024);          \
     if (rc) return rc;                                                                                           \
-    B200_CUDA(launch_overlapped(chunk_scan_kernel<MT, DELTA>, grid, dim3(kChunkThreads), scan, st, p));          \
+    B200_CUDA(launch_overlapped(chunk_scan_kernel<MT, DELTA>, grid, dim3(kScanThreads), scan, st, p));          \
   } while (0)
   if (p.dim <= 64) B200_CHUNK(1);
   else B200_CHUNK(2);

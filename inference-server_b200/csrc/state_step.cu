@@ -89,31 +89,65 @@ state_step_kernel(const StepParams p) {
   const T* act = static_cast<const T*>(p.act) + static_cast<size_t>(row) * p.ld;
   // q, k, v of this head, one value per thread and turn
   const int n = 2 * p.dim + p.vdim;
-  float kk = 0.f, qq = 0.f;
-  for (int i = tid; i < n; i += kStepThreads) {
-    const int ch = i < p.dim ? p.q_off + qh * p.dim + i : i < 2 * p.dim ? p.k_off + qh * p.dim + i - p.dim : p.v_off + h * p.vdim + i - 2 * p.dim;
-    float x = to_f32<T>(act[ch]);
-    if (DELTA) {
-      const T* cw = static_cast<const T*>(p.conv_w) + ch;
-      T* hist = p.taps > 1 ? static_cast<T*>(p.ring) + static_cast<size_t>(slot) * p.taps * p.ld + ch : nullptr;
-      float acc = 0.f;
-      for (int j = 0; j + 1 < p.taps; ++j) {
-        const int at = pos - p.taps + 1 + j;
-        if (at >= 0) acc = fmaf(to_f32<T>(cw[static_cast<size_t>(j) * p.ld]), to_f32<T>(hist[static_cast<size_t>(at % p.taps) * p.ld]), acc);
+  float kk = 0.f, qq = 0.f, b_in = 0.f, a_in = 0.f, alog = 0.f, dtb = 0.f;
+  if (DELTA) {
+    const float* ba = p.ba + static_cast<size_t>(row) * 2 * p.heads;
+    b_in = ba[h];
+    a_in = ba[p.heads + h];
+    alog = p.a_log[h];
+    dtb = p.dt_bias[h];
+  }
+  const T* conv_w = static_cast<const T*>(p.conv_w);
+  T* ring = DELTA && p.taps > 1 ? static_cast<T*>(p.ring) + static_cast<size_t>(slot) * p.taps * p.ld : nullptr;
+  const auto channel = [&](int i) {
+    return i < p.dim ? p.q_off + qh * p.dim + i : i < 2 * p.dim ? p.k_off + qh * p.dim + i - p.dim : p.v_off + h * p.vdim + i - 2 * p.dim;
+  };
+  constexpr int kNear = 4;  // taps whose loads are in flight together, for two channels of the thread
+  for (int i0 = tid; i0 < n; i0 += 2 * kStepThreads) {
+    T x_in[2], w_in[2][kNear], h_in[2][kNear];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = i0 + u * kStepThreads;
+      if (i >= n) break;
+      const int ch = channel(i);
+      x_in[u] = act[ch];
+      if (DELTA) {
+#pragma unroll
+        for (int j = 0; j < kNear; ++j) {  // j positions back
+          w_in[u][j] = j < p.taps ? conv_w[static_cast<size_t>(p.taps - 1 - j) * p.ld + ch] : from_f32<T>(0.f);
+          h_in[u][j] = j > 0 && j < p.taps && pos - j >= 0 ? ring[static_cast<size_t>((pos - j) % p.taps) * p.ld + ch] : from_f32<T>(0.f);
+        }
       }
-      acc = fmaf(to_f32<T>(cw[static_cast<size_t>(p.taps - 1) * p.ld]), x, acc);
-      // the heads that share q and k write the same value once: the first of them
-      if (hist != nullptr && (i >= 2 * p.dim || h == qh * per)) hist[static_cast<size_t>(pos % p.taps) * p.ld] = act[ch];
-      x = to_f32<T>(from_f32<T>(silu_of(acc)));
     }
-    if (i < p.dim) {
-      qs[i] = x;
-      qq = fmaf(x, x, qq);
-    } else if (i < 2 * p.dim) {
-      ks[i - p.dim] = x;
-      kk = fmaf(x, x, kk);
-    } else {
-      vs[i - 2 * p.dim] = x;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = i0 + u * kStepThreads;
+      if (i >= n) break;
+      float x = to_f32<T>(x_in[u]);
+      if (DELTA) {
+        const int ch = channel(i);
+        float acc = 0.f;
+        for (int j = 0; j + kNear < p.taps; ++j) {
+          const int at = pos - p.taps + 1 + j;
+          if (at >= 0)
+            acc = fmaf(to_f32<T>(conv_w[static_cast<size_t>(j) * p.ld + ch]), to_f32<T>(ring[static_cast<size_t>(at % p.taps) * p.ld + ch]), acc);
+        }
+#pragma unroll
+        for (int j = kNear - 1; j > 0; --j) acc = fmaf(to_f32<T>(w_in[u][j]), to_f32<T>(h_in[u][j]), acc);
+        acc = fmaf(to_f32<T>(w_in[u][0]), x, acc);
+        // the heads that share q and k write the same value once: the first of them
+        if (ring != nullptr && (i >= 2 * p.dim || h == qh * per)) ring[static_cast<size_t>(pos % p.taps) * p.ld + ch] = x_in[u];
+        x = to_f32<T>(from_f32<T>(silu_of(acc)));
+      }
+      if (i < p.dim) {
+        qs[i] = x;
+        qq = fmaf(x, x, qq);
+      } else if (i < 2 * p.dim) {
+        ks[i - p.dim] = x;
+        kk = fmaf(x, x, kk);
+      } else {
+        vs[i - 2 * p.dim] = x;
+      }
     }
   }
   if (DELTA) {
@@ -139,9 +173,8 @@ state_step_kernel(const StepParams p) {
     }
     ik = 1.f / sqrtf(kk + 1e-6f);
     iq = p.q_scale / sqrtf(qq + 1e-6f);
-    const float* ba = p.ba + static_cast<size_t>(row) * 2 * p.heads;
-    beta = sigmoid_of(ba[h]);
-    g = expf(step_log_decay(p.a_log[h], ba[p.heads + h], p.dt_bias[h]));
+    beta = sigmoid_of(b_in);
+    g = expf(step_log_decay(alog, a_in, dtb));
   } else {
     g = p.decay[h];
   }
