@@ -283,6 +283,12 @@ __device__ __forceinline__ float clamped_glu_fast(float g, float u, float limit,
 }
 __device__ __forceinline__ float silu_of(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + expf(-z)); }
+// SiLU of a value that is stored as T: the fast forms are good to far more than bf16 keeps.
+template <typename T>
+__device__ __forceinline__ float silu_as(float z) {
+  if constexpr (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-z));
+  else return silu_of(z);
+}
 template <typename T>
 __device__ __forceinline__ float to_f32(T v);
 template <>

@@ -145,9 +145,11 @@ mix_heads_kernel(const float* __restrict__ q, const float* __restrict__ mix, T* 
     const int g = i / hp, h = i - g * hp;
     ms[i] = h < heads ? mix[static_cast<size_t>(h) * heads + c * per + g] : 0.f;
   }
-  for (int i = threadIdx.x * 4; i < rows * row_q; i += blockDim.x * 4) {
-    const int r = i / row_q, x = i - r * row_q;
-    *reinterpret_cast<float4*>(qs + i) = *reinterpret_cast<const float4*>(q + (static_cast<size_t>(m0 + r) * heads + c * per) * D + x);
+  for (int x = threadIdx.x * 4; x < row_q; x += blockDim.x * 4) {
+    const float* src = q + (static_cast<size_t>(m0) * heads + c * per) * D + x;
+#pragma unroll 8
+    for (int r = 0; r < rows; ++r)
+      *reinterpret_cast<float4*>(qs + r * row_q + x) = *reinterpret_cast<const float4*>(src + static_cast<size_t>(r) * heads * D);
   }
   __syncthreads();
   const int d4 = D / 4, per_row = (hp / 4) * d4, items = rows * per_row;
@@ -161,9 +163,9 @@ mix_heads_kernel(const float* __restrict__ q, const float* __restrict__ mix, T* 
       T* dst = out + ((static_cast<size_t>(m0) * heads + h0) * kv_heads + c) * D + d;
 #pragma unroll 2
       for (int r = 0; r < rows; ++r) {
-        float4 acc[4];
+        float2 acc[4][2];
 #pragma unroll
-        for (int u = 0; u < 4; ++u) acc[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int u = 0; u < 4; ++u) acc[u][0] = acc[u][1] = make_float2(0.f, 0.f);
 #pragma unroll
         for (int g = 0; g < 8; ++g) {
           if (g >= per) break;
@@ -171,15 +173,14 @@ mix_heads_kernel(const float* __restrict__ q, const float* __restrict__ mix, T* 
           const float aa[4] = {a[g].x, a[g].y, a[g].z, a[g].w};
 #pragma unroll
           for (int u = 0; u < 4; ++u) {
-            acc[u].x = fmaf(aa[u], v.x, acc[u].x);
-            acc[u].y = fmaf(aa[u], v.y, acc[u].y);
-            acc[u].z = fmaf(aa[u], v.z, acc[u].z);
-            acc[u].w = fmaf(aa[u], v.w, acc[u].w);
+            acc[u][0] = __ffma2_rn(make_float2(aa[u], aa[u]), make_float2(v.x, v.y), acc[u][0]);
+            acc[u][1] = __ffma2_rn(make_float2(aa[u], aa[u]), make_float2(v.z, v.w), acc[u][1]);
           }
         }
 #pragma unroll
         for (int u = 0; u < 4; ++u)
-          if (h0 + u < heads) store4(dst + (static_cast<size_t>(r) * heads + u) * kv_heads * D, acc[u]);
+          if (h0 + u < heads)
+            store4(dst + (static_cast<size_t>(r) * heads + u) * kv_heads * D, make_float4(acc[u][0].x, acc[u][0].y, acc[u][1].x, acc[u][1].y));
       }
     }
     return;
@@ -266,7 +267,7 @@ conv_silu_kernel(const T* __restrict__ in, const T* __restrict__ w, int taps, T*
         for (int e = 0; e < 8; ++e) acc[e] = fmaf(w_r[j][e], a[e], acc[e]);
       }
 #pragma unroll
-      for (int e = 0; e < 8; ++e) acc[e] = silu_of(fmaf(w_r[TAPS > 0 ? TAPS - 1 : 0][e], f[e], acc[e]));
+      for (int e = 0; e < 8; ++e) acc[e] = silu_as<T>(fmaf(w_r[TAPS > 0 ? TAPS - 1 : 0][e], f[e], acc[e]));
 #pragma unroll
       for (int j = 0; j + 2 < TAPS; ++j) win[j] = win[j + 1];
       win[TAPS > 1 ? TAPS - 2 : 0] = x;
@@ -291,7 +292,7 @@ conv_silu_kernel(const T* __restrict__ in, const T* __restrict__ w, int taps, T*
       for (int e = 0; e < 8; ++e) acc[e] = fmaf(b[e], a[e], acc[e]);
     }
 #pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] = silu_of(acc[e]);
+    for (int e = 0; e < 8; ++e) acc[e] = silu_as<T>(acc[e]);
     store8<T>(out + static_cast<size_t>(r) * C + col, acc);
   }
   if (hist == nullptr || (chunk && blockIdx.x != 0)) return;
@@ -418,7 +419,7 @@ extern "C" int b200_conv_silu(const void* in, const void* conv_w, int taps, void
   B200_REQUIRE(aligned16({in, conv_w, ring, out}), "conv_silu: buffers must be 16-byte aligned");
   B200_GLUE_DTYPE("conv_silu");
   if (num_rows == 0) return 0;
-  const int rows_per = chunk ? (taps - 1 > 16 ? taps - 1 : 16) : 1;
+  const int rows_per = chunk ? (taps - 1 > 8 ? taps - 1 : 8) : 1;
   const dim3 grid((num_rows + rows_per - 1) / rows_per, (channels / 8 + 63) / 64);
   int* err = static_cast<int*>(status_word);
 #define B200_CONV(T, TAPS)                                                                                                     \

@@ -155,6 +155,59 @@ moe_route_sigmoid_kernel(const LT* __restrict__ logits, int T, int E, int K, int
 // ---------------------------------------------------------------- permute ---
 constexpr int kRankThreads = 256;
 
+// moe_rank_kernel for more than 16 pairs per thread: a thread's `chunk` ids (a multiple of 4) are read in 16-byte pieces, eight of
+// them in flight, once to count and once to place.
+__device__ __forceinline__ void rank_long(const int* __restrict__ ids, int n_pairs, int chunk, int e, int* __restrict__ rank,
+                                          int* __restrict__ counts, int* warp_tot) {
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int lo = min(n_pairs, tid * chunk), hi = min(n_pairs, lo + chunk);
+  const bool whole = (reinterpret_cast<uintptr_t>(ids) & 15) == 0;
+  unsigned long long seen = 0;  // which of the first 64 are of this expert
+  int c = 0;
+  const auto at = [&](int i, int k, int v) {
+    if (v == e) {
+      ++c;
+      if (i - lo + k < 64) seen |= 1ull << (i - lo + k);
+    }
+  };
+  int i = lo;
+  if (whole) {
+#pragma unroll 8
+    for (; i + 4 <= hi; i += 4) {
+      const int4 v = *reinterpret_cast<const int4*>(ids + i);
+      at(i, 0, v.x);
+      at(i, 1, v.y);
+      at(i, 2, v.z);
+      at(i, 3, v.w);
+    }
+  }
+  for (; i < hi; ++i) at(i, 0, ids[i]);
+  int inc = c;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int y = __shfl_up_sync(0xffffffffu, inc, o);
+    if (lane >= o) inc += y;
+  }
+  if (lane == 31) warp_tot[warp] = inc;
+  __syncthreads();
+  int before = 0, total = 0;
+#pragma unroll
+  for (int w = 0; w < kRankThreads / 32; ++w) {
+    const int t = warp_tot[w];
+    if (w < warp) before += t;
+    total += t;
+  }
+  int run = before + inc - c;
+  while (seen) {
+    const int k = __ffsll(static_cast<long long>(seen)) - 1;
+    seen &= seen - 1;
+    rank[lo + k] = run++;
+  }
+  for (int k = lo + 64; k < hi; ++k)
+    if (ids[k] == e) rank[k] = run++;
+  if (tid == 0) counts[e] = total;
+}
+
 // One CTA per expert: stable rank of every pair routed to this expert.
 __global__ void __launch_bounds__(kRankThreads)
 moe_rank_kernel(const int* __restrict__ topk_ids, int n_pairs, int* __restrict__ rank,
@@ -163,7 +216,11 @@ moe_rank_kernel(const int* __restrict__ topk_ids, int n_pairs, int* __restrict__
   grid_dep_wait();
   grid_dep_launch();
   const int e = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int chunk = (n_pairs + kRankThreads - 1) / kRankThreads;
+  int chunk = (n_pairs + kRankThreads - 1) / kRankThreads;
+  if (chunk > 16) {  // many pairs: whole 16-byte pieces per thread
+    rank_long(topk_ids, n_pairs, (chunk + 3) & ~3, e, rank, counts, warp_tot);
+    return;
+  }
   const int lo = min(n_pairs, tid * chunk), hi = min(n_pairs, lo + chunk);
   // Latency-bound (a few KiB of ids per CTA): a thread's ids are read once, eight at a time into registers
   // (all loads of a group in flight together), and the prefix over the threads is one shuffle scan plus one
@@ -175,7 +232,6 @@ moe_rank_kernel(const int* __restrict__ topk_ids, int n_pairs, int* __restrict__
   for (int u = 0; u < kHold; ++u) held[u] = lo + u < hi ? topk_ids[lo + u] : -2;
 #pragma unroll
   for (int u = 0; u < kHold; ++u) c += held[u] == e;
-  for (int i = lo + kHold; i < hi; ++i) c += topk_ids[i] == e;
   int inc = c;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
@@ -195,8 +251,6 @@ moe_rank_kernel(const int* __restrict__ topk_ids, int n_pairs, int* __restrict__
 #pragma unroll
   for (int u = 0; u < kHold; ++u)
     if (held[u] == e) rank[lo + u] = run++;
-  for (int i = lo + kHold; i < hi; ++i)
-    if (topk_ids[i] == e) rank[i] = run++;
   if (tid == 0) counts[e] = total;
 }
 

@@ -1,7 +1,8 @@
 // One decode step of the recurrences in state_scan.cu (same state, same equations), one CTA per (row, head).
 //
 // The step is bound by the state's bytes: dim x vdim fp32 read and written per row and head.  A thread holds four neighbouring
-// columns of RPT rows; all its loads are asked for before anything else, and the other inputs are prepared while they travel:
+// columns of RPT rows; all loads are asked for before anything is computed, and the other inputs are prepared while the state
+// travels:
 // for the gated delta rule the short convolution with SiLU of this head's q, k and v channels (csrc/gated_glue.cu has it as a
 // kernel of its own), unit norms, step size and decay.  Then one pass gives a = S^T k and b = S^T q, partial sums meet in shared
 // memory, u = beta (v - g a), o = g b + (k . q) u, and S = g S + k u^T is written to the other half of the slot.  The gated
@@ -73,13 +74,6 @@ state_step_kernel(const StepParams p) {
   const size_t half = static_cast<size_t>(p.heads) * p.dim * p.vdim;
   float* st = p.state + static_cast<size_t>(slot) * 2 * half + static_cast<size_t>(h) * p.dim * p.vdim + c;
   const float* src = st + ((pos - 1) & 1) * half;
-  float4 S[RPT];
-#pragma unroll
-  for (int i = 0; i < RPT; ++i) {
-    const int r = rg + i * rgs;
-    S[i] = in && pos > 0 && r < p.dim ? __ldcs(reinterpret_cast<const float4*>(src + static_cast<size_t>(r) * p.vdim))
-                                      : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
   float* ks = st_sm;
   float* qs = ks + p.dim;
   float* vs = qs + p.dim;
@@ -102,9 +96,11 @@ state_step_kernel(const StepParams p) {
   const auto channel = [&](int i) {
     return i < p.dim ? p.q_off + qh * p.dim + i : i < 2 * p.dim ? p.k_off + qh * p.dim + i - p.dim : p.v_off + h * p.vdim + i - 2 * p.dim;
   };
-  constexpr int kNear = 4;  // taps whose loads are in flight together, for two channels of the thread
-  for (int i0 = tid; i0 < n; i0 += 2 * kStepThreads) {
-    T x_in[2], w_in[2][kNear], h_in[2][kNear];
+  // taps whose loads are in flight together, for two channels of the thread
+  constexpr int kNear = 4;
+  T x_in[2], w_in[2][kNear], h_in[2][kNear];
+  const int pos_row = DELTA && p.taps > 1 ? pos % p.taps : 0;
+  const auto ask = [&](int i0) {
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
       const int i = i0 + u * kStepThreads;
@@ -114,11 +110,29 @@ state_step_kernel(const StepParams p) {
       if (DELTA) {
 #pragma unroll
         for (int j = 0; j < kNear; ++j) {  // j positions back
+          const int r = pos_row - j;       // row of the ring
           w_in[u][j] = j < p.taps ? conv_w[static_cast<size_t>(p.taps - 1 - j) * p.ld + ch] : from_f32<T>(0.f);
-          h_in[u][j] = j > 0 && j < p.taps && pos - j >= 0 ? ring[static_cast<size_t>((pos - j) % p.taps) * p.ld + ch] : from_f32<T>(0.f);
+          h_in[u][j] = j > 0 && j < p.taps && pos >= j ? ring[static_cast<size_t>(r < 0 ? r + p.taps : r) * p.ld + ch] : from_f32<T>(0.f);
         }
       }
     }
+  };
+  ask(tid);  // ahead of the state, which is many times as long
+  // the head norm's weight and the gate of this thread's output column
+  float norm_w = 0.f, gate_v = 0.f;
+  if (DELTA && tid < p.vdim) {
+    norm_w = p.norm[tid];
+    gate_v = to_f32<T>(static_cast<const T*>(p.gate)[(static_cast<size_t>(row) * p.heads + h) * p.vdim + tid]);
+  }
+  float4 S[RPT];
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) {
+    const int r = rg + i * rgs;
+    S[i] = in && pos > 0 && r < p.dim ? __ldcs(reinterpret_cast<const float4*>(src + static_cast<size_t>(r) * p.vdim))
+                                      : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  for (int i0 = tid; i0 < n; i0 += 2 * kStepThreads) {
+    if (i0 != tid) ask(i0);
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
       const int i = i0 + u * kStepThreads;
@@ -136,8 +150,8 @@ state_step_kernel(const StepParams p) {
         for (int j = kNear - 1; j > 0; --j) acc = fmaf(to_f32<T>(w_in[u][j]), to_f32<T>(h_in[u][j]), acc);
         acc = fmaf(to_f32<T>(w_in[u][0]), x, acc);
         // the heads that share q and k write the same value once: the first of them
-        if (ring != nullptr && (i >= 2 * p.dim || h == qh * per)) ring[static_cast<size_t>(pos % p.taps) * p.ld + ch] = x_in[u];
-        x = to_f32<T>(from_f32<T>(silu_of(acc)));
+        if (ring != nullptr && (i >= 2 * p.dim || h == qh * per)) ring[static_cast<size_t>(pos_row) * p.ld + ch] = x_in[u];
+        x = to_f32<T>(from_f32<T>(silu_as<T>(acc)));
       }
       if (i < p.dim) {
         qs[i] = x;
@@ -240,9 +254,14 @@ state_step_kernel(const StepParams p) {
   }
   if (DELTA) {
     const float inv = p.out_scale / sqrtf(cta_sum(ss, red) / static_cast<float>(p.norm_size) + p.eps);
-    const T* gt = static_cast<const T*>(p.gate) + (static_cast<size_t>(row) * p.heads + h) * p.vdim;
     T* out = static_cast<T*>(p.out) + static_cast<size_t>(row) * p.out_ld + static_cast<size_t>(h) * p.vdim;
-    for (int j = tid; j < p.vdim; j += kStepThreads) out[j] = from_f32<T>(vs[j] * inv * p.norm[j] * to_f32<T>(gt[j]));
+    for (int j = tid; j < p.vdim; j += kStepThreads) {
+      if (j >= kStepThreads) {
+        norm_w = p.norm[j];
+        gate_v = to_f32<T>(static_cast<const T*>(p.gate)[(static_cast<size_t>(row) * p.heads + h) * p.vdim + j]);
+      }
+      out[j] = from_f32<T>(vs[j] * inv * norm_w * gate_v);
+    }
   }
 }
 

@@ -756,11 +756,15 @@ def pad_distances(table):
 
 
 def mixed_split_tokens(rows: int, window: int, max_ctx: int, num_sms: int = 148) -> int:
-    """Tokens per split of the decode kernel (all heads of a row in one CTA, one CTA per SM for large pages): about four CTAs per
-    SM over the rows' windows, at least 128 tokens each."""
+    """Tokens per split of the decode kernel (all heads of a row in one CTA, one CTA per SM): the number of splits with the
+    shortest sequence of rounds, a CTA costing its tokens and about 150 more (set-up, queries, partials)."""
     seen = min(window, max_ctx) + 15
-    split = -(-seen * rows // (4 * num_sms))
-    return int(min(-(-seen // 32) * 32, max(128, -(-split // 32) * 32)))
+
+    def cost(n):
+        return -(-rows * n // num_sms) * (-(-seen // n) + 150)
+
+    n = min(range(1, max(1, seen // 96) + 1), key=cost)
+    return -(-(-(-seen // n)) // 32) * 32
 
 
 def mixed_attn_workspace(rows, num_q_heads, num_kv_heads, key_dim, value_dim, window, max_pages, split_tokens, device):
