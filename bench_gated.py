@@ -39,11 +39,11 @@ def kernels(eng, rows, positions, ids: dict, decode: bool) -> dict:
         o = torch.empty(n, H, w0.dv, **f32)
         if kind == "parallel":
             a, r = m.left, m.right
-            q, pre, ba = torch.empty(n, a.heads, w0.Dk, **f32), torch.randn(n, w0.channels, **bf), torch.randn(n, 2 * H, **f32)
+            q, pre, ba = torch.empty(n, a.heads, w0.Dk, **bf), torch.randn(n, w0.channels, **bf), torch.randn(n, 2 * H, **f32)
 
             def proj(i):
                 w = eng.layers[i]
-                ops.proj_split(h, w.wproj, [(ops.SEG_F32, q), (ops.SEG_PAGES, eng.k_pools[i]), (ops.SEG_PAGES, eng.v_pools[i]),
+                ops.proj_split(h, w.wproj, [(ops.SEG_ROWS, q), (ops.SEG_PAGES, eng.k_pools[i]), (ops.SEG_PAGES, eng.v_pools[i]),
                                             (ops.SEG_ROWS, pre), (ops.SEG_ROWS, gt, ops.ACT_SILU), (ops.SEG_ROWS, gate, ops.ACT_SIGMOID),
                                             (ops.SEG_F32, ba)], positions=rows.pos, block_table=rows.table, status=eng.status,
                                col_bias=w.proj_bias)
@@ -55,7 +55,7 @@ def kernels(eng, rows, positions, ids: dict, decode: bool) -> dict:
             read = seen * kv if decode else n * kv
             t.add("windowed attention with mixed heads (all its kernels)",
                   [lambda i=i: eng._window_attention(q, eng.k_pools[i], eng.v_pools[i], a, eng.layers[i], rows, 1.0, out) for i in li],
-                  read + n * a.heads * (w0.Dk * 4 + w0.Dv * 2), 2 * seen * a.heads * (w0.Dk + w0.Dv))
+                  read + n * a.heads * (w0.Dk + w0.Dv) * 2, 2 * seen * a.heads * (w0.Dk + w0.Dv))
             pre.normal_()
             if not decode:
                 t.add("convolution + SiLU", [lambda i=i: ops.conv_silu(pre, eng.layers[i].conv, eng.rings[i], rows.slots, rows.pos, True,

@@ -435,34 +435,38 @@ int b200_residual_norm(float* x, const void* delta, const void* expert_rows, con
 /* No counterparts in the reference.  dtype: type of activations, pools and rings (B200_DTYPE_*). */
 
 /* out [num_rows, heads, kv_heads, head_dim]: out[m, h, c] = sum over the query heads g of kv head c of mix[h, g] q[m, g];
- * q [num_rows, heads, head_dim] and mix [heads, heads] fp32; head_dim a multiple of 4. */
-int b200_mix_heads(const float* q, const float* mix, void* out, int num_rows, int heads, int kv_heads, int head_dim,
+ * q [num_rows, heads, head_dim] of the output's type, mix [heads, heads] fp32; head_dim a multiple of 4. */
+int b200_mix_heads(const void* q, const float* mix, void* out, int num_rows, int heads, int kv_heads, int head_dim,
                    int dtype, void* stream);
 
 /*
  * Attention whose scores are mixed over the heads: query head h of a row at position i sees the tokens j with
  * 0 <= i - j < window, with score q[h] . (keys of all kv heads of token j) - bias[h, i - j], and sums values of its own kv
  * head; times out_scale.
- *   q [num_rows, num_q_heads, num_kv_heads * key_dim] (b200_mix_heads); k_pool [num_blocks, num_kv_heads, page_size, key_dim];
- *   v_pool [num_blocks, num_kv_heads, page_size, value_dim]; block_table rows table_stride apart (0: one row for all);
+ *   q [num_rows, num_q_heads, num_kv_heads * key_dim] (b200_mix_heads, mix NULL), or where _mixes says so the raw queries
+ *   [num_rows, num_q_heads, key_dim] with mix [num_q_heads, num_q_heads] fp32; pools cut into 64-wide columns:
+ *   k_pool [num_blocks, num_kv_heads * key_dim / 64, page_size, 64], v_pool likewise with value_dim; block_table rows table_stride apart (0: one row for all);
  *   positions [num_rows]; bias [num_q_heads, bias_ld] fp32 in log2 units: distance d at entry 256 + d, +inf in the 256 entries
  *   before distance 0 and in at least 264 after the last of min(window, positions of the table); bias_ld a multiple of 4;
  *   out [num_rows, out_ld], head h at column h * value_dim.
- * bf16 pools with pages of 16 and sizes in multiples of 64 run on the tensor cores, a row's window in splits of split_tokens (a
+ * key_dim and value_dim are multiples of 64.  bf16 with pages of 16 runs on the tensor cores, a row's window in splits of split_tokens (a
  * multiple of 32) whose partials go through the workspace; split_tokens 0 and every other shape take the generic kernel.
  */
 size_t b200_mixed_attn_workspace_bytes(int num_rows, int num_q_heads, int num_kv_heads, int key_dim, int value_dim, int window,
                                        int max_pages_per_seq, int split_tokens);
-int b200_mixed_attn(const void* q, const void* k_pool, const void* v_pool, const int32_t* block_table, int table_stride,
+int b200_mixed_attn_mixes(int num_q_heads, int num_kv_heads, int key_dim, int value_dim);
+int b200_mixed_attn(const void* q, const float* mix, const void* k_pool, const void* v_pool, const int32_t* block_table, int table_stride,
                     const int32_t* positions, const float* bias, int bias_ld, int window, void* out, int out_ld,
                     float out_scale, void* workspace, size_t workspace_bytes, void* status_word, int num_rows, int num_q_heads,
                     int num_kv_heads, int key_dim, int value_dim, int page_size, int num_blocks, int max_pages_per_seq,
                     int split_tokens, int dtype, void* stream);
 
 /* The same for a chunk of consecutive prompt tokens of one sequence, positions first_position.. (their K/V already in the
- * pages), on the tcgen05 tensor cores; bf16, pages of 16.  _supported: whether it is built for these sizes. */
+ * pages), on the tcgen05 tensor cores; bf16, pages of 16.  _supported: 0 not built for these sizes, 1 for mixed queries (talk not
+ * used), 2 for raw queries [num_tokens, num_q_heads, key_dim], which it mixes with talk [num_q_heads, num_q_heads] bf16 and scores
+ * with the factor `scale`. */
 int b200_mixed_attn_prefill_supported(int num_q_heads, int num_kv_heads, int key_dim, int value_dim);
-int b200_mixed_attn_prefill(const void* q, const void* k_pool, const void* v_pool, const int32_t* block_table_row,
+int b200_mixed_attn_prefill(const void* q, const void* talk, float scale, const void* k_pool, const void* v_pool, const int32_t* block_table_row,
                             const float* bias, int bias_ld, int window, void* out, int out_ld, float out_scale,
                             void* status_word, int num_tokens, int first_position, int num_q_heads, int num_kv_heads,
                             int key_dim, int value_dim, int page_size, int num_blocks, int max_pages_per_seq, void* stream);

@@ -67,10 +67,11 @@ SIGNATURES = {
     "b200_state_step": (c_int, [c_void_p] + [c_int] * 4 + [c_void_p] * 2 + [c_int] + [c_void_p] * 11 + [c_int] * 2 + [c_float] * 2
                         + [c_void_p] + [c_int] * 6 + [c_float, c_int, c_void_p]),
     "b200_mixed_attn_workspace_bytes": (c_size_t, [c_int] * 8),
-    "b200_mixed_attn": (c_int, [c_void_p] * 4 + [c_int] + [c_void_p] * 2 + [c_int] * 2
+    "b200_mixed_attn_mixes": (c_int, [c_int] * 4),
+    "b200_mixed_attn": (c_int, [c_void_p] * 5 + [c_int] + [c_void_p] * 2 + [c_int] * 2
                         + [c_void_p, c_int, c_float, c_void_p, c_size_t, c_void_p] + [c_int] * 10 + [c_void_p]),
     "b200_mixed_attn_prefill_supported": (c_int, [c_int] * 4),
-    "b200_mixed_attn_prefill": (c_int, [c_void_p] * 5 + [c_int] * 2 + [c_void_p, c_int, c_float, c_void_p] + [c_int] * 9 + [c_void_p]),
+    "b200_mixed_attn_prefill": (c_int, [c_void_p] * 2 + [c_float] + [c_void_p] * 4 + [c_int] * 2 + [c_void_p, c_int, c_float, c_void_p] + [c_int] * 9 + [c_void_p]),
     "b200_argmax_rows": (c_int, [c_void_p] * 2 + [c_int] * 2 + [c_void_p]),
     "b200_qkv_rope_append_supported": (c_int, [c_int, c_int]),
     "b200_qkv_rope_append_gemm": (c_int, [c_void_p] * 12 + [c_int] * 5 + [c_float] + [c_int] * 4 + [c_void_p]),

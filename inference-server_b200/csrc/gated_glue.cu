@@ -131,7 +131,7 @@ residual_norm_kernel(float* __restrict__ x, const Pending<T> p, const float* __r
 // four columns of four heads.
 template <typename T>
 __global__ void __launch_bounds__(256)
-mix_heads_kernel(const float* __restrict__ q, const float* __restrict__ mix, T* __restrict__ out, int num_rows, int rows_per,
+mix_heads_kernel(const T* __restrict__ q, const float* __restrict__ mix, T* __restrict__ out, int num_rows, int rows_per,
                  int heads, int kv_heads, int D) {
   grid_dep_wait();
   grid_dep_launch();
@@ -146,10 +146,21 @@ mix_heads_kernel(const float* __restrict__ q, const float* __restrict__ mix, T* 
     ms[i] = h < heads ? mix[static_cast<size_t>(h) * heads + c * per + g] : 0.f;
   }
   for (int x = threadIdx.x * 4; x < row_q; x += blockDim.x * 4) {
-    const float* src = q + (static_cast<size_t>(m0) * heads + c * per) * D + x;
+    const T* src = q + (static_cast<size_t>(m0) * heads + c * per) * D + x;
 #pragma unroll 8
-    for (int r = 0; r < rows; ++r)
-      *reinterpret_cast<float4*>(qs + r * row_q + x) = *reinterpret_cast<const float4*>(src + static_cast<size_t>(r) * heads * D);
+    for (int r = 0; r < rows; ++r) {
+      const T* s = src + static_cast<size_t>(r) * heads * D;
+      float4 v;
+      if constexpr (sizeof(T) == 2) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(s);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        v = make_float4(a.x, a.y, b.x, b.y);
+      } else {
+        v = *reinterpret_cast<const float4*>(s);
+      }
+      *reinterpret_cast<float4*>(qs + r * row_q + x) = v;
+    }
   }
   __syncthreads();
   const int d4 = D / 4, per_row = (hp / 4) * d4, items = rows * per_row;
@@ -380,7 +391,7 @@ extern "C" int b200_residual_norm(float* x, const void* delta, const void* exper
                                                   eps, num_rows, width, ld, center, out, as_stream(stream));
 }
 
-extern "C" int b200_mix_heads(const float* q, const float* mix, void* out, int num_rows, int heads, int kv_heads,
+extern "C" int b200_mix_heads(const void* q, const float* mix, void* out, int num_rows, int heads, int kv_heads,
                               int head_dim, int dtype, void* stream) {
   B200_REQUIRE(q && mix && out, "mix_heads: null pointer");
   B200_REQUIRE(num_rows >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && kv_heads <= 65535 && head_dim > 0 &&
@@ -399,12 +410,12 @@ extern "C" int b200_mix_heads(const float* q, const float* mix, void* out, int n
   if (dtype == 0) {
     int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mix_heads_kernel<__nv_bfloat16>), 200 * 1024);
     if (rc) return rc;
-    B200_CUDA(launch_overlapped(mix_heads_kernel<__nv_bfloat16>, grid, dim3(256), smem, as_stream(stream), q, mix,
-                                static_cast<__nv_bfloat16*>(out), num_rows, rows_per, heads, kv_heads, head_dim));
+    B200_CUDA(launch_overlapped(mix_heads_kernel<__nv_bfloat16>, grid, dim3(256), smem, as_stream(stream),
+                                static_cast<const __nv_bfloat16*>(q), mix, static_cast<__nv_bfloat16*>(out), num_rows, rows_per, heads, kv_heads, head_dim));
   } else {
     int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mix_heads_kernel<float>), 200 * 1024);
     if (rc) return rc;
-    B200_CUDA(launch_overlapped(mix_heads_kernel<float>, grid, dim3(256), smem, as_stream(stream), q, mix,
+    B200_CUDA(launch_overlapped(mix_heads_kernel<float>, grid, dim3(256), smem, as_stream(stream), static_cast<const float*>(q), mix,
                                 static_cast<float*>(out), num_rows, rows_per, heads, kv_heads, head_dim));
   }
   return 0;

@@ -113,12 +113,13 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t,
 struct MapKey {
   int device;
   const void* base;
-  uint64_t rows, cols;
+  uint64_t dim[3];  // innermost first
   int elem_bytes;
-  uint32_t box_rows, box_cols;
+  uint32_t box[3];
   bool operator==(const MapKey& o) const {
-    return device == o.device && base == o.base && rows == o.rows && cols == o.cols &&
-           elem_bytes == o.elem_bytes && box_rows == o.box_rows && box_cols == o.box_cols;
+    for (int i = 0; i < 3; ++i)
+      if (dim[i] != o.dim[i] || box[i] != o.box[i]) return false;
+    return device == o.device && base == o.base && elem_bytes == o.elem_bytes;
   }
 };
 struct MapEntry {
@@ -130,12 +131,10 @@ static std::mutex g_map_mu;
 static std::vector<MapEntry> g_maps;
 static EncodeTiledFn g_encode = nullptr;
 
-int get_tensor_map_2d(const void* base, uint64_t rows, uint64_t cols, int elem_bytes,
-                      uint32_t box_rows, uint32_t box_cols, CUtensorMap* out) {
-  int dev = 0;
-  cudaError_t ce = cudaGetDevice(&dev);
+// Dense row-major tensor of `rank` 2 or 3 dimensions.
+static int get_tensor_map(int rank, MapKey key, CUtensorMap* out) {
+  cudaError_t ce = cudaGetDevice(&key.device);
   if (ce != cudaSuccess) return cuda_fail(ce, "cudaGetDevice");
-  MapKey key{dev, base, rows, cols, elem_bytes, box_rows, box_cols};
   std::lock_guard<std::mutex> lock(g_map_mu);
   for (const MapEntry& e : g_maps) {
     if (e.key == key) {
@@ -153,32 +152,42 @@ int get_tensor_map_2d(const void* base, uint64_t rows, uint64_t cols, int elem_b
     }
     g_encode = reinterpret_cast<EncodeTiledFn>(fn);
   }
-  if (box_cols * static_cast<uint32_t>(elem_bytes) != 128u || box_rows == 0 || box_rows > 256 ||
-      (reinterpret_cast<uintptr_t>(base) & 15) != 0 || (cols * elem_bytes) % 16 != 0) {
-    set_detail("tensor map: base %p rows %llu cols %llu elem %d box %ux%u is not encodable", base,
-               (unsigned long long)rows, (unsigned long long)cols, elem_bytes, box_rows, box_cols);
+  const unsigned long long cols = key.dim[0], rows = key.dim[1];
+  if (key.box[0] * static_cast<uint32_t>(key.elem_bytes) != 128u || key.box[1] == 0 || key.box[1] > 256 || key.box[2] == 0 ||
+      key.box[2] > 256 || (reinterpret_cast<uintptr_t>(key.base) & 15) != 0 || (cols * key.elem_bytes) % 16 != 0) {
+    set_detail("tensor map: base %p rows %llu cols %llu elem %d box %ux%ux%u is not encodable", key.base, rows, cols,
+               key.elem_bytes, key.box[2], key.box[1], key.box[0]);
     return -kErrTensorMap;
   }
-  cuuint64_t gdim[2] = {cols, rows};
-  cuuint64_t gstride[1] = {cols * static_cast<uint64_t>(elem_bytes)};
-  cuuint32_t box[2] = {box_cols, box_rows};
-  cuuint32_t estr[2] = {1, 1};
+  cuuint64_t gdim[3] = {key.dim[0], key.dim[1], key.dim[2]};
+  cuuint64_t gstride[2] = {cols * static_cast<uint64_t>(key.elem_bytes), cols * rows * static_cast<uint64_t>(key.elem_bytes)};
+  cuuint32_t box[3] = {key.box[0], key.box[1], key.box[2]};
+  cuuint32_t estr[3] = {1, 1, 1};
   MapEntry entry;
   entry.key = key;
   CUresult r = g_encode(&entry.map,
-                        elem_bytes == 2 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_UINT8,
-                        2, const_cast<void*>(base), gdim, gstride, box, estr,
+                        key.elem_bytes == 2 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_UINT8,
+                        rank, const_cast<void*>(key.base), gdim, gstride, box, estr,
                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
                         CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r != CUDA_SUCCESS) {
-    set_detail("cuTensorMapEncodeTiled failed with CUresult %d (base %p rows %llu cols %llu)", (int)r,
-               base, (unsigned long long)rows, (unsigned long long)cols);
+    set_detail("cuTensorMapEncodeTiled failed with CUresult %d (base %p rows %llu cols %llu)", (int)r, key.base, rows, cols);
     return -kErrTensorMap;
   }
   if (g_maps.size() >= 4096) g_maps.erase(g_maps.begin(), g_maps.begin() + 2048);
   g_maps.push_back(entry);
   *out = entry.map;
   return 0;
+}
+
+int get_tensor_map_2d(const void* base, uint64_t rows, uint64_t cols, int elem_bytes,
+                      uint32_t box_rows, uint32_t box_cols, CUtensorMap* out) {
+  return get_tensor_map(2, MapKey{0, base, {cols, rows, 1}, elem_bytes, {box_cols, box_rows, 1}}, out);
+}
+
+int get_tensor_map_3d(const void* base, uint64_t planes, uint64_t rows, uint64_t cols, int elem_bytes, uint32_t box_planes,
+                      uint32_t box_rows, uint32_t box_cols, CUtensorMap* out) {
+  return get_tensor_map(3, MapKey{0, base, {cols, rows, planes}, elem_bytes, {box_cols, box_rows, box_planes}}, out);
 }
 
 }  // namespace b200

@@ -28,6 +28,10 @@ int device_sm_count(int* out);
 int get_tensor_map_2d(const void* base, uint64_t rows, uint64_t cols, int elem_bytes,
                       uint32_t box_rows, uint32_t box_cols, CUtensorMap* out);
 
+// The same for a dense [planes, rows, cols] tensor; the box's rows of every plane lie one after the other.
+int get_tensor_map_3d(const void* base, uint64_t planes, uint64_t rows, uint64_t cols, int elem_bytes, uint32_t box_planes,
+                      uint32_t box_rows, uint32_t box_cols, CUtensorMap* out);
+
 // Records the last CUDA error text for b200_last_error_detail().
 int cuda_fail(cudaError_t e, const char* where);
 void set_detail(const char* fmt, ...);

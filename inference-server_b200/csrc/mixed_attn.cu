@@ -9,9 +9,12 @@
 // both sides (kDistPad, kDistTail): outside the window, and for later tokens, it masks.  Every query head then meets the whole
 // of a token's keys, and the values of its own kv head.
 //
-// Decode kernel: bf16, key and value sizes multiples of 64.  grid (rows, splits); a CTA owns up to `split_tokens` consecutive
-// tokens of one row, for all heads, and streams their pages (a producer warp, one TMA box of 16 tokens x 128 B per kv head and
-// 64 columns, mbarrier ring of pages).  Groups of eight consumer warps take two pages (32 tokens) at a time:
+// Pools are cut into 64-wide columns: [num_blocks, kv_heads * size / 64, page, 64], so that a page's keys (or values) of all heads
+// are one run of 128-byte rows.
+//
+// Decode kernel: bf16.  grid (rows, splits); a CTA owns up to `split_tokens` consecutive
+// tokens of one row, for all heads, and streams their pages (a producer warp, TMA boxes of up to 256 rows of 128 B, mbarrier ring
+// of pages).  Groups of eight consumer warps take two pages (32 tokens) at a time:
 //   scores   an item is (page, half of its tokens, 16 query heads): mma.sync m16n8k16 over the keys of all kv heads, queries
 //            from shared memory; times log2 e, less the distance table, masked, into a score tile in shared memory
 //   values   a unit is (kv head, 16 of its query heads, 64 value columns): online softmax over the tile's 32 tokens in the A
@@ -29,9 +32,10 @@ constexpr int kMixWarps = 4;
 constexpr float kMixLog2e = 1.4426950408889634f;
 
 struct MixedAttnParams {
-  const void* q;            // [rows, heads, kv_heads * dk]
-  const void* k_pool;       // [num_blocks, kv_heads, page, dk]
-  const void* v_pool;       // [num_blocks, kv_heads, page, dv]
+  const void* q;            // [rows, heads, dk], or mixed already: [rows, heads, kv_heads * dk]
+  const float* mix;         // [heads, heads]: q is raw and mix applies; NULL: q is mixed
+  const void* k_pool;       // [num_blocks, kv_heads * dk / 64, page, 64]
+  const void* v_pool;       // [num_blocks, kv_heads * dv / 64, page, 64]
   const int* table;         // [rows, max_pages], or one row for all (table_stride 0)
   int table_stride;
   const int* positions;     // [rows]: position of the row's token
@@ -76,20 +80,18 @@ mixed_attn_generic_kernel(const MixedAttnParams p) {
     if (id < 0) continue;
     const int slot = tok % p.page;
     float dot = 0.f;
-    for (int c = 0; c < p.kv_heads; ++c) {
-      const T* kr = kp + ((static_cast<size_t>(id) * p.kv_heads + c) * p.page + slot) * p.dk;
-      for (int d = lane; d < p.dk; d += 32) dot = fmaf(mg_sm[c * p.dk + d], to_f32<T>(kr[d]), dot);
-    }
+    const T* kr = kp + static_cast<size_t>(id) * K * p.page + slot * 64;
+    for (int d = lane; d < K; d += 32) dot = fmaf(mg_sm[d], to_f32<T>(kr[(d >> 6) * p.page * 64 + (d & 63)]), dot);
     dot = fmaf(warp_sum(dot), kMixLog2e, -bias[kDistPad + pos - tok]);
     const float mn = fmaxf(m, dot);
     const float a = exp2f(m - mn), w = exp2f(dot - mn);
     m = mn;
     l = l * a + w;
-    const T* vr = vp + ((static_cast<size_t>(id) * p.kv_heads + kvh) * p.page + slot) * p.dv;
+    const T* vr = vp + (static_cast<size_t>(id) * p.kv_heads + kvh) * p.dv * p.page + slot * 64;
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
       const int d = lane + 32 * j;
-      if (d < p.dv) acc[j] = acc[j] * a + w * to_f32<T>(vr[d]);
+      if (d < p.dv) acc[j] = acc[j] * a + w * to_f32<T>(vr[(d >> 6) * p.page * 64 + (d & 63)]);
     }
   }
   float* o_sm = mg_sm + K;
@@ -127,6 +129,7 @@ struct MixedDecodeParams {
   float* part_o;    // [rows, heads, max_splits, dv]
   float2* part_ml;
   int split_tokens, max_splits, stages;
+  int k_box, v_box;  // rows of a TMA box: they divide a page's rows
 };
 
 // UNITS: units (see above) a warp may own.  GROUPS: groups of eight consumer warps; two of them take the tiles in turn, each with
@@ -183,7 +186,7 @@ mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
       tma_prefetch_desc(&v_map);
     }
     const int* table = p.table + static_cast<size_t>(row) * p.table_stride + first_page;
-    const int kn = p.dk / 64, vn = p.dv / 64;
+    const int k_boxes = (kc * kMdPage + pp.k_box - 1) / pp.k_box, v_boxes = (vc * kMdPage + pp.v_box - 1) / pp.v_box;
     int ids = 0, slot = 0;
     uint32_t phase = 1;
     for (int i = 0; i < npages; ++i) {
@@ -198,12 +201,12 @@ mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
       if (!__all_sync(0xffffffffu, mbar_wait(bar_empty + 8 * slot, phase, p.err))) break;
       if (lane == 0) mbar_arrive_expect_tx(bar_full + 8 * slot, stage_bytes);
       __syncwarp();
-      for (int b = lane; b < kc + vc; b += 32) {
-        const bool is_v = b >= kc;
-        const int bb = is_v ? b - kc : b, n = is_v ? vn : kn;
-        const int head = bb / n;
-        tma_load_2d(ring + slot * stage_bytes + b * 2048u, is_v ? &v_map : &k_map, bar_full + 8 * slot, (bb - head * n) * 64,
-                    (id * p.kv_heads + head) * kMdPage);
+      for (int b = lane; b < k_boxes + v_boxes; b += 32) {
+        if (b < k_boxes)
+          tma_load_2d(ring + slot * stage_bytes + b * pp.k_box * 128u, &k_map, bar_full + 8 * slot, 0, id * kc * kMdPage + b * pp.k_box);
+        else
+          tma_load_2d(ring + slot * stage_bytes + kc * 2048u + (b - k_boxes) * pp.v_box * 128u, &v_map, bar_full + 8 * slot, 0,
+                      id * vc * kMdPage + (b - k_boxes) * pp.v_box);
       }
       if (++slot == stages) {
         slot = 0;
@@ -216,15 +219,50 @@ mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
 
   // ------------------------------------------------------------- consumers --
   const int group = GROUPS > 1 ? warp / kMdWarps : 0, w = warp - group * kMdWarps;
-  {  // the row's mixed queries, zero rows after the last head
+  const int per = p.heads / p.kv_heads;
+  if (p.mix == nullptr) {  // the row's mixed queries, zero rows after the last head
     const uint4* src = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) + static_cast<size_t>(row) * p.heads * K);
     const int per_row = K / 8;
     for (int i = threadIdx.x; i < mt * 16 * per_row; i += GROUPS * kMdWarps * 32) {
       const int h = i / per_row, c = i - h * per_row;
       *reinterpret_cast<uint4*>(q_sm + static_cast<size_t>(h) * q_ld + c * 8) = h < p.heads ? src[i] : make_uint4(0u, 0u, 0u, 0u);
     }
+  } else {  // mix them here: an item is eight columns of one kv head's key and a range of heads (at most 8 raw queries)
+    const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(p.q) + static_cast<size_t>(row) * p.heads * p.dk;
+    const int d8 = p.dk / 8, cols = p.kv_heads * d8;
+    const int ranges = max(1, GROUPS * kMdWarps * 32 / cols), span = (mt * 16 + ranges - 1) / ranges;
+    for (int i = threadIdx.x; i < cols * ranges; i += GROUPS * kMdWarps * 32) {
+      const int rg = i / cols, cd = i - rg * cols, c = cd / d8, d = (cd - c * d8) * 8;
+      const int h_end = min(mt * 16, (rg + 1) * span);
+      float q8[8][8];
+#pragma unroll
+      for (int g = 0; g < 8; ++g) {
+        if (g < per) {
+          load8<__nv_bfloat16>(src + (c * per + g) * p.dk + d, q8[g]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) q8[g][e] = 0.f;
+        }
+      }
+      for (int h = rg * span; h < h_end; ++h) {
+        float acc[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+        if (h < p.heads) {
+          const float* m = p.mix + static_cast<size_t>(h) * p.heads + c * per;
+#pragma unroll
+          for (int g = 0; g < 8; ++g) {
+            if (g >= per) break;
+            const float mv = __ldg(m + g);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) acc[e] = fmaf(mv, q8[g][e], acc[e]);
+          }
+        }
+        store8<__nv_bfloat16>(q_sm + static_cast<size_t>(h) * q_ld + c * p.dk + d, acc);
+      }
+    }
   }
-  const int per = p.heads / p.kv_heads, sub = (per + 15) / 16, dvc = p.dv / 64;
+  const int sub = (per + 15) / 16, dvc = p.dv / 64;
   const int units = p.kv_heads * sub * dvc;
   const int gq = lane >> 2, tq = lane & 3;
   const int lj = lane >> 3, lr = lane & 7;
@@ -562,14 +600,20 @@ extern "C" size_t b200_mixed_attn_workspace_bytes(int num_rows, int num_q_heads,
   return carve(nullptr, num_rows, num_q_heads, value_dim, mixed_max_splits(window, max_pages_per_seq, split_tokens)).bytes;
 }
 
-extern "C" int b200_mixed_attn(const void* q, const void* k_pool, const void* v_pool, const int32_t* block_table,
+extern "C" int b200_mixed_attn_mixes(int num_q_heads, int num_kv_heads, int key_dim, int value_dim) {
+  // a kv head's raw queries sit in registers
+  return num_kv_heads > 0 && num_q_heads % num_kv_heads == 0 && num_q_heads / num_kv_heads <= 8 &&
+         mixed_decode_stages(num_q_heads, num_kv_heads, key_dim, value_dim, nullptr, nullptr) > 0;
+}
+
+extern "C" int b200_mixed_attn(const void* q, const float* mix, const void* k_pool, const void* v_pool, const int32_t* block_table,
                                int table_stride, const int32_t* positions, const float* bias, int bias_ld, int window,
                                void* out, int out_ld, float out_scale, void* workspace, size_t workspace_bytes,
                                void* status_word, int num_rows, int num_q_heads, int num_kv_heads, int key_dim, int value_dim,
                                int page_size, int num_blocks, int max_pages_per_seq, int split_tokens, int dtype, void* stream) {
   B200_REQUIRE(q && k_pool && v_pool && block_table && positions && bias && out, "mixed_attn: null pointer");
   B200_REQUIRE(num_rows >= 0 && num_rows <= 65535 && num_q_heads > 0 && num_kv_heads > 0 && num_q_heads % num_kv_heads == 0 &&
-                   key_dim > 0 && value_dim > 0 && value_dim <= 1024 && page_size > 0 && num_blocks > 0 &&
+                   key_dim > 0 && value_dim > 0 && key_dim % 64 == 0 && value_dim % 64 == 0 && value_dim <= 1024 && page_size > 0 && num_blocks > 0 &&
                    max_pages_per_seq > 0 && window > 0 && (table_stride == 0 || table_stride >= max_pages_per_seq),
                "mixed_attn: %d rows, %d query heads over %d, key size %d, value size %d, window %d", num_rows, num_q_heads,
                num_kv_heads, key_dim, value_dim, window);
@@ -578,9 +622,12 @@ extern "C" int b200_mixed_attn(const void* q, const void* k_pool, const void* v_
                "mixed_attn: bias rows of %d for a window of %d, output rows of %d", bias_ld, window, out_ld);
   B200_GLUE_DTYPE("mixed_attn");
   if (num_rows == 0) return 0;
-  const MixedAttnParams p{q, k_pool, v_pool, block_table, table_stride, positions, bias, bias_ld, window, out, out_ld,
+  const MixedAttnParams p{q, mix, k_pool, v_pool, block_table, table_stride, positions, bias, bias_ld, window, out, out_ld,
                           out_scale, static_cast<int*>(status_word), num_rows, num_q_heads, num_kv_heads, key_dim, value_dim,
                           page_size, num_blocks, max_pages_per_seq};
+  B200_REQUIRE(mix == nullptr || (dtype == 0 && page_size == kMdPage && split_tokens > 0 &&
+                                  b200_mixed_attn_mixes(num_q_heads, num_kv_heads, key_dim, value_dim)),
+               "mixed_attn: raw queries of %d heads over %d cannot be mixed here", num_q_heads, num_kv_heads);
   size_t smem = 0;
   int groups = 1;
   const int stages = dtype == 0 && page_size == kMdPage && split_tokens > 0
@@ -588,7 +635,7 @@ extern "C" int b200_mixed_attn(const void* q, const void* k_pool, const void* v_
   if (stages > 0) {
     B200_REQUIRE(split_tokens % 32 == 0 && out_ld % 2 == 0, "mixed_attn: split_tokens %d is no multiple of 32", split_tokens);
     B200_REQUIRE(aligned16({q, k_pool, v_pool}) && (reinterpret_cast<uintptr_t>(out) & 3) == 0, "mixed_attn: buffers must be aligned");
-    MixedDecodeParams pp{p, nullptr, nullptr, split_tokens, mixed_max_splits(window, max_pages_per_seq, split_tokens), stages};
+    MixedDecodeParams pp{p, nullptr, nullptr, split_tokens, mixed_max_splits(window, max_pages_per_seq, split_tokens), stages, 0, 0};
     B200_REQUIRE(pp.max_splits <= 65535, "mixed_attn: grid too large");
     if (pp.max_splits > 1) {
       const AttnWorkspace w = carve(workspace, num_rows, num_q_heads, value_dim, pp.max_splits);
@@ -600,10 +647,17 @@ extern "C" int b200_mixed_attn(const void* q, const void* k_pool, const void* v_
       pp.part_ml = w.ml;
     }
     CUtensorMap km, vm;
-    const uint64_t pool_rows = static_cast<uint64_t>(num_blocks) * num_kv_heads * kMdPage;
-    int rc = get_tensor_map_2d(k_pool, pool_rows, key_dim, 2, kMdPage, 64, &km);
+    const auto box_rows = [](int rows) {  // of 128 bytes, a page's: the largest equal parts of at most 256
+      int parts = (rows + 255) / 256;
+      while (rows % parts) ++parts;
+      return rows / parts;
+    };
+    const int k_rows = num_kv_heads * key_dim / 64 * kMdPage, v_rows = num_kv_heads * value_dim / 64 * kMdPage;
+    pp.k_box = box_rows(k_rows);
+    pp.v_box = box_rows(v_rows);
+    int rc = get_tensor_map_2d(k_pool, static_cast<uint64_t>(num_blocks) * k_rows, 64, 2, pp.k_box, 64, &km);
     if (rc) return rc;
-    rc = get_tensor_map_2d(v_pool, pool_rows, value_dim, 2, kMdPage, 64, &vm);
+    rc = get_tensor_map_2d(v_pool, static_cast<uint64_t>(num_blocks) * v_rows, 64, 2, pp.v_box, 64, &vm);
     if (rc) return rc;
     const int per = num_q_heads / num_kv_heads, units = num_kv_heads * ((per + 15) / 16) * (value_dim / 64);
     if (groups == 2) return launch_mixed_decode<1, 2>(km, vm, pp, smem, as_stream(stream));

@@ -4,24 +4,29 @@
 //   grid     (query tiles, kv heads).  A CTA owns 128 score rows: 128 / per consecutive positions x the `per` query heads of
 //            its kv head, and walks the key tiles (128 keys = 8 pages) from the one that holds the first key its first row
 //            sees to the one of its last position.
-//   warp 0   K producer: a tile's keys of ALL kv heads, 64 columns (16 KiB: 8 boxes of 16 tokens x 128 B) at a time, into a
-//            ring.
+//   warp 0   K producer: a tile's keys of ALL kv heads, `nc` 64-wide columns (nc x 16 KiB) at a time, into a ring.  A box is 8 tokens
+//            of nc columns; the 16 boxes of a tile lie one after the other, so groups of 8 keys are nc KiB apart and every column is
+//            a K-major B operand as it lands.
 //   warp 1   issuer (one elected lane): S(0), then S(j + 1) and O += P(j) V(j) for every tile j.  S = Q' K^T is 4 x tcgen05.mma
 //            M128 N128 K16 per 64 columns; V is an MN-major B operand straight from its page layout.  While the softmax of
 //            tile j runs, S(j + 1) is in the tensor pipe.
 //   warp 2   the distance table (log2 units): per tile a bulk copy of the slice of B[h][.] that the tile's rows and keys meet.
 //            It is +inf where a distance is negative (a later token) or outside the window, so the mask costs nothing.
-//   warp 3   V producer: the values of the CTA's kv head, one tile at a time.
+//   warp 3   V producer: the values of the CTA's kv head, one tile at a time, a box per page.
 //   warps 4-11  softmax: a thread owns a score row and 64 of the tile's 128 keys (TMEM lanes are bound to warp_id % 4; the two
 //            warps with the same rows meet on a named barrier for the row maximum).  s = score * log2 e - B from the slice in
 //            shared memory, lazy rescale of O as in paged_prefill_tc.cu, P = exp2(s - m) as bf16.
 //
-// The queries meet the keys of all kv heads, so they are kv_heads times as wide as a head, and so is a tile of keys: what a CTA
-// can have in flight decides its speed.  Two forms (QTMEM):
+// The mixed queries meet the keys of all kv heads, so they are kv_heads times as wide as a head, and so is a tile of keys: what a
+// CTA can have in flight decides its speed.  Two forms (QTMEM):
 //   true   Q' is an A operand in TMEM (columns / 2 of it), beside O and one or two S accumulators; P goes through shared memory,
-//          which is left to the ring.  Whenever those fit the 512 columns.
-//   false  Q' in shared memory; S0 columns 0-127, S1 128-255, O from 256 on, P in the last 64 columns; with value size 256, where
-//          none are left, P(j) lies over S(j), and the issuer waits for the product with P(j) before it writes that S again.
+//          which is left to the ring.  Whenever those fit the 512 columns.  The CTA mixes the raw queries itself, on the tensor
+//          cores: per kv head c, Q'_c = T_c q_c, where q_c holds the tile's raw queries of that head (rows position x head) and T_c
+//          repeats the mixing matrix's block (the CTA's heads x the heads of c) along its diagonal, once per position.  q_c comes
+//          through the ring, T_c is written into P's place, the product goes through the S accumulator into Q'.
+//   false  Q', mixed already (b200_mix_heads), in shared memory; S0 columns 0-127, S1 128-255, O from 256 on, P in the last 64
+//          columns; with value size 256, where none are left, P(j) lies over S(j), and the issuer waits for the product with P(j)
+//          before it writes that S again.
 // Every mbarrier wait is bounded; one that runs out records kErrDevWaitTimeout, and the thread stops waiting but keeps the loop
 // structure (the named barriers between partner warps are still met), so the kernel ends.
 
@@ -41,16 +46,17 @@ constexpr float kMpLog2e = 1.4426950408889634f;
 
 struct MixedPrefillParams {
   const int* table_row;
-  const __nv_bfloat16* q;  // [tokens, heads, k_chunks * 64]
+  const __nv_bfloat16* q;  // !QTMEM: [tokens, heads, k_chunks * 64]
+  const __nv_bfloat16* talk;  // QTMEM: the mixing matrix [heads, heads]
   const float* bias;       // [heads, bias_ld]
   __nv_bfloat16* out;      // [tokens, out_ld]
   int* err;
   int bias_ld, window, out_ld;
-  float out_scale;
+  float out_scale, score_scale;  // score_scale: log2 e, with the scores' own factor where that is not in q
   int num_tokens, first_pos, heads, kv_heads, num_blocks;
   int k_chunks;            // 64-wide pieces of a mixed query (all kv heads)
   int dk_chunks;           // of one kv head's keys
-  int stages, s_bufs;
+  int nc, stages, s_bufs;  // 64-wide pieces of a stage
   int bias_stride;         // floats per head of a slice
 };
 
@@ -87,11 +93,22 @@ __device__ __forceinline__ void mp_commit(uint32_t bar) {
 __device__ __forceinline__ bool mp_wait_all(uint32_t bar, uint32_t parity, int* err) {
   return __all_sync(0xffffffffu, mbar_wait(bar, parity, err));
 }
-__device__ __forceinline__ uint64_t mp_desc_mn(uint32_t addr) {  // MN-major, 128-byte swizzle, next 64 columns kMpChunk further
+// Operand descriptors, 128-byte swizzle.  MN-major (16 K rows of it): the next 8 K rows are 1024 bytes, the next 64 columns 2048
+// bytes further.  K-major: groups of 8 rows are `sbo` bytes apart.
+__device__ __forceinline__ uint64_t mp_desc_mn(uint32_t addr) {
   uint64_t d = 0;
   d |= static_cast<uint64_t>((addr & 0x3FFFFu) >> 4);
-  d |= static_cast<uint64_t>(kMpChunk >> 4) << 16;
+  d |= static_cast<uint64_t>(2048 >> 4) << 16;
   d |= static_cast<uint64_t>(1024 >> 4) << 32;
+  d |= static_cast<uint64_t>(1) << 46;
+  d |= static_cast<uint64_t>(2) << 61;
+  return d;
+}
+__device__ __forceinline__ uint64_t mp_desc_k(uint32_t addr, uint32_t sbo) {
+  uint64_t d = 0;
+  d |= static_cast<uint64_t>((addr & 0x3FFFFu) >> 4);
+  d |= static_cast<uint64_t>(1) << 16;
+  d |= static_cast<uint64_t>(sbo >> 4) << 32;
   d |= static_cast<uint64_t>(1) << 46;
   d |= static_cast<uint64_t>(2) << 61;
   return d;
@@ -119,8 +136,8 @@ __device__ __forceinline__ void mp_pair_barrier(int quarter) {
 
 template <int DV, bool QTMEM>
 __global__ void __launch_bounds__(kMpThreads, 1)
-mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
-                        const MixedPrefillParams p) {
+mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
+                        const __grid_constant__ CUtensorMap v_map, const MixedPrefillParams p) {
 #ifdef B200_DEVICE_OK
   constexpr int kVChunks = DV / 64;
   constexpr bool kAlias = !QTMEM && DV > 192;  // P over S
@@ -130,13 +147,15 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
   // Q' or P (two halves of 64 keys), V, the ring of keys
   const int first_chunks = QTMEM ? 2 : p.k_chunks;
   const uint32_t q_sm = base, v_sm = q_sm + first_chunks * kMpChunk, k_sm = v_sm + kVChunks * kMpChunk;
-  uint8_t* extra = base_ptr + (first_chunks + kVChunks + p.stages) * kMpChunk;
-  const uint32_t bars = k_sm + p.stages * kMpChunk;
+  const uint32_t stage_bytes = static_cast<uint32_t>(p.nc) * kMpChunk;
+  uint8_t* extra = base_ptr + (first_chunks + kVChunks + p.stages * p.nc) * kMpChunk;
+  const uint32_t bars = k_sm + p.stages * stage_bytes;
   const uint32_t bar_q = bars, bar_vfull = bars + 8, bar_vempty = bars + 16;
   const uint32_t bar_sfull = bars + 24, bar_sempty = bars + 40;  // [2] each
   const uint32_t bar_pfull = bars + 56, bar_odone = bars + 64;
   const uint32_t bar_bfull = bars + 72, bar_bempty = bars + 88;  // [2] each: slice of the distance table
-  const uint32_t bar_kfull = bars + 104, bar_kempty = bar_kfull + 8 * kMpMaxStages;
+  const uint32_t bar_a = bars + 104, bar_rfull = bars + 112, bar_rempty = bars + 120;  // mixing: T_c written; a round's product
+  const uint32_t bar_kfull = bars + 128, bar_kempty = bar_kfull + 8 * kMpMaxStages;
   uint32_t* tmem_base_sm = reinterpret_cast<uint32_t*>(extra + kMpBarBytes - 16);
   float* mx_sm = reinterpret_cast<float*>(extra + kMpBarBytes);  // [2 tiles][2 halves][128 rows]
   float* l_sm = mx_sm + 2 * 2 * kMpRows;                 // [2 halves][128 rows]
@@ -145,11 +164,15 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int per = p.heads / p.kv_heads, QT = kMpRows / per;
   if (threadIdx.x == 32) {
+    if (QTMEM) tma_prefetch_desc(&q_map);
     tma_prefetch_desc(&k_map);
     tma_prefetch_desc(&v_map);
   }
   if (threadIdx.x == 0) {
     mbar_init(bar_q, kMpSoftmaxWarps);
+    mbar_init(bar_a, kMpSoftmaxWarps);
+    mbar_init(bar_rfull, 1);
+    mbar_init(bar_rempty, kMpSoftmaxWarps);
     mbar_init(bar_vfull, 1);
     mbar_init(bar_vempty, 1);
     mbar_init(bar_pfull, kMpSoftmaxWarps);
@@ -165,6 +188,15 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
       mbar_init(bar_kempty + 8 * s, 1);
     }
     fence_mbar_init();
+    fence_proxy_async();
+  }
+  if (QTMEM && QT * per < kMpRows) {  // raw queries fill QT * per rows of a piece; the rest meets zero columns of T_c and must be finite
+    const int tail = (kMpRows - QT * per) * 8;  // 16-byte pieces
+    for (int i = threadIdx.x; i < p.stages * p.nc * tail; i += kMpThreads) {
+      const int c = i / tail;
+      *reinterpret_cast<uint4*>(base_ptr + (first_chunks + kVChunks + c) * kMpChunk + QT * per * 128 + (i - c * tail) * 16) =
+          make_uint4(0u, 0u, 0u, 0u);
+    }
     fence_proxy_async();
   }
   if (warp == 1) tmem_alloc(smem_u32(tmem_base_sm), 512);
@@ -190,10 +222,27 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     // -------------------------------------------------------- K / V producers ------
     bool alive = true;
     uint32_t slot = 0, kphase = 1;
+    if (QTMEM && warp == 0) {  // the raw queries of all heads, a box per 64-wide piece: rows position x head
+#pragma unroll 1
+      for (int s0 = 0; s0 < p.k_chunks && alive; s0 += p.nc) {
+        alive = mp_wait_all(bar_kempty + 8 * slot, kphase, p.err);
+        if (!alive) break;
+        if (lane == 0) mbar_arrive_expect_tx(bar_kfull + 8 * slot, static_cast<uint32_t>(p.nc * QT * per) * 128u);
+        __syncwarp();
+        if (lane < p.nc) {
+          const int c = (s0 + lane) / p.dk_chunks;
+          tma_load_3d(k_sm + slot * stage_bytes + lane * kMpChunk, &q_map, bar_kfull + 8 * slot, (s0 + lane - c * p.dk_chunks) * 64,
+                      c * per, t0);
+        }
+        if (++slot == static_cast<uint32_t>(p.stages)) {
+          slot = 0;
+          kphase ^= 1;
+        }
+      }
+    }
 #pragma unroll 1
     for (int j = 0; j < n_tiles && alive; ++j) {
-      // lanes 0-7 own a page each; pages past the last position stand in for by it: their keys are masked, their values meet
-      // weights of 0
+      // pages past the last position stand in for by it: their keys are masked, their values meet weights of 0
       int page = 0;
       if (lane < 8) {
         page = __ldg(p.table_row + min((kt0 + j) * 8 + lane, last_page));
@@ -202,22 +251,20 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
           page = 0;
         }
       }
-      const int row0 = page * p.kv_heads * kMpPage;
       if (warp == 0) {
+        const int my_page = __shfl_sync(0xffffffffu, page, (lane >> 1) & 7);  // lanes 0-15: half a page each
 #pragma unroll 1
-        for (int head = 0; head < p.kv_heads && alive; ++head) {
-#pragma unroll 1
-          for (int c = 0; c < p.dk_chunks; ++c) {
-            alive = mp_wait_all(bar_kempty + 8 * slot, kphase, p.err);
-            if (!alive) break;
-            if (lane == 0) mbar_arrive_expect_tx(bar_kfull + 8 * slot, kMpChunk);
-            __syncwarp();
-            if (lane < 8)
-              tma_load_2d(k_sm + slot * kMpChunk + lane * (kMpPage * 128), &k_map, bar_kfull + 8 * slot, c * 64, row0 + head * kMpPage);
-            if (++slot == static_cast<uint32_t>(p.stages)) {
-              slot = 0;
-              kphase ^= 1;
-            }
+        for (int s0 = 0; s0 < p.k_chunks; s0 += p.nc) {
+          alive = mp_wait_all(bar_kempty + 8 * slot, kphase, p.err);
+          if (!alive) break;
+          if (lane == 0) mbar_arrive_expect_tx(bar_kfull + 8 * slot, stage_bytes);
+          __syncwarp();
+          if (lane < 16)
+            tma_load_3d(k_sm + slot * stage_bytes + lane * (p.nc * 1024), &k_map, bar_kfull + 8 * slot, 0, (lane & 1) * 8,
+                        my_page * p.k_chunks + s0);
+          if (++slot == static_cast<uint32_t>(p.stages)) {
+            slot = 0;
+            kphase ^= 1;
           }
         }
       } else {
@@ -226,33 +273,70 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
         if (lane == 0) mbar_arrive_expect_tx(bar_vfull, kVChunks * kMpChunk);
         __syncwarp();
         if (lane < 8)
-#pragma unroll
-          for (int c = 0; c < kVChunks; ++c)
-            tma_load_2d(v_sm + c * kMpChunk + lane * (kMpPage * 128), &v_map, bar_vfull, c * 64, row0 + g * kMpPage);
+          tma_load_2d(v_sm + lane * (kVChunks * 2048), &v_map, bar_vfull, 0, (page * p.kv_heads + g) * kVChunks * kMpPage);
       }
     }
   } else if (warp == 1) {
     // ---------------------------------------------------------------- issuer ------
     constexpr uint32_t idesc_s = mp_idesc(kMpKeys, 0), idesc_o = mp_idesc(DV, 1);
     const uint32_t tmem_o = tmem_base + o_col;
-    bool alive = mp_wait_all(bar_q, 0, p.err);
     uint32_t slot = 0, kphase = 0;
-    const uint64_t q_desc = umma_desc_k128(q_sm), k_desc = umma_desc_k128(k_sm), v_desc = mp_desc_mn(v_sm);
+    const uint64_t q_desc = umma_desc_k128(q_sm), k_desc = mp_desc_k(k_sm, p.nc * 1024), v_desc = mp_desc_mn(v_sm);
+    bool alive = true;
+    if (QTMEM) {  // mix the queries: rounds of up to two 64-wide pieces of a kv head through the first S accumulator
+      constexpr uint32_t idesc_mix = mp_idesc(64, 1);
+      int round = 0, c = 0, cc = 0;
+#pragma unroll 1
+      for (int s0 = 0; s0 < p.k_chunks && alive; s0 += p.nc) {
+        alive = mp_wait_all(bar_kfull + 8 * slot, kphase, p.err);
+#pragma unroll 1
+        for (int i = 0; i < p.nc && alive; ++i) {
+          if (cc == 0) alive = mp_wait_all(bar_a, c & 1, p.err);
+          if ((cc & 1) == 0 && round > 0 && alive) alive = mp_wait_all(bar_rempty, (round - 1) & 1, p.err);
+          if (!alive) break;
+          tc_fence_after();
+          const uint64_t b = mp_desc_mn(k_sm + slot * stage_bytes + i * kMpChunk);
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk)
+            mp_mma_ss(tmem_base + s_col + (cc & 1) * 64, q_desc + (kk >> 2) * (kMpChunk >> 4) + 2 * (kk & 3), b + kk * (2048 >> 4),
+                      idesc_mix, kk > 0 ? 1u : 0u);
+          const bool last = cc + 1 == p.dk_chunks;
+          if ((cc & 1) != 0 || last) {
+            mp_commit(bar_rfull);
+            ++round;
+          }
+          cc = last ? 0 : cc + 1;
+          c += last ? 1 : 0;
+        }
+        mp_commit(bar_kempty + 8 * slot);
+        if (++slot == static_cast<uint32_t>(p.stages)) {
+          slot = 0;
+          kphase ^= 1;
+        }
+      }
+      if (alive) alive = mp_wait_all(bar_rempty, (round - 1) & 1, p.err);  // the last of Q' is in place
+    } else {
+      alive = mp_wait_all(bar_q, 0, p.err);
+    }
     auto scores = [&](int t) {
       const int sb = s_bufs == 2 ? t & 1 : 0;
       const uint32_t ph = (s_bufs == 2 ? t >> 1 : t) & 1, s_acc = tmem_base + s_col + sb * kMpKeys;
       if (alive) alive = mp_wait_all(bar_sempty + 8 * sb, ph ^ 1, p.err);
       if (kAlias && t >= 2 && alive) alive = mp_wait_all(bar_odone, (t - 2) & 1, p.err);  // P(t - 2) lies there
 #pragma unroll 1
-      for (int c = 0; c < p.k_chunks && alive; ++c) {
+      for (int c = 0; c < p.k_chunks && alive; c += p.nc) {
         alive = mp_wait_all(bar_kfull + 8 * slot, kphase, p.err);
         if (!alive) break;
         tc_fence_after();
-        const uint64_t a0 = q_desc + static_cast<uint32_t>(c) * (kMpChunk >> 4), b0 = k_desc + slot * (kMpChunk >> 4);
+#pragma unroll 1
+        for (int i = 0; i < p.nc; ++i) {
+          const uint64_t a0 = q_desc + static_cast<uint32_t>(c + i) * (kMpChunk >> 4);
+          const uint64_t b0 = k_desc + ((slot * stage_bytes + i * 1024u) >> 4);
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          if (QTMEM) mp_mma_ts(s_acc, tmem_base + q_col + c * 32 + k * 8, b0 + 2 * k, idesc_s, (c > 0 || k > 0) ? 1u : 0u);
-          else mp_mma_ss(s_acc, a0 + 2 * k, b0 + 2 * k, idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+          for (int k = 0; k < 4; ++k) {
+            if (QTMEM) mp_mma_ts(s_acc, tmem_base + q_col + (c + i) * 32 + k * 8, b0 + 2 * k, idesc_s, (c + i + k) > 0 ? 1u : 0u);
+            else mp_mma_ss(s_acc, a0 + 2 * k, b0 + 2 * k, idesc_s, (c + i + k) > 0 ? 1u : 0u);
+          }
         }
         mp_commit(bar_kempty + 8 * slot);
         if (++slot == static_cast<uint32_t>(p.stages)) {
@@ -273,7 +357,7 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
       const uint32_t pa = tmem_base + (kAlias ? static_cast<uint32_t>((j & 1) * kMpKeys) : 448u);
 #pragma unroll
       for (int kk = 0; kk < 8; ++kk) {
-        const uint64_t b = v_desc + kk * ((16 * 128) >> 4);
+        const uint64_t b = v_desc + kk * ((kVChunks * 2048) >> 4);  // a page
         if (QTMEM) mp_mma_ss(tmem_o, q_desc + (kk >> 2) * (kMpChunk >> 4) + 2 * (kk & 3), b, idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
         else mp_mma_ts(tmem_o, pa + kk * 8, b, idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
       }
@@ -307,25 +391,47 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     const uint32_t tmem_o = lane_addr + o_col + hf * (DV / 2);
     const int tl = r / per, head = r - tl * per;
     const bool real = tl < QT && t0 + tl < p.num_tokens;
-    // the tile's mixed queries; zero rows past its last position
-    if (QTMEM) {  // 64 columns of this thread's row at a time: one half of them per thread of the row
-      const uint4* src = reinterpret_cast<const uint4*>(p.q + (static_cast<size_t>(t0 + tl) * p.heads + g * per + head) * (p.k_chunks * 64));
-#pragma unroll 2
-      for (int c = hf; c < p.k_chunks; c += 2) {
-        uint32_t v[32];
+    bool alive = true;
+    if (QTMEM) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const uint4 x = real ? __ldg(src + c * 8 + e) : make_uint4(0u, 0u, 0u, 0u);
-          v[4 * e] = x.x;
-          v[4 * e + 1] = x.y;
-          v[4 * e + 2] = x.z;
-          v[4 * e + 3] = x.w;
+      for (int i = 0; i < 8; ++i)
+        *reinterpret_cast<uint4*>(base_ptr + ((sw * 32 + lane) * 8 + i) * 16) = make_uint4(0u, 0u, 0u, 0u);
+      asm volatile("bar.sync 5, %0;" ::"n"(kMpSoftmaxWarps * 32) : "memory");
+      int round = 0;
+#pragma unroll 1
+      for (int c = 0; c < p.kv_heads; ++c) {
+        if (hf == 0 && tl < QT) {  // this row of T_c: the CTA's head against the heads of c, at the row's position
+          const __nv_bfloat16* t = p.talk + static_cast<size_t>(g * per + head) * p.heads + c * per;
+          for (int x = 0; x < per; ++x) {
+            const int col = tl * per + x;
+            *reinterpret_cast<__nv_bfloat16*>(base_ptr + (col >> 6) * kMpChunk + swz128(r, (col & 63) >> 3) + (col & 7) * 2) = t[x];
+          }
         }
-        mp_tmem_st32(lane_addr + q_col + c * 32, v);
+        fence_proxy_async();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(bar_a);
+#pragma unroll 1
+        for (int cc = 0; cc < p.dk_chunks; cc += 2, ++round) {
+          if (alive) alive = mbar_wait(bar_rfull, round & 1, p.err);
+          tc_fence_after();
+          if (cc + hf < p.dk_chunks) {
+            uint32_t v[32], w[32];
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+              tmem_ld32(lane_addr + s_col + hf * 64 + half * 32, v);
+              tmem_ld_wait();
+#pragma unroll
+              for (int e = 0; e < 16; ++e) w[half * 16 + e] = pack_bf16x2(__uint_as_float(v[2 * e]), __uint_as_float(v[2 * e + 1]));
+            }
+            mp_tmem_st32(lane_addr + q_col + (c * p.dk_chunks + cc + hf) * 32, w);
+            mp_tmem_st_wait();
+          }
+          tc_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(bar_rempty);
+        }
       }
-      mp_tmem_st_wait();
-      tc_fence_before();
-    } else {  // neighbouring threads take neighbouring 16-byte pieces of a row
+    } else {  // the mixed queries, zero rows past the tile's last position; neighbouring threads take neighbouring 16-byte pieces
       const int pieces = p.k_chunks * 8;
       for (int i = sw * 32 + lane; i < kMpRows * pieces; i += kMpSoftmaxWarps * 32) {
         const int qr = i / pieces, ch = i - qr * pieces, qtl = qr / per;
@@ -336,14 +442,13 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
         *reinterpret_cast<uint4*>(base_ptr + (ch >> 3) * kMpChunk + swz128(qr, ch & 7)) = v;
       }
       fence_proxy_async();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar_q);
     }
-    __syncwarp();
-    if (lane == 0) mbar_arrive(bar_q);
     // slice entry of this row and key column c: distance (p0 + tl) - (tile key) - c
     const float* b_row = b_sm + head * p.bias_stride + min(tl, QT - 1) + (kMpKeys - 1) - hf * 64 +
                          ((kDistPad + p0 - (kMpKeys - 1)) & 3);  // a tile's first key is a multiple of 128
     float m_run = -INFINITY, l_run = 0.f;
-    bool alive = true;
 #pragma unroll 1
     for (int j = 0; j < n_tiles; ++j) {
       const int buf = j & 1, sb = s_bufs == 2 ? buf : 0;
@@ -361,7 +466,7 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
 #pragma unroll
         for (int c = 0; c < 32; ++c) {
           const int cc = half * 32 + c;
-          s[cc] = fmaf(__uint_as_float(raw[c]), kMpLog2e, -bt[-cc]);
+          s[cc] = fmaf(__uint_as_float(raw[c]), p.score_scale, -bt[-cc]);
           mx4[c & 3] = fmaxf(mx4[c & 3], s[cc]);
         }
       }
@@ -471,11 +576,11 @@ static int mixed_bias_stride(int per) {
 
 // How the kernel runs for a shape: stages of the ring (below 2: not built for it), whether Q' lies in TMEM, S accumulators.
 struct MixedPrefillPlan {
-  int stages, q_tmem, s_bufs;
+  int nc, stages, q_tmem, s_bufs;
   size_t smem;
 };
 static MixedPrefillPlan mixed_prefill_plan(int heads, int kv_heads, int key_dim, int value_dim) {
-  MixedPrefillPlan pl{0, 0, 2, 0};
+  MixedPrefillPlan pl{1, 0, 0, 2, 0};
   if (heads % kv_heads || heads / kv_heads > kMpRows || key_dim % 64 || value_dim % 64 || value_dim > 256) return pl;
   const int per = heads / kv_heads, chunks = kv_heads * key_dim / 64, columns = value_dim + chunks * 32;
   if (columns + kMpKeys <= 512) {
@@ -486,19 +591,25 @@ static MixedPrefillPlan mixed_prefill_plan(int heads, int kv_heads, int key_dim,
                        static_cast<size_t>((pl.q_tmem ? 2 : chunks) + value_dim / 64) * kMpChunk;
   const size_t room = 227 * 1024;
   if (fixed >= room) return pl;
-  pl.stages = static_cast<int>((room - fixed) / kMpChunk);
+  // stages as large as leaves two of them: larger boxes cost the copy engine less
+  for (int nc = 4; nc >= 1; --nc) {
+    if (chunks % nc) continue;
+    pl.nc = nc;
+    pl.stages = static_cast<int>((room - fixed) / (static_cast<size_t>(nc) * kMpChunk));
+    if (pl.stages >= 2) break;
+  }
   if (pl.stages > kMpMaxStages) pl.stages = kMpMaxStages;
-  pl.smem = fixed + static_cast<size_t>(pl.stages) * kMpChunk;
+  pl.smem = fixed + static_cast<size_t>(pl.stages) * pl.nc * kMpChunk;
   return pl;
 }
 
 template <int DV, bool QTMEM>
-static int launch_mixed_prefill(const CUtensorMap& km, const CUtensorMap& vm, const MixedPrefillParams& p, size_t smem, cudaStream_t st) {
+static int launch_mixed_prefill(const CUtensorMap& qm, const CUtensorMap& km, const CUtensorMap& vm, const MixedPrefillParams& p, size_t smem, cudaStream_t st) {
   int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&mixed_prefill_tc_kernel<DV, QTMEM>), 227 * 1024);
   if (rc) return rc;
   const int qt = kMpRows / (p.heads / p.kv_heads);
   B200_CUDA(launch_overlapped(mixed_prefill_tc_kernel<DV, QTMEM>, dim3((p.num_tokens + qt - 1) / qt, p.kv_heads), dim3(kMpThreads),
-                              smem, st, km, vm, p));
+                              smem, st, qm, km, vm, p));
   return 0;
 }
 
@@ -508,10 +619,11 @@ using namespace b200;
 
 extern "C" int b200_mixed_attn_prefill_supported(int num_q_heads, int num_kv_heads, int key_dim, int value_dim) {
   if (num_q_heads <= 0 || num_kv_heads <= 0 || key_dim <= 0 || value_dim <= 0 || num_kv_heads > 65535) return 0;
-  return mixed_prefill_plan(num_q_heads, num_kv_heads, key_dim, value_dim).stages >= 2;
+  const MixedPrefillPlan plan = mixed_prefill_plan(num_q_heads, num_kv_heads, key_dim, value_dim);
+  return plan.stages < 2 ? 0 : plan.q_tmem ? 2 : 1;
 }
 
-extern "C" int b200_mixed_attn_prefill(const void* q, const void* k_pool, const void* v_pool, const int32_t* block_table_row,
+extern "C" int b200_mixed_attn_prefill(const void* q, const void* talk, float scale, const void* k_pool, const void* v_pool, const int32_t* block_table_row,
                                        const float* bias, int bias_ld, int window, void* out, int out_ld, float out_scale,
                                        void* status_word, int num_tokens, int first_position, int num_q_heads, int num_kv_heads,
                                        int key_dim, int value_dim, int page_size, int num_blocks, int max_pages_per_seq,
@@ -530,7 +642,11 @@ extern "C" int b200_mixed_attn_prefill(const void* q, const void* k_pool, const 
   if (rc) return rc;
   const int per = num_q_heads / num_kv_heads;
   const MixedPrefillPlan plan = mixed_prefill_plan(num_q_heads, num_kv_heads, key_dim, value_dim);
+  B200_REQUIRE(!plan.q_tmem || (talk && num_q_heads / num_kv_heads <= 256), "mixed_attn_prefill: raw queries need the mixing matrix");
   MixedPrefillParams p{};
+  p.talk = static_cast<const __nv_bfloat16*>(talk);
+  p.score_scale = (plan.q_tmem ? scale : 1.f) * kMpLog2e;
+  p.nc = plan.nc;
   p.table_row = block_table_row;
   p.q = static_cast<const __nv_bfloat16*>(q);
   p.bias = bias;
@@ -550,16 +666,21 @@ extern "C" int b200_mixed_attn_prefill(const void* q, const void* k_pool, const 
   p.stages = plan.stages;
   p.s_bufs = plan.s_bufs;
   p.bias_stride = mixed_bias_stride(per);
-  CUtensorMap km, vm;
-  const uint64_t rows = static_cast<uint64_t>(num_blocks) * num_kv_heads * kMpPage;
-  rc = get_tensor_map_2d(k_pool, rows, key_dim, 2, kMpPage, 64, &km);
+  CUtensorMap qm, km, vm;
+  rc = get_tensor_map_3d(k_pool, static_cast<uint64_t>(num_blocks) * p.k_chunks, kMpPage, 64, 2, p.nc, 8, 64, &km);
   if (rc) return rc;
-  rc = get_tensor_map_2d(v_pool, rows, value_dim, 2, kMpPage, 64, &vm);
+  const int v_rows = value_dim / 64 * kMpPage;  // of a kv head and page
+  rc = get_tensor_map_2d(v_pool, static_cast<uint64_t>(num_blocks) * num_kv_heads * v_rows, 64, 2, v_rows, 64, &vm);
   if (rc) return rc;
+  qm = km;
+  if (plan.q_tmem) {
+    rc = get_tensor_map_3d(q, num_tokens, num_q_heads, key_dim, 2, kMpRows / per, per, 64, &qm);
+    if (rc) return rc;
+  }
   cudaStream_t st = as_stream(stream);
 #define B200_MIXED_PREFILL(DV)                                                             \
-  return plan.q_tmem ? launch_mixed_prefill<DV, true>(km, vm, p, plan.smem, st)            \
-                     : launch_mixed_prefill<DV, false>(km, vm, p, plan.smem, st)
+  return plan.q_tmem ? launch_mixed_prefill<DV, true>(qm, km, vm, p, plan.smem, st)            \
+                     : launch_mixed_prefill<DV, false>(qm, km, vm, p, plan.smem, st)
   switch (value_dim) {
     case 64: B200_MIXED_PREFILL(64);
     case 128: B200_MIXED_PREFILL(128);

@@ -10,7 +10,7 @@ Sizes are padded with zero rows and columns that change no result: per-head key 
 64, those of a recurrence to 16, an output map's input to 64, an expert's inner size to 128.
 
 Scores mixed over the heads are linear in the queries, so the mixing matrix moves to the queries (``ops.mix_heads``: a head's
-query becomes one vector over the keys of all kv heads) and the distance penalty becomes one table per head over the
+query becomes one vector over the keys of all kv heads, made inside the attention kernels) and the distance penalty becomes one table per head over the
 window (csrc/mixed_attn.cu).
 
 State.  Attention keeps K/V in pages like every other layer.  A recurrence keeps a matrix per head, and its convolution the
@@ -206,7 +206,7 @@ class GatedWeights:
                                           ("v", a.kv_heads, a.vdim, self.Dv)):
                 proj.add(_heads(get("mix.left." + name), heads, size, to), _heads(get(f"mix.left.{name}.b"), heads, size, to))
             talk = get("mix.left.talk").float()
-            self.mix = (talk * a.scale).contiguous()
+            self.mix, self.talk = (talk * a.scale).contiguous(), talk.to(torch.bfloat16).contiguous()
             self.bias = distance_table(talk, get("mix.left.r1"), get("mix.left.r2"), min(a.window, max_positions))
             self.d, self.dv = _up(r.dim, 16), _up(r.vdim, 16)
             convs = []
@@ -343,11 +343,11 @@ class GatedMechanisms:
     def _parallel(self, h, li: int, m: ParallelSpec, w: GatedWeights, rows: Rows) -> Pending:
         a, r, R = m.left, m.right, h.shape[0]
         f32 = torch.float32
-        q = self._act(R, a.heads, w.Dk, dtype=f32)
+        q = self._act(R, a.heads, w.Dk)
         pre, g = self._act(R, w.channels), self._act(R, r.heads * w.dv)
         gate, ba = self._act(R, self.W), self._act(R, 2 * r.heads, dtype=f32)
         kp, vp = self.k_pools[li], self.v_pools[li]
-        ops.proj_split(h, w.wproj, [(ops.SEG_F32, q), (ops.SEG_PAGES, kp), (ops.SEG_PAGES, vp), (ops.SEG_ROWS, pre),
+        ops.proj_split(h, w.wproj, [(ops.SEG_ROWS, q), (ops.SEG_PAGES, kp), (ops.SEG_PAGES, vp), (ops.SEG_ROWS, pre),
                                     (ops.SEG_ROWS, g, ops.ACT_SILU), (ops.SEG_ROWS, gate, ops.ACT_SIGMOID), (ops.SEG_F32, ba)],
                        positions=rows.pos, block_table=rows.table, status=self.status, col_bias=w.proj_bias)
         out = self._act(R, w.out_ld)
@@ -358,15 +358,22 @@ class GatedMechanisms:
         return Pending(gate, dense=self._linear(out, w.wo), bias=w.o_bias)
 
     def _window_attention(self, q, kp, vp, a: WindowAttentionSpec, w: GatedWeights, rows: Rows, scale: float, out) -> None:
-        qm = ops.mix_heads(q, w.mix, a.kv_heads, self.dtype)
-        tiled = ops.mixed_attn_prefill_supported(a.heads, a.kv_heads, w.Dk, w.Dv, self.dtype)
+        shape = (a.heads, a.kv_heads, w.Dk, w.Dv, self.dtype)
+        form, decode_mixes = ops.mixed_attn_prefill_form(*shape), ops.mixed_attn_mixes(*shape)
         for lo, hi, chunk in rows.parts():
-            if chunk and tiled:
-                ops.mixed_attn_prefill(qm[lo:hi], kp, vp, rows.table[0], rows.first, w.bias, a.window, out[lo:hi], scale, self.status)
+            if chunk and form:
+                args = (kp, vp, a.kv_heads, rows.table[0], rows.first, w.bias, a.window, out[lo:hi], scale, self.status)
+                if form == 2:
+                    ops.mixed_attn_prefill(q[lo:hi], *args, talk=w.talk, scale=a.scale)
+                else:
+                    ops.mixed_attn_prefill(ops.mix_heads(q[lo:hi], w.mix, a.kv_heads), *args)
+                continue
+            split, ws = (None, None) if chunk and self.dtype == torch.bfloat16 else self._mixed_plan(hi - lo, a, w)
+            args = (kp, vp, a.kv_heads, rows.table[lo:hi], rows.pos[lo:hi], w.bias, a.window, out[lo:hi], scale, self.status, split, ws)
+            if decode_mixes:
+                ops.mixed_attn(q[lo:hi], *args, mix=w.mix)
             else:
-                split, ws = (None, None) if chunk and self.dtype == torch.bfloat16 else self._mixed_plan(hi - lo, a, w)
-                ops.mixed_attn(qm[lo:hi], kp, vp, rows.table[lo:hi], rows.pos[lo:hi], w.bias, a.window, out[lo:hi], scale, self.status,
-                               split, ws)
+                ops.mixed_attn(ops.mix_heads(q[lo:hi], w.mix, a.kv_heads), *args)
 
     def _mixed_plan(self, rows: int, a: WindowAttentionSpec, w: GatedWeights):
         """(tokens per split, workspace) of the decode attention kernel; one workspace per shape and number of rows, kept for the

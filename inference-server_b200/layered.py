@@ -386,8 +386,9 @@ class LayeredEngine(gated.GatedMechanisms, PagedEngine):
         for spec, w in zip(cfg.layer_list, self.layers):
             if cfg.gated:
                 a = getattr(spec.mixer, "left", None)
-                self.k_pools.append(pool(a.kv_heads, PAGE, w.Dk) if a else None)
-                self.v_pools.append(pool(a.kv_heads, PAGE, w.Dv) if a else None)
+                # 64-wide columns of all heads, see csrc/mixed_attn.cu
+                self.k_pools.append(pool(a.kv_heads * w.Dk // 64, PAGE, 64) if a else None)
+                self.v_pools.append(pool(a.kv_heads * w.Dv // 64, PAGE, 64) if a else None)
                 continue
             attn = isinstance(spec.mixer, AttentionSpec)
             self.k_pools.append(pool(spec.mixer.kv_heads, PAGE, w.D) if attn else None)

@@ -733,14 +733,13 @@ def residual_norm(x, pending, weight, eps: float, width: int, center: bool = Tru
     return out
 
 
-def mix_heads(q, mix, kv_heads: int, dtype):
-    """[M, H, D] fp32 -> [M, H, kv_heads * D]: per kv head the mix-weighted sum of its query heads."""
-    _need(q, "q", torch.float32)
+def mix_heads(q, mix, kv_heads: int):
+    """[M, H, D] -> [M, H, kv_heads * D]: per kv head the mix-weighted (fp32) sum of its query heads."""
+    _need(q, "q")
     _need(mix, "mix", torch.float32)
     M, H, D = q.shape
-    out = torch.empty(M, H, kv_heads * D, dtype=dtype, device=q.device)
-    check(_lib.load().b200_mix_heads(_ptr(q), _ptr(mix), _ptr(out), M, H, kv_heads, D, DTYPE_CODE[dtype], _stream()),
-          "b200_mix_heads")
+    out = torch.empty(M, H, kv_heads * D, dtype=q.dtype, device=q.device)
+    check(_lib.load().b200_mix_heads(_ptr(q), _ptr(mix), _ptr(out), M, H, kv_heads, D, DTYPE_CODE[q.dtype], _stream()), "b200_mix_heads")
     return out
 
 
@@ -772,27 +771,38 @@ def mixed_attn_workspace(rows, num_q_heads, num_kv_heads, key_dim, value_dim, wi
     return torch.zeros(n, dtype=torch.uint8, device=device)
 
 
-def _mixed_shapes(q, k_pool, v_pool, bias, out):
+def _mixed_shapes(q, k_pool, v_pool, bias, out, kv_heads: int, raw: bool):
+    """Pools are cut into 64-wide columns, [blocks, G * D / 64, page, 64]; q holds H * Dk (raw) or H * G * Dk numbers a row."""
     _need(q, "q")
     _need(k_pool, "k_pool", q.dtype)
     _need(v_pool, "v_pool", q.dtype)
     _need(bias, "bias", torch.float32)
     M, H, K = q.shape
-    nb, G, page, Dk = k_pool.shape
-    if K != G * Dk or v_pool.shape[:3] != k_pool.shape[:3] or bias.shape[0] != H:
+    nb, kc, page, _ = k_pool.shape
+    vc = v_pool.shape[1]
+    Dk, Dv = kc * 64 // kv_heads, vc * 64 // kv_heads
+    if k_pool.shape[3] != 64 or v_pool.shape != (nb, vc, page, 64) or Dk * kv_heads != kc * 64 or Dv * kv_heads != vc * 64 or (
+            K != (Dk if raw else kc * 64)) or bias.shape[0] != H:
         raise ValueError("pools or bias do not match q")
     if out.dtype != q.dtype or out.stride(1) != 1 or out.shape[0] != M:
         raise ValueError("out must be rows of q's dtype")
-    return M, H, G, Dk, v_pool.shape[3], page, nb
+    return M, H, kv_heads, Dk, Dv, page, nb
 
 
-def mixed_attn(q, k_pool, v_pool, block_table, positions, bias, window: int, out, out_scale: float, status=None,
-               split_tokens: int | None = None, workspace=None):
-    """Windowed attention of mixed queries [M, H, G * Dk] over pages; writes columns [0, H * Dv) of out [M, ld].  bias: see
-    `pad_distances`.  `split_tokens` 0: the generic kernel."""
-    M, H, G, Dk, Dv, page, nb = _mixed_shapes(q, k_pool, v_pool, bias, out)
+def mixed_attn_mixes(num_q_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, dtype) -> bool:
+    """Whether `mixed_attn` takes raw queries for this shape."""
+    return dtype == torch.bfloat16 and bool(_lib.load().b200_mixed_attn_mixes(num_q_heads, num_kv_heads, key_dim, value_dim))
+
+
+def mixed_attn(q, k_pool, v_pool, kv_heads: int, block_table, positions, bias, window: int, out, out_scale: float, status=None,
+               split_tokens: int | None = None, workspace=None, mix=None):
+    """Windowed attention of mixed queries [M, H, G * Dk] (or raw ones [M, H, Dk] with `mix`, see `mixed_attn_mixes`) over pages;
+    writes columns [0, H * Dv) of out [M, ld].  bias: see `pad_distances`.  `split_tokens` 0: the generic kernel."""
+    M, H, G, Dk, Dv, page, nb = _mixed_shapes(q, k_pool, v_pool, bias, out, kv_heads, mix is not None)
     _need(block_table, "block_table", torch.int32)
     _need(positions, "positions", torch.int32)
+    if mix is not None:
+        _need(mix, "mix", torch.float32)
     if block_table.shape[0] != M or positions.shape[0] != M:
         raise ValueError("block table or positions do not match q")
     mp = block_table.shape[1]
@@ -800,24 +810,29 @@ def mixed_attn(q, k_pool, v_pool, block_table, positions, bias, window: int, out
         split_tokens = mixed_split_tokens(M, window, mp * page)
     if workspace is None and split_tokens:
         workspace = mixed_attn_workspace(M, H, G, Dk, Dv, window, mp, split_tokens, q.device)
-    rc = _lib.load().b200_mixed_attn(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), mp, _ptr(positions), _ptr(bias),
+    rc = _lib.load().b200_mixed_attn(_ptr(q), _ptr(mix), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), mp, _ptr(positions), _ptr(bias),
                                      bias.shape[1], int(window), out.data_ptr(), out.stride(0), float(out_scale), _ptr(workspace),
                                      0 if workspace is None else workspace.numel(), _ptr(status), M, H, G, Dk, Dv, page, nb, mp,
                                      int(split_tokens), DTYPE_CODE[q.dtype], _stream())
     check(rc, "b200_mixed_attn")
 
 
-def mixed_attn_prefill_supported(num_q_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, dtype) -> bool:
-    return dtype == torch.bfloat16 and bool(_lib.load().b200_mixed_attn_prefill_supported(num_q_heads, num_kv_heads, key_dim, value_dim))
+def mixed_attn_prefill_form(num_q_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, dtype) -> int:
+    """0: no prompt kernel for this shape; 1: it takes mixed queries; 2: it takes raw ones and mixes them."""
+    return _lib.load().b200_mixed_attn_prefill_supported(num_q_heads, num_kv_heads, key_dim, value_dim) if dtype == torch.bfloat16 else 0
 
 
-def mixed_attn_prefill(q, k_pool, v_pool, table_row, first_pos: int, bias, window: int, out, out_scale: float, status=None):
-    """`mixed_attn` for consecutive tokens of one sequence, positions first_pos.., on the tensor cores."""
-    M, H, G, Dk, Dv, page, nb = _mixed_shapes(q, k_pool, v_pool, bias, out)
+def mixed_attn_prefill(q, k_pool, v_pool, kv_heads: int, table_row, first_pos: int, bias, window: int, out, out_scale: float, status=None,
+                       talk=None, scale: float = 1.0):
+    """`mixed_attn` for consecutive tokens of one sequence, positions first_pos.., on the tensor cores.  Raw queries [M, H, Dk] with
+    the mixing matrix `talk` (bf16) and the scores' factor, or mixed ones, by `mixed_attn_prefill_form`."""
+    M, H, G, Dk, Dv, page, nb = _mixed_shapes(q, k_pool, v_pool, bias, out, kv_heads, talk is not None)
     _need(table_row, "table_row", torch.int32)
-    rc = _lib.load().b200_mixed_attn_prefill(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(table_row), _ptr(bias), bias.shape[1], int(window),
-                                             out.data_ptr(), out.stride(0), float(out_scale), _ptr(status), M, int(first_pos), H, G, Dk,
-                                             Dv, page, nb, table_row.numel(), _stream())
+    if talk is not None:
+        _need(talk, "talk", torch.bfloat16)
+    rc = _lib.load().b200_mixed_attn_prefill(_ptr(q), _ptr(talk), float(scale), _ptr(k_pool), _ptr(v_pool), _ptr(table_row), _ptr(bias),
+                                             bias.shape[1], int(window), out.data_ptr(), out.stride(0), float(out_scale), _ptr(status), M,
+                                             int(first_pos), H, G, Dk, Dv, page, nb, table_row.numel(), _stream())
     check(rc, "b200_mixed_attn_prefill")
 
 

@@ -64,8 +64,8 @@ def test_residual_norm(ops, width, ld, dtype):
 @pytest.mark.parametrize("dtype", [BF, F32])
 @pytest.mark.parametrize("H,G,D", [(8, 2, 64), (6, 6, 4), (5, 1, 128), (32, 4, 128), (7, 7, 192)])
 def test_mix_heads(ops, H, G, D, dtype):
-    q, mix = randn(9, H, D, seed=1), randn(H, H, seed=2)
-    got = ops.mix_heads(q.to(DEV), mix.to(DEV), G, dtype).cpu().view(9, H, G, D)
+    q, mix = randn(9, H, D, seed=1, dtype=dtype), randn(H, H, seed=2)
+    got = ops.mix_heads(q.to(DEV), mix.to(DEV), G).cpu().view(9, H, G, D)
     per = H // G
     want = torch.stack([torch.einsum("hg,mgd->mhd", mix[:, c * per:(c + 1) * per].double(), q[:, c * per:(c + 1) * per].double())
                         for c in range(G)], 2)
@@ -120,17 +120,32 @@ def test_group_norm_gate(ops, groups, size, ld, shared, dtype):
 # -------------------------------------------------------------- attention
 
 
+def columns(pool):
+    """[blocks, heads, 16, D] -> [blocks, heads * D / 64, 16, 64]."""
+    nb, G, page, D = pool.shape
+    return pool.view(nb, G, page, D // 64, 64).transpose(2, 3).reshape(nb, G * D // 64, page, 64).contiguous()
+
+
 def attention_case(T, H, G, dk, dv, window, dtype, seed, spare=4):
-    """Mixed queries, keys, values, penalties, and the keys and values in shuffled pages."""
-    qm = randn(T, H, G * dk, seed=seed, dtype=dtype, scale=(G * dk) ** -0.5)
+    """Raw queries, the mixing matrix, mixed queries, keys, values, penalties, and the keys and values in shuffled pages."""
+    q = randn(T, H, dk, seed=seed, dtype=dtype)
+    talk = (torch.eye(H) + randn(H, H, seed=seed + 5) * 0.3).bfloat16()
+    per, scale = H // G, dk ** -0.5
+    qm = torch.cat([torch.einsum("hg,tgd->thd", scale * talk[:, c * per:(c + 1) * per].double(), q[:, c * per:(c + 1) * per].double())
+                    for c in range(G)], -1)
     k, v = randn(T, G, dk, seed=seed + 1, dtype=dtype), randn(T, G, dv, seed=seed + 2, dtype=dtype)
     bias = 0.5 * torch.rand(H, min(window, T + 40), generator=torch.Generator().manual_seed(seed + 3)) * torch.arange(min(window, T + 40)).sqrt()
     pages = -(-T // 16)
     order = torch.randperm(pages + spare, generator=torch.Generator().manual_seed(seed + 4))[:pages]
+    for i in (40, 96, 150):  # the score of the row's last seen and of the first unseen key would be far above all others
+        for j in (i - window + 1, i - window):
+            if 0 <= j and i < T:
+                m = qm[i, (i + j) % H].float()
+                k[j] = (m.view(G, dk) * 8 / m.pow(2).sum()).to(dtype)
     kp, vp = torch.full((pages + spare, G, 16, dk), 3.0, dtype=dtype), torch.full((pages + spare, G, 16, dv), 3.0, dtype=dtype)
     for t in range(T):
         kp[order[t // 16], :, t % 16], vp[order[t // 16], :, t % 16] = k[t], v[t]
-    return qm, k, v, bias, kp, vp, order.to(torch.int32)
+    return q, talk, scale, qm, k, v, bias, columns(kp), columns(vp), order.to(torch.int32)
 
 
 def attention_want(qm, k, v, bias, window, rows, positions):
@@ -147,7 +162,7 @@ def attention_want(qm, k, v, bias, window, rows, positions):
     return out
 
 
-SHAPES = [(8, 2, 64, 64), (6, 2, 128, 192), (5, 5, 64, 128), (32, 4, 128, 128), (24, 1, 64, 64), (2, 1, 192, 320), (64, 4, 128, 128),
+SHAPES = [(8, 2, 64, 64), (16, 2, 192, 128), (12, 4, 192, 64), (40, 8, 128, 128), (3, 1, 64, 64), (10, 5, 64, 256), (14, 7, 64, 192), (6, 2, 128, 192), (5, 5, 64, 128), (32, 4, 128, 128), (24, 1, 64, 64), (2, 1, 192, 320), (64, 4, 128, 128),
           (12, 3, 64, 256)]
 
 
@@ -158,41 +173,40 @@ def test_mixed_attention(ops, H, G, dk, dv, window, dtype):
     """Decode rows at page borders, at the sequence's start and around the window's edge, and prompt chunks of several sizes.
     For some rows one key just inside the window and one just outside is made to stand out."""
     T = 170
-    qm, k, v, bias, kp, vp, order = attention_case(T, H, G, dk, dv, window, dtype, seed=H + dk + window)
-    for i in (40, 96, 150):  # the score of the row's last seen and of the first unseen key would be far above all others
-        for j in (i - window + 1, i - window):
-            if j >= 0:
-                k[j] = (qm[i, (i + j) % H].view(G, dk).float() * 8 / qm[i, (i + j) % H].float().pow(2).sum()).to(dtype)
-                kp[order[j // 16], :, j % 16] = k[j]
-    dev = [t.to(DEV) for t in (qm, kp, vp, ops.pad_distances(bias), order)]
-    Q, KP, VP, B, O = dev
+    q, talk, scale, qm, k, v, bias, kp, vp, order = attention_case(T, H, G, dk, dv, window, dtype, seed=H + dk + window)
+    Q, QM, KP, VP, B, O, mix = (t.to(DEV) for t in (q, qm.to(dtype), kp, vp, ops.pad_distances(bias), order, (talk.float() * scale)))
     rows = [0, 1, 15, 16, 17, 31, 32, 40, 47, 48, 96, 99, 100, 150, 169]
     pos = torch.tensor(rows, dtype=torch.int32, device=DEV)
     st = status()
-    out = torch.full((len(rows), H * dv + 32), 7.0, dtype=dtype, device=DEV)
     table = O[None].expand(len(rows), -1).contiguous()
-    ops.mixed_attn(Q[rows].contiguous(), KP, VP, table, pos, B, window, out, 1.3, st)
-    ops.read_status(st, "decode rows")
     want = 1.3 * attention_want(qm, k, v, bias, window, rows, rows)
-    assert rel_err(out[:, : H * dv].cpu().view(-1, H, dv), want) < TOL[dtype] and bool((out[:, H * dv:] == 7.0).all())
-    if not ops.mixed_attn_prefill_supported(H, G, dk, dv, dtype):
+    for raw in (False, True) if ops.mixed_attn_mixes(H, G, dk, dv, dtype) else (False,):
+        for split in (None, 32, 0) if not raw else (None, 64):
+            out = torch.full((len(rows), H * dv + 32), 7.0, dtype=dtype, device=DEV)
+            ops.mixed_attn((Q if raw else QM)[rows].contiguous(), KP, VP, G, table, pos, B, window, out, 1.3, st, split, mix=mix if raw else None)
+            ops.read_status(st, "decode rows")
+            assert rel_err(out[:, : H * dv].cpu().view(-1, H, dv), want) < 1.5 * TOL[dtype], (raw, split)
+            assert bool((out[:, H * dv:] == 7.0).all())
+    form = ops.mixed_attn_prefill_form(H, G, dk, dv, dtype)
+    if not form:
         return
     full = 1.3 * attention_want(qm, k, v, bias, window, range(T), range(T))
     for first, n in ((0, 170), (0, 2), (16, 2), (33, 100), (90, 80), (168, 2), (95, 16)):
         out = torch.full((n, H * dv + 32), 7.0, dtype=dtype, device=DEV)
-        ops.mixed_attn_prefill(Q[first:first + n].contiguous(), KP, VP, O, first, B, window, out, 1.3, st)
+        more = dict(talk=talk.to(DEV), scale=scale) if form == 2 else {}
+        ops.mixed_attn_prefill((Q if form == 2 else QM)[first:first + n].contiguous(), KP, VP, G, O, first, B, window, out, 1.3, st, **more)
         ops.read_status(st, "prompt chunk")
-        assert rel_err(out[:, : H * dv].cpu().view(n, H, dv), full[first:first + n]) < TOL[dtype], (first, n)
+        assert rel_err(out[:, : H * dv].cpu().view(n, H, dv), full[first:first + n]) < 1.5 * TOL[dtype], (first, n)
         assert bool((out[:, H * dv:] == 7.0).all())
 
 
 def test_mixed_attention_reports_bad_pages_and_positions(ops):
-    qm, k, v, bias, kp, vp, order = attention_case(40, 8, 2, 64, 64, 32, BF, 1)
-    Q, KP, VP, B, O = (t.to(DEV) for t in (qm, kp, vp, ops.pad_distances(bias), order))
+    q, talk, scale, qm, k, v, bias, kp, vp, order = attention_case(40, 8, 2, 64, 64, 32, BF, 1)
+    QM, KP, VP, B, O = (t.to(DEV) for t in (qm.to(BF), kp, vp, ops.pad_distances(bias), order))
     out = torch.empty(1, 512, dtype=BF, device=DEV)
     for table, pos in ((torch.full((1, 3), 99, dtype=torch.int32, device=DEV), i32(20)), (O[None].contiguous(), i32(48))):
         st = status()
-        ops.mixed_attn(Q[:1].contiguous(), KP, VP, table, pos, B, 32, out, 1.0, st)
+        ops.mixed_attn(QM[:1].contiguous(), KP, VP, 2, table, pos, B, 32, out, 1.0, st)
         with pytest.raises(RuntimeError):
             ops.read_status(st, "bad page or position")
 
