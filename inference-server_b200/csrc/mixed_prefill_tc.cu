@@ -398,15 +398,27 @@ mixed_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_
         *reinterpret_cast<uint4*>(base_ptr + ((sw * 32 + lane) * 8 + i) * 16) = make_uint4(0u, 0u, 0u, 0u);
       asm volatile("bar.sync 5, %0;" ::"n"(kMpSoftmaxWarps * 32) : "memory");
       int round = 0;
+      const __nv_bfloat16* t = p.talk + static_cast<size_t>(g * per + head) * p.heads;
+      __nv_bfloat16 row[8];  // the row's first factors for the next kv head, asked for ahead
+#pragma unroll
+      for (int x = 0; x < 8; ++x)
+        if (x < per) row[x] = t[x];
 #pragma unroll 1
       for (int c = 0; c < p.kv_heads; ++c) {
         if (hf == 0 && tl < QT) {  // this row of T_c: the CTA's head against the heads of c, at the row's position
-          const __nv_bfloat16* t = p.talk + static_cast<size_t>(g * per + head) * p.heads + c * per;
-          for (int x = 0; x < per; ++x) {
+          const auto put = [&](int x, __nv_bfloat16 v) {
             const int col = tl * per + x;
-            *reinterpret_cast<__nv_bfloat16*>(base_ptr + (col >> 6) * kMpChunk + swz128(r, (col & 63) >> 3) + (col & 7) * 2) = t[x];
-          }
+            *reinterpret_cast<__nv_bfloat16*>(base_ptr + (col >> 6) * kMpChunk + swz128(r, (col & 63) >> 3) + (col & 7) * 2) = v;
+          };
+#pragma unroll
+          for (int x = 0; x < 8; ++x)
+            if (x < per) put(x, row[x]);
+          for (int x = 8; x < per; ++x) put(x, t[c * per + x]);
         }
+        if (c + 1 < p.kv_heads)
+#pragma unroll
+          for (int x = 0; x < 8; ++x)
+            if (x < per) row[x] = t[(c + 1) * per + x];
         fence_proxy_async();
         __syncwarp();
         if (lane == 0) mbar_arrive(bar_a);

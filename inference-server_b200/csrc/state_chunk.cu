@@ -329,25 +329,39 @@ __device__ __forceinline__ void get4(const uint4& v, uint32_t (&a)[4]) {
 }
 
 constexpr int kScanThreads = 9 * 32;
+constexpr int kTileChunk = kBlk * 128;  // 64 tokens x 64 columns, 128-byte swizzle
 
 // Warps 0-3 carry the state (16 tokens each of K S, the residuals and U; MT 16-row tiles each of the state), warps 4-7 make the
-// output (16 tokens each) while the state moves on, warp 8 fetches the next block's k and q.  All meet at two or three barriers
-// per block: state and tiles in place, residuals in place, U in place.
+// output (16 tokens each) while the state moves on, warp 8 asks for the next block's k and q: TMA, boxes of 64 tokens x 64 columns (past
+// a head's size they bring the next one's columns, which nobody reads; past the last token zeros).  All warps meet at two or three
+// barriers per block: state in place, residuals in place, U in place.
 template <int MT, bool DELTA>
 __global__ void __launch_bounds__(kScanThreads)
-chunk_scan_kernel(const ChunkParams p) {
-  extern __shared__ __align__(16) uint8_t cs_sm[];
+chunk_scan_kernel(const __grid_constant__ CUtensorMap act_map, const ChunkParams p) {
+  extern __shared__ uint8_t cs_raw[];
+  __shared__ __align__(8) uint64_t bar_mem[2];
+  const uint32_t cs_base = (smem_u32(cs_raw) + 1023u) & ~1023u;
+  uint8_t* cs_sm = cs_raw + (cs_base - smem_u32(cs_raw));
+  const uint32_t bars = smem_u32(bar_mem);
+  if (threadIdx.x == 0) {
+    tma_prefetch_desc(&act_map);
+    mbar_init(bars, 1);
+    mbar_init(bars + 8, 1);
+    fence_mbar_init();
+    fence_proxy_async();
+  }
+  __syncthreads();
   grid_dep_wait();
   grid_dep_launch();
   const int h = blockIdx.y, c0 = blockIdx.x * 16, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int gq = lane >> 2, tq = lane & 3, lj = lane >> 3, lr = lane & 7;
-  const int qh = h / (p.heads / p.qk_heads), ldk = p.dim + 8, tile_bytes = kBlk * ldk * 2, mtiles = p.dim / 16;
+  const int qh = h / (p.heads / p.qk_heads), chunks = (p.dim + 63) / 64, tile_bytes = chunks * kTileChunk, mtiles = p.dim / 16;
   const int first = p.positions[0], slot = p.slots[0];
   if (slot < 0 || slot >= p.num_slots || first < 0) {
     if (tid == 0) set_error(p.err, kErrDevBadBlockId);
     return;
   }
-  const uint32_t kq_sm = smem_u32(cs_sm);               // [2 buffers][k, q][64][ldk]
+  const uint32_t kq_sm = cs_base;                       // [2 buffers][k, q][chunks][64 tokens][128 bytes]
   const uint32_t s_sm = kq_sm + 4 * tile_bytes;         // state: [high, low][dim][kSmLd]
   const uint32_t s_lo = p.dim * kSmLd * 2;
   const uint32_t u_sm = s_sm + 2 * s_lo;                // residuals, U, scaled U: [3][high, low][64][kSmLd]
@@ -358,24 +372,28 @@ chunk_scan_kernel(const ChunkParams p) {
 
   if (warp == 8) {
     // --------------------------------------------------------------- loader --
-    const TileLoader loader(p.dim, p.ld, lane, 32);
-    const __nv_bfloat16* src = p.act + qh * p.dim;
-    for (int blk = 0; blk <= p.blocks; ++blk) {
-      if (blk < p.blocks) {
-        const size_t at = static_cast<size_t>(blk) * kBlk * p.ld;
-        loader.load(kq_sm + (blk & 1) * 2 * tile_bytes, tile_bytes, src + p.k_off + at, src + p.q_off + at, min(kBlk, p.rows - blk * kBlk), ldk);
+#pragma unroll 1
+    for (int blk = -1; blk < p.blocks; ++blk) {
+      if (blk >= 0) __syncthreads();  // everybody is through with the other tiles
+      if (lane == 0 && blk + 1 < p.blocks) {
+        const uint32_t bar = bars + 8 * ((blk + 1) & 1), dst = kq_sm + ((blk + 1) & 1) * 2 * tile_bytes;
+        mbar_arrive_expect_tx(bar, 2 * tile_bytes);
+        for (int c = 0; c < chunks; ++c) {
+          tma_load_2d(dst + c * kTileChunk, &act_map, bar, p.k_off + qh * p.dim + c * 64, (blk + 1) * kBlk);
+          tma_load_2d(dst + tile_bytes + c * kTileChunk, &act_map, bar, p.q_off + qh * p.dim + c * 64, (blk + 1) * kBlk);
+        }
       }
-      if (blk > 0) {
-        if (DELTA) __syncthreads();  // residuals in place
-        __syncthreads();             // U in place
-      }
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-      if (blk < p.blocks) __syncthreads();  // state and tiles in place; everybody is through with the other tiles
+      __syncwarp();
+      if (blk < 0) continue;
+      if (DELTA) __syncthreads();
+      __syncthreads();
     }
     return;
   }
+  bool alive = true;
   const int w4 = warp & 3, r0 = w4 * 16 + gq, r1 = r0 + 8;
-  const uint32_t a_off = ((w4 * 16 + (lj & 1) * 8 + lr) * ldk + (lj >> 1) * 8) * 2;
+  // A operand of 16 tokens: 16 columns further is ^ 32, ^ 64, ^ 96 inside a chunk
+  const uint32_t a_off = swz128(w4 * 16 + (lj & 1) * 8 + lr, lj >> 1);
 
   if (warp >= 4) {
     // --------------------------------------------------------------- output --
@@ -398,14 +416,15 @@ chunk_scan_kernel(const ChunkParams p) {
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) Q[0][n][e] = Q[1][n][e] = 0.f;
-      __syncthreads();  // state and tiles in place
+      __syncthreads();  // state in place
+      if (alive) alive = mbar_wait(bars + 8 * (blk & 1), (blk >> 1) & 1, p.err);
       const uint32_t q_sm = kq_sm + (blk & 1) * 2 * tile_bytes + tile_bytes;
 #pragma unroll 4
       for (int ks = 0; ks < mtiles; ++ks) {
         uint32_t bh4[4], bl4[4], a[4];
         load_b16(s_sm, ks * 16, lane, bh4);
         load_b16(s_sm + s_lo, ks * 16, lane, bl4);
-        ldmatrix_x4(q_sm + a_off + ks * 32, a[0], a[1], a[2], a[3]);
+        ldmatrix_x4(q_sm + (ks >> 2) * kTileChunk + (a_off ^ ((ks & 3) * 32)), a[0], a[1], a[2], a[3]);
         mma_2(Q[0], a, bh4);
         mma_2(Q[1], a, bl4);
       }
@@ -514,7 +533,8 @@ chunk_scan_kernel(const ChunkParams p) {
           tfr[ks][1] = __ldg(tf + ks * 64 + 32);
         }
     }
-    __syncthreads();  // state and tiles in place
+    __syncthreads();  // state in place
+    if (alive) alive = mbar_wait(bars + 8 * (blk & 1), (blk >> 1) & 1, p.err);
     const uint32_t k_sm = kq_sm + (blk & 1) * 2 * tile_bytes;
     float U[2][4];
     if (DELTA) {
@@ -528,7 +548,7 @@ chunk_scan_kernel(const ChunkParams p) {
         uint32_t bh4[4], bl4[4], a[4];
         load_b16(s_sm, ks * 16, lane, bh4);
         load_b16(s_sm + s_lo, ks * 16, lane, bl4);
-        ldmatrix_x4(k_sm + a_off + ks * 32, a[0], a[1], a[2], a[3]);
+        ldmatrix_x4(k_sm + (ks >> 2) * kTileChunk + (a_off ^ ((ks & 3) * 32)), a[0], a[1], a[2], a[3]);
         mma_2(K[0], a, bh4);
         mma_2(K[1], a, bl4);
       }
@@ -603,7 +623,8 @@ chunk_scan_kernel(const ChunkParams p) {
         const int mt = warp + 4 * i;
         if (mt >= mtiles) break;
         uint32_t a[4];  // K^T: rows = state rows, columns = tokens
-        ldmatrix_x4_trans(k_sm + ((ks * 16 + lr + (lj >> 1) * 8) * ldk + mt * 16 + (lj & 1) * 8) * 2, a[0], a[1], a[2], a[3]);
+        ldmatrix_x4_trans(k_sm + (mt >> 2) * kTileChunk + swz128(ks * 16 + lr + (lj >> 1) * 8, (mt & 3) * 2 + (lj & 1)), a[0], a[1], a[2],
+                          a[3]);
         mma_2(S[i], a, bh4);
         mma_2(D[i], a, bl4);
       }
@@ -643,9 +664,12 @@ static ChunkWorkspace chunk_carve(int rows, int heads, bool delta) {
 
 template <bool DELTA>
 static int launch_chunks(const ChunkParams& p, cudaStream_t st) {
-  const size_t tile = static_cast<size_t>(kBlk) * (p.dim + 8) * 2;
-  const size_t prep = prep_k_bytes(p.dim) + prep_q_bytes(p.dim, DELTA) + (DELTA ? kBlk * 68 * 4 : 0), scan = 4 * tile + 2 * static_cast<size_t>(p.dim) * kSmLd * 2 + 6 * kBlk * kSmLd * 2;
-  int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&chunk_prepare_kernel<DELTA>), 128 * 1024);
+  const size_t prep = prep_k_bytes(p.dim) + prep_q_bytes(p.dim, DELTA) + (DELTA ? kBlk * 68 * 4 : 0);
+  const size_t scan = 1024 + 4 * static_cast<size_t>((p.dim + 63) / 64) * kTileChunk + (2 * p.dim + 6 * kBlk) * kSmLd * 2;
+  CUtensorMap act_map;
+  int rc = get_tensor_map_2d(p.act, p.rows, p.ld, 2, kBlk, 64, &act_map);
+  if (rc) return rc;
+  rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&chunk_prepare_kernel<DELTA>), 128 * 1024);
   if (rc) return rc;
   B200_CUDA(launch_overlapped(chunk_prepare_kernel<DELTA>, dim3(p.blocks, p.heads), dim3(kChunkThreads), prep, st, p));
   const dim3 grid(p.vdim / 16, p.heads);
@@ -653,7 +677,7 @@ static int launch_chunks(const ChunkParams& p, cudaStream_t st) {
   do {                                                                                                           \
     rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&chunk_scan_kernel<MT, DELTA>), 128 * 1024);          \
     if (rc) return rc;                                                                                           \
-    B200_CUDA(launch_overlapped(chunk_scan_kernel<MT, DELTA>, grid, dim3(kScanThreads), scan, st, p));          \
+    B200_CUDA(launch_overlapped(chunk_scan_kernel<MT, DELTA>, grid, dim3(kScanThreads), scan, st, act_map, p)); \
   } while (0)
   if (p.dim <= 64) B200_CHUNK(1);
   else B200_CHUNK(2);
