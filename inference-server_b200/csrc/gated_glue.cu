@@ -317,33 +317,42 @@ conv_silu_kernel(const T* __restrict__ in, const T* __restrict__ w, int taps, T*
   }
 }
 
-// out = o / rms(o over the group) * w * gate * scale, o [M, groups, ldg] fp32 whose columns past `size` are zero.  A warp
-// per (row, group).  `shared_w`: one weight row for all groups.
-template <typename T>
-__global__ void __launch_bounds__(128)
+// out = o / rms(o over the group) * w * gate * scale, o [M, groups, ldg] fp32 whose columns past `size` are zero.  LANES threads
+// per (row, group): a warp (four to a block), or a block of 256 for long groups.  `shared_w`: one weight row for all groups.
+template <typename T, int LANES>
+__global__ void __launch_bounds__(LANES > 32 ? LANES : 128)
 group_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate, float eps,
                        int total, int groups, int size, int ldg, int shared_w, float scale, T* __restrict__ out, int out_ld) {
+  __shared__ float part[LANES / 32];
   grid_dep_wait();
   grid_dep_launch();
-  const int item = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (item >= total) return;
+  const int item = LANES > 32 ? blockIdx.x : blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x % LANES;
+  if (item >= total) return;  // the whole warp or block
   const int m = item / groups, g = item - m * groups;
   const float* src = o + static_cast<size_t>(item) * ldg;
   float ss = 0.f;
-  for (int c = lane * 4; c < ldg; c += 128) {
+#pragma unroll 4
+  for (int c = lane * 4; c < ldg; c += LANES * 4) {
     const float4 v = *reinterpret_cast<const float4*>(src + c);
     ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
   }
   ss = warp_sum(ss);
+  if (LANES > 32) {
+    if ((lane & 31) == 0) part[lane >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < LANES / 32; ++i) ss += part[i];
+  }
   const float inv = scale / sqrtf(ss / static_cast<float>(size) + eps);
   const float* wg = w + (shared_w ? 0 : static_cast<size_t>(g) * ldg);
   const T* gt = gate + static_cast<size_t>(item) * ldg;
   T* dst = out + static_cast<size_t>(m) * out_ld + static_cast<size_t>(g) * ldg;
-  for (int c = lane * 4; c < ldg; c += 128) {
+#pragma unroll 4
+  for (int c = lane * 4; c < ldg; c += LANES * 4) {
     const float4 v = *reinterpret_cast<const float4*>(src + c), a = *reinterpret_cast<const float4*>(wg + c);
     const float g0 = to_f32<T>(gt[c]), g1 = to_f32<T>(gt[c + 1]), g2 = to_f32<T>(gt[c + 2]), g3 = to_f32<T>(gt[c + 3]);
-    const float r[4] = {v.x * inv * a.x * g0, v.y * inv * a.y * g1, v.z * inv * a.z * g2, v.w * inv * a.w * g3};
-    store4(dst + c, make_float4(r[0], r[1], r[2], r[3]));
+    store4(dst + c, make_float4(v.x * inv * a.x * g0, v.y * inv * a.y * g1, v.z * inv * a.z * g2, v.w * inv * a.w * g3));
   }
 }
 
@@ -463,14 +472,14 @@ extern "C" int b200_group_norm_gate(const float* o, const float* weight, const v
   B200_GLUE_DTYPE("group_norm_gate");
   if (num_rows == 0) return 0;
   const int total = num_rows * groups;
-  const dim3 grid((total + 3) / 4);
-  if (dtype == 0)
-    B200_CUDA(launch_overlapped(group_norm_gate_kernel<__nv_bfloat16>, grid, dim3(128), 0, as_stream(stream), o, weight,
-                                static_cast<const __nv_bfloat16*>(gate), eps, total, groups, size, group_ld, shared_weight,
-                                scale, static_cast<__nv_bfloat16*>(out), out_ld));
-  else
-    B200_CUDA(launch_overlapped(group_norm_gate_kernel<float>, grid, dim3(128), 0, as_stream(stream), o, weight,
-                                static_cast<const float*>(gate), eps, total, groups, size, group_ld, shared_weight, scale,
-                                static_cast<float*>(out), out_ld));
+#define B200_GROUP_NORM(T, LANES)                                                                                     \
+  B200_CUDA(launch_overlapped(group_norm_gate_kernel<T, LANES>, dim3(LANES > 32 ? total : (total + 3) / 4),            \
+                              dim3(LANES > 32 ? LANES : 128), 0, as_stream(stream), o, weight, static_cast<const T*>(gate), eps, \
+                              total, groups, size, group_ld, shared_weight, scale, static_cast<T*>(out), out_ld))
+  if (dtype == 0 && group_ld >= 1024) B200_GROUP_NORM(__nv_bfloat16, 256);
+  else if (dtype == 0) B200_GROUP_NORM(__nv_bfloat16, 32);
+  else if (group_ld >= 1024) B200_GROUP_NORM(float, 256);
+  else B200_GROUP_NORM(float, 32);
+#undef B200_GROUP_NORM
   return 0;
 }

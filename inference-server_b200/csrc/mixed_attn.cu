@@ -24,6 +24,8 @@
 //
 // Generic kernel: any sizes, bf16 or fp32, fp32 arithmetic, one CTA per (row, query head).
 
+#include <type_traits>
+
 #include "glue.cuh"
 
 namespace b200 {
@@ -308,41 +310,63 @@ mixed_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_cons
     const int tok_tile = start + tile * 2 * kMdPage;
     if (alive) alive = mbar_wait(bar_full + 8 * slot, phase, p.err);
     if (pages_here > 1 && alive) alive = mbar_wait(bar_full + 8 * slot1, phase1, p.err);
-    // ---- scores: items count up by (page, token half), then by 16 heads
-    const int items = mt * 4;
-#pragma unroll 1
-    for (int item = w; item < items; item += kMdWarps) {
-      const int pg = item & 1, th = (item >> 1) & 1, mi = item >> 2;
-      if (pg >= pages_here) continue;
+    // ---- scores: an item is 16 heads and a page, or half a page where there are too few heads to keep all warps busy so
+    const auto score_item = [&](auto halves, int pg, int th0, int mi) {
+      constexpr int NT = decltype(halves)::value;
       // the distance table's entries travel while the products run
-      const float* bt = p.bias + static_cast<size_t>(mi * 16 + gq) * p.bias_ld + (kDistPad + pos - tok_tile - pg * 16 - th * 8 - 2 * tq);
+      const float* bt = p.bias + static_cast<size_t>(mi * 16 + gq) * p.bias_ld + (kDistPad + pos - tok_tile - pg * 16 - th0 * 8 - 2 * tq);
       const bool h_lo = mi * 16 + gq < p.heads, h_hi = mi * 16 + gq + 8 < p.heads;
       const size_t b_hi = static_cast<size_t>(8) * p.bias_ld;
-      const float b00 = h_lo ? __ldg(bt) : 0.f, b01 = h_lo ? __ldg(bt - 1) : 0.f;
-      const float b10 = h_hi ? __ldg(bt + b_hi) : 0.f, b11 = h_hi ? __ldg(bt + b_hi - 1) : 0.f;
-      float acc0[4] = {0.f, 0.f, 0.f, 0.f}, acc1[4] = {0.f, 0.f, 0.f, 0.f};
+      float b[NT][4], acc[NT][2][4];
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        b[t][0] = h_lo ? __ldg(bt - t * 8) : 0.f;
+        b[t][1] = h_lo ? __ldg(bt - t * 8 - 1) : 0.f;
+        b[t][2] = h_hi ? __ldg(bt - t * 8 + b_hi) : 0.f;
+        b[t][3] = h_hi ? __ldg(bt - t * 8 + b_hi - 1) : 0.f;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[t][0][e] = acc[t][1][e] = 0.f;
+      }
       uint32_t a_addr = a_base + mi * 16 * q_ld * 2;
-      uint32_t k_lo = ring + (pg ? slot1 : slot) * stage_bytes + swz128(th * 8 + lr, lj);
+      uint32_t k_lo = ring + (pg ? slot1 : slot) * stage_bytes + swz128(th0 * 8 + lr, lj);  // 8 tokens further: + 1 KiB
 #pragma unroll 4
       for (int c = 0; c < kc; ++c) {  // 64 of the key columns
-        uint32_t b0, b1, b2, b3, b4, b5, b6, b7, a0[4], a1[4], a2[4], a3[4];
-        ldmatrix_x4(k_lo, b0, b1, b2, b3);
-        ldmatrix_x4(k_lo ^ 64u, b4, b5, b6, b7);
+        uint32_t a0[4], a1[4], a2[4], a3[4];
         ldmatrix_x4(a_addr, a0[0], a0[1], a0[2], a0[3]);
         ldmatrix_x4(a_addr + 32, a1[0], a1[1], a1[2], a1[3]);
         ldmatrix_x4(a_addr + 64, a2[0], a2[1], a2[2], a2[3]);
         ldmatrix_x4(a_addr + 96, a3[0], a3[1], a3[2], a3[3]);
-        mma_bf16_16816(acc0, a0, b0, b1);
-        mma_bf16_16816(acc1, a1, b2, b3);
-        mma_bf16_16816(acc0, a2, b4, b5);
-        mma_bf16_16816(acc1, a3, b6, b7);
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+          uint32_t b0, b1, b2, b3, b4, b5, b6, b7;
+          ldmatrix_x4(k_lo + t * 1024, b0, b1, b2, b3);
+          ldmatrix_x4((k_lo ^ 64u) + t * 1024, b4, b5, b6, b7);
+          mma_bf16_16816(acc[t][0], a0, b0, b1);
+          mma_bf16_16816(acc[t][1], a1, b2, b3);
+          mma_bf16_16816(acc[t][0], a2, b4, b5);
+          mma_bf16_16816(acc[t][1], a3, b6, b7);
+        }
         k_lo += 2048u;
         a_addr += 128u;
       }
-      float* dst = score + (mi * 16 + gq) * kMdScoreLd + pg * 16 + th * 8 + 2 * tq;
-      *reinterpret_cast<float2*>(dst) = make_float2(fmaf(acc0[0] + acc1[0], kMixLog2e, -b00), fmaf(acc0[1] + acc1[1], kMixLog2e, -b01));
-      *reinterpret_cast<float2*>(dst + 8 * kMdScoreLd) =
-          make_float2(fmaf(acc0[2] + acc1[2], kMixLog2e, -b10), fmaf(acc0[3] + acc1[3], kMixLog2e, -b11));
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        const float *x = acc[t][0], *y = acc[t][1];
+        float* dst = score + (mi * 16 + gq) * kMdScoreLd + pg * 16 + (th0 + t) * 8 + 2 * tq;
+        *reinterpret_cast<float2*>(dst) = make_float2(fmaf(x[0] + y[0], kMixLog2e, -b[t][0]), fmaf(x[1] + y[1], kMixLog2e, -b[t][1]));
+        *reinterpret_cast<float2*>(dst + 8 * kMdScoreLd) =
+            make_float2(fmaf(x[2] + y[2], kMixLog2e, -b[t][2]), fmaf(x[3] + y[3], kMixLog2e, -b[t][3]));
+      }
+    };
+    constexpr bool kWide = UNITS <= 2 && GROUPS == 1;  // elsewhere the registers are needed
+    if (kWide && mt * 2 >= kMdWarps) {
+#pragma unroll 1
+      for (int item = w; item < mt * 2; item += kMdWarps)
+        if ((item & 1) < pages_here) score_item(std::integral_constant<int, kWide ? 2 : 1>{}, item & 1, 0, item >> 1);
+    } else {
+#pragma unroll 1
+      for (int item = w; item < mt * 4; item += kMdWarps)
+        if ((item & 1) < pages_here) score_item(std::integral_constant<int, 1>{}, item & 1, (item >> 1) & 1, item >> 2);
     }
     // the group's score tile is complete, and its other one has been read by all its warps
     asm volatile("bar.sync %0, %1;" ::"r"(1 + group), "n"(kMdWarps * 32) : "memory");

@@ -335,8 +335,8 @@ constexpr int kTileChunk = kBlk * 128;  // 64 tokens x 64 columns, 128-byte swiz
 // output (16 tokens each) while the state moves on, warp 8 asks for the next block's k and q: TMA, boxes of 64 tokens x 64 columns (past
 // a head's size they bring the next one's columns, which nobody reads; past the last token zeros).  All warps meet at two or three
 // barriers per block: state in place, residuals in place, U in place.
-template <int MT, bool DELTA>
-__global__ void __launch_bounds__(kScanThreads)
+template <int MT, bool DELTA, int CTAS>
+__global__ void __launch_bounds__(kScanThreads, CTAS)
 chunk_scan_kernel(const __grid_constant__ CUtensorMap act_map, const ChunkParams p) {
   extern __shared__ uint8_t cs_raw[];
   __shared__ __align__(8) uint64_t bar_mem[2];
@@ -673,14 +673,20 @@ static int launch_chunks(const ChunkParams& p, cudaStream_t st) {
   if (rc) return rc;
   B200_CUDA(launch_overlapped(chunk_prepare_kernel<DELTA>, dim3(p.blocks, p.heads), dim3(kChunkThreads), prep, st, p));
   const dim3 grid(p.vdim / 16, p.heads);
-#define B200_CHUNK(MT)                                                                                           \
-  do {                                                                                                           \
-    rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&chunk_scan_kernel<MT, DELTA>), 128 * 1024);          \
-    if (rc) return rc;                                                                                           \
-    B200_CUDA(launch_overlapped(chunk_scan_kernel<MT, DELTA>, grid, dim3(kScanThreads), scan, st, act_map, p)); \
+  int sms = 0;
+  rc = device_sm_count(&sms);
+  if (rc) return rc;
+  const bool two = static_cast<int>(grid.x * grid.y) > sms;  // two CTAs per SM cost registers
+#define B200_CHUNK(MT, CTAS)                                                                                       \
+  do {                                                                                                             \
+    rc = ensure_dynamic_smem(reinterpret_cast<const void*>(&chunk_scan_kernel<MT, DELTA, CTAS>), 110 * 1024);       \
+    if (rc) return rc;                                                                                             \
+    B200_CUDA(launch_overlapped(chunk_scan_kernel<MT, DELTA, CTAS>, grid, dim3(kScanThreads), scan, st, act_map, p)); \
   } while (0)
-  if (p.dim <= 64) B200_CHUNK(1);
-  else B200_CHUNK(2);
+  if (p.dim <= 64 && two) B200_CHUNK(1, 2);
+  else if (p.dim <= 64) B200_CHUNK(1, 1);
+  else if (two) B200_CHUNK(2, 2);
+  else B200_CHUNK(2, 1);
 #undef B200_CHUNK
   return 0;
 }

@@ -101,7 +101,8 @@ def test_conv_silu_in_portions_and_decoded(ops, taps, dtype):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("groups,size,ld,shared", [(4, 64, 64, True), (3, 20, 32, True), (1, 1024, 1024, False), (5, 100, 112, False)])
+@pytest.mark.parametrize("groups,size,ld,shared", [(4, 64, 64, True), (3, 20, 32, True), (1, 1024, 1024, False), (5, 100, 112, False),
+                                                   (1, 1500, 1536, False), (2, 1040, 1040, True)])
 def test_group_norm_gate(ops, groups, size, ld, shared, dtype):
     o, w = torch.zeros(6, groups, ld), torch.zeros(groups, ld)
     o[..., :size] = randn(6, groups, size, seed=1) * torch.logspace(-2, 2, groups)[None, :, None]  # groups of very different sizes
@@ -163,7 +164,7 @@ def attention_want(qm, k, v, bias, window, rows, positions):
 
 
 SHAPES = [(8, 2, 64, 64), (16, 2, 192, 128), (12, 4, 192, 64), (40, 8, 128, 128), (3, 1, 64, 64), (10, 5, 64, 256), (14, 7, 64, 192), (6, 2, 128, 192), (5, 5, 64, 128), (32, 4, 128, 128), (24, 1, 64, 64), (2, 1, 192, 320), (64, 4, 128, 128),
-          (12, 3, 64, 256)]
+          (12, 3, 64, 256), (50, 2, 192, 256)]
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
@@ -253,7 +254,7 @@ def run_recurrence(ops, A, BA, w, state, at, n, d, dv, H, delta, how, st):
 @pytest.mark.parametrize("dtype", [BF, F32])
 @pytest.mark.parametrize("delta", [True, False])
 @pytest.mark.parametrize("H,G,d,dv", [(4, 4, 64, 64), (4, 2, 128, 128), (3, 3, 16, 48), (6, 2, 48, 32), (2, 1, 32, 144), (2, 2, 208, 64),
-                                      (1, 1, 304, 16), (2, 2, 64, 256), (2, 2, 112, 16)])
+                                      (1, 1, 304, 16), (2, 2, 64, 256), (2, 2, 112, 16), (20, 20, 48, 128), (19, 19, 80, 128)])
 def test_recurrence_in_portions_and_decoded(ops, H, G, d, dv, delta, dtype):
     """Any cut of a sequence gives the whole sequence's recurrence, by every kernel that takes the portion: portions from two
     tokens on, over and at the borders of the kernels' inner blocks, decode rows in between (each run twice); other slots keep
