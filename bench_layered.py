@@ -275,8 +275,21 @@ def throughput(eng, args, table, lens, prompt_tokens: int, prompt_blocks: int, c
     B = args.batch
     V = eng.vocab_size
     eng.block_table[:, : table.shape[1]].copy_(torch.from_numpy(table))
-    eng.ctx_lens.copy_(torch.tensor(lens, dtype=torch.int32))
-    eng.tokens.copy_(torch.randint(0, V, (B,), generator=torch.Generator().manual_seed(0)))
+
+    def restart():
+        """Contexts and states as they were: with random weights the states of all rows drift the same way, step by step, and the
+        rows then choose fewer and fewer experts."""
+        eng.ctx_lens.copy_(torch.tensor(lens, dtype=torch.int32))
+        gen = torch.Generator(device=eng.device).manual_seed(7)
+        for pool in [*(getattr(eng, "states", None) or []), *(getattr(eng, "rings", None) or [])]:
+            if pool is not None:
+                pool.normal_(generator=gen)
+
+    restart()
+    # Random weights' own next tokens fall together over the steps, and with them the experts that a step reads: every step is
+    # given new random tokens instead.
+    feeds = torch.randint(0, V, (8, B), generator=torch.Generator().manual_seed(0))
+    on_device, on_host = feeds.to(eng.device), [f.view(B, 1).pin_memory() for f in feeds]
 
     def events(fn, steps):
         torch.cuda.synchronize()
@@ -288,29 +301,31 @@ def throughput(eng, args, table, lens, prompt_tokens: int, prompt_blocks: int, c
         torch.cuda.synchronize()
         return e0.elapsed_time(e1) / steps
 
-    def step(_):
-        eng.tokens[:B].copy_(eng.step(B))
+    def step(i):
+        eng.tokens[:B].copy_(on_device[i % 8])
+        eng.step(B)
 
     for i in range(1 + max(3, args.warmup)):
         step(i)
+    restart()
     if clocks is not None:
         clocks.mark()
     out = {"decode_ms": events(step, args.steps)}
     out["decode_tok_s"] = B / out["decode_ms"] * 1e3
     be = backend_mod.B200Backend(eng)
     be._alloc.free, be._slots.free = [], []
-    now = eng.ctx_lens[:B].cpu().tolist()
-    rows = [backend_mod.SeqKV(block_ids=table[b][: -(-(lens[b] + args.gen_tokens) // PAGE)].tolist(), ctx_len=now[b],
+    rows = [backend_mod.SeqKV(block_ids=table[b][: -(-(lens[b] + args.gen_tokens) // PAGE)].tolist(), ctx_len=lens[b],
                               slot=b if getattr(eng, "num_slots", 0) else None) for b in range(B)]
     batch = backend_mod.PagedBatch(rows=rows)
-    tok = torch.randint(0, V, (B, 1)).pin_memory()
-    for _ in range(3):
-        be.decode_step_batched(tok, batch)
+    for i in range(3):
+        be.decode_step_batched(on_host[i], batch)
+    restart()
+    for row in batch.rows:
+        row.ctx_len -= 3
     torch.cuda.synchronize()
     t0 = time.perf_counter()
-    for _ in range(args.steps):
-        nxt, batch = be.decode_step_batched(tok, batch)
-        tok.copy_(nxt.view(B, 1))
+    for i in range(args.steps):
+        _, batch = be.decode_step_batched(on_host[i % 8], batch)
     torch.cuda.synchronize()
     out["decode_e2e_tok_s"] = B * args.steps / (time.perf_counter() - t0)
     g = torch.Generator().manual_seed(1)

@@ -10,7 +10,8 @@ The directory name contains a hyphen, so import it with
 - ``quant``     load-time e4m3 128x128 block quantisation of expert weights.
 - ``engine``    ``PagedEngine`` (step, graphs, prompt passes) and the Qwen3-MoE
                 ``DecodeEngine`` on it.
-- ``layered``   layer-list decoders (Sulepel) on ``PagedEngine``.
+- ``layered``   layer-list decoders (Sulepel, Sefalorn) on ``PagedEngine``.
+- ``gated``     the mechanisms of gated layer-list decoders (Sefalorn).
 - ``registry``, ``checkpoint``  which engine serves a model; reading model folders.
 - ``backend``   ``B200Backend``: the reference ``InferenceBackend`` interface on
                 block tables instead of dense caches.

@@ -332,9 +332,9 @@ constexpr int kScanThreads = 9 * 32;
 constexpr int kTileChunk = kBlk * 128;  // 64 tokens x 64 columns, 128-byte swizzle
 
 // Warps 0-3 carry the state (16 tokens each of K S, the residuals and U; MT 16-row tiles each of the state), warps 4-7 make the
-// output (16 tokens each) while the state moves on, warp 8 asks for the next block's k and q: TMA, boxes of 64 tokens x 64 columns (past
-// a head's size they bring the next one's columns, which nobody reads; past the last token zeros).  All warps meet at two or three
-// barriers per block: state in place, residuals in place, U in place.
+// output (16 tokens each) while the state moves on, warp 8 asks for the next block's k and q by TMA in boxes of 64 tokens x 64
+// columns (past a head's size they bring the next one's columns, which nobody reads; past the last token zeros).  All warps meet
+// at two or three barriers per block: state in place, residuals in place, U in place.
 template <int MT, bool DELTA, int CTAS>
 __global__ void __launch_bounds__(kScanThreads, CTAS)
 chunk_scan_kernel(const __grid_constant__ CUtensorMap act_map, const ChunkParams p) {

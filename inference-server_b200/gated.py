@@ -10,8 +10,8 @@ Sizes are padded with zero rows and columns that change no result: per-head key 
 64, those of a recurrence to 16, an output map's input to 64, an expert's inner size to 128.
 
 Scores mixed over the heads are linear in the queries, so the mixing matrix moves to the queries (``ops.mix_heads``: a head's
-query becomes one vector over the keys of all kv heads, made inside the attention kernels) and the distance penalty becomes one table per head over the
-window (csrc/mixed_attn.cu).
+query becomes one vector over the keys of all kv heads, made inside the attention kernels where they can) and the distance
+penalty becomes one table per head over the window (csrc/mixed_attn.cu).
 
 State.  Attention keeps K/V in pages like every other layer.  A recurrence keeps a matrix per head, and its convolution the
 last inputs, in a slot per sequence (csrc/state_scan.cu, csrc/gated_glue.cu); both can be stepped twice from the same position,

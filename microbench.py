@@ -9,6 +9,8 @@
     python microbench.py prefill         # tiled causal prompt attention: a chunk of 1024 tokens at several
                                                                # depths of one sequence, beside the row-per-token form
     python microbench.py latent          # decode attention over latents (one vector per token, all heads), 256 sequences
+    python microbench.py mixed           # windowed decode attention with mixed heads, 256 sequences; --chunk N: a prompt
+                                                               # chunk of N tokens at the end of one sequence
     python microbench.py dense           # the bf16 projections (q/k/v, o, router, lm_head + arg-max) at decode
                                                                # sizes, every K split, beside the library GEMM
     ... attn --small / moe --small                             # few launches on a few hundred MB: sized for a profiler
@@ -159,6 +161,53 @@ def run_latent(args) -> None:
         print(json.dumps({"case": "latent", "batch": batch, "heads": H, "rank": R, "mean_ctx": float(np.mean(lens)), "split_tokens": st,
                           "us_median": med, "us_min": mn, "alg_MB": alg / 1e6, "GBs": alg / med / 1e3,
                           "frac_of_hbm_peak": alg / med / 1e3 / peak, "peak_source": src}))
+
+
+def run_mixed(args) -> None:
+    H, G, d, window, chunk = args.q_heads, args.kv_heads, args.head_dim, args.window, args.chunk
+    if args.small:
+        batch, lens = (1, [2 * window]) if chunk else (64, [2 * window] * 64)
+    else:
+        batch = 1 if chunk else args.batch
+        lens = [2 * window] if chunk else np.random.default_rng(0).integers(args.ctx_min, args.ctx_max + 1, size=batch).tolist()
+    q, kp, vp, table, ctx, _ = paged_case(batch, H, G, d, lens, 0)
+    kp, vp = (p.view(p.shape[0], G * d // 64, PAGE, 64) for p in (kp, vp))
+    q = torch.randn(chunk or batch, H, d, device=DEV).bfloat16()
+    talk = (torch.eye(H, device=DEV) + 0.1 * torch.randn(H, H, device=DEV)).bfloat16()
+    mix = (talk.float() * d ** -0.5).contiguous()
+    bias = ops.pad_distances(0.02 * torch.arange(window, device=DEV).float()[None] * torch.rand(H, 1, device=DEV))
+    out = torch.empty(chunk or batch, H * d, device=DEV, dtype=torch.bfloat16)
+    status = torch.zeros(4, dtype=torch.int32, device=DEV)
+    first = lens[0] - chunk if chunk else 0
+    ends = np.arange(first + 1, first + chunk + 1) if chunk else np.asarray(lens)
+    seen = np.minimum(ends, window)
+    read = min(lens[0], window + chunk) if chunk else int(seen.sum())
+    alg, flops = read * G * d * 4 + out.numel() * 4, 4 * int(seen.sum()) * H * d
+    peak, src = measured_hbm_gbs()
+    split = None
+    if chunk:
+        if ops.mixed_attn_prefill_form(H, G, d, d, q.dtype) != 2 or first < 0:
+            raise SystemExit("no prompt kernel on raw queries for this shape, or a chunk longer than two windows")
+        fn = lambda: ops.mixed_attn_prefill(q, kp, vp, G, table[0], first, bias, window, out, 1.0, status, talk, d ** -0.5)
+    else:
+        split = args.split_tokens or ops.mixed_split_tokens(batch, window, table.shape[1] * PAGE)
+        ws = ops.mixed_attn_workspace(batch, H, G, d, d, window, table.shape[1], split, DEV)
+        mixes = ops.mixed_attn_mixes(H, G, d, d, q.dtype)
+        qm = q if mixes else ops.mix_heads(q, mix, G)
+        fn = lambda: ops.mixed_attn(qm, kp, vp, G, table, ctx - 1, bias, window, out, 1.0, status, split, ws, mix=mix if mixes else None)
+    case = {"case": "mixed", "rows": chunk or batch, "q_heads": H, "kv_heads": G, "head_dim": d, "window": window, "split_tokens": split,
+            "alg_MB": alg / 1e6}
+    if args.small:
+        for _ in range(4):
+            fn()
+        torch.cuda.synchronize()
+        ops.read_status(status, "mixed attention")
+        print(json.dumps({**case, "case": "mixed --small", "launches": 4}))
+        return
+    med, mn = Timer(args.iters)(fn)
+    ops.read_status(status, "mixed attention")
+    print(json.dumps({**case, "us_median": med, "us_min": mn, "GBs": alg / med / 1e3, "frac_of_hbm_peak": alg / med / 1e3 / peak,
+                      "TFLOPs": flops / med / 1e6, "peak_source": src}))
 
 
 # ------------------------------------------------------------------------ MoE --
@@ -400,6 +449,16 @@ def main() -> None:
     la.add_argument("--ctx-min", type=int, default=512)
     la.add_argument("--ctx-max", type=int, default=4096)
     la.add_argument("--split-tokens", default="0", help="comma separated; 0 = the default")
+    mx = sub.add_parser("mixed")
+    mx.add_argument("--batch", type=int, default=256)
+    mx.add_argument("--q-heads", type=int, default=32)
+    mx.add_argument("--kv-heads", type=int, default=4)
+    mx.add_argument("--head-dim", type=int, default=128)
+    mx.add_argument("--window", type=int, default=1024)
+    mx.add_argument("--chunk", type=int, default=0)
+    mx.add_argument("--ctx-min", type=int, default=512)
+    mx.add_argument("--ctx-max", type=int, default=4096)
+    mx.add_argument("--split-tokens", type=int, default=0)
     m = sub.add_parser("moe")
     m.add_argument("--tokens", default=MOE_TOKENS_DEFAULT, help="token counts; with --small only the first (default 64)")
     m.add_argument("--tiled", action="store_true", help="weights stored as contiguous 128x128 blocks")
@@ -433,13 +492,13 @@ def main() -> None:
     f.add_argument("--size", type=int, default=8192)
     f.add_argument("--iters", type=int, default=20)
     f.add_argument("--small", action="store_true", help=argparse.SUPPRESS)
-    for p in (a, la, m, e):
+    for p in (a, la, mx, m, e):
         p.add_argument("--iters", type=int, default=20)
         p.add_argument("--small", action="store_true", help="a few launches on a small case (for a profiler)")
     args = ap.parse_args()
     if not torch.cuda.is_available():
         raise SystemExit("microbench.py needs a CUDA device")
-    {"attn": run_attn, "latent": run_latent, "moe": run_moe, "ep": run_ep, "fp8peak": run_fp8peak, "dense": run_dense, "prefill": run_prefill}[args.case](args)
+    {"attn": run_attn, "latent": run_latent, "mixed": run_mixed, "moe": run_moe, "ep": run_ep, "fp8peak": run_fp8peak, "dense": run_dense, "prefill": run_prefill}[args.case](args)
 
 
 if __name__ == "__main__":
