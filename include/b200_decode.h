@@ -481,9 +481,9 @@ int b200_conv_silu(const void* in, const void* conv_w, int taps, void* ring, con
                    int num_rows, int chunk, int channels, int num_slots, void* out, void* status_word, int dtype, void* stream);
 
 /*
- * A matrix state per head, S [dim, vdim] fp32: S <- g S, S <- S + k u^T, o = S^T q per token.
- *   decay given: u = v, g = decay[h].  Otherwise (gated delta rule) q and k are divided by sqrt(sum of squares + 1e-6), q
- *   multiplied by q_scale, u = beta (v - S^T k) with the decayed S, beta = sigmoid(ba[m, h]),
+ * A matrix state per head, S [dim, vdim] fp32: S_t = g S_{t-1} + k (x) e, o = q S_t per token (row vectors).
+ *   decay given: e = v, g = decay[h].  Otherwise (gated delta rule) q and k are divided by sqrt(sum of squares + 1e-6), q
+ *   multiplied by q_scale, e = beta (v - g k S_{t-1}), beta = sigmoid(ba[m, h]),
  *   g = exp(-exp(a_log[h]) softplus(ba[m, heads + h] + dt_bias[h])).
  * act [num_rows, ld] holds q [qk_heads, dim] at q_off, k at k_off and v [heads, vdim] at v_off; head h uses q/k head
  * h / (heads / qk_heads).  state [num_slots, 2, heads, dim, vdim]: the state after position p in half p & 1 of the

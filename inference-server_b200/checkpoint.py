@@ -1,7 +1,7 @@
 """Model folders that hold a config.json and one model.safetensors: reading both without a model library.
 
-A safetensors file is an 8-byte little-endian header length, the header (JSON: name -> dtype, shape, data_offsets), and
-the tensors' bytes.
+The file's layout: the header's length in 8 bytes (little-endian), the header as JSON with every tensor's dtype, shape and
+data_offsets, then the tensors' bytes.
 """
 from __future__ import annotations
 

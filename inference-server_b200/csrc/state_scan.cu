@@ -1,8 +1,8 @@
 // Recurrences over a matrix state per head (csrc of the layer-list decoders' lightning attention and gated delta rule):
 //
-//     S <- g S;   u = DELTA ? beta (v - S^T k) : v;   S <- S + k u^T;   o = S^T q
+//     S_t = g_t S_{t-1} + k_t (x) e_t,    e_t = DELTA ? beta_t (v_t - g_t k_t S_{t-1}) : v_t,    o_t = q_t S_t
 //
-// with S [dim, vdim] fp32, kept from step to step in a slot per sequence:  state [slots, 2, heads, dim, vdim].  The state
+// with row vectors, (x) the outer product and S [dim, vdim] fp32, kept from step to step in a slot per sequence:  state [slots, 2, heads, dim, vdim].  The state
 // after position p is in half p & 1 of the slot, so a decode step reads one half and writes the other and may be run
 // again; position 0 starts from zeros whatever the slot holds, so a slot needs no clearing when it changes hands.
 //
@@ -10,8 +10,8 @@
 // + dt_bias)).  Otherwise g = decay[h] and q, k are taken as they are.
 //
 // The columns of S do not meet, so a head's columns are spread over warps.  Scan kernel: a warp owns 4 * CPL columns; its
-// lanes are 8 row groups x 4 column groups, a lane holds 4 * R4 rows of CPL columns in registers.  With a = S^T k, b = S^T q of the
-// state before the token, u = beta (v - g a) and o = g b + (k . q) u: both products are taken in one pass over the state
+// lanes are 8 row groups x 4 column groups, a lane holds 4 * R4 rows of CPL columns in registers.  With a = k S, b = q S of the
+// state before the token, e = beta (v - g a) and o = g b + (k . q) e: both products are taken in one pass over the state
 // and reduced together, and the update follows.
 
 #include "glue.cuh"

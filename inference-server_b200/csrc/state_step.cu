@@ -4,8 +4,8 @@
 // columns of RPT rows; all loads are asked for before anything is computed, and the other inputs are prepared while the state
 // travels:
 // for the gated delta rule the short convolution with SiLU of this head's q, k and v channels (csrc/gated_glue.cu has it as a
-// kernel of its own), unit norms, step size and decay.  Then one pass gives a = S^T k and b = S^T q, partial sums meet in shared
-// memory, u = beta (v - g a), o = g b + (k . q) u, and S = g S + k u^T is written to the other half of the slot.  The gated
+// kernel of its own), unit norms, step size and decay.  Then one pass gives a = k S and b = q S, partial sums meet in shared
+// memory, e = beta (v - g a), o = g b + (k . q) e, and g S + k (x) e is written to the other half of the slot.  The gated
 // delta rule's output is normed per head, gated and scaled here as well; lightning's, whose norm spans the heads, goes out
 // as fp32.
 
